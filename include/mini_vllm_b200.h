@@ -312,6 +312,100 @@ int mvb_act_mul(const void* gate_up, int64_t in_row_stride, void* out, int64_t o
 int mvb_add_rmsnorm(void* x, const void* y, int64_t y_row_stride, const void* y_weight, const void* weight,
                     void* out, int rows, int hidden, float eps, int unit_offset, void* stream);
 
+/*
+ * Attention with capped scores, for models whose scores pass c tanh(s / c) before the softmax (softcap = c > 0; 0 = none)
+ * and mixers whose output carries a constant factor (out_scale; 1 = none).  Otherwise mvb_prefill_attn_items (items may be
+ * NULL here: the grid form) and mvb_decode_attn.  The cap is computed to a few fp32 ulps of c.
+ */
+int mvb_prefill_attn_capped(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* v,
+                            int64_t v_row_stride, int64_t kv_rows, const int32_t* cu_seqlens_q,
+                            const int32_t* cu_seqlens_k, const int32_t* block_table, int64_t table_stride,
+                            int block_size, int num_seqs, int total_q, int max_seqlen_q, int num_q_heads,
+                            int num_kv_heads, int head_dim, float scale, int window_left, void* out,
+                            int64_t out_row_stride, const int32_t* items, int num_items, float softcap, float out_scale,
+                            int32_t* dev_status, void* stream);
+int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
+                           int64_t num_blocks, int block_size, const int32_t* cache_seqlens, const int32_t* block_table,
+                           int64_t table_stride, int table_width, int num_seqs, int num_q_heads, int num_kv_heads,
+                           int head_dim, float scale, int window_left, void* out, int64_t out_row_stride, void* workspace,
+                           size_t workspace_bytes, float softcap, float out_scale, int32_t* dev_status, void* stream);
+
+/*
+ * The entry points below take dtype 0 (activations, weights and K/V in bf16) or 1 (fp32); the arithmetic between loads and
+ * stores is fp32 in both.  A "ragged step" has cu_seqlens_q [num_seqs + 1]; with cu_seqlens_q == NULL every sequence
+ * brings one token and row t is sequence t.  positions [num_tokens] are absolute; a sequence whose first token of the
+ * step has position 0 starts from a zero state whatever its slot holds, so slots need no clearing.  state_slots
+ * [num_seqs] picks a sequence's slot, negative = no state is read or kept (padding rows, warm-up).
+ *
+ * mvb_any_attn: attention of any head size (<= 1024), group size and dtype, one warp per (token, head), for what the
+ *   tensor-core kernels do not take.  block_table == NULL: dense K/V rows cu_seqlens_k[s] + j (row strides); else a pool of
+ *   kv_rows slots (k_row_stride = v_row_stride = num_kv_heads * head_dim).  cache_seqlens (optional): rows of length 0 give 0.
+ * mvb_rope_kv_write_f32: mvb_rope_kv_write for fp32 activations and pools.
+ */
+int mvb_any_attn(int dtype, const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* v,
+                 int64_t v_row_stride, int64_t kv_rows, const int32_t* block_table, int64_t table_stride, int table_width,
+                 int block_size, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const int64_t* positions,
+                 const int32_t* cache_seqlens, int num_seqs, int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                 float scale, int window_left, float softcap, float out_scale, void* out, int64_t out_row_stride,
+                 int32_t* dev_status, void* stream);
+int mvb_rope_kv_write_f32(float* q, int64_t q_row_stride, float* k, int64_t k_row_stride, const float* v,
+                          int64_t v_row_stride, const int64_t* positions, const float* cos_sin, int64_t max_pos,
+                          const int32_t* slot_mapping, float* k_cache, float* v_cache, int64_t num_slots, int num_tokens,
+                          int num_q_heads, int num_kv_heads, int head_dim, int k_in_place, int32_t* dev_status, void* stream);
+
+/*
+ * Glue around an fp32 residual stream x [rows, width].  rmsnorm(v, w) = v * rsqrt(mean(v^2) + eps) * w.
+ * mvb_residual_norm: x += (y_weight ? rmsnorm(y, y_weight) : y) in place; out = rmsnorm(x, weight).  row_ends != NULL: output
+ *   row r is computed from source row row_ends[r + 1] - 1 and x is left as it is.
+ * mvb_embed_norm: x[r] = table[ids[r]]; out = rmsnorm(x, weight).
+ * mvb_clamped_glu: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1) on a packed
+ *   [rows, 2 * intermediate] projection.
+ * mvb_cap_logits: out = cap tanh(in / cap) (cap == 0: a copy), each side bf16 or fp32.
+ * mvb_argmax_f32: the greedy token of fp32 logits (lowest column wins ties); scatter_* as for mvb_sample.
+ */
+int mvb_argmax_f32(const float* logits, int64_t row_stride, int rows, int cols, int64_t* out, int64_t* scatter_table,
+                   const int32_t* scatter_index, void* stream);
+int mvb_residual_norm(int dtype, float* x, const void* y, int64_t y_row_stride, const void* y_weight, const void* weight,
+                      void* out, const int32_t* row_ends, int rows, int width, float eps, void* stream);
+int mvb_embed_norm(int dtype, const int64_t* ids, const void* table, int64_t vocab, float* x, const void* weight, void* out,
+                   int rows, int width, float eps, int32_t* dev_status, void* stream);
+int mvb_clamped_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows,
+                    int intermediate, float limit, float alpha, void* stream);
+int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_stride, void* out, int64_t out_row_stride,
+                   int rows, int cols, float cap, void* stream);
+
+/*
+ * Recurrent mixers with per-sequence state slots.
+ * mvb_short_conv_silu: out[t, c] = silu(bias[c] + sum_j weight[j, c] u[t - j, c]), j < taps <= 32; inputs from before the
+ *   step come from state [num_slots, taps - 1, channels] (dtype; oldest input first), which is then brought up to date.
+ * mvb_selective_scan: S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n, out_c = (sum_n S[c, n] C_n + D_c u_c) silu(z_c),
+ *   dt = softplus(raw + dt_bias).  a_log2e [channels, state_stride] = A * log2(e), zero past num_states; state [num_slots,
+ *   channels, state_stride] fp32; state_stride a multiple of 4, num_states <= 256.
+ * mvb_gated_delta: per head S <- g * S, e = beta (v - S^T k), S <- S + k e^T, o = S^T q, with q, k made unit vectors
+ *   (1e-6 inside the root; q times q_scale), g = exp(-exp_a softplus(a + dt_bias)) per key channel, beta = sigmoid(b);
+ *   out = o / rms(o) * norm_weight * sigmoid(gate) * out_scale.  Head h reads q/k head h / (heads / kv_heads).  q, k
+ *   [tokens, kv_heads, dim], v [tokens, heads, vdim] share one row stride; dim <= 256.  state [num_slots, heads, dim,
+ *   vdim rounded up to 4] fp32.  scratch: mvb_gated_delta_scratch_bytes(...) bytes.
+ */
+int mvb_short_conv_silu(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias, void* out,
+                        int64_t out_row_stride, void* state, const int32_t* state_slots, int64_t num_slots,
+                        const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int channels,
+                        int taps, int32_t* dev_status, void* stream);
+int mvb_selective_scan(int dtype, const void* u, int64_t u_row_stride, const void* dt, int64_t dt_row_stride, const void* z,
+                       int64_t z_row_stride, const void* b, const void* c, int64_t bc_row_stride, const float* dt_bias,
+                       const float* a_log2e, const float* d, void* out, int64_t out_row_stride, float* state,
+                       const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions,
+                       int num_seqs, int num_tokens, int channels, int num_states, int state_stride, int32_t* dev_status,
+                       void* stream);
+size_t mvb_gated_delta_scratch_bytes(int num_tokens, int heads, int kv_heads, int dim, int vdim, int ragged);
+int mvb_gated_delta(int dtype, const void* q, const void* k, const void* v, int64_t qkv_row_stride, const void* a,
+                    int64_t a_row_stride, const void* b, int64_t b_row_stride, const void* gate, int64_t gate_row_stride,
+                    const float* exp_a, const float* dt_bias, const float* norm_weight, void* out, int64_t out_row_stride,
+                    float* state, const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q,
+                    const int64_t* positions, int num_seqs, int num_tokens, int heads, int kv_heads, int dim, int vdim,
+                    float q_scale, float eps, float out_scale, void* scratch, size_t scratch_bytes, int32_t* dev_status,
+                    void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -40,6 +40,25 @@ SIGNATURES = {
     "mvb_lm_head_argmax_scratch_bytes": (sz, [i32]),
     "mvb_lm_head_argmax": (i32, [vp, i64, vp, i64, i32, i32, i32, vp, vp, vp, vp, sz, vp, vp]),
     "mvb_sample": (i32, [vp, i64, i32, i32, vp, vp, vp, u64, u64, vp, vp, vp, vp, vp]),
+    "mvb_argmax_f32": (i32, [vp, i64, i32, i32, vp, vp, vp, vp]),
+    "mvb_prefill_attn_capped": (i32, [vp, i64, vp, i64, vp, i64, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32,
+                                      i32, f32, i32, vp, i64, vp, i32, f32, f32, vp, vp]),
+    "mvb_decode_attn_capped": (i32, [vp, i64, vp, vp, i64, i32, vp, vp, i64, i32, i32, i32, i32, i32, f32, i32, vp,
+                                     i64, vp, sz, f32, f32, vp, vp]),
+    "mvb_any_attn": (i32, [i32, vp, i64, vp, i64, vp, i64, i64, vp, i64, i32, i32, vp, vp, vp, vp, i32, i32, i32,
+                           i32, i32, f32, i32, f32, f32, vp, i64, vp, vp]),
+    "mvb_rope_kv_write_f32": (i32, [vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32,
+                                    vp, vp]),
+    "mvb_residual_norm": (i32, [i32, vp, vp, i64, vp, vp, vp, vp, i32, i32, f32, vp]),
+    "mvb_embed_norm": (i32, [i32, vp, vp, i64, vp, vp, vp, i32, i32, f32, vp, vp]),
+    "mvb_clamped_glu": (i32, [i32, vp, i64, vp, i64, i32, i32, f32, f32, vp]),
+    "mvb_cap_logits": (i32, [i32, i32, vp, i64, vp, i64, i32, i32, f32, vp]),
+    "mvb_short_conv_silu": (i32, [i32, vp, i64, vp, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, vp, vp]),
+    "mvb_selective_scan": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp,
+                                 vp, i32, i32, i32, i32, i32, vp, vp]),
+    "mvb_gated_delta_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32]),
+    "mvb_gated_delta": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp,
+                              vp, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, sz, vp, vp]),
 }
 
 _lib = None

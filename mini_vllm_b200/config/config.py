@@ -6,7 +6,8 @@ path-free way to describe a model, since random-init runs have no checkpoint dir
 ``hidden_size``, ``intermediate_size``, ``vocab_size``, ``rms_norm_eps``, ``attention_bias``,
 ``max_position_embeddings``, ``rope_theta``, ``tie_word_embeddings``, ``eos_token_id`` and, for
 Gemma3, ``query_pre_attn_scalar``, ``sliding_window``, ``rope_local_base_freq``).  When only
-``model`` (a Hugging Face directory) is given it is read with ``AutoConfig`` as the reference does.
+``model`` (a Hugging Face directory) is given it is read with ``AutoConfig`` as the reference does; a directory whose
+``config.json`` names an ``architecture`` of the package's own is read by ``config/native.py``.
 """
 from __future__ import annotations
 
@@ -17,12 +18,17 @@ from typing import Any, Optional, Set
 
 import torch
 
+from .native import read_native
+
 
 @dataclass
 class Config:
     model: Optional[str] = None
     hf_config: Any = None
     max_model_len: int = 4096
+    # activations, weights and KV pool; None: what the model description says (bfloat16 for a native checkpoint).  float32
+    # (no reduced-precision matrix products) is for the models of models/hybrid.py.
+    dtype: Optional[torch.dtype] = None
 
     # scheduler
     max_num_batched_tokens: int = 16384
@@ -35,6 +41,8 @@ class Config:
     gpu_memory_utilization: float = 0.5
     enable_prefix_cache: bool = False        # the reference ships with prefix caching switched off
     enable_mixed_steps: bool = False         # extension: new prompts join a step of running decodes (scheduler.py)
+    enable_chunked_prefill: bool = False     # extension: prompts enter in portions of at most the token budget
+    num_state_slots: Optional[int] = None    # recurrent models: sequences that can hold state (None: max_num_batched_seqs)
 
     # executor
     use_cuda_graph: bool = True
@@ -56,8 +64,12 @@ class Config:
             path = os.path.expanduser(self.model)
             if not os.path.isdir(path):
                 raise ValueError(f"Model path {self.model} is not a directory.")
-            from transformers import AutoConfig
-            self.hf_config = _flatten_hf(AutoConfig.from_pretrained(path))
+            self.hf_config = read_native(path, self.dtype, self.max_model_len)
+            if self.hf_config is None:
+                from transformers import AutoConfig
+                self.hf_config = _flatten_hf(AutoConfig.from_pretrained(path))
+        if self.dtype is not None:
+            self.hf_config.dtype = self.dtype
         if self.eos_token_ids is None:
             eos = getattr(self.hf_config, "eos_token_id", None)
             if eos is None:
@@ -120,3 +132,11 @@ def gemma3_shape(num_hidden_layers: int = 26, hidden_size: int = 1152, intermedi
                            rope_theta=rope_theta, rope_local_base_freq=rope_local_base_freq,
                            sliding_window=sliding_window, query_pre_attn_scalar=query_pre_attn_scalar,
                            tie_word_embeddings=tie_word_embeddings, eos_token_id=None, **extra)
+
+
+def fupupel_shape(layers: list[dict], width: int, vocab: int, eps: float = 1e-6, logit_softcap: float | None = 15.0,
+                  max_position_embeddings: int = 32768, dtype: torch.dtype = torch.bfloat16) -> SimpleNamespace:
+    """A Fupupel description without a checkpoint; ``layers`` as in its config.json."""
+    from .native import fupupel_config
+    return fupupel_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
+                           "logit_softcap": logit_softcap}, None, dtype, max_position_embeddings)

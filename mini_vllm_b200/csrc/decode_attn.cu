@@ -86,11 +86,14 @@ struct DecodeCfg {
   static_assert(NW % HPC == 0, "warps must divide evenly over the heads of a CTA");
 };
 
-static int cta_tokens_for(int hkv, int d) {
-  const int nw = d == 128 ? 8 : 4;
-  const int hpc = hkv < nw ? hkv : nw;
-  return (nw / hpc) * 16;
+// KV heads per CTA: the largest power of two that divides the head count, at most one per warp
+static int heads_per_cta(int hkv, int d) {
+  int hpc = d == 128 ? 8 : 4;
+  while (hkv % hpc != 0) hpc >>= 1;
+  return hpc;
 }
+
+static int cta_tokens_for(int hkv, int d) { return ((d == 128 ? 8 : 4) / heads_per_cta(hkv, d)) * 16; }
 
 // ---- plan -------------------------------------------------------------------------------------
 __device__ __forceinline__ int visible_start(int n, int window_left) {
@@ -183,6 +186,8 @@ struct DecodeParams {
   int num_seqs, hq, group, block_size;
   int64_t num_blocks;
   float scale_log2;
+  float cap_in, cap_log2;       // score cap c > 0: s -> c tanh(s scale / c), in log2 units; cap_log2 = 0: none
+  float out_scale;
   int window_left;
   const DecodeHeader* hdr;
   const CtaDesc* descs;
@@ -389,10 +394,14 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
       }
       const int j0 = token0 + (lane >> 2), j1 = j0 + 8;
       const bool v0 = j0 < cs.n && j0 >= cs.start, v1 = j1 < cs.n && j1 >= cs.start;
-      const float x0 = v0 ? (s0[0] + s1[0]) * p.scale_log2 : -INFINITY;
-      const float x1 = v0 ? (s0[1] + s1[1]) * p.scale_log2 : -INFINITY;
-      const float x2 = v1 ? (s0[2] + s1[2]) * p.scale_log2 : -INFINITY;
-      const float x3 = v1 ? (s0[3] + s1[3]) * p.scale_log2 : -INFINITY;
+      auto score = [&](float s) -> float {
+        if (p.cap_log2 == 0.f) return s * p.scale_log2;
+        return fmaf(-2.f * p.cap_log2, fast_rcp(1.f + fast_exp2(s * p.cap_in)), p.cap_log2);
+      };
+      const float x0 = v0 ? score(s0[0] + s1[0]) : -INFINITY;
+      const float x1 = v0 ? score(s0[1] + s1[1]) : -INFINITY;
+      const float x2 = v1 ? score(s0[2] + s1[2]) : -INFINITY;
+      const float x3 = v1 ? score(s0[3] + s1[3]) : -INFINITY;
       float ta = fmaxf(x0, x2), tb = fmaxf(x1, x3);
 #pragma unroll
       for (int off = 4; off < 32; off <<= 1) {
@@ -477,7 +486,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
         const int qh = blockIdx.y * heads + h;
         if (whole) {
           uint2 w2;
-          w2.x = pack_bf16(acc.x, acc.y); w2.y = pack_bf16(acc.z, acc.w);
+          w2.x = pack_bf16(acc.x * p.out_scale, acc.y * p.out_scale);
+          w2.y = pack_bf16(acc.z * p.out_scale, acc.w * p.out_scale);
           *reinterpret_cast<uint2*>(outp + b * p.out_stride + static_cast<int64_t>(qh) * D + dim) = w2;
         } else {
           const int64_t pi = (static_cast<int64_t>(c) * 2 + slot) * p.hq + qh;
@@ -558,7 +568,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
           const int it = threadIdx.x + k * NW * 32;
           if (it < items) {
             const int h = (it * 4) / D, dim = (it * 4) % D, qh = blockIdx.y * heads + h;
-            const float inv = wsum[k] > 0.f ? 1.f / wsum[k] : 0.f;
+            const float inv = wsum[k] > 0.f ? p.out_scale / wsum[k] : 0.f;
             uint2 w2;
             w2.x = pack_bf16(acc[k].x * inv, acc[k].y * inv); w2.y = pack_bf16(acc[k].z * inv, acc[k].w * inv);
             *reinterpret_cast<uint2*>(outp + b * p.out_stride + static_cast<int64_t>(qh) * D + dim) = w2;
@@ -602,10 +612,7 @@ static int decode_shape_ok(int hq, int hkv, int d) {
   if (hq <= 0 || hkv <= 0 || hq % hkv != 0) return 0;
   if (d != 128 && d != 256) return 0;
   const int g = hq / hkv;
-  if (g > 8) return 0;
-  const int nw = d == 128 ? 8 : 4;
-  if (hkv < nw) return (hkv == 1 || hkv == 2 || hkv == 4);
-  return hkv % nw == 0;
+  return g <= 8;
 }
 
 // Everything about a decode-attention call that can be rejected before anything is enqueued.
@@ -660,14 +667,14 @@ extern "C" int mvb_decode_plan_with_table(const int32_t* cache_seqlens, const in
                           num_kv_heads, head_dim, workspace, workspace_bytes, stream);
 }
 
-extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
-                               int64_t num_blocks, int block_size, const int32_t* cache_seqlens,
-                               const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
-                               int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left,
-                               void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
-                               int32_t* dev_status, void* stream) {
+extern "C" int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
+                                      int64_t num_blocks, int block_size, const int32_t* cache_seqlens,
+                                      const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
+                                      int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left,
+                                      void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                                      float softcap, float out_scale, int32_t* dev_status, void* stream) {
   using namespace mvb;
-  if (!workspace) return kInvalidArgument;
+  if (!workspace || !(softcap >= 0.f)) return kInvalidArgument;
   int rc = decode_check_args(q, q_row_stride, k_cache, v_cache, num_blocks, block_size, cache_seqlens, block_table,
                              table_stride, table_width, num_seqs, num_q_heads, num_kv_heads, head_dim, out,
                              out_row_stride);
@@ -690,7 +697,11 @@ extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* 
   p.table_width = table_width;
   p.num_seqs = num_seqs; p.hq = num_q_heads; p.group = num_q_heads / num_kv_heads; p.block_size = block_size;
   p.num_blocks = num_blocks;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  const float kLog2e = 1.4426950408889634f;
+  p.scale_log2 = scale * kLog2e;
+  p.cap_in = softcap > 0.f ? 2.f * scale * kLog2e / softcap : 0.f;
+  p.cap_log2 = softcap * kLog2e;
+  p.out_scale = out_scale;
   p.window_left = window_left;
   p.hdr = reinterpret_cast<const DecodeHeader*>(ws);
   p.descs = reinterpret_cast<const CtaDesc*>(ws + l.descs);
@@ -703,8 +714,7 @@ extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* 
   int num_ctas = sm_count();
   if (num_ctas > kMaxCtas) num_ctas = kMaxCtas;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int nw = head_dim == 128 ? 8 : 4;
-  const int hpc = num_kv_heads < nw ? num_kv_heads : nw;
+  const int hpc = heads_per_cta(num_kv_heads, head_dim);
   rc = kUnsupportedShape;
   if (head_dim == 128) {
     if (hpc == 8) rc = launch_decode<128, 8>(km, vm, p, num_kv_heads, num_ctas, st);
@@ -717,6 +727,17 @@ extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* 
     else if (hpc == 1) rc = launch_decode<256, 1>(km, vm, p, num_kv_heads, num_ctas, st);
   }
   return rc;
+}
+
+extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
+                               int64_t num_blocks, int block_size, const int32_t* cache_seqlens,
+                               const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
+                               int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left,
+                               void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                               int32_t* dev_status, void* stream) {
+  return mvb_decode_attn_capped(q, q_row_stride, k_cache, v_cache, num_blocks, block_size, cache_seqlens, block_table,
+                                table_stride, table_width, num_seqs, num_q_heads, num_kv_heads, head_dim, scale,
+                                window_left, out, out_row_stride, workspace, workspace_bytes, 0.f, 1.f, dev_status, stream);
 }
 
 // ---- decode attention without caller-supplied scratch ------------------------------------------------

@@ -55,7 +55,9 @@ struct PrefillParams {
   int64_t kv_rows;
   int num_seqs, hq, group;
   int pair_heads;               // 1: an item's query tiles are the heads of one GQA group over the same rows
-  float scale_log2;
+  float scale_log2;             // (with a score cap: 1, the cap's own factors carry the scale)
+  float cap_in, cap_log2;       // score cap c: s -> c tanh(s scale / c), in log2 units; 2 scale log2(e) / c and c log2(e)
+  float out_scale;              // factor of the whole output (applied with 1 / row sum)
   int window_left;
   __nv_bfloat16* out;
   int64_t out_stride;
@@ -165,7 +167,8 @@ struct PrefillItem {
 
 // LIST: the work comes as a list of (sequence, query block) pairs (PrefillParams::items) instead of a 3-D grid; a
 // kernel of its own, so that the grid form carries none of the list's code.
-template <int D, int BN, int NQ, bool LIST>
+// CAP: scores pass c tanh(s / c) before the softmax.
+template <int D, int BN, int NQ, bool LIST, bool CAP>
 __global__ void __launch_bounds__(PrefillCfg<D, BN, NQ>::THREADS, 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                     const __grid_constant__ CUtensorMap v_map, const PrefillParams p) {
@@ -536,6 +539,11 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
     const uint32_t lane_addr = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const uint32_t s_base = lane_addr + C::S_COL + t * C::S_BUFS * BN;
     const uint32_t o_addr = lane_addr + C::O_COL + t * D;
+    // c tanh(x / c) in log2 units as c - 2 c / (1 + 2^(2 x / c ...)): absolute error of a few fp32 ulps of c
+    auto cap_score = [&](uint32_t s_bits) -> uint32_t {
+      const float e = fast_exp2(__uint_as_float(s_bits) * p.cap_in);
+      return __float_as_uint(fmaf(-2.f * p.cap_log2, fast_rcp(1.f + e), p.cap_log2));
+    };
     uint32_t n_s = 0, n_epi = 0;                              // S tiles consumed (S / P parity), epilogues done (O parity)
     bool ok = true;
     Item item;
@@ -627,6 +635,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
 #pragma unroll
           for (int c = 0; c < NCH; ++c) tmem_ld_32x32(s_addr + c * 32, sreg[c]);
           tmem_wait_ld();
+          if constexpr (CAP) {
+#pragma unroll
+            for (int c = 0; c < NCH; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; ++i) sreg[c][i] = cap_score(sreg[c][i]);
+          }
           float max0 = -INFINITY, max1 = -INFINITY;
 #pragma unroll
           for (int c = 0; c < NCH; ++c)
@@ -659,6 +673,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             uint32_t r[32];
             tmem_ld_32x32(s_addr + c * 32, r);
             tmem_wait_ld();
+            if constexpr (CAP) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) r[i] = cap_score(r[i]);
+            }
             if (cl == 0) {
               float max0 = -INFINITY, max1 = -INFINITY;
 #pragma unroll
@@ -687,6 +705,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
               uint32_t r[32];
               tmem_ld_32x32(s_addr + c * 32, r);
               tmem_wait_ld();
+              if constexpr (CAP) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) r[i] = cap_score(r[i]);
+              }
               if (cl == 1) {
                 const uint32_t bits = visible_bits(c * 32);
 #pragma unroll
@@ -712,7 +734,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
       ++n_epi;
       if (ok) {
         tc_fence_after();
-        const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        const float inv = l_run > 0.f ? p.out_scale / l_run : 0.f;
         // the whole row of O, normalised, as bf16 pairs in registers; then O_t belongs to the next item
         uint32_t packed[D / 2];
 #pragma unroll
@@ -768,7 +790,7 @@ struct PrefillOperands {            // what the tensor maps are built from
   int total_q, hq, hkv;
 };
 
-template <int D, int BN, int NQ, bool LIST>
+template <int D, int BN, int NQ, bool LIST, bool CAP>
 static int launch_prefill(const PrefillOperands& op, const PrefillParams& p, int max_seqlen_q, cudaStream_t stream) {
   using C = PrefillCfg<D, BN, NQ>;
   if (p.block_table != nullptr && p.block_size % BN != 0) return kUnsupportedShape;   // a KV tile must not straddle blocks
@@ -780,8 +802,8 @@ static int launch_prefill(const PrefillOperands& op, const PrefillParams& p, int
   if (rc != kOk) return rc;
   rc = make_kv_tensor_map(&vm, op.v, op.kv_rows, op.hkv, D, op.v_stride, BN);
   if (rc != kOk) return rc;
-  using KernelTag = std::integral_constant<int, D * 8 + NQ * 2 + (LIST ? 1 : 0)>;   // one opt-in record per kernel
-  rc = opt_in_dynamic_smem<KernelTag>(reinterpret_cast<const void*>(&prefill_attn_kernel<D, BN, NQ, LIST>), C::SMEM);
+  using KernelTag = std::integral_constant<int, D * 16 + NQ * 4 + (LIST ? 2 : 0) + (CAP ? 1 : 0)>;   // one opt-in record per kernel
+  rc = opt_in_dynamic_smem<KernelTag>(reinterpret_cast<const void*>(&prefill_attn_kernel<D, BN, NQ, LIST, CAP>), C::SMEM);
   if (rc != kOk) return rc;
   PrefillParams pp = p;
   pp.pair_heads = (NQ > 1 && p.group % NQ == 0) ? 1 : 0;
@@ -793,7 +815,7 @@ static int launch_prefill(const PrefillOperands& op, const PrefillParams& p, int
     grid.y = p.num_items;
     grid.z = 1;
   }
-  prefill_attn_kernel<D, BN, NQ, LIST><<<grid, C::THREADS, C::SMEM, stream>>>(qm, km, vm, pp);
+  prefill_attn_kernel<D, BN, NQ, LIST, CAP><<<grid, C::THREADS, C::SMEM, stream>>>(qm, km, vm, pp);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
@@ -813,9 +835,10 @@ static int prefill_attn_impl(const void* q, int64_t q_row_stride, const void* k,
                              const int32_t* cu_seqlens_k, const int32_t* block_table, int64_t table_stride,
                              int block_size, int num_seqs, int total_q, int max_seqlen_q, int num_q_heads,
                              int num_kv_heads, int head_dim, float scale, int window_left, void* out,
-                             int64_t out_row_stride, const int32_t* items, int num_items, int32_t* dev_status,
-                             void* stream) {
+                             int64_t out_row_stride, const int32_t* items, int num_items, float softcap,
+                             float out_scale, int32_t* dev_status, void* stream) {
   using namespace mvb;
+  if (!(softcap >= 0.f)) return kInvalidArgument;
   if (!q || !k || !v || !cu_seqlens_q || !cu_seqlens_k || !out) return kInvalidArgument;
   if (num_seqs <= 0 || total_q < 0 || max_seqlen_q < 0 || kv_rows <= 0) return kInvalidArgument;
   if (num_q_heads <= 0 || num_kv_heads <= 0 || num_q_heads % num_kv_heads != 0) return kInvalidArgument;
@@ -833,25 +856,35 @@ static int prefill_attn_impl(const void* q, int64_t q_row_stride, const void* k,
   p.block_size = block_size; p.kv_rows = kv_rows; p.num_seqs = num_seqs; p.hq = num_q_heads;
   p.group = num_q_heads / num_kv_heads;
   p.pair_heads = 0;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  const float kLog2e = 1.4426950408889634f;
+  const bool cap = softcap > 0.f;
+  p.scale_log2 = cap ? 1.f : scale * kLog2e;
+  p.cap_in = cap ? 2.f * scale * kLog2e / softcap : 0.f;
+  p.cap_log2 = softcap * kLog2e;
+  p.out_scale = out_scale;
   p.window_left = window_left;
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_row_stride;
   p.dev_status = dev_status;
   p.items = items; p.num_items = num_items;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  // The list form pays when the grid would be mostly empty indices (a ragged batch).  When the list fills the
+  // grid - sequences of about one length - both forms take the items in the same order and the grid form,
+  // which reads no list, measured 2-3 % faster: run that one (a complete list gives identical results).
+  bool list = false;
   if (items != nullptr) {
-    // The list form pays when the grid would be mostly empty indices (a ragged batch).  When the list fills the
-    // grid - sequences of about one length - both forms take the items in the same order and the grid form,
-    // which reads no list, measured 2-3 % faster: run that one (a complete list gives identical results).
     const int rows = prefill_item_rows(num_q_heads, num_kv_heads, head_dim);
     const int64_t grid_items = static_cast<int64_t>(num_seqs) * ((max_seqlen_q + rows - 1) / rows);
-    if (static_cast<int64_t>(num_items) * 100 < grid_items * 85) {
-      if (head_dim == 128) return launch_prefill<128, 128, 2, true>(op, p, max_seqlen_q, st);
-      return launch_prefill<256, 64, 1, true>(op, p, max_seqlen_q, st);
-    }
+    list = static_cast<int64_t>(num_items) * 100 < grid_items * 85;
   }
-  if (head_dim == 128) return launch_prefill<128, 128, 2, false>(op, p, max_seqlen_q, st);
-  return launch_prefill<256, 64, 1, false>(op, p, max_seqlen_q, st);
+  auto launch = [&](auto cap_tag) {
+    constexpr bool CAP = decltype(cap_tag)::value;
+    if (head_dim == 128)
+      return list ? launch_prefill<128, 128, 2, true, CAP>(op, p, max_seqlen_q, st)
+                  : launch_prefill<128, 128, 2, false, CAP>(op, p, max_seqlen_q, st);
+    return list ? launch_prefill<256, 64, 1, true, CAP>(op, p, max_seqlen_q, st)
+                : launch_prefill<256, 64, 1, false, CAP>(op, p, max_seqlen_q, st);
+  };
+  return cap ? launch(std::true_type{}) : launch(std::false_type{});
 }
 
 extern "C" int mvb_prefill_attn(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride,
@@ -863,8 +896,8 @@ extern "C" int mvb_prefill_attn(const void* q, int64_t q_row_stride, const void*
                                 int32_t* dev_status, void* stream) {
   return prefill_attn_impl(q, q_row_stride, k, k_row_stride, v, v_row_stride, kv_rows, cu_seqlens_q, cu_seqlens_k,
                            block_table, table_stride, block_size, num_seqs, total_q, max_seqlen_q, num_q_heads,
-                           num_kv_heads, head_dim, scale, window_left, out, out_row_stride, nullptr, 0, dev_status,
-                           stream);
+                           num_kv_heads, head_dim, scale, window_left, out, out_row_stride, nullptr, 0, 0.f, 1.f,
+                           dev_status, stream);
 }
 
 extern "C" int mvb_prefill_item_rows(int num_q_heads, int num_kv_heads, int head_dim) {
@@ -881,6 +914,20 @@ extern "C" int mvb_prefill_attn_items(const void* q, int64_t q_row_stride, const
   if (items == nullptr) return mvb::kInvalidArgument;
   return prefill_attn_impl(q, q_row_stride, k, k_row_stride, v, v_row_stride, kv_rows, cu_seqlens_q, cu_seqlens_k,
                            block_table, table_stride, block_size, num_seqs, total_q, max_seqlen_q, num_q_heads,
-                           num_kv_heads, head_dim, scale, window_left, out, out_row_stride, items, num_items,
+                           num_kv_heads, head_dim, scale, window_left, out, out_row_stride, items, num_items, 0.f, 1.f,
                            dev_status, stream);
+}
+
+extern "C" int mvb_prefill_attn_capped(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride,
+                                       const void* v, int64_t v_row_stride, int64_t kv_rows,
+                                       const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
+                                       const int32_t* block_table, int64_t table_stride, int block_size, int num_seqs,
+                                       int total_q, int max_seqlen_q, int num_q_heads, int num_kv_heads, int head_dim,
+                                       float scale, int window_left, void* out, int64_t out_row_stride,
+                                       const int32_t* items, int num_items, float softcap, float out_scale,
+                                       int32_t* dev_status, void* stream) {
+  return prefill_attn_impl(q, q_row_stride, k, k_row_stride, v, v_row_stride, kv_rows, cu_seqlens_q, cu_seqlens_k,
+                           block_table, table_stride, block_size, num_seqs, total_q, max_seqlen_q, num_q_heads,
+                           num_kv_heads, head_dim, scale, window_left, out, out_row_stride, items, num_items, softcap,
+                           out_scale, dev_status, stream);
 }

@@ -1,0 +1,271 @@
+// Decoder glue around an fp32 residual stream (activations in bf16 or fp32): embedding lookup + first norm, branch
+// norm + residual add + next norm, the clamped gated activation, and the tanh cap of the logits.
+//
+// One CTA per row for the norms; a row stays in registers between the reductions, so the residual stream is read and
+// written once per sublayer.  Roofline: HBM at prefill (rows * hidden * (8 + 2 * sizeof(T)) bytes for the add + norm),
+// launch latency at decode.
+#include "dtype.cuh"
+#include "host_util.cuh"
+#include "mini_vllm_b200.h"
+
+namespace mvb {
+
+struct NormParams {
+  float* x;                     // residual stream [rows, width], fp32
+  const void* y;                // branch output (add form) or the embedding table (lookup form)
+  int64_t y_stride;
+  const int64_t* ids;           // lookup form: row r of x becomes table[ids[r]]
+  int64_t vocab;
+  const void* y_weight;         // nullptr: the branch output is added as it is
+  const void* weight;
+  void* out;
+  const int32_t* row_ends;      // nullptr, or: output row r comes from source row row_ends[r + 1] - 1 and x is left alone
+  int width;
+  float eps;
+  int* dev_status;
+};
+
+__device__ __forceinline__ float row_sum(float v, float* scratch) {
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  if (nw == 1) return v;
+  __syncthreads();                                          // scratch may still be read from a previous call
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  float s = lane < nw ? scratch[lane] : 0.f;
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+  return s;
+}
+
+template <class T, int V, int ITEMS>
+__global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p) {
+  __shared__ float scratch[32];
+  const int out_row = blockIdx.x;
+  const int row = p.row_ends != nullptr ? p.row_ends[out_row + 1] - 1 : out_row;
+  if (row < 0) return;
+  const int nvec = p.width / V, nt = blockDim.x;
+  float* xrow = p.x + static_cast<int64_t>(row) * p.width;
+  const T* yrow = static_cast<const T*>(p.y) + static_cast<int64_t>(row) * p.y_stride;
+  if (p.ids != nullptr) {
+    int64_t id = p.ids[row];
+    if (id < 0 || id >= p.vocab) {
+      if (threadIdx.x == 0) report(p.dev_status, kDevBadPosition, row);
+      id = 0;
+    }
+    yrow = static_cast<const T*>(p.y) + id * p.y_stride;
+  }
+  float v[ITEMS][V], res[ITEMS][V];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < ITEMS; ++k) {
+    const int i = threadIdx.x + k * nt;
+    if (i >= nvec) continue;
+    load_vec<T, V>(yrow + i * V, v[k]);
+    if (p.ids == nullptr) load_f32<V>(xrow + i * V, res[k]);
+  }
+  if (p.y_weight != nullptr) {
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k)
+      if (threadIdx.x + k * nt < nvec) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss += v[k][j] * v[k][j];
+      }
+    const float r = rsqrtf(row_sum(ss, scratch) / static_cast<float>(p.width) + p.eps);
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+      const int i = threadIdx.x + k * nt;
+      if (i >= nvec) continue;
+      float w[V];
+      load_vec<T, V>(static_cast<const T*>(p.y_weight) + i * V, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[k][j] = v[k][j] * r * w[j];
+    }
+  }
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < ITEMS; ++k) {
+    const int i = threadIdx.x + k * nt;
+    if (i >= nvec) continue;
+    if (p.ids == nullptr) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[k][j] += res[k][j];
+    }
+    if (p.row_ends == nullptr) store_f32<V>(xrow + i * V, v[k]);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += v[k][j] * v[k][j];
+  }
+  const float r = rsqrtf(row_sum(ss, scratch) / static_cast<float>(p.width) + p.eps);
+  T* orow = static_cast<T*>(p.out) + static_cast<int64_t>(out_row) * p.width;
+#pragma unroll
+  for (int k = 0; k < ITEMS; ++k) {
+    const int i = threadIdx.x + k * nt;
+    if (i >= nvec) continue;
+    float w[V];
+    load_vec<T, V>(static_cast<const T*>(p.weight) + i * V, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) w[j] = v[k][j] * r * w[j];
+    store_vec<T, V>(orow + i * V, w);
+  }
+}
+
+template <class T, int V>
+static int launch_norm_v(const NormParams& p, int rows, cudaStream_t st) {
+  const int nvec = p.width / V;
+  // about four vectors in flight per thread for wide rows, a whole warp at least for narrow ones
+  int items = nvec <= 128 ? 1 : (nvec <= 512 ? 2 : 4);
+  while (items < 8 && (nvec + items - 1) / items > 1024) items *= 2;
+  const int nt = ((nvec + items - 1) / items + 31) / 32 * 32;
+  if (nt > 1024) return kUnsupportedShape;
+  if (items == 1) residual_norm_kernel<T, V, 1><<<rows, nt, 0, st>>>(p);
+  else if (items == 2) residual_norm_kernel<T, V, 2><<<rows, nt, 0, st>>>(p);
+  else if (items == 4) residual_norm_kernel<T, V, 4><<<rows, nt, 0, st>>>(p);
+  else residual_norm_kernel<T, V, 8><<<rows, nt, 0, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+template <class T>
+static int launch_norm(const NormParams& p, int rows, cudaStream_t st) {
+  constexpr int V = kVec<T>;
+  const bool vec = p.width % V == 0 && p.width % 4 == 0 && p.y_stride % V == 0 && is_aligned(p.x, 16) && is_aligned(p.y, 16) &&
+                   is_aligned(p.y_weight, 16) && is_aligned(p.weight, 16) && is_aligned(p.out, 16);
+  return vec ? launch_norm_v<T, V>(p, rows, st) : launch_norm_v<T, 1>(p, rows, st);
+}
+
+// out = g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+template <class T, int V>
+__global__ void __launch_bounds__(128) clamped_glu_kernel(const T* __restrict__ gate_up, int64_t in_stride, T* __restrict__ out,
+                                                          int64_t out_stride, int rows, int inter, float limit, float alpha) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
+  if (c >= inter) return;
+  const float k = -alpha * 1.4426950408889634f;
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    const T* r = gate_up + t * in_stride + c;
+    float g[V], u[V];
+    load_vec<T, V>(r, g);
+    load_vec<T, V>(r + inter, u);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float gi = fminf(g[i], limit), ui = fminf(fmaxf(u[i], -limit), limit);
+      // gi -> -inf: exp2 -> inf, the reciprocal -> 0 and the product with the finite gi -> 0
+      g[i] = gi * fast_rcp(1.f + fast_exp2(k * gi)) * (ui + 1.f);
+    }
+    store_vec<T, V>(out + t * out_stride + c, g);
+  }
+}
+
+template <class T>
+static int launch_glu(const void* gu, int64_t is, void* out, int64_t os, int rows, int inter, float limit, float alpha,
+                      cudaStream_t st) {
+  constexpr int V = kVec<T>;
+  const bool vec = inter % V == 0 && is % V == 0 && os % V == 0 && is_aligned(gu, 16) && is_aligned(out, 16);
+  const int v = vec ? V : 1, bx = (inter + 128 * v - 1) / (128 * v);
+  int by = rows, cap = (sm_count() * 16 + bx - 1) / bx;
+  if (by > cap) by = cap;
+  if (by > 65535) by = 65535;
+  if (vec) clamped_glu_kernel<T, V><<<dim3(bx, by), 128, 0, st>>>(static_cast<const T*>(gu), is, static_cast<T*>(out), os, rows, inter, limit, alpha);
+  else clamped_glu_kernel<T, 1><<<dim3(bx, by), 128, 0, st>>>(static_cast<const T*>(gu), is, static_cast<T*>(out), os, rows, inter, limit, alpha);
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+template <class TI, class TO>
+__global__ void __launch_bounds__(256) cap_logits_kernel(const TI* __restrict__ in, int64_t in_stride, TO* __restrict__ out,
+                                                         int64_t out_stride, int cols, float cap, float inv_cap) {
+  const int64_t row = blockIdx.y;
+  for (int c = blockIdx.x * 256 + threadIdx.x; c < cols; c += gridDim.x * 256) {
+    const float v = to_f(in[row * in_stride + c]);
+    out[row * out_stride + c] = from_f<TO>(cap > 0.f ? cap * tanhf(v * inv_cap) : v);
+  }
+}
+
+// greedy token of fp32 logits: one CTA per row, the lowest column winning ties
+__global__ void __launch_bounds__(1024) argmax_f32_kernel(const float* __restrict__ logits, int64_t stride, int cols,
+                                                          int64_t* __restrict__ out, int64_t* __restrict__ scatter_table,
+                                                          const int32_t* __restrict__ scatter_index) {
+  __shared__ float bv[32];
+  __shared__ int bi[32];
+  const float* row = logits + blockIdx.x * stride;
+  float v = -INFINITY;
+  int idx = cols;
+  auto take = [&](float x, int i) { if (x > v || (x == v && i < idx)) { v = x; idx = i; } };
+  for (int c = threadIdx.x; c < cols; c += 1024) take(row[c], c);
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) {
+    const float x = __shfl_xor_sync(0xffffffffu, v, off);
+    const int i = __shfl_xor_sync(0xffffffffu, idx, off);
+    take(x, i);
+  }
+  if ((threadIdx.x & 31) == 0) { bv[threadIdx.x >> 5] = v; bi[threadIdx.x >> 5] = idx; }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    for (int w = 1; w < 32; ++w) take(bv[w], bi[w]);
+    const int64_t tok = idx < cols ? idx : 0;
+    out[blockIdx.x] = tok;
+    if (scatter_table != nullptr) scatter_table[scatter_index[blockIdx.x]] = tok;
+  }
+}
+
+}  // namespace mvb
+
+extern "C" int mvb_argmax_f32(const float* logits, int64_t row_stride, int rows, int cols, int64_t* out, int64_t* scatter_table,
+                              const int32_t* scatter_index, void* stream) {
+  using namespace mvb;
+  if (!logits || !out || rows < 0 || cols <= 0 || (scatter_table == nullptr) != (scatter_index == nullptr)) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  argmax_f32_kernel<<<rows, 1024, 0, static_cast<cudaStream_t>(stream)>>>(logits, row_stride, cols, out, scatter_table, scatter_index);
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+extern "C" int mvb_residual_norm(int dtype, float* x, const void* y, int64_t y_row_stride, const void* y_weight,
+                                 const void* weight, void* out, const int32_t* row_ends, int rows, int width, float eps,
+                                 void* stream) {
+  using namespace mvb;
+  if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  const NormParams p{x, y, y_row_stride, nullptr, 0, y_weight, weight, out, row_ends, width, eps, nullptr};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
+}
+
+extern "C" int mvb_embed_norm(int dtype, const int64_t* ids, const void* table, int64_t vocab, float* x, const void* weight,
+                              void* out, int rows, int width, float eps, int32_t* dev_status, void* stream) {
+  using namespace mvb;
+  if (!ids || !table || !x || !weight || !out || rows < 0 || width <= 0 || vocab <= 0 || (dtype != kBf16 && dtype != kF32))
+    return kInvalidArgument;
+  if (rows == 0) return kOk;
+  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, dev_status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
+}
+
+extern "C" int mvb_clamped_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride,
+                               int rows, int intermediate, float limit, float alpha, void* stream) {
+  using namespace mvb;
+  if (!gate_up || !out || rows < 0 || intermediate <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_glu<__nv_bfloat16>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, st)
+                        : launch_glu<float>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, st);
+}
+
+extern "C" int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_stride, void* out,
+                              int64_t out_row_stride, int rows, int cols, float cap, void* stream) {
+  using namespace mvb;
+  if (!in || !out || rows < 0 || cols <= 0 || !(cap >= 0.f)) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  if (rows > 65535) return kUnsupportedShape;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  int bx = (cols + 1023) / 1024;
+  if (bx > 64) bx = 64;
+  const dim3 grid(bx, rows);
+  const float inv = cap > 0.f ? 1.f / cap : 0.f;
+  auto bi = static_cast<const __nv_bfloat16*>(in); auto fi = static_cast<const float*>(in);
+  auto bo = static_cast<__nv_bfloat16*>(out); auto fo = static_cast<float*>(out);
+  if (in_dtype == kBf16 && out_dtype == kBf16) cap_logits_kernel<<<grid, 256, 0, st>>>(bi, in_row_stride, bo, out_row_stride, cols, cap, inv);
+  else if (in_dtype == kBf16 && out_dtype == kF32) cap_logits_kernel<<<grid, 256, 0, st>>>(bi, in_row_stride, fo, out_row_stride, cols, cap, inv);
+  else if (in_dtype == kF32 && out_dtype == kBf16) cap_logits_kernel<<<grid, 256, 0, st>>>(fi, in_row_stride, bo, out_row_stride, cols, cap, inv);
+  else if (in_dtype == kF32 && out_dtype == kF32) cap_logits_kernel<<<grid, 256, 0, st>>>(fi, in_row_stride, fo, out_row_stride, cols, cap, inv);
+  else return kInvalidArgument;
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}

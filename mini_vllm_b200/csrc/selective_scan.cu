@@ -1,0 +1,246 @@
+// Selective state-space scan (input-dependent diagonal recurrence) on a packed ragged batch, state carried per sequence.
+//
+//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n        dt_c = softplus(raw_c + bias_c)
+//   out_c   = (sum_n S[c, n] C_n + D_c u_c) * silu(z_c)
+//
+// Everything between the projections and the output is fp32; the state lives in fp32 slots [slots, channels, N'] (N' =
+// N rounded up to 4).  A lane owns 4 R consecutive states of one channel, L lanes a channel; the sum over n is a shuffle
+// reduction.  exp(dt A) is one ex2 with A pre-multiplied by log2(e).
+//
+// Ragged step (scan_tokens_kernel): a CTA of 4 warps walks the tokens of one sequence for 128 / L channels, TT tokens at a
+// time: raw operands of the next tile are requested into registers before the current tile is worked on, dt and dt*u
+// are computed once per (token, channel) into shared memory.
+// One token per sequence (scan_step_kernel): bound by reading and writing the state; no shared memory.
+//
+// Roofline: a ragged step is bound by the special-function unit (channels * N exponentials per token, 16 per clock and SM)
+// or, for few states, by HBM (4 activations of channels elements per token); a decode step by HBM (2 * 4 * channels * N bytes
+// per sequence).
+#include "dtype.cuh"
+#include "host_util.cuh"
+#include "mini_vllm_b200.h"
+
+namespace mvb {
+
+struct ScanParams {
+  const void* u; int64_t u_stride;
+  const void* dt; int64_t dt_stride;       // raw, before bias and softplus
+  const void* z; int64_t z_stride;
+  const void* b; const void* c; int64_t bc_stride;
+  const float* dt_bias;                    // [channels]
+  const float* a_log2e;                    // [channels, np] = A log2(e), zero in the padding
+  const float* d;                          // [channels]
+  void* out; int64_t out_stride;
+  float* state;                            // [slots, channels, np] or nullptr
+  const int32_t* slots; int64_t num_slots;
+  const int32_t* cu; const int64_t* positions;
+  int num_seqs, tokens, channels, n, np;
+  int* dev_status;
+};
+
+__device__ __forceinline__ int64_t scan_slot(const ScanParams& p, int s) {
+  if (p.state == nullptr) return -1;
+  const int64_t slot = p.slots[s];
+  if (slot >= p.num_slots) { report(p.dev_status, kDevBadSlot, s); return -1; }
+  return slot;
+}
+__device__ __forceinline__ float silu_f(float z) { return z * fast_rcp(1.f + fast_exp2(z * -1.4426950408889634f)); }
+
+// S 2^x + in.  A decay close to 1 acts over thousands of tokens, where the couple of ulps of the hardware exponential would
+// add up to more than an fp32 model's own rounding: there the decrement is computed instead of the factor.
+template <class T>
+__device__ __forceinline__ float advance(float S, float x, float in) {
+  if constexpr (sizeof(T) == 4) return fmaf(S, expm1f(x * 0.6931471805599453f), S) + in;
+  else return fmaf(fast_exp2(x), S, in);
+}
+
+template <class T, int L, int R>
+__global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
+  constexpr int CHW = 32 / L, CH = 4 * CHW, NP = 4 * L * R, TT = L <= 8 ? 32 : 16;
+  constexpr int EPT = TT * CH >= 128 ? TT * CH / 128 : 1, BPT = TT * 2 * NP / 128;
+  __shared__ float dt_s[TT][CH], du_s[TT][CH], y_s[TT][CH];
+  __shared__ __align__(16) float b_s[TT][NP];
+  __shared__ __align__(16) float c_s[TT][NP];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, sub = lane % L;
+  const int chl = warp * CHW + lane / L, c0 = blockIdx.y * CH, c = c0 + chl, s = blockIdx.x;
+  const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin;
+  if (n_tok <= 0) return;
+  const int64_t slot = scan_slot(p, s);
+  const bool fresh = p.positions[begin] == 0 || slot < 0;
+
+  float a[R][4], S[R][4];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int n0 = (sub + L * r) * 4;
+    float4 av = make_float4(0.f, 0.f, 0.f, 0.f), sv = av;
+    if (c < p.channels && n0 < p.np) {
+      av = *reinterpret_cast<const float4*>(p.a_log2e + static_cast<int64_t>(c) * p.np + n0);
+      if (!fresh) sv = *reinterpret_cast<const float4*>(p.state + (slot * p.channels + c) * p.np + n0);
+    }
+    a[r][0] = av.x; a[r][1] = av.y; a[r][2] = av.z; a[r][3] = av.w;
+    S[r][0] = sv.x; S[r][1] = sv.y; S[r][2] = sv.z; S[r][3] = sv.w;
+  }
+
+  // element e of a tile: token e / CH, channel e % CH; a thread keeps the same channel throughout
+  static_assert(128 % CH == 0 || CH == 128, "");
+  const int ech = tid % CH, etok = tid / CH;
+  constexpr int ESTEP = 128 / CH;
+  const bool ech_ok = c0 + ech < p.channels;
+  const float bias = ech_ok ? p.dt_bias[c0 + ech] : 0.f, dskip = ech_ok ? p.d[c0 + ech] : 0.f;
+  T ru[EPT], rdt[EPT], rz[EPT], rbc[BPT];
+  auto request = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < EPT; ++k) {
+      const int tl = etok + k * ESTEP, t = t0 + tl;
+      const bool ok = ech_ok && tl < TT && t < n_tok;
+      const int64_t row = begin + t;
+      ru[k] = ok ? static_cast<const T*>(p.u)[row * p.u_stride + c0 + ech] : from_f<T>(0.f);
+      rdt[k] = ok ? static_cast<const T*>(p.dt)[row * p.dt_stride + c0 + ech] : from_f<T>(0.f);
+      rz[k] = ok ? static_cast<const T*>(p.z)[row * p.z_stride + c0 + ech] : from_f<T>(0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < BPT; ++k) {
+      const int e = tid + k * 128, t = t0 + e / (2 * NP), j = e % (2 * NP), nn = j % NP;
+      const T* src = static_cast<const T*>(j < NP ? p.b : p.c);
+      rbc[k] = t < n_tok && nn < p.n ? src[(begin + t) * p.bc_stride + nn] : from_f<T>(0.f);
+    }
+  };
+  request(0);
+  for (int t0 = 0; t0 < n_tok; t0 += TT) {
+    float cu_[EPT], cz[EPT];
+#pragma unroll
+    for (int k = 0; k < EPT; ++k) {
+      const int tl = etok + k * ESTEP;
+      cu_[k] = to_f(ru[k]); cz[k] = to_f(rz[k]);
+      const float dt = softplus_f(to_f(rdt[k]) + bias);
+      if (TT * CH < 128 && tl >= TT) continue;
+      dt_s[tl][ech] = dt;
+      du_s[tl][ech] = dt * cu_[k];
+    }
+#pragma unroll
+    for (int k = 0; k < BPT; ++k) {
+      const int e = tid + k * 128, tl = e / (2 * NP), j = e % (2 * NP);
+      if (j < NP) b_s[tl][j] = to_f(rbc[k]); else c_s[tl][j - NP] = to_f(rbc[k]);
+    }
+    __syncthreads();
+    if (t0 + TT < n_tok) request(t0 + TT);
+    const int nt = min(TT, n_tok - t0);
+#pragma unroll 4
+    for (int tl = 0; tl < nt; ++tl) {
+      const float dt = dt_s[tl][chl], du = du_s[tl][chl];
+      float acc = 0.f;
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const float4 bv = *reinterpret_cast<const float4*>(&b_s[tl][(sub + L * r) * 4]);
+        const float4 cv = *reinterpret_cast<const float4*>(&c_s[tl][(sub + L * r) * 4]);
+        S[r][0] = advance<T>(S[r][0], dt * a[r][0], du * bv.x); acc = fmaf(S[r][0], cv.x, acc);
+        S[r][1] = advance<T>(S[r][1], dt * a[r][1], du * bv.y); acc = fmaf(S[r][1], cv.y, acc);
+        S[r][2] = advance<T>(S[r][2], dt * a[r][2], du * bv.z); acc = fmaf(S[r][2], cv.z, acc);
+        S[r][3] = advance<T>(S[r][3], dt * a[r][3], du * bv.w); acc = fmaf(S[r][3], cv.w, acc);
+      }
+#pragma unroll
+      for (int off = 1; off < L; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+      if (sub == 0) y_s[tl][chl] = acc;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < EPT; ++k) {
+      const int tl = etok + k * ESTEP;
+      if (ech_ok && tl < nt)
+        static_cast<T*>(p.out)[(begin + t0 + tl) * p.out_stride + c0 + ech] =
+            from_f<T>(fmaf(dskip, cu_[k], y_s[tl][ech]) * silu_f(cz[k]));
+    }
+  }
+  if (slot >= 0 && c < p.channels) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int n0 = (sub + L * r) * 4;
+      if (n0 < p.np)
+        *reinterpret_cast<float4*>(p.state + (slot * p.channels + c) * p.np + n0) = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+    }
+  }
+}
+
+template <class T, int L, int R>
+__global__ void __launch_bounds__(256) scan_step_kernel(const ScanParams p) {
+  const int s = blockIdx.y, i = blockIdx.x * 256 + threadIdx.x, c = i / L, sub = i % L;
+  const int64_t slot = scan_slot(p, s);
+  const bool fresh = slot < 0 || p.positions[s] == 0, ok = c < p.channels;
+  float acc = 0.f, u = 0.f;
+  if (ok) {
+    u = to_f(static_cast<const T*>(p.u)[s * p.u_stride + c]);
+    const float dt = softplus_f(to_f(static_cast<const T*>(p.dt)[s * p.dt_stride + c]) + p.dt_bias[c]), du = dt * u;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int n0 = (sub + L * r) * 4;
+      if (n0 >= p.np) continue;
+      float* st = p.state + (slot * p.channels + c) * p.np + n0;
+      const float4 av = *reinterpret_cast<const float4*>(p.a_log2e + static_cast<int64_t>(c) * p.np + n0);
+      const float4 sv = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
+      const float a[4] = {av.x, av.y, av.z, av.w};
+      float S[4] = {sv.x, sv.y, sv.z, sv.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const bool in = n0 + j < p.n;
+        const float bn = in ? to_f(static_cast<const T*>(p.b)[s * p.bc_stride + n0 + j]) : 0.f;
+        const float cn = in ? to_f(static_cast<const T*>(p.c)[s * p.bc_stride + n0 + j]) : 0.f;
+        S[j] = advance<T>(S[j], dt * a[j], du * bn);
+        acc = fmaf(S[j], cn, acc);
+      }
+      if (slot >= 0) *reinterpret_cast<float4*>(st) = make_float4(S[0], S[1], S[2], S[3]);
+    }
+  }
+#pragma unroll
+  for (int off = 1; off < L; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+  if (ok && sub == 0) {
+    const float z = to_f(static_cast<const T*>(p.z)[s * p.z_stride + c]);
+    static_cast<T*>(p.out)[s * p.out_stride + c] = from_f<T>(fmaf(p.d[c], u, acc) * silu_f(z));
+  }
+}
+
+template <class T, int L, int R>
+static int launch_scan_lr(const ScanParams& p, cudaStream_t st) {
+  if (p.cu == nullptr) {
+    const int64_t threads = static_cast<int64_t>(p.channels) * L;
+    if (p.num_seqs > 65535) return kUnsupportedShape;
+    scan_step_kernel<T, L, R><<<dim3(static_cast<unsigned>((threads + 255) / 256), p.num_seqs), 256, 0, st>>>(p);
+  } else {
+    constexpr int CH = 4 * (32 / L);
+    const int gy = (p.channels + CH - 1) / CH;
+    if (gy > 65535) return kUnsupportedShape;
+    scan_tokens_kernel<T, L, R><<<dim3(p.num_seqs, gy), 128, 0, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+template <class T>
+static int launch_scan(const ScanParams& p, cudaStream_t st) {
+  if (p.np <= 16) return launch_scan_lr<T, 4, 1>(p, st);
+  if (p.np <= 32) return launch_scan_lr<T, 8, 1>(p, st);
+  if (p.np <= 64) return launch_scan_lr<T, 16, 1>(p, st);
+  if (p.np <= 128) return launch_scan_lr<T, 32, 1>(p, st);
+  if (p.np <= 256) return launch_scan_lr<T, 32, 2>(p, st);
+  return kUnsupportedShape;
+}
+
+}  // namespace mvb
+
+extern "C" int mvb_selective_scan(int dtype, const void* u, int64_t u_row_stride, const void* dt, int64_t dt_row_stride,
+                                  const void* z, int64_t z_row_stride, const void* b, const void* c, int64_t bc_row_stride,
+                                  const float* dt_bias, const float* a_log2e, const float* d, void* out,
+                                  int64_t out_row_stride, float* state, const int32_t* state_slots, int64_t num_slots,
+                                  const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens,
+                                  int channels, int num_states, int state_stride, int32_t* dev_status, void* stream) {
+  using namespace mvb;
+  if (!u || !dt || !z || !b || !c || !dt_bias || !a_log2e || !d || !out || !positions) return kInvalidArgument;
+  if (num_seqs < 0 || num_tokens < 0 || channels <= 0 || num_states <= 0 || state_stride < num_states) return kInvalidArgument;
+  if (state != nullptr && (state_slots == nullptr || num_slots <= 0)) return kInvalidArgument;
+  if (cu_seqlens_q == nullptr && num_seqs != num_tokens) return kInvalidArgument;
+  if (dtype != kBf16 && dtype != kF32) return kInvalidArgument;
+  if (state_stride % 4 != 0 || !is_aligned(state, 16) || !is_aligned(a_log2e, 16)) return kMisaligned;
+  if (num_tokens == 0 || num_seqs == 0) return kOk;
+  const ScanParams p{u, u_row_stride, dt, dt_row_stride, z, z_row_stride, b, c, bc_row_stride, dt_bias, a_log2e, d, out,
+                     out_row_stride, state, state_slots, num_slots, cu_seqlens_q, positions, num_seqs, num_tokens, channels,
+                     num_states, state_stride, dev_status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_scan<__nv_bfloat16>(p, st) : launch_scan<float>(p, st);
+}

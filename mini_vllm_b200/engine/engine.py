@@ -5,6 +5,7 @@ random-init shape configs (no tokenizer on disk) ``prompt``/``completion`` are l
 """
 from __future__ import annotations
 
+import os
 from collections import deque
 
 import numpy as np
@@ -19,11 +20,17 @@ from .metrics import Metrics
 from .request import Request
 
 
+def has_tokenizer(path: str) -> bool:
+    """A checkpoint of weights and shapes alone is served by token ids; one with tokenizer files gets text as well."""
+    names = ("tokenizer.json", "tokenizer_config.json", "tokenizer.model", "vocab.json")
+    return any(os.path.exists(os.path.join(os.path.expanduser(path), n)) for n in names)
+
+
 class Engine:
     def __init__(self, config: Config):
         self.config = config
         self.tokenizer = None
-        if config.model is not None:
+        if config.model is not None and has_tokenizer(config.model):
             from transformers import AutoTokenizer
             self.tokenizer = AutoTokenizer.from_pretrained(config.model, use_fast=True)
         self.executor = Executor(config)       # may lower config.kv_cache_num_blocks to what fits
@@ -43,6 +50,34 @@ class Engine:
         self.scheduler.update(batch, tokens)
         self.metrics.update(batch)
         return batch
+
+    def replay_step(self, entries: list[tuple[Request, list[int], list[int]]]):
+        """One step over GIVEN tokens instead of sampled ones: each entry is (request, its next tokens, the places among
+        them whose logits are wanted).  All entries are one batch - portions of prompts of any length beside single
+        tokens - continuing from what earlier steps left in the cache and the state slots.  Returns fp32 logits, rows in
+        the order of the entries and places (None if no place is wanted).  ``release`` gives a request's memory back."""
+        for req, tokens, _ in entries:
+            if not tokens:
+                raise ValueError("an entry brings at least one token")
+            req.num_cached_tokens = len(req.tokens)
+            req.tokens.extend(tokens)
+            req.prompt_token_count = len(req.tokens)
+            req.state = Request.RUNNING
+            self.scheduler.block_manager.extend(req)
+        order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]) == 1)      # prompts, then single tokens
+        split = sum(len(e[1]) > 1 for e in entries)
+        first, row = {}, 0
+        for i in order:
+            first[i] = row
+            row += len(entries[i][1])
+        reqs = [entries[i][0] for i in order]
+        return self.executor.replay_logits(reqs[:split], reqs[split:],
+                                           [first[i] + k for i, e in enumerate(entries) for k in e[2]])
+
+    def release(self, req: Request) -> None:
+        """Ends a request that was driven by ``replay_step``."""
+        self.scheduler.block_manager.deallocate(req)
+        req.state = Request.FINISHED
 
     @property
     def finished(self) -> bool:
@@ -80,6 +115,8 @@ class Engine:
             batch_reqs, positions, host, event = item
             event.synchronize()
             for r, pos, tok in zip(batch_reqs, positions, host.tolist()):
+                if pos < 0:                           # a portion of a prompt yields no token
+                    continue
                 unresolved[r.id] -= 1
                 if r.id in stopped_at:                # a step that ran past the request's EOS
                     continue
@@ -121,13 +158,14 @@ class Engine:
                     if not head and not tail:
                         continue
                     batch.requests, batch.num_decode = head + tail, len(tail)
+                    batch.mark_partial()
                     if batch.type == Batch.MIXED and not (head and tail):
                         batch.type = Batch.PREFILL if head else Batch.DECODE
             slots = np.fromiter((slot_of[r.id] for r in batch.requests), np.int32, len(batch.requests))
             host, event = ex.launch(batch, slots)
-            positions = [len(r.tokens) for r in batch.requests]
-            for r in batch.requests:
-                unresolved[r.id] += 1
+            positions = [-1 if partial else len(r.tokens) for r, partial in zip(batch.requests, batch.partial)]
+            for r, pos in zip(batch.requests, positions):
+                unresolved[r.id] += pos >= 0
             sch.update(batch, [self.PLACEHOLDER] * len(batch.requests), defer_cache=True)
             self.metrics.update(batch)
             pending.append((list(batch.requests), positions, host, event))

@@ -34,7 +34,8 @@ class Metrics:
         dt = time.perf_counter() - batch.create_time
         if batch.type == Batch.MIXED:                 # counted as a decode step that also prefilled
             bp = len(batch.requests) - batch.num_decode
-            self.prefill_tokens += sum(len(r.tokens) - 1 - r.num_cached_tokens for r in batch.requests[:bp])
+            self.prefill_tokens += (batch.prefill_tokens if batch.prefill_tokens is not None else
+                                    sum(len(r.tokens) - 1 - r.num_cached_tokens for r in batch.requests[:bp]))
             self.decode_steps += 1
             self.decode_time += dt
             self.decode_tokens += batch.num_decode
@@ -42,7 +43,8 @@ class Metrics:
         elif batch.type == Batch.PREFILL:
             self.prefill_steps += 1
             self.prefill_time += dt
-            self.prefill_tokens += sum(len(r.tokens) - r.num_cached_tokens for r in batch.requests)
+            self.prefill_tokens += (batch.prefill_tokens if batch.prefill_tokens is not None else
+                                    sum(len(r.tokens) - r.num_cached_tokens for r in batch.requests))
         else:
             self.decode_steps += 1
             self.decode_time += dt

@@ -39,6 +39,12 @@ class Context:
     prefill_items: Optional[torch.Tensor] = field(default=None, repr=False, compare=False)
     prefill_item_rows: int = 0
 
+    # extension (models with recurrent layers): the state slot of every sequence, int32 [B], -1 = no state
+    state_slots: Optional[torch.Tensor] = None
+    # extension: the rows a ragged step's head reads, int32 [n + 1] with row r = logit_rows[r + 1] - 1 (None: the last
+    # token of every sequence, i.e. cu_seqlens_q itself)
+    logit_rows: Optional[torch.Tensor] = None
+
     # filled by the attention layer on first use within this forward pass
     decode_plans: dict = field(default_factory=dict, repr=False, compare=False)
     # optional device int32[4]; kernels record out-of-range slots / block ids here

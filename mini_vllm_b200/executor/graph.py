@@ -33,6 +33,7 @@ class CudaGraphRunner:
         self.slot_mapping = torch.full((m,), -1, dtype=torch.int32, device=dev)
         self.cache_seqlens = torch.zeros(m, dtype=torch.int32, device=dev)
         self.block_table = torch.full((m, config.kv_cache_num_blocks), -1, dtype=torch.int32, device=dev)
+        self.state_slots = torch.full((m,), -1, dtype=torch.int32, device=dev)     # (read by recurrent layers only)
         # The captured step ends at the rows the lm_head reads (final norm applied); the head itself - the GEMM and
         # the sampler, or the fused argmax kernel - runs behind the replay, where the executor knows whether the
         # batch samples greedily.  (The reference captures the logits, graph.py:21.)
@@ -44,7 +45,8 @@ class CudaGraphRunner:
     def static_context(self, batch_size: int) -> Context:
         return Context(prefill=False, positions=self.positions[:batch_size],
                        slot_mapping=self.slot_mapping[:batch_size], cache_seqlens=self.cache_seqlens[:batch_size],
-                       block_table=self.block_table[:batch_size], status=self.status)
+                       block_table=self.block_table[:batch_size], status=self.status,
+                       state_slots=self.state_slots[:batch_size])
 
     @torch.inference_mode()
     def capture(self) -> None:
@@ -80,6 +82,9 @@ class CudaGraphRunner:
             self.cache_seqlens.zero_()
             self.cache_seqlens[:bs] = ctx.cache_seqlens
             self.block_table[:bs, :ctx.block_table.size(1)] = ctx.block_table
+            if ctx.state_slots is not None:
+                self.state_slots.fill_(-1)
+                self.state_slots[:bs] = ctx.state_slots
         padded = self.padded_size(bs)
         self.graphs[padded].replay()
         LaunchCounter.add(self.launches[padded])

@@ -26,6 +26,7 @@ import xxhash
 
 from ..engine.request import Request
 from ..utils import cdiv
+from .state_slots import StateSlots
 
 NO_HASH = -1
 
@@ -45,8 +46,9 @@ class KVCacheBlock:
 
 class KVCacheBlockManager:
     def __init__(self, capacity: int, block_size: int, support_prefix_cache: bool = False,
-                 keep_last_block_uncached: bool = False):
+                 keep_last_block_uncached: bool = False, state_slots: StateSlots | None = None):
         self.block_size = block_size
+        self.state_slots = state_slots       # recurrent models: a request's state slot comes and goes with its blocks
         self.capacity = capacity
         self.support_prefix_cache = support_prefix_cache
         # When a whole prompt is found in the cache the reference marks every token cached, which
@@ -74,7 +76,13 @@ class KVCacheBlockManager:
         return cdiv(len(req.tokens), self.block_size) - len(req.blocks)
 
     def can_allocate_new_block(self, req: Request) -> bool:
+        if self.state_slots is not None and req.state_slot < 0 and not self.state_slots.num_free:
+            return False
         return len(self._free) >= self.request_required_blocks(req)
+
+    def _take_state_slot(self, req: Request) -> None:
+        if self.state_slots is not None and req.state_slot < 0:
+            req.state_slot = self.state_slots.take()
 
     # ---- allocation ----------------------------------------------------------------------------
     def _take(self, bid: int = -1) -> int:
@@ -98,6 +106,7 @@ class KVCacheBlockManager:
 
     def allocate_blocks_for_prefill(self, req: Request) -> None:
         assert req.state == Request.WAITING and not req.blocks
+        self._take_state_slot(req)
         bs, n = self.block_size, len(req.tokens)
         toks = np.asarray(req.tokens, dtype="<i4")
         chain, missed = NO_HASH, False
@@ -139,7 +148,18 @@ class KVCacheBlockManager:
         if self.request_required_blocks(req) > 0:
             req.blocks.append(self._take())
 
+    def extend(self, req: Request) -> None:
+        """Blocks (and the state slot) for every token the request holds now, none of them looked up or published."""
+        if not self.can_allocate_new_block(req):
+            raise RuntimeError("KV cache exhausted")
+        self._take_state_slot(req)
+        while self.request_required_blocks(req) > 0:
+            req.blocks.append(self._take())
+
     def deallocate(self, req: Request) -> None:
+        if req.state_slot >= 0:
+            self.state_slots.give(req.state_slot)
+            req.state_slot = -1
         for bid in reversed(req.blocks):
             assert self._refcount[bid] > 0
             self._refcount[bid] -= 1
@@ -148,6 +168,7 @@ class KVCacheBlockManager:
                 self._free[bid] = None
         req.blocks = []
         req.num_cached_tokens = 0
+        req.portion_end = None
 
     def cache_block_at(self, req: Request, index: int) -> None:
         """Publish block ``index`` of the request, which has become full some steps ago (the pipelined

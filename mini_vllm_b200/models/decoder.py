@@ -164,8 +164,17 @@ class DecoderLM(nn.Module):
             nxt = self.layers[i + 1].input_layernorm if i < last else self.norm
             # at prefill the lm_head reads one row per sequence: the last layer's closing add + final norm gather
             # those rows themselves instead of normalising every token and indexing afterwards
-            h = layer(ctx, x, h, positions, nxt, ctx.cu_seqlens_q if (i == last and ctx.prefill) else None)
+            rows = ctx.logit_rows if ctx.logit_rows is not None else ctx.cu_seqlens_q
+            h = layer(ctx, x, h, positions, nxt, rows if (i == last and ctx.prefill) else None)
         return self.lm_head(h) if head else h                  # the final norm is already applied
+
+    def logits(self, hidden_rows: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+        """The head on rows that ``forward(head=False)`` returned."""
+        logits = self.lm_head(hidden_rows)
+        return logits if out_dtype is None else logits.to(out_dtype)
+
+    fuses_greedy_head = True          # the head's shape suits the fused lm_head + argmax kernel
+    recurrent = False
 
     def greedy_tokens(self, hidden_rows: torch.Tensor, scratch: torch.Tensor, out: torch.Tensor | None = None,
                       scatter_table: torch.Tensor | None = None, scatter_index: torch.Tensor | None = None,

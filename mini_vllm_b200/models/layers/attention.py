@@ -9,6 +9,10 @@ embedding inside the KV-write kernel, saving one round trip of q and k through H
 
 Unlike the reference, ``scaling`` and ``sliding_window`` are honoured (the reference stores both
 and passes neither to its attention calls, ``attention.py:84-91``).
+
+Beyond the reference: ``softcap`` (scores pass ``c tanh(s / c)``), ``out_scale`` (a constant factor of the output) and,
+for activations or head layouts the tensor-core kernels do not take (fp32, head sizes other than 128 / 256, more than
+eight query heads per KV head in a decode step), the general attention kernel over the same cache.
 """
 from __future__ import annotations
 
@@ -22,11 +26,12 @@ _workspaces: dict = {}
 _superseded: list = []      # outgrown buffers stay allocated: captured CUDA graphs keep writing through their pointers
 
 
-def _decode_workspace(device, max_seqs: int, num_heads: int, head_dim: int, window_left: int) -> torch.Tensor:
+def _decode_workspace(device, max_seqs: int, num_heads: int, num_kv_heads: int, head_dim: int,
+                      window_left: int) -> torch.Tensor:
     """One scratch buffer per (device, head shape, window); a larger one takes its place when a larger batch
     arrives.  The smaller buffer is never freed: a graph captured while it was current has its address
     baked in, and a replay after the memory went back to the allocator would scribble over someone else."""
-    key = (device, num_heads, head_dim, window_left)
+    key = (device, num_heads, num_kv_heads, head_dim, window_left)
     ws = _workspaces.get(key)
     need = ops._cabi.load().mvb_decode_workspace_bytes(max_seqs, num_heads, head_dim)
     if ws is None or ws.numel() < need:
@@ -42,13 +47,14 @@ def _decode_workspace(device, max_seqs: int, num_heads: int, head_dim: int, wind
 
 class FlashAttention(nn.Module):
     def __init__(self, num_heads: int, head_dim: int, scaling: float, num_kv_heads: int,
-                 sliding_window=(-1, -1)):
+                 sliding_window=(-1, -1), softcap: float = 0.0, out_scale: float = 1.0):
         super().__init__()
         self.num_heads = num_heads
         self.head_dim = head_dim
         self.scaling = scaling
         self.num_kv_heads = num_kv_heads
         self.sliding_window = tuple(sliding_window)
+        self.softcap, self.out_scale = float(softcap), float(out_scale)
         # placeholders the executor replaces with views of its KV pool (found by hasattr)
         self.k_cache = self.v_cache = torch.tensor([])
         self._item_rows = None            # query-block size of the prefill kernel's work items for this head layout
@@ -68,13 +74,29 @@ class FlashAttention(nn.Module):
         return self._attend(ctx, q, k, v)
 
     def forward_fused(self, ctx: Context, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
-                      positions: torch.Tensor, cos_sin_cache: torch.Tensor) -> torch.Tensor:
+                      positions: torch.Tensor, cos_sin_cache: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
         """q, k NOT yet rotated: RoPE (in place on q and k) + cache write in one kernel, then attention."""
         has_cache = self._has_cache()
-        ops.rope_kv_write(q, k, v, positions, cos_sin_cache, ctx.slot_mapping if has_cache else None,
-                          self.k_cache if has_cache else None, self.v_cache if has_cache else None,
-                          k_in_place=ctx.prefill and ctx.block_table is None, status=ctx.status)
-        return self._attend(ctx, q, k, v)
+        write = ops.rope_kv_write if q.dtype == torch.bfloat16 else ops.rope_kv_write_f32
+        write(q, k, v, positions, cos_sin_cache, ctx.slot_mapping if has_cache else None,
+              self.k_cache if has_cache else None, self.v_cache if has_cache else None,
+              k_in_place=ctx.prefill and ctx.block_table is None, status=ctx.status)
+        if not self.tensor_cores(q.dtype, decode=not ctx.prefill or ctx.num_decode > 0):
+            return self._attend_any(ctx, q, k, v, positions, out)
+        return self._attend(ctx, q, k, v, out)
+
+    def tensor_cores(self, dtype: torch.dtype, decode: bool) -> bool:
+        """Whether the tensor-core kernels take this layer's activations and head layout."""
+        return (dtype == torch.bfloat16 and self.head_dim in (128, 256) and
+                (not decode or self.num_heads <= 8 * self.num_kv_heads))
+
+    def _attend_any(self, ctx: Context, q, k, v, positions, out) -> torch.Tensor:
+        paged = ctx.block_table is not None
+        return ops.any_attn(q, self.k_cache if paged else k, self.v_cache if paged else v, positions, self.scaling,
+                            self.window_left, cu_seqlens_q=ctx.cu_seqlens_q if ctx.prefill else None,
+                            cu_seqlens_k=ctx.cu_seqlens_k, block_table=ctx.block_table,
+                            cache_seqlens=None if ctx.prefill else ctx.cache_seqlens, softcap=self.softcap,
+                            out_scale=self.out_scale, out=out, status=ctx.status)
 
     def forward_fused_norm(self, ctx: Context, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
                            positions: torch.Tensor, cos_sin_cache: torch.Tensor, q_weight: torch.Tensor,
@@ -96,46 +118,43 @@ class FlashAttention(nn.Module):
             self._item_rows = ops.prefill_item_rows(self.num_heads, self.num_kv_heads, self.head_dim)
         return ctx.prefill_items if ctx.prefill_item_rows == self._item_rows else None
 
-    def _attend_mixed(self, ctx: Context, q: torch.Tensor) -> torch.Tensor:
+    def _decode(self, ctx: Context, q: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+        wl = self.window_left
+        key = (wl, self.num_heads, self.num_kv_heads, self.head_dim)
+        ws = ctx.decode_plans.get(key)
+        if ws is None:
+            ws = _decode_workspace(q.device, ctx.cache_seqlens.numel(), self.num_heads, self.num_kv_heads, self.head_dim, wl)
+            ops.decode_plan(ctx.cache_seqlens, wl, self.num_heads, self.num_kv_heads, self.head_dim, ws,
+                            block_table=table, block_size=self.k_cache.shape[1])
+            ctx.decode_plans[key] = ws
+        return ops.decode_attn(q, self.k_cache, self.v_cache, ctx.cache_seqlens, table, self.scaling, wl, ws, out=out,
+                               status=ctx.status, softcap=self.softcap, out_scale=self.out_scale)
+
+    def _prefill(self, ctx: Context, q, k, v, cu_q, cu_k, table, out=None) -> torch.Tensor:
+        return ops.prefill_attn(q, k, v, cu_q, cu_k, ctx.max_seqlen_q, self.scaling, self.window_left, block_table=table,
+                                out=out, status=ctx.status, items=self._items(ctx), softcap=self.softcap,
+                                out_scale=self.out_scale)
+
+    def _attend_mixed(self, ctx: Context, q: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
         """A step holding both kinds of sequence (an extension; the reference's Context is one or the
         other): the prompts go through the prefill kernel, the single-token sequences at the end through
         the decode kernel, both over the paged pool the write kernel has just filled."""
         nd = ctx.num_decode
         bp, tp = ctx.cu_seqlens_q.numel() - 1 - nd, q.shape[0] - nd
-        out = torch.empty(q.shape, dtype=q.dtype, device=q.device)
-        ops.prefill_attn(q[:tp], self.k_cache, self.v_cache, ctx.cu_seqlens_q[:bp + 1], ctx.cu_seqlens_k[:bp + 1],
-                         ctx.max_seqlen_q, self.scaling, self.window_left, block_table=ctx.block_table[:bp],
-                         out=out[:tp], status=ctx.status, items=self._items(ctx))
-        wl = self.window_left
-        table = ctx.block_table[bp:]
-        ws = ctx.decode_plans.get(wl)
-        if ws is None:
-            ws = _decode_workspace(q.device, nd, self.num_heads, self.head_dim, wl)
-            ops.decode_plan(ctx.cache_seqlens, wl, self.num_heads, self.num_kv_heads, self.head_dim, ws,
-                            block_table=table, block_size=self.k_cache.shape[1])
-            ctx.decode_plans[wl] = ws
-        ops.decode_attn(q[tp:], self.k_cache, self.v_cache, ctx.cache_seqlens, table, self.scaling, wl, ws, out=out[tp:],
-                        status=ctx.status)
+        if out is None:
+            out = torch.empty(q.shape, dtype=q.dtype, device=q.device)
+        self._prefill(ctx, q[:tp], self.k_cache, self.v_cache, ctx.cu_seqlens_q[:bp + 1], ctx.cu_seqlens_k[:bp + 1],
+                      ctx.block_table[:bp], out[:tp])
+        self._decode(ctx, q[tp:], ctx.block_table[bp:], out[tp:])
         return out
 
-    def _attend(self, ctx: Context, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> torch.Tensor:
+    def _attend(self, ctx: Context, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
+                out: torch.Tensor | None = None) -> torch.Tensor:
         if ctx.prefill and ctx.num_decode:
-            return self._attend_mixed(ctx, q)
+            return self._attend_mixed(ctx, q, out)
         if ctx.prefill:
             if ctx.block_table is not None:        # prefix cache in play: keys come from the pool
-                return ops.prefill_attn(q, self.k_cache, self.v_cache, ctx.cu_seqlens_q, ctx.cu_seqlens_k,
-                                        ctx.max_seqlen_q, self.scaling, self.window_left,
-                                        block_table=ctx.block_table, status=ctx.status, items=self._items(ctx))
-            return ops.prefill_attn(q, k, v, ctx.cu_seqlens_q, ctx.cu_seqlens_k, ctx.max_seqlen_q, self.scaling,
-                                    self.window_left, status=ctx.status, items=self._items(ctx))
+                k, v = self.k_cache, self.v_cache
+            return self._prefill(ctx, q, k, v, ctx.cu_seqlens_q, ctx.cu_seqlens_k, ctx.block_table, out)
         # decode: q [B,Hq,D] -> [B,1,Hq,D] like flash_attn_with_kvcache on q.unsqueeze(1)
-        wl = self.window_left
-        ws = ctx.decode_plans.get(wl)
-        if ws is None:
-            ws = _decode_workspace(q.device, ctx.cache_seqlens.numel(), self.num_heads, self.head_dim, wl)
-            ops.decode_plan(ctx.cache_seqlens, wl, self.num_heads, self.num_kv_heads, self.head_dim, ws,
-                            block_table=ctx.block_table, block_size=self.k_cache.shape[1])
-            ctx.decode_plans[wl] = ws
-        o = ops.decode_attn(q, self.k_cache, self.v_cache, ctx.cache_seqlens, ctx.block_table, self.scaling, wl, ws,
-                            status=ctx.status)
-        return o.unsqueeze(1)
+        return self._decode(ctx, q, ctx.block_table, out).unsqueeze(1)

@@ -1,0 +1,239 @@
+"""Mixer branches for decoders whose layers are assembled from parts.
+
+A branch is one token mixer (attention, selective scan, gated delta rule) without its outer projections: it declares how
+many rows it needs in the layer's packed input projection and how many columns it brings to the packed output
+projection, and works between the two.  ``PackedMixer`` puts any number of branches side by side on the same input: ONE
+input GEMM over the concatenated rows, the branches, ONE output GEMM over the concatenated columns, which also adds the
+branches up.  A branch's constant factor is applied where it writes its columns (in fp32, before rounding).
+
+Layout rules: every block a branch takes from the packed projection starts at a multiple of 8 rows, so that its view is
+16-byte aligned; padding rows have zero weights.  Recurrent branches name their per-sequence state in ``state_specs``;
+the executor owns the buffers (one row per state slot) and binds them to the attributes of the same names.
+"""
+from __future__ import annotations
+
+import math
+from typing import Callable
+
+import torch
+import torch.nn.functional as F
+from torch import nn
+
+from ... import ops
+from ...executor.context import Context
+from .attention import FlashAttention
+from .rotary import RotaryEmbedding
+
+LOG2E = 1.0 / math.log(2.0)
+Weights = Callable[[str], torch.Tensor]        # tensor of this branch by its name
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def pad_rows(w: torch.Tensor, rows: int) -> torch.Tensor:
+    return w if w.shape[0] == rows else F.pad(w, (0, 0, 0, rows - w.shape[0]))
+
+
+def pad_cols(w: torch.Tensor, cols: int) -> torch.Tensor:
+    return w if w.shape[1] == cols else F.pad(w, (0, cols - w.shape[1]))
+
+
+def weight(*shape: int) -> nn.Parameter:
+    return nn.Parameter(torch.zeros(*shape), requires_grad=False)
+
+
+def weight_f32(*shape: int) -> nn.Parameter:
+    return nn.Parameter(torch.zeros(*shape, dtype=torch.float32), requires_grad=False)
+
+
+def ragged(ctx: Context) -> torch.Tensor | None:
+    """Row boundaries of the step's sequences; None when every sequence brings one token."""
+    return ctx.cu_seqlens_q if ctx.prefill else None
+
+
+class Branch(nn.Module):
+    in_rows: int        # rows of the packed input projection, a multiple of 8
+    out_cols: int       # columns of the packed output projection, a multiple of 8
+    out_used: int       # of these, the ones the branch writes (the rest stay zero)
+
+    def state_specs(self, dtype: torch.dtype) -> dict[str, tuple[tuple[int, ...], torch.dtype]]:
+        return {}
+
+    def load(self, w: Weights) -> tuple[torch.Tensor, torch.Tensor]:
+        """Load the branch's own parameters; returns its input rows [in_rows, width] and output columns [width, out_cols]."""
+        raise NotImplementedError
+
+    def forward(self, ctx: Context, proj: torch.Tensor, out: torch.Tensor, positions: torch.Tensor) -> None:
+        raise NotImplementedError
+
+
+class AttentionBranch(Branch):
+    """Grouped-query attention with rotation, optional window and score cap, and a value size of its own.
+
+    The kernels know one head size, so q/k heads (``dim``) and v heads (``vdim``) are both padded to it inside the packed
+    projections: zero rows cost nothing but projection width, leave every score unchanged and give zero output columns
+    that meet zero columns of the output projection.  The rotated pairs (i, i + dims/2) are laid out at (i, i + D/2) - a
+    permutation common to q and k, which no score sees - so the kernel that pairs the halves of a head serves any
+    ``rot_dims``; the coordinates that are not rotated fill the other pairs and get angle 0."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rotary: RotaryEmbedding, rot_dims: int,
+                 padded: int, window: int | None = None, softcap: float | None = None, factor: float = 1.0):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim, self.d, self.rot_dims = heads, kv_heads, dim, vdim, padded, rot_dims
+        self.rotary = rotary
+        self.attn = FlashAttention(heads, padded, scale, kv_heads, (-1 if window is None else window - 1, -1),
+                                   softcap=softcap or 0.0, out_scale=factor)
+        self.in_rows = (heads + 2 * kv_heads) * padded
+        self.out_cols = self.out_used = heads * padded
+
+    @staticmethod
+    def padded_size(dim: int, vdim: int, dtype: torch.dtype) -> int:
+        d = max(dim, vdim)
+        if dtype == torch.bfloat16 and d <= 256:
+            return 128 if d <= 128 else 256
+        return -(-d // 16) * 16
+
+    def _layout(self) -> torch.Tensor:
+        """Where coordinate i of a q/k head goes inside the padded head."""
+        half, r = self.d // 2, self.rot_dims // 2
+        free = [j for j in range(self.d) if not (j < r or half <= j < half + r)]
+        place = list(range(r)) + [half + i for i in range(r)] + free[:self.dim - 2 * r]
+        return torch.tensor(place, dtype=torch.long)
+
+    def load(self, w: Weights):
+        rows = []
+        place = self._layout()
+        for name, n, used in (("q", self.heads, self.dim), ("k", self.kv_heads, self.dim), ("v", self.kv_heads, self.vdim)):
+            src = w(name)
+            dst = src.new_zeros(n, self.d, src.shape[1])
+            dst[:, place.to(src.device) if name != "v" else slice(0, used)] = src.view(n, used, -1)
+            rows.append(dst.view(n * self.d, -1))
+        o = w("o")
+        cols = o.new_zeros(o.shape[0], self.heads, self.d)
+        cols[:, :, :self.vdim] = o.view(o.shape[0], self.heads, self.vdim)
+        return torch.cat(rows), cols.view(o.shape[0], -1)
+
+    def forward(self, ctx, proj, out, positions):
+        h, g, d = self.heads, self.kv_heads, self.d
+        q, k, v = (t.unflatten(1, (-1, d)) for t in proj.split([h * d, g * d, g * d], dim=1))
+        self.attn.forward_fused(ctx, q, k, v, positions, self.rotary.cos_sin_cache, out=out.unflatten(1, (h, d)))
+
+
+class SelectiveScanBranch(Branch):
+    """Mamba's selective scan: short convolution, input-dependent step and B / C, diagonal recurrence, gate."""
+
+    def __init__(self, inner: int, states: int, dt_rank: int, taps: int):
+        super().__init__()
+        self.inner, self.states, self.rank, self.taps = inner, states, dt_rank, taps
+        self.ip, self.rp, self.sp = pad8(inner), pad8(dt_rank), pad8(states)
+        self.np = -(-states // 4) * 4
+        self.in_rows, self.out_cols, self.out_used = 2 * self.ip, self.ip, inner
+        self.conv_weight, self.conv_bias = weight(taps, self.ip), weight(self.ip)
+        self.x_proj, self.dt_proj = weight(self.rp + 2 * self.sp, self.ip), weight(inner, self.rp)
+        self.dt_bias, self.a_log2e, self.skip = weight_f32(inner), weight_f32(inner, self.np), weight_f32(inner)
+        self.conv_state = self.scan_state = None
+
+    def state_specs(self, dtype):
+        return {"conv_state": ((self.taps - 1, self.ip), dtype), "scan_state": ((self.inner, self.np), torch.float32)}
+
+    def load(self, w: Weights):
+        x, z = w("in").split([self.inner, self.inner])
+        self.conv_weight.copy_(pad_cols(w("conv").flip(1).T, self.ip))
+        self.conv_bias.copy_(F.pad(w("conv.b"), (0, self.ip - self.inner)))
+        dt, b, c = (pad_cols(t, self.ip) for t in w("x").split([self.rank, self.states, self.states]))
+        self.x_proj.copy_(torch.cat([pad_rows(dt, self.rp), pad_rows(b, self.sp), pad_rows(c, self.sp)]))
+        self.dt_proj.copy_(pad_cols(w("dt"), self.rp))
+        self.dt_bias.copy_(w("dt.b").float())
+        self.a_log2e.copy_(pad_cols(-torch.exp(w("A_log").float()) * LOG2E, self.np))
+        self.skip.copy_(w("D").float())
+        return torch.cat([pad_rows(x, self.ip), pad_rows(z, self.ip)]), pad_cols(w("o"), self.out_cols)
+
+    def forward(self, ctx, proj, out, positions):
+        cu = ragged(ctx)
+        u = ops.short_conv_silu(proj[:, :self.ip], self.conv_weight, self.conv_bias, self.conv_state, ctx.state_slots, cu,
+                                positions, status=ctx.status)
+        x = F.linear(u, self.x_proj)
+        dt = F.linear(x[:, :self.rp], self.dt_proj)
+        ops.selective_scan(u[:, :self.inner], dt, proj[:, self.ip:self.ip + self.inner], x[:, self.rp:self.rp + self.states],
+                           x[:, self.rp + self.sp:self.rp + self.sp + self.states], self.dt_bias, self.a_log2e, self.skip,
+                           out[:, :self.inner], self.scan_state, ctx.state_slots, cu, positions, status=ctx.status)
+
+
+class GatedDeltaBranch(Branch):
+    """Gated delta rule with a decay per head and key channel, short convolutions on q, k, v and a gated output norm.
+
+    The two low-rank pairs (decay, output gate) share one second GEMM with a block-diagonal weight."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, decay_rank: int, gate_rank: int, eps: float,
+                 factor: float = 1.0):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim, self.taps = heads, kv_heads, dim, vdim, taps
+        self.eps, self.factor = eps, factor
+        self.decay_rank, self.gate_rank = decay_rank, gate_rank
+        self.kp, self.vp = pad8(kv_heads * dim), pad8(heads * vdim)            # conv channels: q | k | v
+        self.channels = 2 * self.kp + self.vp
+        self.bp, self.ap, self.gp = pad8(heads), pad8(decay_rank), pad8(gate_rank)
+        self.hp = pad8(heads * dim)
+        self.in_rows = self.channels + self.bp + self.ap + self.gp
+        self.out_cols, self.out_used = self.vp, heads * vdim
+        self.conv_weight = weight(taps, self.channels)
+        self.low_rank = weight(self.hp + self.vp, self.ap + self.gp)
+        self.exp_a, self.dt_bias, self.norm_weight = weight_f32(heads), weight_f32(heads * dim), weight_f32(vdim)
+        self.conv_state = self.delta_state = None
+
+    def state_specs(self, dtype):
+        return {"conv_state": ((self.taps - 1, self.channels), dtype),
+                "delta_state": ((self.heads, self.dim, -(-self.vdim // 4) * 4), torch.float32)}
+
+    def load(self, w: Weights):
+        sizes = {"q": self.kp, "k": self.kp, "v": self.vp}
+        self.conv_weight.copy_(torch.cat([pad_cols(w(n + ".conv").flip(1).T, c) for n, c in sizes.items()], dim=1))
+        self.low_rank.zero_()
+        a2, g2 = w("a2"), w("g2")
+        self.low_rank[:a2.shape[0], :self.decay_rank].copy_(a2)
+        self.low_rank[self.hp:self.hp + g2.shape[0], self.ap:self.ap + self.gate_rank].copy_(g2)
+        self.exp_a.copy_(torch.exp(w("A_log").float()).reshape(-1))
+        self.dt_bias.copy_(w("dt_bias").float().reshape(-1))
+        self.norm_weight.copy_(w("norm").float())
+        rows = [pad_rows(w(n), c) for n, c in sizes.items()]
+        rows += [pad_rows(w(n), c) for n, c in (("b", self.bp), ("a1", self.ap), ("g1", self.gp))]
+        return torch.cat(rows), pad_cols(w("o"), self.out_cols)
+
+    def forward(self, ctx, proj, out, positions):
+        cu, c, kv, h = ragged(ctx), self.channels, self.kv_heads * self.dim, self.heads
+        low = F.linear(proj[:, c + self.bp:], self.low_rank)
+        qkv = ops.short_conv_silu(proj[:, :c], self.conv_weight, None, self.conv_state, ctx.state_slots, cu, positions,
+                                  status=ctx.status)
+        q, k = (qkv[:, i * self.kp:i * self.kp + kv].unflatten(1, (self.kv_heads, self.dim)) for i in (0, 1))
+        v = qkv[:, 2 * self.kp:2 * self.kp + h * self.vdim].unflatten(1, (h, self.vdim))
+        ops.gated_delta(q, k, v, low[:, :h * self.dim], proj[:, c:c + h], low[:, self.hp:self.hp + h * self.vdim], self.exp_a,
+                        self.dt_bias, self.norm_weight, out[:, :h * self.vdim].unflatten(1, (h, self.vdim)), self.delta_state,
+                        ctx.state_slots, cu, positions, self.dim ** -0.5, self.eps, self.factor, status=ctx.status)
+
+
+class PackedMixer(nn.Module):
+    """Branches side by side on one input; their outputs meet in one output projection."""
+
+    def __init__(self, width: int, branches: dict[str, Branch]):
+        super().__init__()
+        self.branches = nn.ModuleDict(branches)
+        self.in_sizes = [b.in_rows for b in branches.values()]
+        self.out_sizes = [b.out_cols for b in branches.values()]
+        self.in_proj, self.out_proj = weight(sum(self.in_sizes), width), weight(width, sum(self.out_sizes))
+        self.dense_out = all(b.out_used == b.out_cols for b in branches.values())
+
+    @torch.no_grad()
+    def load(self, prefixes: dict[str, str], w: Weights) -> None:
+        parts = [b.load(lambda n, p=prefixes[key]: w(p + n)) for key, b in self.branches.items()]
+        self.in_proj.copy_(torch.cat([p[0] for p in parts]))
+        self.out_proj.copy_(torch.cat([p[1] for p in parts], dim=1))
+
+    def forward(self, ctx: Context, h: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+        proj = F.linear(h, self.in_proj)
+        make = torch.empty if self.dense_out else torch.zeros     # columns nobody writes meet zero weights and must be finite
+        y = make(h.shape[0], self.out_proj.shape[1], dtype=h.dtype, device=h.device)
+        for b, pi, yi in zip(self.branches.values(), proj.split(self.in_sizes, dim=1), y.split(self.out_sizes, dim=1)):
+            b(ctx, pi, yi, positions)
+        return F.linear(y, self.out_proj)

@@ -27,6 +27,8 @@ class Sampler(nn.Module):
                 top_p: Optional[torch.Tensor] = None, top_k: Optional[torch.Tensor] = None,
                 scatter_table: Optional[torch.Tensor] = None, scatter_index: Optional[torch.Tensor] = None
                 ) -> torch.Tensor:
+        if logits.dtype == torch.float32 and top_k is None and top_p is None:
+            return ops.argmax_f32(logits, scatter_table=scatter_table, scatter_index=scatter_index)
         if logits.dtype != torch.bfloat16:
             logits = logits.to(torch.bfloat16)
         if top_k is None and top_p is None:

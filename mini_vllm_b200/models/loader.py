@@ -32,6 +32,8 @@ def load_model(config, device="cuda") -> torch.nn.Module:
     finally:
         torch.set_default_dtype(prev)
     model.to(device)          # moves the CPU-built fp32 cos/sin tables; parameters are already there
+    if getattr(model, "recurrent", False) and getattr(config, "enable_prefix_cache", False):
+        raise ValueError("prefix caching needs a model without recurrent state (cached blocks hold no state)")
     fuse = bool(getattr(config, "fuse_qk_norm", True))
     for module in model.modules():
         if hasattr(module, "fuse_qk_norm"):

@@ -12,6 +12,7 @@ from . import _cabi
 _DEV_ERRORS = {1: "slot outside the KV pool", 2: "block id outside the KV pool",
                3: "position outside the cos/sin table", 4: "a bounded device wait ran out",
                5: "sequence length does not fit its block list"}
+_DTYPE = {torch.bfloat16: 0, torch.float32: 1}      # the dtype argument of the entry points that take either
 
 
 class LaunchCounter:
@@ -215,8 +216,10 @@ def decode_plan(cache_seqlens: torch.Tensor, window_left: int, num_q_heads: int,
 
 def decode_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cache_seqlens: torch.Tensor,
                 block_table: torch.Tensor, scale: float, window_left: int, workspace: torch.Tensor,
-                out: torch.Tensor | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
-    """q [B,Hq,D]; the plan for (cache_seqlens, window_left) must already be in ``workspace``."""
+                out: torch.Tensor | None = None, status: torch.Tensor | None = None, softcap: float = 0.0,
+                out_scale: float = 1.0) -> torch.Tensor:
+    """q [B,Hq,D]; the plan for (cache_seqlens, window_left) must already be in ``workspace``.  ``softcap`` > 0: scores
+    pass ``softcap * tanh(score / softcap)``; ``out_scale`` multiplies the output."""
     _need(q, torch.bfloat16, "q"); _heads_contiguous(q, "q")
     _need(cache_seqlens, torch.int32, "cache_seqlens"); _need(block_table, torch.int32, "block_table")
     B, hq, d = q.shape
@@ -226,11 +229,11 @@ def decode_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
     assert cache_seqlens.numel() >= B
     if out is None:
         out = torch.empty(B, hq, d, dtype=torch.bfloat16, device=q.device)
-    rc = _cabi.load().mvb_decode_attn(
+    rc = _cabi.load().mvb_decode_attn_capped(
         _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), nblk, bs, _ptr(cache_seqlens), _ptr(block_table),
         block_table.stride(0), block_table.shape[1], B, hq, hkv, d, float(scale), window_left, _ptr(out),
-        out.stride(0), _ptr(workspace), workspace.numel(), _ptr(status), _stream())
-    _cabi.check(rc, "mvb_decode_attn")
+        out.stride(0), _ptr(workspace), workspace.numel(), float(softcap), float(out_scale), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_decode_attn_capped")
     LaunchCounter.add(1)
     return out
 
@@ -288,7 +291,8 @@ def build_prefill_items(q_lens, k_lens, item_rows: int):
 def prefill_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q: torch.Tensor,
                  cu_seqlens_k: torch.Tensor, max_seqlen_q: int, scale: float, window_left: int = -1,
                  block_table: torch.Tensor | None = None, out: torch.Tensor | None = None,
-                 status: torch.Tensor | None = None, items: torch.Tensor | None = None) -> torch.Tensor:
+                 status: torch.Tensor | None = None, items: torch.Tensor | None = None, softcap: float = 0.0,
+                 out_scale: float = 1.0) -> torch.Tensor:
     """q [Tq,Hq,D]; k/v dense [Tk,Hkv,D] (block_table None) or the paged pool [blocks,bs,Hkv,D].
 
     ``items`` (int32 [n, 2] on the device, from ``build_prefill_items``) gives the launch its work as a list of
@@ -307,21 +311,16 @@ def prefill_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q
         kv_rows, k_stride, v_stride, tstride = nblk * bs, hkv * d, hkv * d, block_table.stride(0)
     if out is None:
         out = torch.empty(Tq, hq, d, dtype=torch.bfloat16, device=q.device)
-    if items is not None and 0 < items.shape[0] <= 65535:
+    use = items is not None and 0 < items.shape[0] <= 65535
+    if use:
         _need(items, torch.int32, "items")
         assert items.dim() == 2 and items.shape[1] == 2 and items.is_contiguous()
-        rc = _cabi.load().mvb_prefill_attn_items(
-            _ptr(q), q.stride(0), _ptr(k), k_stride, _ptr(v), v_stride, kv_rows, _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
-            _ptr(block_table), tstride, bs, cu_seqlens_q.numel() - 1, Tq, int(max_seqlen_q), hq, hkv, d, float(scale),
-            window_left, _ptr(out), out.stride(0), _ptr(items), items.shape[0], _ptr(status), _stream())
-        _cabi.check(rc, "mvb_prefill_attn_items")
-        LaunchCounter.add(1)
-        return out
-    rc = _cabi.load().mvb_prefill_attn(
+    rc = _cabi.load().mvb_prefill_attn_capped(
         _ptr(q), q.stride(0), _ptr(k), k_stride, _ptr(v), v_stride, kv_rows, _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
         _ptr(block_table), tstride, bs, cu_seqlens_q.numel() - 1, Tq, int(max_seqlen_q), hq, hkv, d, float(scale),
-        window_left, _ptr(out), out.stride(0), _ptr(status), _stream())
-    _cabi.check(rc, "mvb_prefill_attn")
+        window_left, _ptr(out), out.stride(0), _ptr(items) if use else None, items.shape[0] if use else 0,
+        float(softcap), float(out_scale), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_prefill_attn_capped")
     LaunchCounter.add(1)
     return out
 
@@ -426,4 +425,241 @@ def lm_head_argmax(hidden_states: torch.Tensor, weight: torch.Tensor, scratch: t
                                          scratch.numel(), _ptr(status), _stream())
     _cabi.check(rc, "mvb_lm_head_argmax")
     LaunchCounter.add(1)
+    return out
+
+
+# ---- kernels that run in bf16 or fp32 -----------------------------------------------------------------------
+def _dtype_of(t: torch.Tensor, name: str) -> int:
+    if not t.is_cuda:
+        raise ValueError(f"{name} must be a CUDA tensor (the kernels have no CPU path)")
+    if t.dtype not in _DTYPE:
+        raise TypeError(f"{name} must be bfloat16 or float32, got {t.dtype}")
+    return _DTYPE[t.dtype]
+
+
+def _same(dtype, **tensors) -> None:
+    for name, t in tensors.items():
+        if t is not None:
+            _need(t, dtype, name)
+
+
+def any_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: torch.Tensor, scale: float,
+             window_left: int = -1, cu_seqlens_q: torch.Tensor | None = None, cu_seqlens_k: torch.Tensor | None = None,
+             block_table: torch.Tensor | None = None, cache_seqlens: torch.Tensor | None = None, softcap: float = 0.0,
+             out_scale: float = 1.0, out: torch.Tensor | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Attention of any head size, group size and dtype (one warp per token and head).  k/v are the paged pool with a
+    ``block_table``, else dense rows; without ``cu_seqlens_q`` every row is a sequence of its own."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v)
+    _heads_contiguous(q, "q")
+    _need(positions, torch.int64, "positions")
+    tokens, hq, d = q.shape
+    if block_table is not None:
+        _need(block_table, torch.int32, "block_table")
+        assert k.dim() == 4 and k.is_contiguous() and v.is_contiguous() and v.shape == k.shape and block_table.stride(1) == 1
+        nblk, bs, hkv, _ = k.shape
+        kv_rows, ks, vs, tstride, width = nblk * bs, hkv * d, hkv * d, block_table.stride(0), block_table.shape[1]
+    else:
+        _heads_contiguous(k, "k"); _heads_contiguous(v, "v")
+        _need(cu_seqlens_k, torch.int32, "cu_seqlens_k")
+        kv_rows, hkv, ks, vs, bs, tstride, width = k.shape[0], k.shape[1], k.stride(0), v.stride(0), 0, 0, 0
+    num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
+    if out is None:
+        out = torch.empty(tokens, hq, d, dtype=q.dtype, device=q.device)
+    rc = _cabi.load().mvb_any_attn(
+        code, _ptr(q), q.stride(0), _ptr(k), ks, _ptr(v), vs, kv_rows, _ptr(block_table), tstride, width, bs,
+        _ptr(cu_seqlens_q), _ptr(cu_seqlens_k), _ptr(positions), _ptr(cache_seqlens), num_seqs, tokens, hq, hkv, d,
+        float(scale), window_left, float(softcap), float(out_scale), _ptr(out), out.stride(0), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_any_attn")
+    LaunchCounter.add(1)
+    return out
+
+
+def rope_kv_write_f32(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tensor,
+                      slot_mapping: torch.Tensor | None, k_cache: torch.Tensor | None, v_cache: torch.Tensor | None,
+                      k_in_place: bool = True, status: torch.Tensor | None = None) -> None:
+    """``rope_kv_write`` for fp32 activations and pools."""
+    _same(torch.float32, q=q, k=k, v=v, cos_sin=cos_sin)
+    for t, n in ((q, "q"), (k, "k"), (v, "v")):
+        _heads_contiguous(t, n)
+    _need(positions, torch.int64, "positions")
+    tokens, hkv, d = k.shape
+    assert cos_sin.is_contiguous() and cos_sin.shape[1] == d and q.shape[2] == d
+    num_slots = 0
+    if slot_mapping is not None:
+        _need(slot_mapping, torch.int32, "slot_mapping")
+        _same(torch.float32, k_cache=k_cache, v_cache=v_cache)
+        assert k_cache.is_contiguous() and v_cache.is_contiguous()
+        num_slots = k_cache.shape[0] * k_cache.shape[1]
+    rc = _cabi.load().mvb_rope_kv_write_f32(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(positions), _ptr(cos_sin), cos_sin.shape[0],
+        _ptr(slot_mapping), _ptr(k_cache) if slot_mapping is not None else None,
+        _ptr(v_cache) if slot_mapping is not None else None, num_slots, tokens, q.shape[1], hkv, d, 1 if k_in_place else 0,
+        _ptr(status), _stream())
+    _cabi.check(rc, "mvb_rope_kv_write_f32")
+    LaunchCounter.add(1)
+
+
+def residual_norm(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, y_weight: torch.Tensor | None = None,
+                  row_ends: torch.Tensor | None = None) -> torch.Tensor:
+    """fp32 residual stream: ``x += y`` (or ``x += rmsnorm(y, y_weight)``) in place, returns ``rmsnorm(x, weight)`` in y's
+    dtype.  With ``row_ends`` (int32 [n + 1]) only rows ``row_ends[1:] - 1`` are produced and ``x`` is left as it is."""
+    code = _dtype_of(y, "y")
+    _need(x, torch.float32, "x"); _same(y.dtype, weight=weight, y_weight=y_weight)
+    assert x.dim() == 2 and x.is_contiguous() and y.shape == x.shape and y.stride(1) == 1
+    rows = x.shape[0]
+    if row_ends is not None:
+        _need(row_ends, torch.int32, "row_ends")
+        rows = row_ends.numel() - 1
+    out = torch.empty(rows, x.shape[1], dtype=y.dtype, device=x.device)
+    if rows == 0:
+        return out
+    rc = _cabi.load().mvb_residual_norm(code, _ptr(x), _ptr(y), y.stride(0), _ptr(y_weight), _ptr(weight), _ptr(out),
+                                        _ptr(row_ends), rows, x.shape[1], float(eps), _stream())
+    _cabi.check(rc, "mvb_residual_norm")
+    LaunchCounter.add(1)
+    return out
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float,
+               status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """(fp32 residual stream ``table[ids]``, ``rmsnorm`` of it in the table's dtype)."""
+    code = _dtype_of(table, "table")
+    _need(ids, torch.int64, "ids"); _same(table.dtype, weight=weight)
+    assert table.is_contiguous() and ids.dim() == 1 and ids.is_contiguous()
+    rows, width = ids.numel(), table.shape[1]
+    x = torch.empty(rows, width, dtype=torch.float32, device=table.device)
+    out = torch.empty(rows, width, dtype=table.dtype, device=table.device)
+    rc = _cabi.load().mvb_embed_norm(code, _ptr(ids), _ptr(table), table.shape[0], _ptr(x), _ptr(weight), _ptr(out), rows,
+                                     width, float(eps), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_embed_norm")
+    LaunchCounter.add(1)
+    return x, out
+
+
+def clamped_glu(gate_up: torch.Tensor, intermediate: int, limit: float, alpha: float) -> torch.Tensor:
+    """``g sigmoid(alpha g) (u + 1)``, ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, packed ``[gate | up]``."""
+    code = _dtype_of(gate_up, "gate_up")
+    assert gate_up.dim() == 2 and gate_up.stride(1) == 1 and gate_up.shape[1] == 2 * intermediate
+    rows = gate_up.shape[0]
+    out = torch.empty(rows, intermediate, dtype=gate_up.dtype, device=gate_up.device)
+    rc = _cabi.load().mvb_clamped_glu(code, _ptr(gate_up), gate_up.stride(0), _ptr(out), out.stride(0), rows, intermediate,
+                                      float(limit), float(alpha), _stream())
+    _cabi.check(rc, "mvb_clamped_glu")
+    LaunchCounter.add(1)
+    return out
+
+
+def cap_logits(logits: torch.Tensor, cap: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """``cap * tanh(logits / cap)`` (``cap`` 0: the logits as they are) in ``out_dtype``."""
+    code = _dtype_of(logits, "logits")
+    assert logits.dim() == 2 and logits.stride(1) == 1
+    out = torch.empty(logits.shape, dtype=out_dtype, device=logits.device)
+    rc = _cabi.load().mvb_cap_logits(code, _DTYPE[out_dtype], _ptr(logits), logits.stride(0), _ptr(out), out.stride(0),
+                                     logits.shape[0], logits.shape[1], float(cap), _stream())
+    _cabi.check(rc, "mvb_cap_logits")
+    LaunchCounter.add(1)
+    return out
+
+
+def argmax_f32(logits: torch.Tensor, scatter_table: torch.Tensor | None = None,
+               scatter_index: torch.Tensor | None = None) -> torch.Tensor:
+    """Greedy tokens of fp32 logits (the lowest column wins ties)."""
+    _need(logits, torch.float32, "logits")
+    assert logits.dim() == 2 and logits.stride(1) == 1
+    out = torch.empty(logits.shape[0], dtype=torch.int64, device=logits.device)
+    if scatter_table is not None:
+        _need(scatter_table, torch.int64, "scatter_table"); _need(scatter_index, torch.int32, "scatter_index")
+    rc = _cabi.load().mvb_argmax_f32(_ptr(logits), logits.stride(0), logits.shape[0], logits.shape[1], _ptr(out),
+                                     _ptr(scatter_table), _ptr(scatter_index), _stream())
+    _cabi.check(rc, "mvb_argmax_f32")
+    LaunchCounter.add(1)
+    return out
+
+
+def _state_args(state: torch.Tensor | None, slots: torch.Tensor | None):
+    """(state pointer, slot-index pointer, number of slots); a step without slots keeps no state."""
+    if state is None or slots is None:
+        return None, None, 0
+    _need(slots, torch.int32, "state_slots")
+    assert state.is_contiguous()
+    return _ptr(state), _ptr(slots), state.shape[0]
+
+
+def short_conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor | None,
+                    state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor,
+                    status: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal depthwise convolution + SiLU.  ``u`` [T, C] (free row stride), ``weight`` [taps, C] (row j weighs the input j
+    tokens back), ``state`` [slots, taps - 1, C]."""
+    code = _dtype_of(u, "u")
+    _same(u.dtype, weight=weight, bias=bias, state=state)
+    _need(positions, torch.int64, "positions")
+    tokens, channels = u.shape
+    taps = weight.shape[0]
+    assert u.stride(1) == 1 and weight.is_contiguous() and weight.shape[1] == channels
+    assert state is None or state.shape[1:] == (taps - 1, channels)
+    out = torch.empty(tokens, channels, dtype=u.dtype, device=u.device)
+    st, sl, n = _state_args(state, state_slots)
+    num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
+    rc = _cabi.load().mvb_short_conv_silu(code, _ptr(u), u.stride(0), _ptr(weight), _ptr(bias), _ptr(out), out.stride(0), st, sl,
+                                          n, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, channels, taps,
+                                          _ptr(status), _stream())
+    _cabi.check(rc, "mvb_short_conv_silu")
+    LaunchCounter.add(2 if cu_seqlens_q is not None and st is not None and taps > 1 else 1)
+    return out
+
+
+def selective_scan(u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, b: torch.Tensor, c: torch.Tensor,
+                   dt_bias: torch.Tensor, a_log2e: torch.Tensor, d: torch.Tensor, out: torch.Tensor,
+                   state: torch.Tensor | None, state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None,
+                   positions: torch.Tensor, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Selective scan with its gate: u, dt (raw), z, out [T, channels]; b, c [T, N] with one row stride; fp32 ``dt_bias``,
+    ``d`` [channels] and ``a_log2e`` [channels, N padded to 4]; ``state`` fp32 [slots, channels, N padded]."""
+    code = _dtype_of(u, "u")
+    _same(u.dtype, dt=dt, z=z, b=b, c=c, out=out)
+    _same(torch.float32, dt_bias=dt_bias, a_log2e=a_log2e, d=d, state=state)
+    _need(positions, torch.int64, "positions")
+    tokens, channels = u.shape
+    assert b.stride(0) == c.stride(0) or tokens <= 1
+    assert a_log2e.is_contiguous() and a_log2e.shape[0] == channels
+    st, sl, n = _state_args(state, state_slots)
+    num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
+    rc = _cabi.load().mvb_selective_scan(
+        code, _ptr(u), u.stride(0), _ptr(dt), dt.stride(0), _ptr(z), z.stride(0), _ptr(b), _ptr(c), b.stride(0),
+        _ptr(dt_bias), _ptr(a_log2e), _ptr(d), _ptr(out), out.stride(0), st, sl, n, _ptr(cu_seqlens_q), _ptr(positions),
+        num_seqs, tokens, channels, b.shape[1], a_log2e.shape[1], _ptr(status), _stream())
+    _cabi.check(rc, "mvb_selective_scan")
+    LaunchCounter.add(1)
+    return out
+
+
+def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, gate: torch.Tensor,
+                exp_a: torch.Tensor, dt_bias: torch.Tensor, norm_weight: torch.Tensor, out: torch.Tensor,
+                state: torch.Tensor | None, state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None,
+                positions: torch.Tensor, q_scale: float, eps: float, out_scale: float = 1.0,
+                status: torch.Tensor | None = None) -> torch.Tensor:
+    """Gated delta rule with its gated output norm: q, k [T, kv_heads, dim], v and out [T, heads, vdim], raw decay ``a``
+    [T, heads * dim], raw ``b`` [T, heads], raw ``gate`` [T, heads * vdim]; ``state`` fp32 [slots, heads, dim, vdim padded to 4]."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v, a=a, b=b, gate=gate, out=out)
+    _same(torch.float32, exp_a=exp_a, dt_bias=dt_bias, norm_weight=norm_weight, state=state)
+    _need(positions, torch.int64, "positions")
+    for t, name in ((q, "q"), (k, "k"), (v, "v"), (out, "out")):
+        _heads_contiguous(t, name)
+    tokens, kv_heads, dim = q.shape
+    heads, vdim = v.shape[1:]
+    assert q.stride(0) == k.stride(0) == v.stride(0) or tokens <= 1
+    st, sl, n = _state_args(state, state_slots)
+    ragged = cu_seqlens_q is not None
+    num_seqs = cu_seqlens_q.numel() - 1 if ragged else tokens
+    lib = _cabi.load()
+    scratch = torch.empty(lib.mvb_gated_delta_scratch_bytes(tokens, heads, kv_heads, dim, vdim, int(ragged)), dtype=torch.uint8,
+                          device=q.device)
+    rc = lib.mvb_gated_delta(
+        code, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(a), a.stride(0), _ptr(b), b.stride(0), _ptr(gate), gate.stride(0),
+        _ptr(exp_a), _ptr(dt_bias), _ptr(norm_weight), _ptr(out), out.stride(0), st, sl, n, _ptr(cu_seqlens_q),
+        _ptr(positions), num_seqs, tokens, heads, kv_heads, dim, vdim, float(q_scale), float(eps), float(out_scale),
+        _ptr(scratch), scratch.numel(), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_gated_delta")
+    LaunchCounter.add(3 if ragged else (2 if vdim > 128 else 1))
     return out
