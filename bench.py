@@ -594,6 +594,151 @@ def config2_parity() -> dict:
             "unscreened_identical_of_64": int(z["unscreened_identical"])}
 
 
+# ---- Fupupel: prefill and decode beside the closest existing model, and the kernels of its own ----------------
+FUPUPEL_SIZES = {      # width, heads / KV heads (128 wide), feed-forward, layers (half of them selective scans)
+    "w1024": (1024, 16, 8, 3072, 12), "w2048": (2048, 16, 8, 6144, 12), "w4096": (4096, 32, 8, 12288, 8)}
+
+
+def fupupel_bench_shape(size: str, window: int = 1024):
+    from mini_vllm_b200.config import fupupel_shape
+    width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
+    scan = {"type": "mamba1", "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}, "mlp": None}
+    both = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff, "limit": 7.0},
+            "mixer": {"left": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "mask": {"size": window},
+                               "rot": {"base": 1e6, "dims": 128}, "scale": 128 ** -0.5, "softcap": 30.0},
+                      "right": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128,
+                                "gate_rank": 128}, "left_scale": 0.5, "right_scale": 0.5}}
+    return fupupel_shape([scan if i % 2 == 0 else both for i in range(layers)], width, 32768)
+
+
+def fupupel_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
+    """Prefill (8 prompts of 2048 tokens) and decode (32 and 256 sequences) through ``Engine.generate`` with random weights,
+    beside Qwen3 layers of the same width, heads, feed-forward and count."""
+    from mini_vllm_b200.engine.engine import Engine
+    out = {}
+    for size in sizes:
+        width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
+        twin = qwen3_shape(num_hidden_layers=layers, hidden_size=width, intermediate_size=ff, num_attention_heads=heads,
+                           num_key_value_heads=kv, vocab_size=32768)
+        for name, hf in (("fupupel", fupupel_bench_shape(size)), ("qwen3", twin)):
+            eng = Engine(Config(hf_config=hf, kv_cache_num_blocks=1024, max_num_batched_seqs=256, max_graph_batch_size=256,
+                                max_num_batched_tokens=16384, gpu_memory_utilization=0.85, seed=0))
+            params = sum(p.numel() for p in eng.executor.model.parameters())
+            job = lambda n, length, new: (eng.generate([[(7 * i + j) % 32768 for j in range(length)] for i in range(n)],
+                                                       SamplingParams(max_tokens=new, ignore_eos=True), use_tqdm=False),
+                                          eng.last_job_device_ms)[1]
+            med = lambda *a: statistics.median(job(*a) for _ in range(3))
+            job(8, 2048, 1)
+            row = {"parameters": params, "prefill_tok_s": round(8 * 2048 / med(8, 2048, 1) * 1e3)}
+            for n in (32, 256):
+                job(n, 512, 2)
+                row[f"decode{n}_step_ms"] = round((med(n, 512, 65) - med(n, 512, 1)) / 64, 4)
+                row[f"decode{n}_tok_s"] = round(n / row[f"decode{n}_step_ms"] * 1e3)
+            out[f"{size}_{name}"] = row
+            del eng
+            torch.cuda.empty_cache()
+    return out
+
+
+def fupupel_kernel_legs(dev, peaks) -> dict:
+    """Each kernel of the design against its roofline, next to the like kernel of the existing models where there is one.
+    16 heads of 128 (8 KV heads), width 2048, scan of 4096 channels x 16 states, 8192 prefill tokens, 256 decode rows."""
+    from mini_vllm_b200 import ops
+    out, bf = {}, torch.bfloat16
+    sms, ghz = torch.cuda.get_device_properties(dev).multi_processor_count, 1.9
+    rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
+
+    def leg(name, call, nbuf, byts=None, flops=None, mufu=None, fp32=None):
+        ms = graph_time_ms(lambda: [call(i) for i in range(nbuf)], nbuf)
+        row = {"us": round(ms * 1e3, 2)}
+        if byts:
+            row.update({"GB/s": round(byts / ms / 1e6, 1), "frac_of_measured_hbm": round(byts / ms / 1e6 / peaks["hbm_gbs"], 4)})
+        if flops:
+            row.update({"TFLOP/s": round(flops / ms / 1e9, 1), "frac_of_measured_bf16": round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)})
+        if mufu:
+            row["frac_of_special_function_rate"] = round(mufu / (sms * 16 * ghz * 1e9) / (ms * 1e-3), 4)
+        if fp32:
+            row["frac_of_fp32_fma_rate"] = round(fp32 / (sms * 128 * ghz * 1e9) / (ms * 1e-3), 4)
+        out[name] = row
+
+    heads, kv, d, width, ff, window = 16, 8, 128, 2048, 6144, 1024
+    for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
+        tokens = sum(lens)
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        pos = torch.cat([torch.arange(n, device=dev) for n in lens])
+        q, k, v = rnd(tokens, heads, d), rnd(tokens, kv, d), rnd(tokens, kv, d)
+        pairs = sum(sum(min(i + 1, window) for i in range(n)) for n in lens)
+        for name, cap in (("prefill_attn_window1024", 0.0), ("prefill_attn_window1024_capped", 30.0)):
+            leg(f"{name}_{tag}", lambda i: ops.prefill_attn(q, k, v, cu, cu, max(lens), d ** -0.5, window - 1, softcap=cap), 4,
+                flops=4 * heads * d * pairs)
+        full = sum(n * (n + 1) // 2 for n in lens)
+        for name, cap in (("prefill_attn_full", 0.0), ("prefill_attn_full_capped", 30.0)):
+            leg(f"{name}_{tag}", lambda i: ops.prefill_attn(q, k, v, cu, cu, max(lens), d ** -0.5, -1, softcap=cap), 4,
+                flops=4 * heads * d * full)
+        inner, n = 4096, 16
+        state = torch.zeros(len(lens), inner, n, device=dev)
+        slots = torch.arange(len(lens), dtype=torch.int32, device=dev)
+        u, dt, z, y = (rnd(tokens, inner) for _ in range(4))
+        bc = rnd(tokens, 2 * n)
+        a = -torch.arange(1, n + 1, device=dev).float().expand(inner, n).contiguous() * 1.44
+        bias, skip = torch.full((inner,), -4.0, device=dev), torch.ones(inner, device=dev)
+        leg(f"selective_scan_{tag}", lambda i: ops.selective_scan(u, dt, z, bc[:, :n], bc[:, n:], bias, a, skip, y, state, slots,
+                                                                  cu, pos), 2,
+            byts=tokens * (inner * 4 + 2 * n) * 2, mufu=tokens * inner * n)
+        w4, cstate = rnd(4, inner), torch.zeros(len(lens), 3, inner, device=dev, dtype=bf)
+        leg(f"short_conv_{tag}", lambda i: ops.short_conv_silu(u, w4, None, cstate, slots, cu, pos), 4, byts=tokens * inner * 4)
+        qd, kd, vd, gate, od = (rnd(tokens, heads, d) for _ in range(5))
+        raw_a, raw_b = rnd(tokens, heads * d), rnd(tokens, heads)
+        ea, db, nw = torch.rand(heads, device=dev) * 8 + 1, torch.full((heads * d,), -4.0, device=dev), torch.ones(d, device=dev)
+        dstate = torch.zeros(len(lens), heads, d, d, device=dev)
+        leg(f"gated_delta_{tag}", lambda i: ops.gated_delta(qd, kd, vd, raw_a, raw_b, gate.flatten(1), ea, db, nw, od, dstate,
+                                                            slots, cu, pos, d ** -0.5, 1e-6), 1,
+            byts=tokens * heads * d * 6 * 2, fp32=tokens * heads * d * d * 4)
+    tokens = 8192
+    gu = [rnd(tokens, 2 * ff) for _ in range(2)]
+    leg("act_mul_8192", lambda i: ops.act_mul(gu[i], ff, False), 2, byts=tokens * ff * 6)
+    leg("clamped_glu_8192", lambda i: ops.clamped_glu(gu[i], ff, 7.0, 1.702), 2, byts=tokens * ff * 6)
+    del gu
+    w, ys = torch.ones(width, device=dev, dtype=bf), [rnd(tokens, width) for _ in range(4)]
+    xs16, xs32 = [rnd(tokens, width) for _ in range(4)], [torch.randn(tokens, width, device=dev) for _ in range(4)]
+    leg("add_rmsnorm_branch_norm_8192", lambda i: ops.add_rmsnorm(xs16[i], ys[i], w, 1e-6, True, y_weight=w), 4, byts=tokens * width * 8)
+    leg("residual_norm_f32_8192", lambda i: ops.residual_norm(xs32[i], ys[i], w, 1e-6, y_weight=w), 4, byts=tokens * width * 12)
+    # decode: 256 sequences, contexts of 1024 and more (a window layer reads 1024 keys of each)
+    b, blocks = 256, 256 * 5
+    pools = [torch.randn(2, blocks, 256, kv, d, device=dev, dtype=bf) for _ in range(2)]
+    lens = torch.full((b,), 1200, dtype=torch.int32, device=dev)
+    bt = torch.arange(blocks, dtype=torch.int32, device=dev).view(b, 5)
+    q, o = rnd(b, heads, d), rnd(b, heads, d)
+    ws = ops.decode_workspace(b, heads, d, dev)
+    ops.decode_plan(lens, window - 1, heads, kv, d, ws, block_table=bt, block_size=256)
+    for name, cap in (("decode_attn_window1024", 0.0), ("decode_attn_window1024_capped", 30.0)):
+        leg(f"{name}_256", lambda i: ops.decode_attn(q, pools[i][0], pools[i][1], lens, bt, d ** -0.5, window - 1, ws, out=o,
+                                                     softcap=cap), 2, byts=b * window * 2 * kv * d * 2)
+    del pools
+    pos, slots = torch.full((b,), 1199, device=dev), torch.arange(b, dtype=torch.int32, device=dev)
+    inner, n = 4096, 16
+    states = [torch.randn(b, inner, n, device=dev) for _ in range(4)]
+    u, dt, z, y, bc = rnd(b, inner), rnd(b, inner), rnd(b, inner), rnd(b, inner), rnd(b, 2 * n)
+    a = -torch.arange(1, n + 1, device=dev).float().expand(inner, n).contiguous() * 1.44
+    bias, skip = torch.full((inner,), -4.0, device=dev), torch.ones(inner, device=dev)
+    leg("selective_scan_decode256", lambda i: ops.selective_scan(u, dt, z, bc[:, :n], bc[:, n:], bias, a, skip, y, states[i], slots,
+                                                                 None, pos), 4, byts=b * inner * n * 8)
+    del states
+    dstates = [torch.randn(b, heads, d, d, device=dev) * 0.01 for _ in range(2)]
+    qd, kd, vd, gate, od = (rnd(b, heads, d) for _ in range(5))
+    raw_a, raw_b = rnd(b, heads * d), rnd(b, heads)
+    ea, db, nw = torch.rand(heads, device=dev) * 8 + 1, torch.full((heads * d,), -4.0, device=dev), torch.ones(d, device=dev)
+    leg("gated_delta_decode256", lambda i: ops.gated_delta(qd, kd, vd, raw_a, raw_b, gate.flatten(1), ea, db, nw, od, dstates[i],
+                                                           slots, None, pos, d ** -0.5, 1e-6), 2, byts=b * heads * d * d * 8)
+    w4, cstate, uc = rnd(4, 6144), torch.zeros(b, 3, 6144, device=dev, dtype=bf), rnd(b, 6144)
+    leg("short_conv_decode256", lambda i: ops.short_conv_silu(uc, w4, None, cstate, slots, None, pos), 4, byts=b * 6144 * 2 * 8)
+    x32, y16, w = torch.randn(b, width, device=dev), rnd(b, width), torch.ones(width, device=dev, dtype=bf)
+    x16 = rnd(b, width)
+    leg("add_rmsnorm_branch_norm_256", lambda i: ops.add_rmsnorm(x16, y16, w, 1e-6, True, y_weight=w), 8, byts=b * width * 8)
+    leg("residual_norm_f32_256", lambda i: ops.residual_norm(x32, y16, w, 1e-6, y_weight=w), 8, byts=b * width * 12)
+    return out
+
+
 # ---- CPU leg: the oracle restatement of the reference path on the host cores ------------------------
 class CpuReference:
     """The oracle model (restatement of the reference's PyTorch path, pinned to the reference's own engine loop by
@@ -707,6 +852,9 @@ def main():
                          "config-2 model (64 screened prompts)")
     ap.add_argument("--config4-step", action="store_true",
                     help="engine-level config 4: a decode step of 128 sequences on Gemma3-1B shapes")
+    ap.add_argument("--fupupel", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
+                    help="the Fupupel design with random weights: prefill and decode throughput beside Qwen3 layers of equal "
+                         "size, and its kernels against their rooflines beside the like kernels")
     ap.add_argument("--engine-steps", type=int, default=0,
                     help="profiling aid: prefill + N decode steps of the workload without CUDA graphs, then exit")
     args = ap.parse_args()
@@ -727,6 +875,15 @@ def main():
     if args.config4_step:
         torch.cuda.set_device(0)
         print(json.dumps({"config4_engine_step": config4_engine_step()}))
+        return
+    if args.fupupel:
+        torch.cuda.set_device(0)
+        line = {}
+        if args.fupupel in ("all", "kernels"):
+            line["kernels"] = fupupel_kernel_legs(torch.device("cuda", 0), measured_peaks()[0])
+        if args.fupupel in ("all", "engine"):
+            line["engine"] = fupupel_throughput()
+        print(json.dumps({"fupupel": line}))
         return
     if args.kernel_legs:
         peaks, _ = measured_peaks()
