@@ -1,0 +1,267 @@
+"""Fupupel through the engine's own step, cache and scheduler: whole prompts, portions, mixed batches, reused memory and greedy
+generation, against the plain oracle on small models with weights of the tests' making."""
+import random
+from functools import lru_cache
+
+import pytest
+import torch
+
+from mini_vllm_b200.config import Config, SamplingParams
+from oracle.fupupel import OracleFupupel
+from tests.fupupel_helpers import CONFIGS, both_layer, config, row_errors, scan_layer, tensors, write_checkpoint
+
+pytestmark = pytest.mark.gpu
+BF, F32 = torch.bfloat16, torch.float32
+# bf16: a branch output near zero is blown up by the norm behind it, so single positions of these tiny models stray far above the
+# mean; fp32 is the sharp comparison
+TOL = {BF: 0.25, F32: 1e-4}
+MEAN_TOL = {BF: 0.03, F32: 2e-5}
+LENS = [1, 2, 3, 23, 130, 257, 310]
+
+
+@lru_cache(maxsize=None)
+def reference(name):
+    """(config, tensors, prompts, logits of every position in float64)"""
+    cfg, rnd = CONFIGS[name], random.Random(name)
+    w = tensors(cfg, seed=len(name))
+    prompts = [[rnd.randrange(cfg["vocab"]) for _ in range(n)] for n in LENS]
+    model = OracleFupupel(w, cfg)
+    return cfg, w, prompts, [model.forward(p) for p in prompts]
+
+
+def make_engine(path, dtype, blocks=12, slots=4, seqs=4, **extra):
+    from mini_vllm_b200.engine.engine import Engine
+    return Engine(Config(model=path, dtype=dtype, kv_cache_num_blocks=blocks, kv_cache_block_size=128, max_model_len=1024,
+                         max_num_batched_seqs=seqs, num_state_slots=slots, gpu_memory_utilization=0.5, **extra))
+
+
+@pytest.fixture(scope="module", params=[(n, d) for n in CONFIGS for d in (BF, F32)], ids=lambda p: f"{p[0]}-{str(p[1])[6:]}")
+def served(request, cuda, tmp_path_factory):
+    name, dtype = request.param
+    ref = reference(name)
+    eng = make_engine(write_checkpoint(tmp_path_factory.mktemp("m") / name, ref[0], ref[1]), dtype)
+    yield eng, dtype, ref
+    del eng
+    torch.cuda.empty_cache()
+
+
+def feed(eng, prompts, plan):
+    """Runs a plan - steps of (prompt index, number of tokens) - and returns each prompt's logits; a prompt fed to its end
+    gives its memory back at once."""
+    from mini_vllm_b200.engine.request import Request
+    live, at, got = {}, {}, {}
+    for step in plan:
+        entries = []
+        for i, n in step:
+            lo = at.get(i, 0)
+            at[i] = lo + n
+            entries.append((live.setdefault(i, Request([])), prompts[i][lo:lo + n], list(range(n))))
+        out, row = eng.replay_step(entries).cpu(), 0
+        for i, n in step:
+            got.setdefault(i, []).append(out[row:row + n])
+            row += n
+            if at[i] == len(prompts[i]):
+                eng.release(live.pop(i))
+                at.pop(i)
+    eng.executor.check_device_status()
+    bm = eng.scheduler.block_manager
+    if not live:                                                     # everything was given back
+        assert bm.num_free_blocks == bm.capacity and bm.state_slots.num_free == bm.state_slots.capacity
+    return {i: torch.cat(v) for i, v in got.items()}
+
+
+def portions(n, sizes):
+    out = []
+    while sum(out) < n:
+        out.append(min(sizes[len(out) % len(sizes)], n - sum(out)))
+    return out
+
+
+def check(got, want, dtype):
+    errs = {i: row_errors(g, want[i][:g.shape[0]]) for i, g in got.items()}
+    for i, e in errs.items():
+        assert e.max() < TOL[dtype], (i, int(e.argmax()), float(e.max()))
+    assert torch.cat(list(errs.values())).mean() < MEAN_TOL[dtype]
+
+
+def test_whole_prompts_alone(served):
+    eng, dtype, (_, _, prompts, want) = served
+    check(feed(eng, prompts, [[(i, len(p))] for i, p in enumerate(prompts)]), want, dtype)
+
+
+def test_token_by_token(served):
+    eng, dtype, (_, _, prompts, want) = served
+    check(feed(eng, prompts, [[(i, 1)] for i in (0, 2, 3, 5) for _ in prompts[i]]), want, dtype)
+
+
+@pytest.mark.parametrize("sizes", [[2], [100, 69, 2, 3, 1], [128], [127, 2, 1, 1, 130]])
+def test_portions(served, sizes):
+    eng, dtype, (_, _, prompts, want) = served
+    picked = [5] if sizes == [2] else [4, 6]
+    check(feed(eng, prompts, [[(i, n)] for i in picked for n in portions(len(prompts[i]), sizes)]), want, dtype)
+
+
+def test_mixed_batches_with_reused_blocks_and_slots(served):
+    """Unequal requests in one batch, portions beside single tokens, requests that pause, end, and leave their blocks and slot
+    to the next; the pool holds four requests at a time."""
+    eng, dtype, (_, _, prompts, want) = served
+    rnd, todo, live, plan = random.Random(3), [6, 0, 4, 5, 2, 3, 1], {}, []
+    while todo or live:
+        while todo and len(live) < 4:
+            i = todo.pop(0)
+            live[i] = len(prompts[i])
+        step = []
+        for i in sorted(live, key=lambda _: rnd.random()):
+            if rnd.random() < 0.25 and len(live) > 1:
+                continue                                             # left out of this step
+            n = min(live[i], rnd.choice([1, 1, 1, 2, 3, 16, 64, 128]))
+            step.append((i, n))
+            live[i] -= n
+        live = {i: n for i, n in live.items() if n}
+        if step:
+            plan.append(step)
+    got = feed(eng, prompts, plan)
+    check(got, want, dtype)
+    alone = feed(eng, prompts, [[(i, len(prompts[i]))] for i in (4, 6)])     # the same positions however they were cut
+    for i in (4, 6):
+        assert row_errors(got[i], alone[i].double()).max() < TOL[dtype]
+
+
+@pytest.mark.parametrize("window", [1, 2, 64, 127, 128, 129])
+@pytest.mark.parametrize("dtype", [BF, F32])
+def test_a_key_at_the_window_edge(cuda, tmp_path, window, dtype):
+    """Token 7's key is made to win every softmax (its embedding points along the query direction), so whether it is just inside or
+    just outside the window decides the logits - in a prompt, in portions and in decoding."""
+    cfg = config([both_layer(window=window, softcap=30.0, rot=2, ff=None, rs=0.05)], width=64, vocab=40)
+    w = tensors(cfg, seed=9)
+    g = torch.Generator().manual_seed(1)
+    u = torch.randn(64, generator=g)
+    u = u / u.norm()
+    for n, heads in (("q", 4), ("k", 2)):
+        t = torch.zeros(heads, 32, 64)
+        t[:, 20] = u * (8.0 if n == "k" else 0.0)
+        if n == "q":
+            t[:, 20] = torch.ones(64) * 0.3
+        w[f"l0.mix.left.{n}"] = t.view(heads * 32, 64).to(torch.bfloat16)
+    w["embed"] = (torch.rand(40, 64, generator=g) * 0.5 + 0.5 + (torch.arange(40) == 7)[:, None] * 6 * u).to(torch.bfloat16)
+    rnd = random.Random(2)
+    prompt = [rnd.randrange(8, 40) for _ in range(140 + window)]
+    prompt[130] = 7                                                  # seen up to position 130 + window - 1
+    want = OracleFupupel(w, cfg).forward(prompt)
+    moved = OracleFupupel(w, {**cfg, "layers": [both_layer(window=window + 1, softcap=30.0, rot=2, ff=None, rs=0.05)]}).forward(prompt)
+    assert row_errors(moved[130 + window:131 + window], want[130 + window:131 + window]).max() > 0.2, "the edge does not show"
+    eng = make_engine(write_checkpoint(tmp_path / "m", cfg, w), dtype)
+    for plan in ([[(0, len(prompt))]], [[(0, 129)]] + [[(0, 1)]] * (len(prompt) - 129), [[(0, n)] for n in portions(len(prompt), [50, 2])]):
+        check(feed(eng, [prompt], plan), [want], dtype)
+
+
+def test_long_decoding_from_graphs(cuda, tmp_path):
+    """Hundreds of decoded tokens: far beyond every window, over block borders, with a slow decay that remembers the start."""
+    cfg = config([scan_layer(inner=24, state=4), both_layer(window=9)], vocab=60)
+    w = tensors(cfg, seed=4)
+    w["l0.mix.dt.b"] = torch.full((24,), -7.0, dtype=torch.bfloat16)
+    rnd = random.Random(7)
+    prompt = [rnd.randrange(60) for _ in range(520)]
+    want = OracleFupupel(w, cfg).forward(prompt)
+    for dtype in (BF, F32):
+        eng = make_engine(write_checkpoint(tmp_path / "m", cfg, w), dtype)
+        check(feed(eng, [prompt], [[(0, 3)]] + [[(0, 1)]] * 517), [want], dtype)
+        del eng
+
+
+def test_residual_stream_of_every_layer(cuda, tmp_path):
+    cfg, w, prompts, _ = reference("grouped")
+    streams, taps = [], []
+    OracleFupupel(w, cfg).forward(prompts[4], streams)
+    eng = make_engine(write_checkpoint(tmp_path / "m", cfg, w), F32)
+    eng.executor.model.residual_tap = lambda i, x: taps.append(x.clone())
+    feed(eng, prompts, [[(4, len(prompts[4]))]])
+    assert len(taps) == len(streams) and all((t.double().cpu() - s).abs().max() < 1e-4 for t, s in zip(taps, streams))
+
+
+# ---- greedy generation through Engine.generate and the scheduler -----------------------------------------------
+def greedy_case(n, seed, lens, new):
+    cfg = config([scan_layer(inner=32, state=6), both_layer(window=12), both_layer(window=40, heads=2, kv_heads=1)], vocab=70)
+    w = tensors(cfg, seed=seed)
+    rnd = random.Random(seed)
+    prompts = [[rnd.randrange(70) for _ in range(rnd.choice(lens))] for _ in range(n)]
+    model = OracleFupupel(w, cfg)
+    return cfg, w, prompts, [model.greedy(p, new) for p in prompts]
+
+
+def assert_tokens(got, want, margin):
+    """Equal until the oracle's own two best logits come closer than rounding can keep apart."""
+    compared = 0
+    for toks, (ref, margins) in zip(got, want):
+        for t, r, m in zip(toks, ref, margins):
+            if m < margin:
+                break
+            assert t == r
+            compared += 1
+    return compared
+
+
+@pytest.mark.parametrize("dtype,margin", [(F32, 1e-3), (BF, 0.5)])
+@pytest.mark.parametrize("extra", [{}, {"enable_mixed_steps": True}, {"enable_chunked_prefill": True, "max_num_batched_tokens": 48},
+                                   {"enable_chunked_prefill": True, "enable_mixed_steps": True, "max_num_batched_tokens": 33},
+                                   {"use_cuda_graph": False, "fused_greedy_head": False}], ids=["plain", "mixed", "chunked", "chunked-mixed", "eager"])
+@pytest.mark.parametrize("pipelined", [True, False])
+def test_greedy_generation(cuda, tmp_path, dtype, margin, extra, pipelined):
+    cfg, w, prompts, want = greedy_case(7, 11, [1, 5, 30, 75], 12)
+    eng = make_engine(write_checkpoint(tmp_path / "m", cfg, w), dtype, blocks=4, slots=3, **extra)     # three live at a time at most
+    out = eng.generate(prompts, SamplingParams(max_tokens=12, ignore_eos=True), use_tqdm=not pipelined)
+    assert all(len(o["tokens"]) == 12 for o in out)
+    compared = assert_tokens([o["tokens"] for o in out], want, margin)
+    assert compared >= (80 if dtype == F32 else 4)
+    bm = eng.scheduler.block_manager
+    assert bm.num_free_blocks == bm.capacity and bm.state_slots.num_free == 3
+
+
+def test_preempted_requests_start_over_from_zero_state(cuda, tmp_path):
+    """Two blocks for three requests that each grow into a second: somebody is preempted, loses slot and blocks, and is computed
+    again from its first token."""
+    cfg, w, prompts, want = greedy_case(3, 13, [120, 126], 12)
+    eng = make_engine(write_checkpoint(tmp_path / "m", cfg, w), F32, blocks=4, slots=3)
+    preempted, preempt = [], eng.scheduler.preempt
+    eng.scheduler.preempt = lambda r: (preempted.append(r.id), preempt(r))[1]
+    out = eng.generate(prompts, SamplingParams(max_tokens=12, ignore_eos=True), use_tqdm=False)
+    assert preempted and assert_tokens([o["tokens"] for o in out], want, 1e-3) > 20
+
+
+def test_sampling_and_random_init(cuda):
+    from mini_vllm_b200.config import fupupel_shape
+    from mini_vllm_b200.engine.engine import Engine
+    from tests.fupupel_helpers import both_layer as both, scan_layer as scan
+    hf = fupupel_shape([scan(), both()], 64, 96)
+    eng = Engine(Config(hf_config=hf, kv_cache_num_blocks=8, max_num_batched_seqs=4, seed=3))
+    out = eng.generate([[1, 2, 3], [4]], SamplingParams(max_tokens=6, ignore_eos=True, temperature=0.8, top_k=20, top_p=0.9), use_tqdm=False)
+    assert all(len(o["tokens"]) == 6 and all(0 <= t < 96 for t in o["tokens"]) for o in out)
+
+
+def test_prefix_cache_is_refused(cuda):
+    from mini_vllm_b200.config import fupupel_shape
+    from mini_vllm_b200.engine.engine import Engine
+    with pytest.raises(ValueError, match="state"):
+        Engine(Config(hf_config=fupupel_shape([scan_layer()], 64, 96), enable_prefix_cache=True))
+
+
+def test_trace_program(cuda, tmp_path):
+    """bin/trace_run end to end: acknowledgements, files only where something is wanted, exit code."""
+    import json
+    import subprocess
+    from pathlib import Path
+
+    import numpy as np
+    cfg, w, prompts, want = reference("grouped")
+    path = write_checkpoint(tmp_path / "m", cfg, w)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": prompts[4][:50], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": prompts[2], "want": [2]}, {"id": "a", "tokens": prompts[4][50:], "want": [0, 79]}],
+              "end": ["a", "b"]}]
+    r = subprocess.run([str(Path(__file__).resolve().parent.parent / "bin" / "trace_run"), "--model", path, "--dtype", "float32", "--out",
+                        str(tmp_path), "--max-tokens", "256"], input="\n".join(map(json.dumps, steps)) + "\n", capture_output=True, text=True,
+                       timeout=300)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1"]
+    assert not (tmp_path / "0.f32").exists()
+    got = torch.from_numpy(np.fromfile(tmp_path / "1.f32", dtype="<f4").reshape(3, -1))
+    assert row_errors(got, torch.stack([want[2][2], want[4][50], want[4][129]])).max() < 1e-4
