@@ -67,6 +67,19 @@ __device__ __forceinline__ void store_f32(float* p, const float (&v)[V]) {
 
 // z >= -inf: log(1 + e^z) without overflow; 1 / (1 + e^-z)
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// The same for bf16 activations, where a few fp32 ulps do not matter but instructions do: with y = e^-|z| in (0, 1] and
+// w = y / (2 + y), log(1 + y) = 2 artanh(w) = 2 w (1 + w^2/3 + w^4/5 + ...), w <= 1/3, so eight terms reach fp32.
+__device__ __forceinline__ float softplus_fast(float z) {
+  const float y = fast_exp2(-1.4426950408889634f * fabsf(z)), w = y * fast_rcp(2.f + y), q = w * w;
+  float t = 1.f / 15.f;
+  t = fmaf(t, q, 1.f / 13.f); t = fmaf(t, q, 1.f / 11.f); t = fmaf(t, q, 1.f / 9.f); t = fmaf(t, q, 1.f / 7.f);
+  t = fmaf(t, q, 1.f / 5.f); t = fmaf(t, q, 1.f / 3.f); t = fmaf(t, q, 1.f);
+  return fmaf(2.f * w, t, fmaxf(z, 0.f));
+}
+template <class T> __device__ __forceinline__ float softplus_of(float z) {
+  if constexpr (sizeof(T) == 2) return softplus_fast(z);
+  else return softplus_f(z);
+}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 
 // the sequence of packed row t: the largest s with cu[s] <= t (cu ascending, cu[0] = 0, t < cu[n]); rows of a step

@@ -167,8 +167,9 @@ struct PrefillItem {
 
 // LIST: the work comes as a list of (sequence, query block) pairs (PrefillParams::items) instead of a 3-D grid; a
 // kernel of its own, so that the grid form carries none of the list's code.
-// CAP: scores pass c tanh(s / c) before the softmax.
-template <int D, int BN, int NQ, bool LIST, bool CAP>
+// CAP: scores pass c tanh(s / c) before the softmax.  1: c is small enough that c itself serves as the maximum of every row
+// (2^(score - c) stays a normal number), so a tile takes a single pass and O is never rescaled; 2: any c, online maximum.
+template <int D, int BN, int NQ, bool LIST, int CAP>
 __global__ void __launch_bounds__(PrefillCfg<D, BN, NQ>::THREADS, 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                     const __grid_constant__ CUtensorMap v_map, const PrefillParams p) {
@@ -539,10 +540,23 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
     const uint32_t lane_addr = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const uint32_t s_base = lane_addr + C::S_COL + t * C::S_BUFS * BN;
     const uint32_t o_addr = lane_addr + C::O_COL + t * D;
-    // c tanh(x / c) in log2 units as c - 2 c / (1 + 2^(2 x / c ...)): absolute error of a few fp32 ulps of c
-    auto cap_score = [&](uint32_t s_bits) -> uint32_t {
-      const float e = fast_exp2(__uint_as_float(s_bits) * p.cap_in);
-      return __float_as_uint(fmaf(-2.f * p.cap_log2, fast_rcp(1.f + e), p.cap_log2));
+    // c tanh(x / c) = c - 2 c / (1 + 2^y), y = 2 x log2(e) / c, to a few fp32 ulps of c.  Four reciprocals come from one (of
+    // the product), which spares the special-function unit three; y is cut at 29, where tanh has rounded to 1.
+    auto cap_terms = [&](uint32_t (&s)[32]) {                 // s -> 1 / (1 + 2^y)
+#pragma unroll
+      for (int i = 0; i < 32; i += 4) {
+        float a[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a[k] = 1.f + fast_exp2(fminf(__uint_as_float(s[i + k]) * p.cap_in, 29.f));
+        const float ab = a[0] * a[1], cd = a[2] * a[3], r = fast_rcp(ab * cd), iab = r * cd, icd = r * ab;
+        s[i] = __float_as_uint(iab * a[1]); s[i + 1] = __float_as_uint(iab * a[0]);
+        s[i + 2] = __float_as_uint(icd * a[3]); s[i + 3] = __float_as_uint(icd * a[2]);
+      }
+    };
+    auto cap_scores = [&](uint32_t (&s)[32]) {                // s -> capped score in log2 units (CAP 2)
+      cap_terms(s);
+#pragma unroll
+      for (int i = 0; i < 32; ++i) s[i] = __float_as_uint(fmaf(-2.f * p.cap_log2, __uint_as_float(s[i]), p.cap_log2));
     };
     uint32_t n_s = 0, n_epi = 0;                              // S tiles consumed (S / P parity), epilogues done (O parity)
     bool ok = true;
@@ -635,11 +649,24 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
 #pragma unroll
           for (int c = 0; c < NCH; ++c) tmem_ld_32x32(s_addr + c * 32, sreg[c]);
           tmem_wait_ld();
-          if constexpr (CAP) {
+          if constexpr (CAP == 1) {
 #pragma unroll
-            for (int c = 0; c < NCH; ++c)
+            for (int c = 0; c < NCH; ++c) {
+              uint32_t pk[16];
+              cap_terms(sreg[c]);
 #pragma unroll
-              for (int i = 0; i < 32; ++i) sreg[c][i] = cap_score(sreg[c][i]);
+              for (int i = 0; i < 32; i += 2) {
+                const float e0 = fast_exp2(__uint_as_float(sreg[c][i]) * (-2.f * p.cap_log2));
+                const float e1 = fast_exp2(__uint_as_float(sreg[c][i + 1]) * (-2.f * p.cap_log2));
+                sum0 += e0; sum1 += e1;
+                pk[i >> 1] = pack_bf16(e0, e1);
+              }
+              publish_p(c, pk);
+            }
+          } else {
+          if constexpr (CAP == 2) {
+#pragma unroll
+            for (int c = 0; c < NCH; ++c) cap_scores(sreg[c]);
           }
           float max0 = -INFINITY, max1 = -INFINITY;
 #pragma unroll
@@ -663,9 +690,11 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             }
             publish_p(c, pk);
           }
+          }
         } else {
           // chunks every row of the warp sees completely run the plain code here too
           float tile_max = -INFINITY;
+          if constexpr (CAP != 1) {
 #pragma unroll 1
           for (int c = 0; c < NCH; ++c) {
             const int cl = chunk_class(c * 32);
@@ -673,10 +702,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             uint32_t r[32];
             tmem_ld_32x32(s_addr + c * 32, r);
             tmem_wait_ld();
-            if constexpr (CAP) {
-#pragma unroll
-              for (int i = 0; i < 32; ++i) r[i] = cap_score(r[i]);
-            }
+            if constexpr (CAP == 2) cap_scores(r);
             if (cl == 0) {
               float max0 = -INFINITY, max1 = -INFINITY;
 #pragma unroll
@@ -693,6 +719,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             }
           }
           new_max(tile_max);
+          }
           const float m_safe = m_use == -INFINITY ? 0.f : m_use;
 #pragma unroll 1
           for (int c = 0; c < NCH; ++c) {
@@ -705,20 +732,20 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
               uint32_t r[32];
               tmem_ld_32x32(s_addr + c * 32, r);
               tmem_wait_ld();
-              if constexpr (CAP) {
-#pragma unroll
-                for (int i = 0; i < 32; ++i) r[i] = cap_score(r[i]);
-              }
+              if constexpr (CAP == 1) cap_terms(r);
+              if constexpr (CAP == 2) cap_scores(r);
               if (cl == 1) {
                 const uint32_t bits = visible_bits(c * 32);
 #pragma unroll
                 for (int i = 0; i < 32; ++i)
-                  if (!((bits >> i) & 1u)) r[i] = 0xff800000u;  // -inf
+                  if (!((bits >> i) & 1u)) r[i] = CAP == 1 ? 0x7f800000u : 0xff800000u;  // CAP 1 multiplies by a negative factor
               }
 #pragma unroll
               for (int i = 0; i < 32; i += 2) {
-                const float e0 = fast_exp2(fmaf(__uint_as_float(r[i]), p.scale_log2, -m_safe));
-                const float e1 = fast_exp2(fmaf(__uint_as_float(r[i + 1]), p.scale_log2, -m_safe));
+                const float e0 = CAP == 1 ? fast_exp2(__uint_as_float(r[i]) * (-2.f * p.cap_log2))
+                                          : fast_exp2(fmaf(__uint_as_float(r[i]), p.scale_log2, -m_safe));
+                const float e1 = CAP == 1 ? fast_exp2(__uint_as_float(r[i + 1]) * (-2.f * p.cap_log2))
+                                          : fast_exp2(fmaf(__uint_as_float(r[i + 1]), p.scale_log2, -m_safe));
                 sum0 += e0; sum1 += e1;
                 pk[i >> 1] = pack_bf16(e0, e1);
               }
@@ -790,7 +817,7 @@ struct PrefillOperands {            // what the tensor maps are built from
   int total_q, hq, hkv;
 };
 
-template <int D, int BN, int NQ, bool LIST, bool CAP>
+template <int D, int BN, int NQ, bool LIST, int CAP>
 static int launch_prefill(const PrefillOperands& op, const PrefillParams& p, int max_seqlen_q, cudaStream_t stream) {
   using C = PrefillCfg<D, BN, NQ>;
   if (p.block_table != nullptr && p.block_size % BN != 0) return kUnsupportedShape;   // a KV tile must not straddle blocks
@@ -802,7 +829,7 @@ static int launch_prefill(const PrefillOperands& op, const PrefillParams& p, int
   if (rc != kOk) return rc;
   rc = make_kv_tensor_map(&vm, op.v, op.kv_rows, op.hkv, D, op.v_stride, BN);
   if (rc != kOk) return rc;
-  using KernelTag = std::integral_constant<int, D * 16 + NQ * 4 + (LIST ? 2 : 0) + (CAP ? 1 : 0)>;   // one opt-in record per kernel
+  using KernelTag = std::integral_constant<int, D * 32 + NQ * 8 + (LIST ? 4 : 0) + CAP>;   // one opt-in record per kernel
   rc = opt_in_dynamic_smem<KernelTag>(reinterpret_cast<const void*>(&prefill_attn_kernel<D, BN, NQ, LIST, CAP>), C::SMEM);
   if (rc != kOk) return rc;
   PrefillParams pp = p;
@@ -877,14 +904,15 @@ static int prefill_attn_impl(const void* q, int64_t q_row_stride, const void* k,
     list = static_cast<int64_t>(num_items) * 100 < grid_items * 85;
   }
   auto launch = [&](auto cap_tag) {
-    constexpr bool CAP = decltype(cap_tag)::value;
+    constexpr int CAP = decltype(cap_tag)::value;
     if (head_dim == 128)
       return list ? launch_prefill<128, 128, 2, true, CAP>(op, p, max_seqlen_q, st)
                   : launch_prefill<128, 128, 2, false, CAP>(op, p, max_seqlen_q, st);
     return list ? launch_prefill<256, 64, 1, true, CAP>(op, p, max_seqlen_q, st)
                 : launch_prefill<256, 64, 1, false, CAP>(op, p, max_seqlen_q, st);
   };
-  return cap ? launch(std::true_type{}) : launch(std::false_type{});
+  if (!cap) return launch(std::integral_constant<int, 0>{});
+  return p.cap_log2 <= 50.f ? launch(std::integral_constant<int, 1>{}) : launch(std::integral_constant<int, 2>{});
 }
 
 extern "C" int mvb_prefill_attn(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride,

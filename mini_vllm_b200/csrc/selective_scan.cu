@@ -34,6 +34,7 @@ struct ScanParams {
   const int32_t* slots; int64_t num_slots;
   const int32_t* cu; const int64_t* positions;
   int num_seqs, tokens, channels, n, np;
+  bool bc_vec;                             // four consecutive elements of b or c may be read as one vector
   int* dev_status;
 };
 
@@ -51,6 +52,23 @@ template <class T>
 __device__ __forceinline__ float advance(float S, float x, float in) {
   if constexpr (sizeof(T) == 4) return fmaf(S, expm1f(x * 0.6931471805599453f), S) + in;
   else return fmaf(fast_exp2(x), S, in);
+}
+
+// four values at p[0..n), zeros past n; vec: p is aligned for one vector access
+template <class T>
+__device__ __forceinline__ void load4(const T* p, int n, bool vec, float (&v)[4]) {
+  if (vec && n >= 4) {
+    if constexpr (sizeof(T) == 2) {
+      const uint2 w = *reinterpret_cast<const uint2*>(p);
+      v[0] = bf16_lo(w.x); v[1] = bf16_hi(w.x); v[2] = bf16_lo(w.y); v[3] = bf16_hi(w.y);
+    } else {
+      const float4 w = *reinterpret_cast<const float4*>(p);
+      v[0] = w.x; v[1] = w.y; v[2] = w.z; v[3] = w.w;
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = j < n ? to_f(p[j]) : 0.f;
+  }
 }
 
 template <class T, int L, int R>
@@ -111,7 +129,7 @@ __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
     for (int k = 0; k < EPT; ++k) {
       const int tl = etok + k * ESTEP;
       cu_[k] = to_f(ru[k]); cz[k] = to_f(rz[k]);
-      const float dt = softplus_f(to_f(rdt[k]) + bias);
+      const float dt = t0 + tl < n_tok ? softplus_of<T>(to_f(rdt[k]) + bias) : 0.f;   // (a token past the end changes nothing)
       if (TT * CH < 128 && tl >= TT) continue;
       dt_s[tl][ech] = dt;
       du_s[tl][ech] = dt * cu_[k];
@@ -124,22 +142,36 @@ __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
     __syncthreads();
     if (t0 + TT < n_tok) request(t0 + TT);
     const int nt = min(TT, n_tok - t0);
-#pragma unroll 4
-    for (int tl = 0; tl < nt; ++tl) {
-      const float dt = dt_s[tl][chl], du = du_s[tl][chl];
-      float acc = 0.f;
+    // four tokens at a time: all operands and exponentials first, so that only the multiply-adds of S are a chain
+    for (int tb = 0; tb < nt; tb += 4) {
+      float dt[4], du[4], acc[4];
+#pragma unroll
+      for (int m = 0; m < 4; ++m) { dt[m] = dt_s[tb + m][chl]; du[m] = du_s[tb + m][chl]; acc[m] = 0.f; }
 #pragma unroll
       for (int r = 0; r < R; ++r) {
-        const float4 bv = *reinterpret_cast<const float4*>(&b_s[tl][(sub + L * r) * 4]);
-        const float4 cv = *reinterpret_cast<const float4*>(&c_s[tl][(sub + L * r) * 4]);
-        S[r][0] = advance<T>(S[r][0], dt * a[r][0], du * bv.x); acc = fmaf(S[r][0], cv.x, acc);
-        S[r][1] = advance<T>(S[r][1], dt * a[r][1], du * bv.y); acc = fmaf(S[r][1], cv.y, acc);
-        S[r][2] = advance<T>(S[r][2], dt * a[r][2], du * bv.z); acc = fmaf(S[r][2], cv.z, acc);
-        S[r][3] = advance<T>(S[r][3], dt * a[r][3], du * bv.w); acc = fmaf(S[r][3], cv.w, acc);
+        const int n0 = (sub + L * r) * 4;
+        float4 bv[4], cv[4];
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          bv[m] = *reinterpret_cast<const float4*>(&b_s[tb + m][n0]);
+          cv[m] = *reinterpret_cast<const float4*>(&c_s[tb + m][n0]);
+        }
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          S[r][0] = advance<T>(S[r][0], dt[m] * a[r][0], du[m] * bv[m].x); acc[m] = fmaf(S[r][0], cv[m].x, acc[m]);
+          S[r][1] = advance<T>(S[r][1], dt[m] * a[r][1], du[m] * bv[m].y); acc[m] = fmaf(S[r][1], cv[m].y, acc[m]);
+          S[r][2] = advance<T>(S[r][2], dt[m] * a[r][2], du[m] * bv[m].z); acc[m] = fmaf(S[r][2], cv[m].z, acc[m]);
+          S[r][3] = advance<T>(S[r][3], dt[m] * a[r][3], du[m] * bv[m].w); acc[m] = fmaf(S[r][3], cv[m].w, acc[m]);
+        }
       }
 #pragma unroll
-      for (int off = 1; off < L; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
-      if (sub == 0) y_s[tl][chl] = acc;
+      for (int off = 1; off < L; off <<= 1)
+#pragma unroll
+        for (int m = 0; m < 4; ++m) acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], off);
+      if (sub == 0) {
+#pragma unroll
+        for (int m = 0; m < 4; ++m) y_s[tb + m][chl] = acc[m];
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -167,26 +199,30 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanParams p) {
   const bool fresh = slot < 0 || p.positions[s] == 0, ok = c < p.channels;
   float acc = 0.f, u = 0.f;
   if (ok) {
+    float4 sv[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) {                            // what the kernel waits for goes out first
+      const int n0 = (sub + L * r) * 4;
+      sv[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!fresh && n0 < p.np) sv[r] = *reinterpret_cast<const float4*>(p.state + (slot * p.channels + c) * p.np + n0);
+    }
     u = to_f(static_cast<const T*>(p.u)[s * p.u_stride + c]);
-    const float dt = softplus_f(to_f(static_cast<const T*>(p.dt)[s * p.dt_stride + c]) + p.dt_bias[c]), du = dt * u;
+    const float dt = softplus_of<T>(to_f(static_cast<const T*>(p.dt)[s * p.dt_stride + c]) + p.dt_bias[c]), du = dt * u;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int n0 = (sub + L * r) * 4;
       if (n0 >= p.np) continue;
-      float* st = p.state + (slot * p.channels + c) * p.np + n0;
       const float4 av = *reinterpret_cast<const float4*>(p.a_log2e + static_cast<int64_t>(c) * p.np + n0);
-      const float4 sv = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
       const float a[4] = {av.x, av.y, av.z, av.w};
-      float S[4] = {sv.x, sv.y, sv.z, sv.w};
+      float S[4] = {sv[r].x, sv[r].y, sv[r].z, sv[r].w}, bn[4], cn[4];
+      load4(static_cast<const T*>(p.b) + s * p.bc_stride + n0, p.n - n0, p.bc_vec, bn);
+      load4(static_cast<const T*>(p.c) + s * p.bc_stride + n0, p.n - n0, p.bc_vec, cn);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const bool in = n0 + j < p.n;
-        const float bn = in ? to_f(static_cast<const T*>(p.b)[s * p.bc_stride + n0 + j]) : 0.f;
-        const float cn = in ? to_f(static_cast<const T*>(p.c)[s * p.bc_stride + n0 + j]) : 0.f;
-        S[j] = advance<T>(S[j], dt * a[j], du * bn);
-        acc = fmaf(S[j], cn, acc);
+        S[j] = advance<T>(S[j], dt * a[j], du * bn[j]);
+        acc = fmaf(S[j], cn[j], acc);
       }
-      if (slot >= 0) *reinterpret_cast<float4*>(st) = make_float4(S[0], S[1], S[2], S[3]);
+      if (slot >= 0) *reinterpret_cast<float4*>(p.state + (slot * p.channels + c) * p.np + n0) = make_float4(S[0], S[1], S[2], S[3]);
     }
   }
 #pragma unroll
@@ -240,7 +276,9 @@ extern "C" int mvb_selective_scan(int dtype, const void* u, int64_t u_row_stride
   if (num_tokens == 0 || num_seqs == 0) return kOk;
   const ScanParams p{u, u_row_stride, dt, dt_row_stride, z, z_row_stride, b, c, bc_row_stride, dt_bias, a_log2e, d, out,
                      out_row_stride, state, state_slots, num_slots, cu_seqlens_q, positions, num_seqs, num_tokens, channels,
-                     num_states, state_stride, dev_status};
+                     num_states, state_stride,
+                     bc_row_stride % 4 == 0 && is_aligned(b, 16 / (dtype == kBf16 ? 2 : 1)) && is_aligned(c, 16 / (dtype == kBf16 ? 2 : 1)),
+                     dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_scan<__nv_bfloat16>(p, st) : launch_scan<float>(p, st);
 }

@@ -30,7 +30,7 @@ struct ConvParams {
   int* dev_status;
 };
 
-constexpr int kConvRun = 32;     // tokens a thread walks
+constexpr int kConvRun = 16;     // tokens a thread walks
 
 __device__ __forceinline__ int64_t conv_slot(const ConvParams& p, int s) {
   if (p.state == nullptr) return -1;
@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvParams p) {
   int s = seq_of_row(p.cu, p.num_seqs, t_begin);
   int begin = p.cu == nullptr ? t_begin : p.cu[s], end = p.cu == nullptr ? t_begin + 1 : p.cu[s + 1];
   bool fill = true;
-  for (int t = t_begin; t < t_end; ++t) {
+  for (int t = t_begin; t < t_end;) {
     while (t >= end) {                                       // (a sequence may bring no token)
       ++s; begin = end; end = p.cu[s + 1]; fill = true;
     }
@@ -81,29 +81,41 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvParams p) {
           load_vec<T, V>(static_cast<const T*>(p.state) + (slot * (taps - 1) + (taps - 1 - (j - (t - begin)))) * C + c, hist[j]);
       }
     }
-    load_vec<T, V>(u + t * p.u_stride, hist[0]);
-    float acc[V];
+    // the rest of this run inside the sequence, four tokens at a time so that four loads are in flight
+    const int stop = min(t_end, end);
+    for (; t < stop; t += 4) {
+      float in[4][V];
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = bias[i];
+      for (int m = 0; m < 4; ++m)
+        if (t + m < stop) load_vec<T, V>(u + (t + m) * p.u_stride, in[m]);
 #pragma unroll
-    for (int j = TAPS - 1; j >= 0; --j)
+      for (int m = 0; m < 4; ++m) {
+        if (t + m >= stop) break;
+        float acc[V];
 #pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], hist[j][i], acc[i]);
+        for (int i = 0; i < V; ++i) { hist[0][i] = in[m][i]; acc[i] = bias[i]; }
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = acc[i] * fast_rcp(1.f + fast_exp2(acc[i] * -1.4426950408889634f));
-    store_vec<T, V>(out + t * p.out_stride, acc);
-    if (p.cu == nullptr) {                                   // the slot's rows are this thread's alone
-      const int64_t slot = conv_slot(p, s);
-      if (slot >= 0) {
+        for (int j = TAPS - 1; j >= 0; --j)
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j)
-          if (j < taps - 1) store_vec<T, V>(static_cast<T*>(p.state) + (slot * (taps - 1) + (taps - 2 - j)) * C + c, hist[j]);
+          for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], hist[j][i], acc[i]);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = acc[i] * fast_rcp(1.f + fast_exp2(acc[i] * -1.4426950408889634f));
+        store_vec<T, V>(out + (t + m) * p.out_stride, acc);
+        if (p.cu == nullptr) {                               // the slot's rows are this thread's alone
+          const int64_t slot = conv_slot(p, s);
+          if (slot >= 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+              if (j < taps - 1) store_vec<T, V>(static_cast<T*>(p.state) + (slot * (taps - 1) + (taps - 2 - j)) * C + c, hist[j]);
+          }
+        }
+#pragma unroll
+        for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+          for (int i = 0; i < V; ++i) hist[j][i] = hist[j - 1][i];
       }
     }
-#pragma unroll
-    for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-      for (int i = 0; i < V; ++i) hist[j][i] = hist[j - 1][i];
+    t = stop;
   }
 }
 
