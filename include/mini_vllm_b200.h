@@ -397,7 +397,8 @@ int mvb_selective_scan(int dtype, const void* u, int64_t u_row_stride, const voi
                        const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions,
                        int num_seqs, int num_tokens, int channels, int num_states, int state_stride, int32_t* dev_status,
                        void* stream);
-size_t mvb_gated_delta_scratch_bytes(int num_tokens, int heads, int kv_heads, int dim, int vdim, int ragged);
+size_t mvb_gated_delta_scratch_bytes(int dtype, int num_tokens, int num_seqs, int heads, int kv_heads, int dim, int vdim,
+                                     int ragged);
 int mvb_gated_delta(int dtype, const void* q, const void* k, const void* v, int64_t qkv_row_stride, const void* a,
                     int64_t a_row_stride, const void* b, int64_t b_row_stride, const void* gate, int64_t gate_row_stride,
                     const float* exp_a, const float* dt_bias, const float* norm_weight, void* out, int64_t out_row_stride,

@@ -56,7 +56,7 @@ SIGNATURES = {
     "mvb_short_conv_silu": (i32, [i32, vp, i64, vp, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, vp, vp]),
     "mvb_selective_scan": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp,
                                  vp, i32, i32, i32, i32, i32, vp, vp]),
-    "mvb_gated_delta_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32]),
+    "mvb_gated_delta_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32, i32, i32]),
     "mvb_gated_delta": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp,
                               vp, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, sz, vp, vp]),
 }

@@ -10,9 +10,11 @@
 // One token per sequence (delta_step_kernel): a CTA per (sequence, head, tile of at most 128 columns); a thread holds RPT
 // rows x 4 columns of S in registers, so the state is read once and written once (the roofline: HBM, 8 * dim * vdim bytes per
 // head and sequence); gates, norms and, when one tile covers the head, the gated output norm are in the same kernel.
-// Ragged step: delta_prep_kernel writes q, k, g as fp32 [tokens, heads, dp] once per token; delta_tokens_kernel walks a
-// sequence's tokens with S in registers (8 row groups x 4 columns per warp, the sum over rows is three shuffles), operands staged
-// TT tokens ahead with cp.async; gated_norm_kernel finishes the rows.
+// Ragged step, bf16 activations: chunks of 16 tokens on the tensor cores (delta_chunks.cuh).
+// Ragged step, fp32 activations: plain fp32 throughout.  delta_prep_kernel writes q, k, g as [tokens, heads, dp] once per token;
+// delta_tokens_kernel walks a sequence's tokens with S in registers (8 row groups x 4 columns per warp, the sum over rows is
+// three shuffles), operands staged TT tokens ahead with cp.async.
+// gated_norm_kernel finishes the rows of either.
 #include "dtype.cuh"
 #include "host_util.cuh"
 #include "mini_vllm_b200.h"
@@ -292,18 +294,40 @@ __global__ void __launch_bounds__(128) delta_tokens_kernel(const DeltaParams p) 
 
 // out[t, h, :] = o / rms(o) * w * sigmoid(gate) * factor; one warp per (token, head)
 template <class T>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(256) gated_norm_kernel(const DeltaParams p, bool vec) {
   const int64_t w = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31, t = static_cast<int>(w / p.heads), h = static_cast<int>(w % p.heads);
   if (t >= p.tokens) return;
   const float* o = p.o + w * p.vdim;
+  const T* gate = static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<int64_t>(h) * p.vdim;
+  T* out = static_cast<T*>(p.out) + t * p.out_stride + static_cast<int64_t>(h) * p.vdim;
+  auto sig = [](float z) { return sizeof(T) == 2 ? fast_rcp(1.f + fast_exp2(z * -1.4426950408889634f)) : sigmoid_f(z); };
+  if (sizeof(T) == 2 && vec && p.vdim <= 128) {               // a lane keeps its four columns
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    uint2 gw = make_uint2(0u, 0u);
+    const int i = lane * 4;
+    if (i < p.vdim) { x = *reinterpret_cast<const float4*>(o + i); gw = *reinterpret_cast<const uint2*>(gate + i); }
+    const float r = p.out_scale * rsqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) / static_cast<float>(p.vdim) + p.eps);
+    if (i < p.vdim) {
+      const float4 nw = *reinterpret_cast<const float4*>(p.norm_w + i);
+      uint2 y;
+      y.x = pack_bf16(x.x * r * nw.x * sig(bf16_lo(gw.x)), x.y * r * nw.y * sig(bf16_hi(gw.x)));
+      y.y = pack_bf16(x.z * r * nw.z * sig(bf16_lo(gw.y)), x.w * r * nw.w * sig(bf16_hi(gw.y)));
+      *reinterpret_cast<uint2*>(out + i) = y;
+    }
+    return;
+  }
   float ss = 0.f;
   for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
   const float r = p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.vdim) + p.eps);
-  const T* gate = static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<int64_t>(h) * p.vdim;
-  T* out = static_cast<T*>(p.out) + t * p.out_stride + static_cast<int64_t>(h) * p.vdim;
-  for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * r * p.norm_w[i] * sigmoid_f(to_f(gate[i])));
+  for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * r * p.norm_w[i] * sig(to_f(gate[i])));
 }
+
+}  // namespace mvb
+
+#include "delta_chunks.cuh"
+
+namespace mvb {
 
 static int delta_row_pad(int dim) { return (dim + 31) / 32 * 32; }
 
@@ -311,7 +335,9 @@ template <class T>
 static int launch_gated_norm(const DeltaParams& p, cudaStream_t st) {
   const int64_t blocks = (static_cast<int64_t>(p.tokens) * p.heads * 32 + 255) / 256;
   if (blocks > 0x7fffffffLL) return kUnsupportedShape;
-  gated_norm_kernel<T><<<static_cast<unsigned>(blocks), 256, 0, st>>>(p);
+  const bool vec = p.vdim % 4 == 0 && p.gate_stride % 4 == 0 && p.out_stride % 4 == 0 && is_aligned(p.gate, 8) &&
+                   is_aligned(p.out, 8) && is_aligned(p.norm_w, 16) && is_aligned(p.o, 16);
+  gated_norm_kernel<T><<<static_cast<unsigned>(blocks), 256, 0, st>>>(p, vec);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
@@ -357,6 +383,22 @@ template <class T>
 static int launch_delta(const DeltaParams& p, cudaStream_t st) {
   if (p.cu == nullptr) return launch_step<T>(p, st);
   if (p.heads > 65535 || p.num_seqs > 65535) return kUnsupportedShape;
+  if constexpr (sizeof(T) == 2) {
+    uint8_t* records = reinterpret_cast<uint8_t*>(p.qn);
+    int rc = kUnsupportedShape;
+    switch (chunk_ks(p.dim)) {
+      case 1: rc = launch_delta_chunks<T, 1>(p, records, st); break;
+      case 2: rc = launch_delta_chunks<T, 2>(p, records, st); break;
+      case 3: rc = launch_delta_chunks<T, 3>(p, records, st); break;
+      case 4: rc = launch_delta_chunks<T, 4>(p, records, st); break;
+      case 6: rc = launch_delta_chunks<T, 6>(p, records, st); break;
+      case 8: rc = launch_delta_chunks<T, 8>(p, records, st); break;
+      case 12: rc = launch_delta_chunks<T, 12>(p, records, st); break;
+      case 16: rc = launch_delta_chunks<T, 16>(p, records, st); break;
+      default: break;
+    }
+    return rc == kOk ? launch_gated_norm<T>(p, st) : rc;
+  } else {
   delta_prep_kernel<T><<<p.tokens, 256, 0, st>>>(p);
   if (cudaGetLastError() != cudaSuccess) return kLaunchFailed;
   int rc = kUnsupportedShape;
@@ -373,19 +415,28 @@ static int launch_delta(const DeltaParams& p, cudaStream_t st) {
   }
   if (rc != kOk) return rc;
   return launch_gated_norm<T>(p, st);
+  }
 }
 
 static size_t up64(size_t n) { return (n + 63) / 64 * 64; }
 
 }  // namespace mvb
 
-extern "C" size_t mvb_gated_delta_scratch_bytes(int num_tokens, int heads, int kv_heads, int dim, int vdim, int ragged) {
+// floats in front of o in the scratch of a ragged step: the chunk records, or q, k, g and beta
+static size_t delta_operand_floats(int dtype, size_t t, size_t num_seqs, int heads, int kv_heads, int dim, int vdim) {
   using namespace mvb;
-  if (num_tokens <= 0 || heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0) return 0;
+  if (dtype == kBf16) return up64((t / kChunk + num_seqs) * heads * (chunk_layout(chunk_ks(dim), vdim).total / 4));
+  const size_t dp = delta_row_pad(dim);
+  return 2 * up64(t * kv_heads * dp) + up64(t * heads * dp) + up64(t * heads);
+}
+
+extern "C" size_t mvb_gated_delta_scratch_bytes(int dtype, int num_tokens, int num_seqs, int heads, int kv_heads, int dim, int vdim,
+                                                int ragged) {
+  using namespace mvb;
+  if (num_tokens <= 0 || num_seqs <= 0 || heads <= 0 || kv_heads <= 0 || dim <= 0 || dim > 256 || vdim <= 0) return 0;
   const size_t t = num_tokens, o = up64(t * heads * vdim);
   if (!ragged) return (vdim + 3) / 4 * 4 > 128 ? o * sizeof(float) : 64;
-  const size_t dp = delta_row_pad(dim);
-  return (2 * up64(t * kv_heads * dp) + up64(t * heads * dp) + up64(t * heads) + o) * sizeof(float);
+  return (delta_operand_floats(dtype, t, num_seqs, heads, kv_heads, dim, vdim) + o) * sizeof(float);
 }
 
 extern "C" int mvb_gated_delta(int dtype, const void* q, const void* k, const void* v, int64_t qkv_row_stride, const void* a,
@@ -404,7 +455,7 @@ extern "C" int mvb_gated_delta(int dtype, const void* q, const void* k, const vo
   if (!is_aligned(state, 16) || !is_aligned(scratch, 16)) return kMisaligned;
   if (dim > 256) return kUnsupportedShape;
   if (num_tokens == 0 || num_seqs == 0) return kOk;
-  if (!scratch || scratch_bytes < mvb_gated_delta_scratch_bytes(num_tokens, heads, kv_heads, dim, vdim, cu_seqlens_q != nullptr))
+  if (!scratch || scratch_bytes < mvb_gated_delta_scratch_bytes(dtype, num_tokens, num_seqs, heads, kv_heads, dim, vdim, cu_seqlens_q != nullptr))
     return kInvalidArgument;
   DeltaParams p;
   p.q = q; p.k = k; p.v = v; p.qkv_stride = qkv_row_stride;
@@ -421,7 +472,10 @@ extern "C" int mvb_gated_delta(int dtype, const void* q, const void* k, const vo
   float* f = static_cast<float*>(scratch);
   const size_t t = num_tokens;
   p.qn = p.kn = p.gn = p.beta = nullptr;
-  if (cu_seqlens_q != nullptr) {
+  if (cu_seqlens_q != nullptr && dtype == kBf16) {
+    p.qn = f;                                                  // (the records)
+    f += delta_operand_floats(dtype, t, num_seqs, heads, kv_heads, dim, vdim);
+  } else if (cu_seqlens_q != nullptr) {
     p.qn = f; f += up64(t * kv_heads * p.dp);
     p.kn = f; f += up64(t * kv_heads * p.dp);
     p.gn = f; f += up64(t * heads * p.dp);

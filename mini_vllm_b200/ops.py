@@ -653,7 +653,7 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tens
     ragged = cu_seqlens_q is not None
     num_seqs = cu_seqlens_q.numel() - 1 if ragged else tokens
     lib = _cabi.load()
-    scratch = torch.empty(lib.mvb_gated_delta_scratch_bytes(tokens, heads, kv_heads, dim, vdim, int(ragged)), dtype=torch.uint8,
+    scratch = torch.empty(lib.mvb_gated_delta_scratch_bytes(code, tokens, num_seqs, heads, kv_heads, dim, vdim, int(ragged)), dtype=torch.uint8,
                           device=q.device)
     rc = lib.mvb_gated_delta(
         code, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(a), a.stride(0), _ptr(b), b.stride(0), _ptr(gate), gate.stride(0),
