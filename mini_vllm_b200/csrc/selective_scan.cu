@@ -71,11 +71,30 @@ __device__ __forceinline__ void load4(const T* p, int n, bool vec, float (&v)[4]
   }
 }
 
-template <class T, int L, int R>
+// E neighbouring elements as they lie in memory
+template <class T, int E> struct Raw { T v[E]; };
+template <class T, int E> __device__ __forceinline__ Raw<T, E> load_raw(const T* p, bool ok) {
+  Raw<T, E> r;
+  if constexpr (E == 1) {
+    r.v[0] = ok ? *p : from_f<T>(0.f);
+  } else if constexpr (sizeof(T) == 2) {
+    const uint32_t w = ok ? *reinterpret_cast<const uint32_t*>(p) : 0u;
+    *reinterpret_cast<uint32_t*>(r.v) = w;
+  } else {
+    const float2 w = ok ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
+    r.v[0] = w.x; r.v[1] = w.y;
+  }
+  return r;
+}
+
+// E: channels per thread in the elementwise part (2 where the operands are aligned for it)
+template <class T, int L, int R, int E>
 __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
   constexpr int CHW = 32 / L, CH = 4 * CHW, NP = 4 * L * R, TT = L <= 8 ? 32 : 16;
-  constexpr int EPT = TT * CH >= 128 ? TT * CH / 128 : 1, BPT = TT * 2 * NP / 128;
-  __shared__ float dt_s[TT][CH], du_s[TT][CH], y_s[TT][CH];
+  constexpr int ECH = CH / E, EPT = TT * ECH >= 128 ? TT * ECH / 128 : 1, BPT = TT * 2 * NP / 128;
+  __shared__ __align__(8) float dt_s[TT][CH];
+  __shared__ __align__(8) float du_s[TT][CH];
+  __shared__ __align__(8) float y_s[TT][CH];
   __shared__ __align__(16) float b_s[TT][NP];
   __shared__ __align__(16) float c_s[TT][NP];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, sub = lane % L;
@@ -98,23 +117,33 @@ __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
     S[r][0] = sv.x; S[r][1] = sv.y; S[r][2] = sv.z; S[r][3] = sv.w;
   }
 
-  // element e of a tile: token e / CH, channel e % CH; a thread keeps the same channel throughout
-  static_assert(128 % CH == 0 || CH == 128, "");
-  const int ech = tid % CH, etok = tid / CH;
-  constexpr int ESTEP = 128 / CH;
+  // a thread keeps its E channels throughout and takes every ESTEP-th token of a tile
+  constexpr int ESTEP = 128 / ECH;
+  const int ech = tid % ECH * E, etok = tid / ECH;
   const bool ech_ok = c0 + ech < p.channels;
-  const float bias = ech_ok ? p.dt_bias[c0 + ech] : 0.f, dskip = ech_ok ? p.d[c0 + ech] : 0.f;
-  T ru[EPT], rdt[EPT], rz[EPT], rbc[BPT];
+  float bias[E], dskip[E];
+#pragma unroll
+  for (int j = 0; j < E; ++j) {
+    bias[j] = ech_ok ? p.dt_bias[c0 + ech + j] : 0.f;
+    dskip[j] = ech_ok ? p.d[c0 + ech + j] : 0.f;
+  }
+  const int64_t first = begin + etok;
+  const T* pu = static_cast<const T*>(p.u) + first * p.u_stride + c0 + ech;
+  const T* pd = static_cast<const T*>(p.dt) + first * p.dt_stride + c0 + ech;
+  const T* pz = static_cast<const T*>(p.z) + first * p.z_stride + c0 + ech;
+  T* po = static_cast<T*>(p.out) + first * p.out_stride + c0 + ech;
+  Raw<T, E> ru[EPT], rdt[EPT], rz[EPT];
+  T rbc[BPT];
   auto request = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < EPT; ++k) {
-      const int tl = etok + k * ESTEP, t = t0 + tl;
-      const bool ok = ech_ok && tl < TT && t < n_tok;
-      const int64_t row = begin + t;
-      ru[k] = ok ? static_cast<const T*>(p.u)[row * p.u_stride + c0 + ech] : from_f<T>(0.f);
-      rdt[k] = ok ? static_cast<const T*>(p.dt)[row * p.dt_stride + c0 + ech] : from_f<T>(0.f);
-      rz[k] = ok ? static_cast<const T*>(p.z)[row * p.z_stride + c0 + ech] : from_f<T>(0.f);
+      const int tl = etok + k * ESTEP;
+      const bool ok = ech_ok && tl < TT && t0 + tl < n_tok;
+      ru[k] = load_raw<T, E>(pu + k * ESTEP * p.u_stride, ok);
+      rdt[k] = load_raw<T, E>(pd + k * ESTEP * p.dt_stride, ok);
+      rz[k] = load_raw<T, E>(pz + k * ESTEP * p.z_stride, ok);
     }
+    pu += TT * p.u_stride; pd += TT * p.dt_stride; pz += TT * p.z_stride;
 #pragma unroll
     for (int k = 0; k < BPT; ++k) {
       const int e = tid + k * 128, t = t0 + e / (2 * NP), j = e % (2 * NP), nn = j % NP;
@@ -124,15 +153,26 @@ __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
   };
   request(0);
   for (int t0 = 0; t0 < n_tok; t0 += TT) {
-    float cu_[EPT], cz[EPT];
+    Raw<T, E> cu_[EPT], cz[EPT];
 #pragma unroll
     for (int k = 0; k < EPT; ++k) {
       const int tl = etok + k * ESTEP;
-      cu_[k] = to_f(ru[k]); cz[k] = to_f(rz[k]);
-      const float dt = t0 + tl < n_tok ? softplus_of<T>(to_f(rdt[k]) + bias) : 0.f;   // (a token past the end changes nothing)
-      if (TT * CH < 128 && tl >= TT) continue;
-      dt_s[tl][ech] = dt;
-      du_s[tl][ech] = dt * cu_[k];
+      cu_[k] = ru[k]; cz[k] = rz[k];
+      if (TT * ECH < 128 && tl >= TT) continue;
+      const bool in = t0 + tl < n_tok;                       // (a token past the end changes nothing)
+      float dt[E], du[E];
+#pragma unroll
+      for (int j = 0; j < E; ++j) {
+        dt[j] = in ? softplus_of<T>(to_f(rdt[k].v[j]) + bias[j]) : 0.f;
+        du[j] = dt[j] * to_f(ru[k].v[j]);
+      }
+      if constexpr (E == 2) {
+        *reinterpret_cast<float2*>(&dt_s[tl][ech]) = make_float2(dt[0], dt[1]);
+        *reinterpret_cast<float2*>(&du_s[tl][ech]) = make_float2(du[0], du[1]);
+      } else {
+        dt_s[tl][ech] = dt[0];
+        du_s[tl][ech] = du[0];
+      }
     }
 #pragma unroll
     for (int k = 0; k < BPT; ++k) {
@@ -177,10 +217,16 @@ __global__ void __launch_bounds__(128) scan_tokens_kernel(const ScanParams p) {
 #pragma unroll
     for (int k = 0; k < EPT; ++k) {
       const int tl = etok + k * ESTEP;
-      if (ech_ok && tl < nt)
-        static_cast<T*>(p.out)[(begin + t0 + tl) * p.out_stride + c0 + ech] =
-            from_f<T>(fmaf(dskip, cu_[k], y_s[tl][ech]) * silu_f(cz[k]));
+      if (!ech_ok || tl >= nt) continue;
+      float y[E];
+#pragma unroll
+      for (int j = 0; j < E; ++j) y[j] = fmaf(dskip[j], to_f(cu_[k].v[j]), y_s[tl][ech + j]) * silu_f(to_f(cz[k].v[j]));
+      T* dst = po + k * ESTEP * p.out_stride;
+      if constexpr (E == 1) *dst = from_f<T>(y[0]);
+      else if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16(y[0], y[1]);
+      else *reinterpret_cast<float2*>(dst) = make_float2(y[0], y[1]);
     }
+    po += TT * p.out_stride;
   }
   if (slot >= 0 && c < p.channels) {
 #pragma unroll
@@ -243,7 +289,11 @@ static int launch_scan_lr(const ScanParams& p, cudaStream_t st) {
     constexpr int CH = 4 * (32 / L);
     const int gy = (p.channels + CH - 1) / CH;
     if (gy > 65535) return kUnsupportedShape;
-    scan_tokens_kernel<T, L, R><<<dim3(p.num_seqs, gy), 128, 0, st>>>(p);
+    constexpr uintptr_t A = 2 * sizeof(T);
+    const bool pairs = p.channels % 2 == 0 && p.u_stride % 2 == 0 && p.dt_stride % 2 == 0 && p.z_stride % 2 == 0 && p.out_stride % 2 == 0 &&
+                       is_aligned(p.u, A) && is_aligned(p.dt, A) && is_aligned(p.z, A) && is_aligned(p.out, A);
+    if (pairs) scan_tokens_kernel<T, L, R, 2><<<dim3(p.num_seqs, gy), 128, 0, st>>>(p);
+    else scan_tokens_kernel<T, L, R, 1><<<dim3(p.num_seqs, gy), 128, 0, st>>>(p);
   }
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }

@@ -265,3 +265,15 @@ def test_trace_program(cuda, tmp_path):
     assert not (tmp_path / "0.f32").exists()
     got = torch.from_numpy(np.fromfile(tmp_path / "1.f32", dtype="<f4").reshape(3, -1))
     assert row_errors(got, torch.stack([want[2][2], want[4][50], want[4][129]])).max() < 1e-4
+
+
+def test_command_line_generation(cuda, tmp_path, capsys):
+    import json
+
+    from mini_vllm_b200.__main__ import main
+    cfg, w, prompts, want = greedy_case(2, 17, [5, 9], 6)
+    path = write_checkpoint(tmp_path / "m", cfg, w)
+    args = ["--model", path, "--dtype", "float32", "--max-tokens", "6", "--ignore-eos", "--max-model-len", "256", "--chunked-prefill"]
+    assert main(args + [x for p in prompts for x in ("--prompt", " ".join(map(str, p)))]) == 0
+    out = [json.loads(x)["tokens"] for x in capsys.readouterr().out.splitlines() if x.startswith("{")]
+    assert assert_tokens(out, want, 1e-3) > 4
