@@ -51,7 +51,7 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
   float* q_s = sm;                               // [16][ROW]
   float* k_s = q_s + kChunk * ROW;
   float* g_s = k_s + kChunk * ROW;               // log2 of the decay, then its running sum
-  uint32_t* rec_s = reinterpret_cast<uint32_t*>(g_s + kChunk * ROW);   // W, Q, K operand words
+  float* u_s = g_s + kChunk * ROW;               // [columns of U][17]
   __shared__ float am[kChunk][kChunk + 1], bm[kChunk][kChunk + 1], beta_s[kChunk];
   __shared__ __align__(16) float tm[kChunk][kChunk];
   const int slot = blockIdx.x, h = blockIdx.y, kvh = h / (p.heads / p.kv_heads);
@@ -70,6 +70,18 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
   // a warp takes every fourth token; the raw operands of U tokens are requested before any is worked on
   constexpr int U = NI <= 4 ? 4 : 2;
   const float ea = -p.exp_a[h] * 1.4426950408889634f;
+  float bias[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) bias[i] = i * 32 + lane < p.dim ? p.dt_bias[h * p.dim + i * 32 + lane] : 0.f;
+  const float raw_b = tid < nt ? to_f(static_cast<const T*>(p.b)[(begin + t0 + tid) * p.b_stride + h]) : 0.f;
+  for (int v = tid; v < lay.vtp * 16; v += 128) {              // v waits in the columns that U will take
+    T vv[kChunk];
+#pragma unroll
+    for (int s = 0; s < kChunk; ++s)
+      vv[s] = v < p.vdim && s < nt ? static_cast<const T*>(p.v)[(begin + t0 + s) * p.qkv_stride + h * p.vdim + v] : from_f<T>(0.f);
+#pragma unroll
+    for (int s = 0; s < kChunk; ++s) u_s[v * 17 + s] = to_f(vv[s]);
+  }
 #pragma unroll 1
   for (int tb = warp; tb < kChunk; tb += 4 * U) {
     T rq[U][NI], rk[U][NI], ra[U][NI];
@@ -97,7 +109,7 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
       for (int i = 0; i < NI; ++i) {
         const int d = i * 32 + lane;
         const bool in = t < nt && d < p.dim;
-        g_s[t * ROW + d] = in ? ea * softplus_of<T>(to_f(ra[m][i]) + p.dt_bias[h * p.dim + d]) : 0.f;
+        g_s[t * ROW + d] = in ? ea * softplus_of<T>(to_f(ra[m][i]) + bias[i]) : 0.f;
         const float q = to_f(rq[m][i]), k = to_f(rk[m][i]);
         qq += q * q; kk += k * k;
       }
@@ -108,9 +120,9 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
         q_s[t * ROW + i * 32 + lane] = to_f(rq[m][i]) * nq;
         k_s[t * ROW + i * 32 + lane] = to_f(rk[m][i]) * nk;
       }
-      if (lane == 0) beta_s[t] = t < nt ? sigmoid_f(to_f(static_cast<const T*>(p.b)[(begin + t0 + t) * p.b_stride + h])) : 0.f;
     }
   }
+  if (tid < kChunk) beta_s[tid] = tid < nt ? sigmoid_f(raw_b) : 0.f;
   __syncthreads();
   for (int d = tid; d < D32; d += 128) {
     float run = 0.f;
@@ -184,62 +196,61 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
     }
   }
   __syncthreads();
-  for (int d = tid; d < D32; d += 128) {         // (whole warps: D32 is a multiple of 32)
+  // a thread owns a key channel: its columns of q, k, g turn into those of Q = q e^G, K = k e^{G_16 - G} and W in place
+  for (int d = tid; d < D32; d += 128) {
     float kh[kChunk];
     const float g_end = g_s[(kChunk - 1) * ROW + d];
-    uint32_t* wq = rec_s;
-    const int ks = d >> 4, kk = d & 15, col = (kk & 7) >> 1, part = (kk < 8 ? 0 : 1) + (d & 1 ? 2 : 0);
-    auto put = [&](int base, int t, float x) {   // even channel writes the pair's high parts, odd channel the low parts
-      const float y = __shfl_xor_sync(0xffffffffu, x, 1);
-      const float e = d & 1 ? y : x, o = d & 1 ? x : y;
-      uint32_t hi_w, lo_w;
-      split_pair(e, o, hi_w, lo_w);
-      if (d < DP) wq[base + ((ks * 2 + (t >> 3)) * 32 + (t & 7) * 4 + col) * 4 + part] = d & 1 ? lo_w : hi_w;
-    };
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      const float g = g_s[t * ROW + d], eg = fast_exp2(g);
-      kh[t] = k_s[t * ROW + d] * eg;
-      put(KS * 256, t, q_s[t * ROW + d] * eg);
+      const float g = g_s[t * ROW + d], eg = fast_exp2(g), k = k_s[t * ROW + d];
+      kh[t] = k * eg;
+      q_s[t * ROW + d] *= eg;
+      k_s[t * ROW + d] = k * fast_exp2(g_end - g);
     }
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
       float acc = 0.f;
 #pragma unroll
       for (int s = 0; s <= t; ++s) acc = fmaf(tm[t][s], kh[s], acc);
-      put(0, t, acc);
+      g_s[t * ROW + d] = acc;
     }
-    if (d < DP) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        uint32_t hi_w, lo_w;
-        split_pair(k_s[2 * i * ROW + d] * fast_exp2(g_end - g_s[2 * i * ROW + d]),
-                   k_s[(2 * i + 1) * ROW + d] * fast_exp2(g_end - g_s[(2 * i + 1) * ROW + d]), hi_w, lo_w);
-        uint32_t* dst = wq + 2 * KS * 256 + ((d >> 3) * 32 + (d & 7) * 4 + (i & 3)) * 4 + (i < 4 ? 0 : 1);
-        dst[0] = hi_w; dst[2] = lo_w;
-      }
-      reinterpret_cast<float*>(rec + lay.decay)[d] = fast_exp2(g_end);
-    }
+    if (d < DP) reinterpret_cast<float*>(rec + lay.decay)[d] = fast_exp2(g_end);
   }
   for (int v = tid; v < lay.vtp * 16; v += 128) {
     float vv[kChunk];
 #pragma unroll
-    for (int s = 0; s < kChunk; ++s)
-      vv[s] = v < p.vdim && s < nt ? to_f(static_cast<const T*>(p.v)[(begin + t0 + s) * p.qkv_stride + static_cast<int64_t>(h) * p.vdim + v]) : 0.f;
-    float* dst = reinterpret_cast<float*>(rec + lay.u) + (v >> 4) * 256 + (v & 7) * 16 + ((v & 15) < 8 ? 0 : 2);
+    for (int s = 0; s < kChunk; ++s) vv[s] = u_s[v * 17 + s];
 #pragma unroll
-    for (int t = 0; t < kChunk; t += 2) {
-      float u0 = 0.f, u1 = 0.f;
+    for (int t = 0; t < kChunk; ++t) {
+      float u = 0.f;
 #pragma unroll
-      for (int s = 0; s <= t + 1; ++s) {
-        if (s <= t) u0 = fmaf(tm[t][s], vv[s], u0);
-        u1 = fmaf(tm[t + 1][s], vv[s], u1);
-      }
-      *reinterpret_cast<float2*>(dst + (t >> 3) * 128 + ((t & 7) >> 1) * 4) = make_float2(u0, u1);
+      for (int s = 0; s <= t; ++s) u = fmaf(tm[t][s], vv[s], u);
+      u_s[v * 17 + t] = u;
     }
   }
   __syncthreads();
-  for (int i = tid; i < 3 * KS * 64; i += 128) reinterpret_cast<uint4*>(rec)[i] = reinterpret_cast<const uint4*>(rec_s)[i];
+  // the record, 16 bytes at a time in the order in which lanes will read it
+  for (int i = tid; i < 2 * KS * 64; i += 128) {
+    const int w = i < KS * 64 ? i : i - KS * 64, ln = w & 31, n = (w >> 5) & 1, ks = w >> 6;
+    const float* src = (i < KS * 64 ? g_s : q_s) + (n * 8 + (ln >> 2)) * ROW + ks * 16 + (ln & 3) * 2;
+    const float2 x = *reinterpret_cast<const float2*>(src), y = *reinterpret_cast<const float2*>(src + 8);
+    uint4 o;
+    split_pair(x.x, x.y, o.x, o.z);
+    split_pair(y.x, y.y, o.y, o.w);
+    reinterpret_cast<uint4*>(rec)[i] = o;
+  }
+  for (int i = tid; i < KS * 64; i += 128) {
+    const int ln = i & 31, d = (i >> 5) * 8 + (ln >> 2), t = (ln & 3) * 2;
+    uint4 o;
+    split_pair(k_s[t * ROW + d], k_s[(t + 1) * ROW + d], o.x, o.z);
+    split_pair(k_s[(t + 8) * ROW + d], k_s[(t + 9) * ROW + d], o.y, o.w);
+    reinterpret_cast<uint4*>(rec + lay.k)[i] = o;
+  }
+  for (int i = tid; i < lay.vtp * 64; i += 128) {
+    const int ln = i & 31, t = ((i >> 5) & 1) * 8 + (ln & 3) * 2, v = (i >> 6) * 16 + (ln >> 2);
+    reinterpret_cast<float4*>(rec + lay.u)[i] =
+        make_float4(u_s[v * 17 + t], u_s[v * 17 + t + 1], u_s[(v + 8) * 17 + t], u_s[(v + 8) * 17 + t + 1]);
+  }
 }
 
 // d += a * b with a, b given as high and low parts
@@ -380,14 +391,15 @@ __global__ void __launch_bounds__(WARPS * 32) delta_chunk_scan(const DeltaParams
 template <class T, int KS>
 static int launch_delta_chunks(const DeltaParams& p, uint8_t* records, cudaStream_t st) {
   constexpr int D32 = (16 * KS + 31) / 32 * 32;
-  constexpr size_t prep_smem = 3 * kChunk * (D32 + 4) * sizeof(float) + 3 * KS * 1024;
+  const ChunkLayout lay = chunk_layout(KS, p.vdim);
+  const size_t prep_smem = (3 * kChunk * (D32 + 4) + lay.vtp * 16 * 17) * sizeof(float);
+  if (prep_smem > 200 * 1024) return kUnsupportedShape;
   struct PrepTag {};
   int rc = opt_in_dynamic_smem<PrepTag>(reinterpret_cast<const void*>(&delta_chunk_prep<T, KS>), prep_smem);
   if (rc != kOk) return rc;
   const int slots = p.tokens / kChunk + p.num_seqs;
   delta_chunk_prep<T, KS><<<dim3(slots, p.heads), 128, prep_smem, st>>>(p, records);
   if (cudaGetLastError() != cudaSuccess) return kLaunchFailed;
-  const ChunkLayout lay = chunk_layout(KS, p.vdim);
   auto scan = [&](auto tag) -> int {
     constexpr int WARPS = decltype(tag)::value;
     struct ScanTag {};
