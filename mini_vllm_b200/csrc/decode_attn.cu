@@ -33,6 +33,8 @@
 #include "mini_vllm_b200.h"
 #include "scan.cuh"
 
+#include <type_traits>
+
 namespace mvb {
 
 constexpr int kMaxCtas = 160;          // workspace is sized for this many persistent CTAs
@@ -212,7 +214,8 @@ __device__ __forceinline__ void load_seq(SeqView& s, int b, const DecodeParams& 
   s.start_al = s.start / CT * CT;
 }
 
-template <int D, int HPC>
+// CAP: scores pass c tanh(s / c) before the softmax.
+template <int D, int HPC, bool CAP>
 __global__ void __launch_bounds__(DecodeCfg<D, HPC>::NW * 32, 1)
 decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                    const DecodeParams p) {
@@ -395,8 +398,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
       const int j0 = token0 + (lane >> 2), j1 = j0 + 8;
       const bool v0 = j0 < cs.n && j0 >= cs.start, v1 = j1 < cs.n && j1 >= cs.start;
       auto score = [&](float s) -> float {
-        if (p.cap_log2 == 0.f) return s * p.scale_log2;
-        return fmaf(-2.f * p.cap_log2, fast_rcp(1.f + fast_exp2(s * p.cap_in)), p.cap_log2);
+        if constexpr (CAP) return fmaf(-2.f * p.cap_log2, fast_rcp(1.f + fast_exp2(s * p.cap_in)), p.cap_log2);
+        else return s * p.scale_log2;
       };
       const float x0 = v0 ? score(s0[0] + s1[0]) : -INFINITY;
       const float x1 = v0 ? score(s0[1] + s1[1]) : -INFINITY;
@@ -594,11 +597,15 @@ static int launch_decode(const CUtensorMap& km, const CUtensorMap& vm, const Dec
                       C::NW * C::NSTAGES * sizeof(uint64_t) +
                       static_cast<size_t>(C::NW) * p.group * C::FIN_STRIDE * sizeof(float);
   if (smem + 64 > 227 * 1024) return kUnsupportedShape;       // static shared memory counts too
-  const int rc = opt_in_dynamic_smem<C>(reinterpret_cast<const void*>(&decode_attn_kernel<D, HPC>), smem);
-  if (rc != kOk) return rc;
-  dim3 grid(num_ctas, hkv / HPC);
-  decode_attn_kernel<D, HPC><<<grid, C::NW * 32, smem, stream>>>(km, vm, p);
-  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+  auto launch = [&](auto tag) -> int {
+    constexpr bool CAP = decltype(tag)::value;
+    struct Tag {};
+    const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&decode_attn_kernel<D, HPC, CAP>), smem);
+    if (rc != kOk) return rc;
+    decode_attn_kernel<D, HPC, CAP><<<dim3(num_ctas, hkv / HPC), C::NW * 32, smem, stream>>>(km, vm, p);
+    return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+  };
+  return p.cap_log2 > 0.f ? launch(std::true_type{}) : launch(std::false_type{});
 }
 
 }  // namespace mvb
