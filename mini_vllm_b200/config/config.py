@@ -134,7 +134,7 @@ def gemma3_shape(num_hidden_layers: int = 26, hidden_size: int = 1152, intermedi
                            tie_word_embeddings=tie_word_embeddings, eos_token_id=None, **extra)
 
 
-def fupupel_shape(layers: list[dict], width: int, vocab: int, eps: float = 1e-6, logit_softcap: float | None = 15.0,
+def fupupel_shape(layers: list[dict], width: int, vocab: int, eps: float = 1e-6, logit_softcap: float | None = 30.0,
                   max_position_embeddings: int = 32768, dtype: torch.dtype = torch.bfloat16) -> SimpleNamespace:
     """A Fupupel description without a checkpoint; ``layers`` as in its config.json."""
     from .native import fupupel_config

@@ -4,7 +4,7 @@
 //
 // The taps - 1 inputs in front of a step's tokens come from the sequence's state slot ([slots, taps - 1, channels], row
 // taps - 1 - d = the input d tokens before the step), zeros before the start of the sequence; afterwards the slot holds the
-// last taps - 1 inputs again.  A thread owns a 16-byte vector of channels and walks a run of tokens with the window in
+// last taps - 1 inputs again.  A thread owns four channels and walks a run of tokens with the window in
 // registers, so every input is read once.  A step in which every sequence brings one token (cu == nullptr) reads and
 // rewrites its slots in the same kernel; a ragged step writes them in a second small kernel, because the tokens that read
 // the old inputs and those that leave the new ones may be worked on by different CTAs.
@@ -15,6 +15,20 @@
 #include "mini_vllm_b200.h"
 
 namespace mvb {
+
+// V elements as they lie in memory
+template <class T, int V> struct alignas(sizeof(T) * V) RawVec { T v[V]; };
+template <class T, int V> __device__ __forceinline__ void get(const T* p, float (&out)[V]) {
+  const RawVec<T, V> r = *reinterpret_cast<const RawVec<T, V>*>(p);
+#pragma unroll
+  for (int i = 0; i < V; ++i) out[i] = to_f(r.v[i]);
+}
+template <class T, int V> __device__ __forceinline__ void put(T* p, const float (&in)[V]) {
+  RawVec<T, V> r;
+#pragma unroll
+  for (int i = 0; i < V; ++i) r.v[i] = from_f<T>(in[i]);
+  *reinterpret_cast<RawVec<T, V>*>(p) = r;
+}
 
 struct ConvParams {
   const void* u; int64_t u_stride;
@@ -40,7 +54,7 @@ __device__ __forceinline__ int64_t conv_slot(const ConvParams& p, int s) {
 }
 
 template <class T, int V, int TAPS>
-__global__ void __launch_bounds__(128) short_conv_kernel(const ConvParams p) {
+__global__ void __launch_bounds__(128, TAPS <= 4 ? 7 : 1) short_conv_kernel(const ConvParams p) {
   const int c = (blockIdx.y * 128 + threadIdx.x) * V;
   if (c >= p.channels) return;
   const int t_begin = blockIdx.x * (p.cu == nullptr ? 1 : kConvRun);
@@ -51,12 +65,12 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvParams p) {
   float w[TAPS][V], bias[V];
 #pragma unroll
   for (int i = 0; i < V; ++i) bias[i] = 0.f;
-  if (p.bias != nullptr) load_vec<T, V>(static_cast<const T*>(p.bias) + c, bias);
+  if (p.bias != nullptr) get<T, V>(static_cast<const T*>(p.bias) + c, bias);
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) {
 #pragma unroll
     for (int i = 0; i < V; ++i) w[j][i] = 0.f;
-    if (j < taps) load_vec<T, V>(static_cast<const T*>(p.w) + static_cast<int64_t>(j) * C + c, w[j]);
+    if (j < taps) get<T, V>(static_cast<const T*>(p.w) + static_cast<int64_t>(j) * C + c, w[j]);
   }
 
   float hist[TAPS][V];                                       // hist[j]: the input j tokens back (hist[0]: this token's)
@@ -76,37 +90,38 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvParams p) {
 #pragma unroll
         for (int i = 0; i < V; ++i) hist[j][i] = 0.f;
         if (j >= taps || pos - j < 0) continue;
-        if (t - j >= begin) load_vec<T, V>(u + (t - j) * p.u_stride, hist[j]);
+        if (t - j >= begin) get<T, V>(u + (t - j) * p.u_stride, hist[j]);
         else if (slot >= 0)
-          load_vec<T, V>(static_cast<const T*>(p.state) + (slot * (taps - 1) + (taps - 1 - (j - (t - begin)))) * C + c, hist[j]);
+          get<T, V>(static_cast<const T*>(p.state) + (slot * (taps - 1) + (taps - 1 - (j - (t - begin)))) * C + c, hist[j]);
       }
     }
-    // the rest of this run inside the sequence, four tokens at a time so that four loads are in flight
+    // the rest of this run inside the sequence, B tokens at a time so that B loads are in flight
+    constexpr int B = 4;
     const int stop = min(t_end, end);
-    for (; t < stop; t += 4) {
-      float in[4][V];
+    for (; t < stop; t += B) {
+      RawVec<T, V> in[B];
 #pragma unroll
-      for (int m = 0; m < 4; ++m)
-        if (t + m < stop) load_vec<T, V>(u + (t + m) * p.u_stride, in[m]);
+      for (int m = 0; m < B; ++m)
+        if (t + m < stop) in[m] = *reinterpret_cast<const RawVec<T, V>*>(u + (t + m) * p.u_stride);
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
+      for (int m = 0; m < B; ++m) {
         if (t + m >= stop) break;
         float acc[V];
 #pragma unroll
-        for (int i = 0; i < V; ++i) { hist[0][i] = in[m][i]; acc[i] = bias[i]; }
+        for (int i = 0; i < V; ++i) { hist[0][i] = to_f(in[m].v[i]); acc[i] = bias[i]; }
 #pragma unroll
         for (int j = TAPS - 1; j >= 0; --j)
 #pragma unroll
           for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], hist[j][i], acc[i]);
 #pragma unroll
         for (int i = 0; i < V; ++i) acc[i] = acc[i] * fast_rcp(1.f + fast_exp2(acc[i] * -1.4426950408889634f));
-        store_vec<T, V>(out + (t + m) * p.out_stride, acc);
+        put<T, V>(out + (t + m) * p.out_stride, acc);
         if (p.cu == nullptr) {                               // the slot's rows are this thread's alone
           const int64_t slot = conv_slot(p, s);
           if (slot >= 0) {
 #pragma unroll
             for (int j = 0; j < TAPS; ++j)
-              if (j < taps - 1) store_vec<T, V>(static_cast<T*>(p.state) + (slot * (taps - 1) + (taps - 2 - j)) * C + c, hist[j]);
+              if (j < taps - 1) put<T, V>(static_cast<T*>(p.state) + (slot * (taps - 1) + (taps - 2 - j)) * C + c, hist[j]);
           }
         }
 #pragma unroll
@@ -135,12 +150,12 @@ __global__ void __launch_bounds__(128) conv_state_kernel(const ConvParams p) {
 #pragma unroll
     for (int i = 0; i < V; ++i) v[d][i] = 0.f;
     if (d >= taps || next - d < 0) continue;
-    if (n - d >= 0) load_vec<T, V>(static_cast<const T*>(p.u) + (begin + n - d) * p.u_stride + c, v[d]);
-    else load_vec<T, V>(st + static_cast<int64_t>(taps - 1 - (d - n)) * p.channels, v[d]);
+    if (n - d >= 0) get<T, V>(static_cast<const T*>(p.u) + (begin + n - d) * p.u_stride + c, v[d]);
+    else get<T, V>(st + static_cast<int64_t>(taps - 1 - (d - n)) * p.channels, v[d]);
   }
 #pragma unroll
   for (int d = 1; d < TAPS; ++d)
-    if (d < taps) store_vec<T, V>(st + static_cast<int64_t>(taps - 1 - d) * p.channels, v[d]);
+    if (d < taps) put<T, V>(st + static_cast<int64_t>(taps - 1 - d) * p.channels, v[d]);
 }
 
 template <class T, int V, int TAPS>
@@ -155,7 +170,7 @@ static int launch_conv_t(const ConvParams& p, cudaStream_t st) {
 
 template <class T>
 static int launch_conv(const ConvParams& p, cudaStream_t st) {
-  constexpr int V = kVec<T>;
+  constexpr int V = 4;                                       // (8 bf16 would double the registers and halve the warps)
   const bool vec = p.channels % V == 0 && p.u_stride % V == 0 && p.out_stride % V == 0 && is_aligned(p.u, 16) &&
                    is_aligned(p.out, 16) && is_aligned(p.state, 16) && is_aligned(p.w, 16) && is_aligned(p.bias, 16);
   if (p.taps <= 4) return vec ? launch_conv_t<T, V, 4>(p, st) : launch_conv_t<T, 1, 4>(p, st);

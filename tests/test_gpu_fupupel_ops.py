@@ -86,7 +86,7 @@ def scan_inputs(g, lens, inner, n, dtype):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("inner,n", [(40, 16), (33, 5), (128, 24), (20, 40), (12, 100), (9, 130), (70, 1)])
+@pytest.mark.parametrize("inner,n", [(40, 16), (33, 5), (128, 20), (20, 40), (12, 100), (9, 130), (70, 1)])
 @pytest.mark.parametrize("portions", ["whole", "single", "mixed", "long"])
 def test_selective_scan(cuda, dtype, inner, n, portions):
     g, lens = gen(2), [70, 3, 300, 1]
@@ -117,7 +117,7 @@ def test_selective_scan(cuda, dtype, inner, n, portions):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("heads,kv,dim,vdim", [(4, 2, 64, 32), (3, 3, 20, 12), (2, 1, 128, 128), (2, 2, 40, 136), (1, 1, 200, 24), (6, 2, 8, 50),
+@pytest.mark.parametrize("heads,kv,dim,vdim", [(4, 2, 64, 40), (3, 3, 20, 12), (2, 1, 128, 128), (2, 2, 40, 136), (1, 1, 200, 24), (6, 2, 8, 50),
                                                (2, 2, 96, 96)])
 @pytest.mark.parametrize("portions", ["whole", "single", "mixed", "long"])
 def test_gated_delta(cuda, dtype, heads, kv, dim, vdim, portions):
@@ -177,12 +177,12 @@ def plant_key(q, k, dist, strength=6.0):
         k[i - dist, h] = (u / u.norm() * strength).to(k.dtype)
 
 
-@pytest.mark.parametrize("heads,kv,d,window,cap", [(4, 2, 128, 96, 20.0), (3, 3, 128, 33, 5.0), (8, 1, 256, 128, 30.0), (6, 3, 128, None, 50.0),
+@pytest.mark.parametrize("heads,kv,d,window,cap", [(4, 2, 128, 80, 18.0), (3, 3, 128, 33, 5.0), (8, 1, 256, 128, 30.0), (6, 3, 128, None, 50.0),
                                                    (4, 2, 128, 129, 0.0), (4, 4, 128, 1, 2.0)])
 @pytest.mark.parametrize("edge", [-1, 0])
 def test_capped_window_attention_prefill_and_decode(cuda, heads, kv, d, window, cap, edge):
     """edge 0: the planted key is just outside the window; -1: just inside."""
-    g, lens, scale, factor = gen(4), [130, 1, 300, 257, 40], 0.4, 0.8
+    g, lens, scale, factor = gen(4), [130, 1, 300, 257, 40], 0.4, 0.75
     seqs = window_case(g, lens, heads, kv, d, BF)
     for q, k, _ in seqs:
         plant_key(q, k, (window or 120) + edge)
@@ -248,7 +248,7 @@ def test_scores_do_not_lose_the_cap_far_out(cuda):
     k = torch.stack([torch.full((1, 128), 8.0), torch.full((1, 128), 4.0)]).to(BF).to(cuda)
     v = torch.stack([torch.full((1, 128), 1.0), torch.full((1, 128), 3.0)]).to(BF).to(cuda)
     cu = torch.tensor([0, 2], dtype=torch.int32, device=cuda)
-    out = ops.prefill_attn(q, k, v, cu, cu, 2, 1.0, -1, softcap=20.0)
+    out = ops.prefill_attn(q, k, v, cu, cu, 2, 1.0, -1, softcap=25.0)
     assert torch.allclose(out[1].float(), torch.full_like(out[1], 2.0).float(), atol=1e-2)
 
 
@@ -311,7 +311,7 @@ def test_clamped_glu(cuda, dtype, inter):
 
 def test_capped_logits_and_fp32_argmax(cuda):
     x = torch.randn(5, 1003, generator=gen(9)) * 30
-    assert rel(ops.cap_logits(x.to(cuda), 15.0, F32), plain.soft_cap(x.double(), 15.0)) < 1e-6
+    assert rel(ops.cap_logits(x.to(cuda), 12.0, F32), plain.soft_cap(x.double(), 12.0)) < 1e-6
     assert torch.equal(ops.cap_logits(x.to(cuda), 0.0, F32).cpu(), x)
     y = x.clone()
     y[0, 700] = y[0, 3] = 1e3                                   # a tie: the lower column wins
