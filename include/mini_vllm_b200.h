@@ -407,6 +407,73 @@ int mvb_gated_delta(int dtype, const void* q, const void* k, const void* v, int6
                     float q_scale, float eps, float out_scale, void* scratch, size_t scratch_bytes, int32_t* dev_status,
                     void* stream);
 
+/*
+ * Linear attention with decay (per-sequence state slots as above): per head S <- D S + w k v^T, o = S^T q, then
+ * out = o / rms(o) * norm_weight * gate function.  q, k [tokens, heads, dim], v [tokens, heads, vdim] share one row stride; q is
+ * multiplied by q_scale; dim <= 256; state [num_slots, heads, dim, vdim rounded up to 4] fp32.
+ * mvb_gated_linear: D = diag(sigmoid(decay + decay_bias)^inv_tau) per key channel (decay [tokens, heads * dim]), w = 1; SiLU gate;
+ *   norm_weight [vdim].
+ * mvb_mlstm: log gates i = cap tanh((input + input_bias) / cap), f = log sigmoid(cap tanh((forget + forget_bias) / cap)) per head; with
+ *   the running maximum m' = max(f + m, i) (m from 0): D = e^{f + m - m'}, w = e^{i - m'}; n <- D n + w k; o over
+ *   max(|n . q|, e^{-m'}) + 1e-6; sigmoid gate; norm_weight [heads * vdim].  normaliser [num_slots, heads, dim], maximum
+ *   [num_slots, heads] fp32.
+ * scratch: mvb_linear_attn_scratch_bytes(...) bytes (exp_gates: 1 for mvb_mlstm; ragged: cu_seqlens_q != NULL).
+ */
+size_t mvb_linear_attn_scratch_bytes(int dtype, int num_tokens, int num_seqs, int heads, int dim, int vdim, int exp_gates, int ragged);
+int mvb_gated_linear(int dtype, const void* q, const void* k, const void* v, int64_t qkv_row_stride, const void* decay,
+                     int64_t decay_row_stride, const float* decay_bias, float inv_tau, const void* gate, int64_t gate_row_stride,
+                     const float* norm_weight, void* out, int64_t out_row_stride, float* state, const int32_t* state_slots,
+                     int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int heads,
+                     int dim, int vdim, float q_scale, float eps, void* scratch, size_t scratch_bytes, int32_t* dev_status, void* stream);
+int mvb_mlstm(int dtype, const void* q, const void* k, const void* v, int64_t qkv_row_stride, const void* forget,
+              int64_t forget_row_stride, const float* forget_bias, const void* input, int64_t input_row_stride, const float* input_bias,
+              float cap, const void* gate, int64_t gate_row_stride, const float* norm_weight, void* out, int64_t out_row_stride,
+              float* state, float* normaliser, float* maximum, const int32_t* state_slots, int64_t num_slots,
+              const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int heads, int dim, int vdim,
+              float q_scale, float eps, void* scratch, size_t scratch_bytes, int32_t* dev_status, void* stream);
+
+/*
+ * Hyper-connected residual streams x [rows, streams, width] fp32; norms in `groups` equal consecutive parts of a row.
+ * mvb_hyper_embed_norm: every stream = table[ids] + pos_table[positions]; h = norm(sum_s in[s] x_s) * weight.
+ * mvb_hyper_norm: x_t <- sum_s mix[s, t] x_s + out[t] y; h = norm(sum_s in[s] x_s) * weight (in NULL: the plain sum).  row_ends != NULL:
+ *   output row r comes from source row row_ends[r + 1] - 1 and x is left as it is.  streams <= 16.
+ * mvb_poly_norm: out = a N(z) + b N(z^2) + c N(z^3) + e over the row's `cols` values, N(v) = v / sqrt(mean(v^2) + eps), act = {a, b, c,
+ *   e} on the device; columns cols..out_cols-1 become 0.
+ */
+int mvb_hyper_embed_norm(int dtype, const int64_t* ids, const int64_t* positions, const void* table, int64_t vocab,
+                         const void* pos_table, int64_t max_positions, float* x, const float* in_weights, const void* weight, void* h,
+                         int rows, int width, int streams, int groups, float eps, int32_t* dev_status, void* stream);
+int mvb_hyper_norm(int dtype, float* x, const void* y, int64_t y_row_stride, const float* mix, const float* out_weights,
+                   const float* in_weights, const void* weight, void* h, const int32_t* row_ends, int rows, int width, int streams,
+                   int groups, float eps, void* stream);
+int mvb_poly_norm(int dtype, const void* z, int64_t z_row_stride, void* out, int64_t out_row_stride, int rows, int cols, int out_cols,
+                  const float* act, float eps, void* stream);
+
+/*
+ * Attention over a cached latent (pool [num_blocks, block_size, width], one row per token for all heads).
+ * mvb_latent_norm: q_out = rmsnorm(q) [tokens, q_pad] and, with c != NULL, c_out = rmsnorm(c) [tokens, c_pad], also into
+ *   cache[slot_mapping[t]] (slots < 0: not written; cache NULL: no cache); columns behind q_cols / c_cols become 0.
+ * mvb_gather_latents: the contexts cu_seqlens_k describes as dense rows.
+ * mvb_gate_mul: out = o * sigmoid(gate).
+ * mvb_latent_decode: one query row per sequence in the absorbed form: out[b, h] = softmax(scale q[b, h] . c) c, bf16; width one of 64,
+ *   128, 192, 256, 384, 512; block_size a multiple of 64.  The workspace (mvb_decode_workspace_bytes(num_seqs, num_heads, width)) must
+ *   hold the plan of mvb_latent_decode_plan for the same cache_seqlens.
+ */
+int mvb_latent_norm(int dtype, const void* q, int64_t q_row_stride, const void* q_weight, void* q_out, int q_cols, int q_pad,
+                    const void* c, int64_t c_row_stride, const void* c_weight, void* c_out, int c_cols, int c_pad, void* cache,
+                    const int32_t* slot_mapping, int64_t num_slots, int num_tokens, float eps, int32_t* dev_status, void* stream);
+int mvb_gather_latents(const void* cache, int64_t num_slots, int row_bytes, const int32_t* block_table, int64_t table_stride,
+                       int table_width, int block_size, const int32_t* cu_seqlens_k, int num_seqs, int num_rows, void* out,
+                       int32_t* dev_status, void* stream);
+int mvb_gate_mul(int dtype, const void* o, int64_t o_row_stride, const void* gate, int64_t gate_row_stride, void* out,
+                 int64_t out_row_stride, int rows, int cols, void* stream);
+int mvb_latent_decode_plan(const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int block_size, int num_seqs,
+                           int num_heads, int width, void* workspace, size_t workspace_bytes, void* stream);
+int mvb_latent_decode(const void* q, int64_t q_row_stride, int64_t q_head_stride, const void* cache, int64_t num_blocks, int block_size,
+                      const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
+                      int num_heads, int width, float scale, void* out, int64_t out_row_stride, int64_t out_head_stride, void* workspace,
+                      size_t workspace_bytes, int32_t* dev_status, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

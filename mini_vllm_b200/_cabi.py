@@ -59,6 +59,20 @@ SIGNATURES = {
     "mvb_gated_delta_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32, i32, i32]),
     "mvb_gated_delta": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp,
                               vp, i32, i32, i32, i32, i32, i32, f32, f32, f32, vp, sz, vp, vp]),
+    "mvb_linear_attn_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32, i32, i32]),
+    "mvb_gated_linear": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, f32, vp, i64, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32,
+                               i32, i32, i32, f32, f32, vp, sz, vp, vp]),
+    "mvb_mlstm": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, vp, i64, vp, f32, vp, i64, vp, vp, i64, vp, vp, vp, vp, i64, vp,
+                        vp, i32, i32, i32, i32, i32, f32, f32, vp, sz, vp, vp]),
+    "mvb_hyper_embed_norm": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp, vp]),
+    "mvb_hyper_norm": (i32, [i32, vp, vp, i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp]),
+    "mvb_poly_norm": (i32, [i32, vp, i64, vp, i64, i32, i32, i32, vp, f32, vp]),
+    "mvb_latent_norm": (i32, [i32, vp, i64, vp, vp, i32, i32, vp, i64, vp, vp, i32, i32, vp, vp, i64, i32, f32, vp, vp]),
+    "mvb_gather_latents": (i32, [vp, i64, i32, vp, i64, i32, i32, vp, i32, i32, vp, vp, vp]),
+    "mvb_gate_mul": (i32, [i32, vp, i64, vp, i64, vp, i64, i32, i32, vp]),
+    "mvb_latent_decode_plan": (i32, [vp, vp, i64, i32, i32, i32, i32, vp, sz, vp]),
+    "mvb_latent_decode": (i32, [vp, i64, i64, vp, i64, i32, vp, vp, i64, i32, i32, i32, i32, f32, vp, i64, i64, vp, sz, vp,
+                                vp]),
 }
 
 _lib = None

@@ -140,3 +140,11 @@ def fupupel_shape(layers: list[dict], width: int, vocab: int, eps: float = 1e-6,
     from .native import fupupel_config
     return fupupel_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
                            "logit_softcap": logit_softcap}, None, dtype, max_position_embeddings)
+
+
+def vebonex_shape(layers: list[dict], width: int, vocab: int, streams: int = 4, groups: int = 1, eps: float = 1e-6,
+                  max_positions: int = 8192, dtype: torch.dtype = torch.bfloat16) -> SimpleNamespace:
+    """A Vebonex description without a checkpoint; ``layers`` as in its config.json."""
+    from .native import vebonex_config
+    return vebonex_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": groups}, "streams": streams,
+                           "max_positions": max_positions}, None, dtype)

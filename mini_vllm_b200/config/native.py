@@ -45,7 +45,26 @@ def fupupel_config(config: dict, shapes: dict[str, list[int]] | None = None, dty
         max_position_embeddings=max_position_embeddings, eos_token_id=config.get("eos_token_id"))
 
 
-_READERS = {"Fupupel": fupupel_config}
+def vebonex_config(config: dict, shapes: dict[str, list[int]] | None = None, dtype: torch.dtype = torch.bfloat16,
+                   max_position_embeddings: int = 4096) -> SimpleNamespace:
+    """Positions are a learned table, so its size is the model's and not the engine's.  The rank of a decay's low-rank pair is given by
+    tensor shapes alone; without a checkpoint it comes from the mixer's ``decay_rank`` (default: its ``dim``)."""
+    layers = copy.deepcopy(config["layers"])
+    for i, layer in enumerate(layers):
+        if layer["type"] != "gla":
+            continue
+        tensor = f"l{i}.mix.a1"
+        if shapes and tensor in shapes:
+            layer["mixer"]["decay_rank"] = shapes[tensor][0]
+        else:
+            layer["mixer"].setdefault("decay_rank", layer["mixer"]["dim"])
+    return SimpleNamespace(
+        architectures=["Vebonex"], dtype=dtype, layers=layers, num_hidden_layers=len(layers), hidden_size=config["width"],
+        vocab_size=config["vocab"], rms_norm_eps=config["norm"]["eps"], norm_groups=config["norm"]["groups"], streams=config["streams"],
+        max_position_embeddings=config["max_positions"], learned_positions=config["max_positions"], eos_token_id=config.get("eos_token_id"))
+
+
+_READERS = {"Fupupel": fupupel_config, "Vebonex": vebonex_config}
 
 
 def read_native(path: str, dtype: torch.dtype | None, max_position_embeddings: int) -> Any:

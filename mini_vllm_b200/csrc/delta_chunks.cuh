@@ -15,14 +15,9 @@
 // Every fp32 operand enters as bf16 high + low part and every product as high*high + high*low + low*high: 16 significant bits
 // per factor with fp32 accumulation; the state itself is never rounded below fp32.
 #pragma once
-#include "dtype.cuh"
+#include "chunk_common.cuh"
 
 namespace mvb {
-
-constexpr int kChunk = 16;
-
-// sequence s owns chunk slots chunk_base(s) .. + ceil(n / 16): never overlapping, no prefix sum needed
-__host__ __device__ __forceinline__ int chunk_base(int row, int s) { return row / kChunk + s; }
 
 struct ChunkLayout {              // bytes inside a record
   int ks, vtp, q, k, b, decay, u, total;
@@ -35,13 +30,6 @@ __host__ __device__ inline ChunkLayout chunk_layout(int ks, int vdim) {
   l.u = l.decay + ks * 64;
   l.total = l.u + l.vtp * 1024;
   return l;
-}
-
-__device__ __forceinline__ float bf16_round(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
-// (x, y) as packed bf16: the rounded values, and what the rounding left over
-__device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(x, y);
-  lo = pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));
 }
 
 template <class T, int KS>
@@ -253,13 +241,6 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) delta_chunk_prep(const D
   }
 }
 
-// d += a * b with a, b given as high and low parts
-struct Split { uint32_t hi[4], lo[4]; };
-__device__ __forceinline__ void split_tile(const float (&x)[4], const float (&y)[4], Split& s) {   // two adjacent 8-column tiles
-  split_pair(x[0], x[1], s.hi[0], s.lo[0]); split_pair(x[2], x[3], s.hi[1], s.lo[1]);
-  split_pair(y[0], y[1], s.hi[2], s.lo[2]); split_pair(y[2], y[3], s.hi[3], s.lo[3]);
-}
-
 template <int KS, int WARPS>
 struct ChunkScanCfg {
   static constexpr int STAGES = 3;
@@ -289,10 +270,8 @@ __global__ void __launch_bounds__(WARPS * 32) delta_chunk_scan(const DeltaParams
     const uint8_t* src = rec + c * rec_step;
     const uint32_t dst = smem_u32(smem + st * C::STAGE), bar = smem_u32(&full[st]);
     mbar_arrive_expect_tx(&full[st], C::STAGE);
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 ::"r"(dst), "l"(src), "r"(C::SHARED), "r"(bar) : "memory");
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 ::"r"(dst + C::SHARED), "l"(src + lay.u + blockIdx.x * (WARPS * 1024)), "r"(WARPS * 1024), "r"(bar) : "memory");
+    bulk_copy(dst, src, C::SHARED, bar);
+    bulk_copy(dst + C::SHARED, src + lay.u + blockIdx.x * (WARPS * 1024), WARPS * 1024, bar);
   };
   if (tid == 0)
     for (int c = 0; c < min(C::STAGES, n_chunks); ++c) fetch(c);
@@ -412,14 +391,6 @@ static int launch_delta_chunks(const DeltaParams& p, uint8_t* records, cudaStrea
   // few (sequence, head) pairs: one warp per CTA, so that they spread over the SMs
   const bool few = static_cast<int64_t>(lay.vtp) * p.heads * p.num_seqs <= sm_count() * 2;
   return few ? scan(std::integral_constant<int, 1>{}) : scan(std::integral_constant<int, 4>{});
-}
-
-// the instance that holds a key size
-static int chunk_ks(int dim) {
-  const int need = (dim + 15) / 16;
-  for (int ks : {1, 2, 3, 4, 6, 8, 12, 16})
-    if (need <= ks) return ks;
-  return 0;
 }
 
 }  // namespace mvb

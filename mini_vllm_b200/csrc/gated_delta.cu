@@ -14,8 +14,9 @@
 // Ragged step, fp32 activations: plain fp32 throughout.  delta_prep_kernel writes q, k, g as [tokens, heads, dp] once per token;
 // delta_tokens_kernel walks a sequence's tokens with S in registers (8 row groups x 4 columns per warp, the sum over rows is
 // three shuffles), operands staged TT tokens ahead with cp.async.
-// gated_norm_kernel finishes the rows of either.
-#include "dtype.cuh"
+// head_norm_kernel (head_norm.cuh) finishes the rows of either.
+#include "chunk_common.cuh"
+#include "head_norm.cuh"
 #include "host_util.cuh"
 #include "mini_vllm_b200.h"
 
@@ -47,11 +48,6 @@ __device__ __forceinline__ int64_t delta_slot(const DeltaParams& p, int s) {
   const int64_t slot = p.slots[s];
   if (slot >= p.num_slots) { report(p.dev_status, kDevBadSlot, s); return -1; }
   return slot;
-}
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-  return v;
 }
 __device__ __forceinline__ float decay_of(float raw, float bias, float exp_a) { return expf(-exp_a * softplus_f(raw + bias)); }
 
@@ -189,12 +185,6 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
 }
 
 // ---- ragged step: the recurrence -------------------------------------------------------------------------
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 // NI: 32-row groups of S per column (dim <= 32 NI); a CTA owns 16 columns of one (sequence, head)
 template <class T, int NI>
 __global__ void __launch_bounds__(128) delta_tokens_kernel(const DeltaParams p) {
@@ -292,54 +282,21 @@ __global__ void __launch_bounds__(128) delta_tokens_kernel(const DeltaParams p) 
   }
 }
 
-// out[t, h, :] = o / rms(o) * w * sigmoid(gate) * factor; one warp per (token, head)
-template <class T>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const DeltaParams p, bool vec) {
-  const int64_t w = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31, t = static_cast<int>(w / p.heads), h = static_cast<int>(w % p.heads);
-  if (t >= p.tokens) return;
-  const float* o = p.o + w * p.vdim;
-  const T* gate = static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<int64_t>(h) * p.vdim;
-  T* out = static_cast<T*>(p.out) + t * p.out_stride + static_cast<int64_t>(h) * p.vdim;
-  auto sig = [](float z) { return sizeof(T) == 2 ? fast_rcp(1.f + fast_exp2(z * -1.4426950408889634f)) : sigmoid_f(z); };
-  if (sizeof(T) == 2 && vec && p.vdim <= 128) {               // a lane keeps its four columns
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    uint2 gw = make_uint2(0u, 0u);
-    const int i = lane * 4;
-    if (i < p.vdim) { x = *reinterpret_cast<const float4*>(o + i); gw = *reinterpret_cast<const uint2*>(gate + i); }
-    const float r = p.out_scale * rsqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) / static_cast<float>(p.vdim) + p.eps);
-    if (i < p.vdim) {
-      const float4 nw = *reinterpret_cast<const float4*>(p.norm_w + i);
-      uint2 y;
-      y.x = pack_bf16(x.x * r * nw.x * sig(bf16_lo(gw.x)), x.y * r * nw.y * sig(bf16_hi(gw.x)));
-      y.y = pack_bf16(x.z * r * nw.z * sig(bf16_lo(gw.y)), x.w * r * nw.w * sig(bf16_hi(gw.y)));
-      *reinterpret_cast<uint2*>(out + i) = y;
-    }
-    return;
-  }
-  float ss = 0.f;
-  for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
-  const float r = p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.vdim) + p.eps);
-  for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * r * p.norm_w[i] * sig(to_f(gate[i])));
-}
-
 }  // namespace mvb
 
 #include "delta_chunks.cuh"
 
 namespace mvb {
 
-static int delta_row_pad(int dim) { return (dim + 31) / 32 * 32; }
-
 template <class T>
 static int launch_gated_norm(const DeltaParams& p, cudaStream_t st) {
-  const int64_t blocks = (static_cast<int64_t>(p.tokens) * p.heads * 32 + 255) / 256;
-  if (blocks > 0x7fffffffLL) return kUnsupportedShape;
-  const bool vec = p.vdim % 4 == 0 && p.gate_stride % 4 == 0 && p.out_stride % 4 == 0 && is_aligned(p.gate, 8) &&
-                   is_aligned(p.out, 8) && is_aligned(p.norm_w, 16) && is_aligned(p.o, 16);
-  gated_norm_kernel<T><<<static_cast<unsigned>(blocks), 256, 0, st>>>(p, vec);
-  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+  HeadNormParams n{};
+  n.o = p.o; n.gate = p.gate; n.gate_stride = p.gate_stride; n.norm_w = p.norm_w; n.out = p.out; n.out_stride = p.out_stride;
+  n.tokens = p.tokens; n.heads = p.heads; n.vdim = p.vdim; n.eps = p.eps; n.out_scale = p.out_scale;
+  return launch_head_norm<T, kGateSigmoid>(n, st);
 }
+
+static int delta_row_pad(int dim) { return (dim + 31) / 32 * 32; }
 
 static int step_tile_cols(int vp) {                            // columns per CTA: the whole head up to 128, else 128
   return vp <= 128 ? vp : 128;

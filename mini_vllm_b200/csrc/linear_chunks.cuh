@@ -1,0 +1,509 @@
+// Linear attention with decay over chunks of 16 tokens on the tensor cores (ragged steps with bf16 activations).
+//
+// Channel decay: with log-decays summed inside a chunk, G_t = sum_{s <= t} log a_s (per key channel), and the chunk's initial S0:
+//   o_t = (q_t e^{G_t}) S0 + sum_{s <= t} B_ts v_s          B_ts = sum_d q_t k_s e^{G_t - G_s}
+//   S  <- e^{G_16} S0 + sum_s (k_s e^{G_16 - G_s}) v_s^T
+// Exponential gates: F_t = sum_{s <= t} f_s (a scalar per head), M_t = max_{s <= t} (F_t - F_s + i_s), m_t = max(F_t + m_0, M_t):
+//   o_t = e^{F_t + m_0 - m_t} q_t S0 + e^{M_t - m_t} sum_{s <= t} B_ts v_s          B_ts = (q_t . k_s) e^{F_t - F_s + i_s - M_t}
+//   S  <- e^{F_16 + m_0 - m_16} S0 + e^{M_16 - m_16} sum_s (k_s e^{F_16 - F_s + i_s - M_16}) v_s^T
+// B, M and the scaled keys do not depend on what came before the chunk; only the row factors do, through the one scalar m_0.
+// All exponents are <= 0, whatever the gates are.  The normaliser n is column vdim of S, with value 1.
+//
+// The prep kernels (parallel over chunks and heads) leave one contiguous record per (chunk, head) with everything the recurrence
+// needs, already in the register order of mma.sync operands.  linear_chunk_scan (sequential over the chunks of a sequence, parallel
+// over heads and 16-column tiles) keeps S^T in the fp32 accumulator registers of one warp per 16 columns, whose fragments are operand
+// fragments of the next product as they stand; records arrive by bulk copies, three chunks ahead.
+// v (and, with exponential gates, q) is a bf16 projection and enters exactly; every other operand enters as bf16 high + low part:
+// 16 significant bits per factor with fp32 accumulation.  The state itself is never rounded below fp32.
+#pragma once
+#include "chunk_common.cuh"
+
+namespace mvb {
+
+struct LinearLayout {             // bytes inside a record
+  int k, b, extra, v, total;      // q at 0; extra: decay of the chunk per key channel, or F and M of its tokens
+};
+__host__ __device__ inline LinearLayout linear_layout(int ks, int vtp, bool exp_gates) {
+  LinearLayout l;
+  l.k = ks * (exp_gates ? 512 : 1024);
+  l.b = l.k + ks * 1024;
+  l.extra = l.b + 1024;
+  l.v = l.extra + (exp_gates ? 128 : ks * 64);
+  l.total = l.v + vtp * 512;
+  return l;
+}
+
+static inline int linear_warps(const LinearParams& p, bool exp_gates) {      // 16-column tiles per CTA
+  const int tiles = (p.vdim + (exp_gates ? 1 : 0) + 15) / 16;
+  // few (sequence, head) pairs: one warp per CTA, so that they spread over the SMs
+  if (static_cast<int64_t>(tiles) * p.heads * p.num_seqs <= sm_count() * 2) return 1;
+  int best = 4;
+  for (int w = 4; w >= 2; --w)
+    if ((tiles + w - 1) / w * w < (tiles + best - 1) / best * best) best = w;
+  return tiles == 1 ? 1 : best;
+}
+static inline int linear_tiles(const LinearParams& p, bool exp_gates) {
+  const int tiles = (p.vdim + (exp_gates ? 1 : 0) + 15) / 16, w = linear_warps(p, exp_gates);
+  return (tiles + w - 1) / w * w;
+}
+
+struct ChunkSite { int seq, row, n; };        // the sequence, first row and token count of a chunk slot; n = 0: an unused slot
+__device__ __forceinline__ ChunkSite chunk_site(const LinearParams& p, int slot) {
+  int lo = 0, hi = p.num_seqs;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (chunk_base(p.cu[mid], mid) <= slot) lo = mid; else hi = mid;
+  }
+  const int begin = p.cu[lo], t0 = (slot - chunk_base(begin, lo)) * kChunk;
+  return {lo, begin + t0, min(kChunk, p.cu[lo + 1] - begin - t0)};
+}
+
+__device__ __forceinline__ float bf_at(const void* base, int64_t i) { return __bfloat162float(static_cast<const __nv_bfloat16*>(base)[i]); }
+
+// v of a chunk as [16][cols] bf16 in shared memory: zeros behind the tokens and columns there are, ones in column `one`
+__device__ __forceinline__ void stage_values(const LinearParams& p, const ChunkSite& c, int h, int cols, int one, __nv_bfloat16* v_s) {
+  const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(p.v) + c.row * p.qkv_stride + static_cast<int64_t>(h) * p.vdim;
+  if (p.vdim % 8 == 0 && p.qkv_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(p.v) & 15) == 0) {
+    const int vec = cols / 8;
+    for (int e = threadIdx.x; e < kChunk * vec; e += blockDim.x) {
+      const int t = e / vec, col = (e % vec) * 8;
+      uint4 w = make_uint4(0u, 0u, 0u, 0u);
+      if (t < c.n && col < p.vdim) w = *reinterpret_cast<const uint4*>(v + t * p.qkv_stride + col);
+      if (t < c.n && col == one) w.x = 0x3f80u;               // (one = vdim is a multiple of 8 here)
+      *reinterpret_cast<uint4*>(v_s + t * cols + col) = w;
+    }
+  } else {
+    for (int e = threadIdx.x; e < kChunk * cols; e += blockDim.x) {
+      const int t = e / cols, col = e % cols;
+      v_s[e] = t < c.n && col < p.vdim ? v[t * p.qkv_stride + col] : __float2bfloat16_rn(t < c.n && col == one ? 1.f : 0.f);
+    }
+  }
+}
+// the values as first operand of V^T (.): rows = columns of v, k = tokens
+__device__ __forceinline__ void write_values(const __nv_bfloat16* v_s, int cols, uint8_t* dst) {
+  const uint16_t* v = reinterpret_cast<const uint16_t*>(v_s);
+  auto two = [&](int t, int c) { return static_cast<uint32_t>(v[t * cols + c]) | static_cast<uint32_t>(v[(t + 1) * cols + c]) << 16; };
+  for (int i = threadIdx.x; i < cols / 16 * 32; i += blockDim.x) {
+    const int ln = i & 31, t = (ln & 3) * 2, c = (i >> 5) * 16 + (ln >> 2);
+    reinterpret_cast<uint4*>(dst)[i] = make_uint4(two(t, c), two(t, c + 8), two(t + 8, c), two(t + 8, c + 8));
+  }
+}
+// B as second operand of (.) B^T; at(t, s) for s <= t, one warp
+template <class F>
+__device__ __forceinline__ void write_triangle(F at, int lane, uint8_t* dst) {
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const int t = n * 8 + (lane >> 2), s = (lane & 3) * 2;
+    auto below = [&](int c) { return c <= t ? at(t, c) : 0.f; };
+    uint4 w;
+    split_pair(below(s), below(s + 1), w.x, w.z);
+    split_pair(below(s + 8), below(s + 9), w.y, w.w);
+    reinterpret_cast<uint4*>(dst)[n * 32 + lane] = w;
+  }
+}
+// scaled keys k_s [16][row] (fp32) as second operand of V^T K: 8-channel tiles
+__device__ __forceinline__ void write_keys(const float* k_s, int row, int ks, uint8_t* dst) {
+  for (int i = threadIdx.x; i < ks * 64; i += blockDim.x) {
+    const int ln = i & 31, d = (i >> 5) * 8 + (ln >> 2), t = (ln & 3) * 2;
+    uint4 o;
+    split_pair(k_s[t * row + d], k_s[(t + 1) * row + d], o.x, o.z);
+    split_pair(k_s[(t + 8) * row + d], k_s[(t + 9) * row + d], o.y, o.w);
+    reinterpret_cast<uint4*>(dst)[i] = o;
+  }
+}
+
+// ---- channel decay ----------------------------------------------------------------------------------------
+template <int KS>
+__global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const LinearParams p) {
+  constexpr int D32 = (16 * KS + 31) / 32 * 32, ROW = D32 + 4, NI = D32 / 32;
+  extern __shared__ __align__(16) float sm[];
+  float* q_s = sm;                               // [16][ROW]
+  float* k_s = q_s + kChunk * ROW;
+  float* g_s = k_s + kChunk * ROW;               // log2 of the decay, then its running sum
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(g_s + kChunk * ROW);
+  __shared__ float bm[kChunk][kChunk + 1];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const ChunkSite c = chunk_site(p, blockIdx.x);
+  if (c.n <= 0) return;
+  const LinearLayout lay = linear_layout(KS, p.vtp, false);
+  uint8_t* rec = p.records + (static_cast<int64_t>(blockIdx.x) * p.heads + h) * lay.total;
+
+  // a warp takes every fourth token; the raw operands of U tokens are requested before any is worked on
+  constexpr int U = NI <= 4 ? 4 : 2;
+  const float to_log2 = p.inv_tau * kLog2e;
+  float bias[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) bias[i] = i * 32 + lane < p.dim ? p.decay_bias[h * p.dim + i * 32 + lane] : 0.f;
+  stage_values(p, c, h, p.vtp * 16, -1, v_s);
+#pragma unroll 1
+  for (int tb = warp; tb < kChunk; tb += 4 * U) {
+    float rq[U][NI], rk[U][NI], ra[U][NI];
+#pragma unroll
+    for (int m = 0; m < U; ++m) {
+      const int t = tb + 4 * m;
+      const int64_t qk = (c.row + t) * p.qkv_stride + h * p.dim, a = (c.row + t) * p.decay_stride + h * p.dim;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int d = i * 32 + lane;
+        const bool in = t < c.n && d < p.dim;
+        rq[m][i] = in ? bf_at(p.q, qk + d) : 0.f;
+        rk[m][i] = in ? bf_at(p.k, qk + d) : 0.f;
+        ra[m][i] = in ? bf_at(p.decay, a + d) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < U; ++m) {
+      const int t = tb + 4 * m;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int d = i * 32 + lane, x = t * ROW + d;
+        g_s[x] = t < c.n && d < p.dim ? to_log2 * log_sigmoid_of<__nv_bfloat16>(ra[m][i] + bias[i]) : 0.f;
+        q_s[x] = rq[m][i] * p.q_scale;
+        k_s[x] = rk[m][i];
+      }
+    }
+  }
+  __syncthreads();
+  for (int d = tid; d < D32; d += 128) {
+    float run = 0.f;
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) { run += g_s[t * ROW + d]; g_s[t * ROW + d] = run; }
+  }
+  __syncthreads();
+  // B below and on the diagonal: a warp takes every fourth row, eight columns at a time (those past the diagonal are not stored)
+  for (int t = warp; t < kChunk; t += 4) {
+    float q[NI], g[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) { const int x = t * ROW + i * 32 + lane; q[i] = q_s[x]; g[i] = g_s[x]; }
+#pragma unroll 1
+    for (int s0 = 0; s0 <= t; s0 += 8) {
+      float v[8];
+#pragma unroll
+      for (int m = 0; m < 8; ++m) {
+        float b = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int x = (s0 + m) * ROW + i * 32 + lane;
+          b = fmaf(q[i], k_s[x] * fast_exp2(fminf(g[i] - g_s[x], 0.f)), b);
+        }
+        v[m] = b;
+      }
+      // halving exchanges leave lane groups of four with one sum each
+      const bool up16 = lane & 16, up8 = lane & 8, up4 = lane & 4;
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        const float send = up16 ? v[m] : v[4 + m];
+        v[m] = (up16 ? v[4 + m] : v[m]) + __shfl_xor_sync(0xffffffffu, send, 16);
+      }
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const float send = up8 ? v[m] : v[2 + m];
+        v[m] = (up8 ? v[2 + m] : v[m]) + __shfl_xor_sync(0xffffffffu, send, 8);
+      }
+      {
+        const float send = up4 ? v[0] : v[1];
+        v[0] = (up4 ? v[1] : v[0]) + __shfl_xor_sync(0xffffffffu, send, 4);
+      }
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], 2);
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+      const int sc = s0 + (up16 ? 4 : 0) + (up8 ? 2 : 0) + (up4 ? 1 : 0);
+      if ((lane & 3) == 0 && sc <= t) bm[t][sc] = v[0];
+    }
+  }
+  __syncthreads();
+  if (warp == 0) write_triangle([&](int t, int s) { return bm[t][s]; }, lane, rec + lay.b);
+  for (int d = tid; d < D32; d += 128) {         // a thread owns a key channel: q e^G and k e^{G_16 - G} in place
+    const float g_end = g_s[(kChunk - 1) * ROW + d];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      const float g = g_s[t * ROW + d];
+      q_s[t * ROW + d] *= fast_exp2(g);
+      k_s[t * ROW + d] *= fast_exp2(g_end - g);
+    }
+    if (d < 16 * KS) reinterpret_cast<float*>(rec + lay.extra)[d] = fast_exp2(g_end);
+  }
+  __syncthreads();
+  for (int i = tid; i < KS * 64; i += 128) {
+    const int ln = i & 31, n = (i >> 5) & 1, ks = i >> 6;
+    const float* src = q_s + (n * 8 + (ln >> 2)) * ROW + ks * 16 + (ln & 3) * 2;
+    const float2 x = *reinterpret_cast<const float2*>(src), y = *reinterpret_cast<const float2*>(src + 8);
+    uint4 o;
+    split_pair(x.x, x.y, o.x, o.z);
+    split_pair(y.x, y.y, o.y, o.w);
+    reinterpret_cast<uint4*>(rec)[i] = o;
+  }
+  write_keys(k_s, ROW, KS, rec + lay.k);
+  write_values(v_s, p.vtp * 16, rec + lay.v);
+}
+
+// ---- exponential gates -------------------------------------------------------------------------------------
+template <int KS>
+__global__ void __launch_bounds__(128) exp_chunk_prep(const LinearParams p) {
+  constexpr int DP = 16 * KS, ROW = DP + 2;
+  extern __shared__ __align__(16) float sm[];
+  float* k_s = sm;                               // [16][ROW], scaled
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(k_s + kChunk * ROW);
+  __shared__ float part[4][kChunk][kChunk + 1], e_s[kChunk], top_s[kChunk];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const ChunkSite c = chunk_site(p, blockIdx.x);
+  if (c.n <= 0) return;
+  const LinearLayout lay = linear_layout(KS, p.vtp, true);
+  uint8_t* rec = p.records + (static_cast<int64_t>(blockIdx.x) * p.heads + h) * lay.total;
+  if (tid == 0 && c.row == p.cu[c.seq]) stash_maximum(p, c.seq, h);
+  stage_values(p, c, h, p.vtp * 16, p.vdim, v_s);
+  // gates, every warp for itself (lanes 0..15): F, the running maximum of i - F, and with them M, all in log2 units
+  float f = 0.f, i = -INFINITY;
+  if (lane < c.n) {
+    f = log_forget<__nv_bfloat16>(p, c.row + lane, h) * kLog2e;
+    i = log_input<__nv_bfloat16>(p, c.row + lane, h) * kLog2e;
+  }
+#pragma unroll
+  for (int off = 1; off < kChunk; off <<= 1) {
+    const float x = __shfl_up_sync(0xffffffffu, f, off);
+    if (lane >= off) f += x;
+  }
+  const float e = i - f;                         // -inf behind the last token
+  float top = e;
+#pragma unroll
+  for (int off = 1; off < kChunk; off <<= 1) {
+    const float x = __shfl_up_sync(0xffffffffu, top, off);
+    if (lane >= off) top = fmaxf(top, x);
+  }
+  if (warp == 0 && lane < kChunk) {
+    e_s[lane] = e; top_s[lane] = top;
+    reinterpret_cast<float*>(rec + lay.extra)[lane] = f;
+    reinterpret_cast<float*>(rec + lay.extra)[kChunk + lane] = f + top;
+  }
+  const float key_w = fast_exp2(e - __shfl_sync(0xffffffffu, top, kChunk - 1));      // lane s: e^{F_16 - F_s + i_s - M_16}
+  // q . k: a warp takes every fourth 16-channel step.  The second operand of (.) q^T is the first operand of q k^T with its
+  // middle registers exchanged
+  float acc[2][4];
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[n][j] = 0.f;
+  const bool pairs = p.dim % 2 == 0 && p.qkv_stride % 2 == 0 && ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k)) & 3) == 0;
+  auto two = [&](const void* base, int t, int d) -> uint32_t {
+    if (t >= c.n || d >= p.dim) return 0u;
+    const uint16_t* x = static_cast<const uint16_t*>(base) + (c.row + t) * p.qkv_stride + static_cast<int64_t>(h) * p.dim + d;
+    if (pairs) return *reinterpret_cast<const uint32_t*>(x);
+    return static_cast<uint32_t>(x[0]) | (d + 1 < p.dim ? static_cast<uint32_t>(x[1]) << 16 : 0u);
+  };
+  const float w0 = __shfl_sync(0xffffffffu, key_w, lane >> 2), w1 = __shfl_sync(0xffffffffu, key_w, (lane >> 2) + 8);
+#pragma unroll
+  for (int ks = warp; ks < KS; ks += 4) {
+    const int t = lane >> 2, d = ks * 16 + (lane & 3) * 2;
+    const uint2 q0 = make_uint2(two(p.q, t, d), two(p.q, t, d + 8)), q1 = make_uint2(two(p.q, t + 8, d), two(p.q, t + 8, d + 8));
+    const uint2 k0 = make_uint2(two(p.k, t, d), two(p.k, t, d + 8)), k1 = make_uint2(two(p.k, t + 8, d), two(p.k, t + 8, d + 8));
+    reinterpret_cast<uint2*>(rec)[(ks * 2) * 32 + lane] = q0;
+    reinterpret_cast<uint2*>(rec)[(ks * 2 + 1) * 32 + lane] = q1;
+    const uint32_t a[4] = {q0.x, q1.x, q0.y, q1.y};
+    mma_bf16_16816(acc[0], a, k0.x, k0.y);
+    mma_bf16_16816(acc[1], a, k1.x, k1.y);
+    float* row0 = k_s + t * ROW + d;
+    float* row1 = row0 + 8 * ROW;
+    *reinterpret_cast<float2*>(row0) = make_float2(bf16_lo(k0.x) * w0, bf16_hi(k0.x) * w0);
+    *reinterpret_cast<float2*>(row0 + 8) = make_float2(bf16_lo(k0.y) * w0, bf16_hi(k0.y) * w0);
+    *reinterpret_cast<float2*>(row1) = make_float2(bf16_lo(k1.x) * w1, bf16_hi(k1.x) * w1);
+    *reinterpret_cast<float2*>(row1 + 8) = make_float2(bf16_lo(k1.y) * w1, bf16_hi(k1.y) * w1);
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) part[warp][(lane >> 2) + (j >> 1) * 8][n * 8 + (lane & 3) * 2 + (j & 1)] = acc[n][j];
+  __syncthreads();
+  if (warp == 0)
+    write_triangle([&](int t, int s) {
+      const float dot = (part[0][t][s] + part[1][t][s]) + (part[2][t][s] + part[3][t][s]);
+      return dot * p.q_scale * fast_exp2(e_s[s] - top_s[t]);
+    }, lane, rec + lay.b);
+  write_keys(k_s, ROW, KS, rec + lay.k);
+  write_values(v_s, p.vtp * 16, rec + lay.v);
+}
+
+// ---- the recurrence over chunks ------------------------------------------------------------------------------
+template <bool EXP, int KS, int WARPS>
+struct LinearScanCfg {
+  static constexpr int STAGES = 3;
+  static constexpr int SHARED = KS * (EXP ? 512 : 1024) + KS * 1024 + 1024 + (EXP ? 128 : KS * 64);
+  static constexpr int STAGE = SHARED + WARPS * 512;           // common part + a tile of values per warp
+  static constexpr int SMEM = STAGES * STAGE + 64;
+  static_assert(STAGE % 16 == 0, "stages start at multiples of 16 bytes");
+};
+
+template <bool EXP, int KS, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearParams p) {
+  using C = LinearScanCfg<EXP, KS, WARPS>;
+  extern __shared__ __align__(128) uint8_t smem[];
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::STAGES * C::STAGE);
+  const int s = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin;
+  if (n_tok <= 0) return;
+  const int n_chunks = (n_tok + kChunk - 1) / kChunk, vt = blockIdx.x * WARPS + warp;
+  const LinearLayout lay = linear_layout(KS, p.vtp, EXP);
+  const uint8_t* rec = p.records + (static_cast<int64_t>(chunk_base(begin, s)) * p.heads + h) * lay.total;
+  const int64_t rec_step = static_cast<int64_t>(p.heads) * lay.total;
+  if (tid == 0) {
+    for (int i = 0; i < C::STAGES; ++i) mbar_init(&full[i], 1);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  auto fetch = [&](int c) {                       // one thread
+    const int st = c % C::STAGES;
+    const uint8_t* src = rec + c * rec_step;
+    const uint32_t dst = smem_u32(smem + st * C::STAGE), bar = smem_u32(&full[st]);
+    mbar_arrive_expect_tx(&full[st], C::STAGE);
+    bulk_copy(dst, src, C::SHARED, bar);
+    bulk_copy(dst + C::SHARED, src + lay.v + blockIdx.x * (WARPS * 512), WARPS * 512, bar);
+  };
+  if (tid == 0)
+    for (int c = 0; c < min(C::STAGES, n_chunks); ++c) fetch(c);
+
+  const int64_t slot = linear_slot(p, s), hbase = (slot * p.heads + h) * static_cast<int64_t>(p.dim);
+  const bool fresh = slot < 0 || p.positions[begin] == 0;
+  const int v0 = vt * 16 + (lane >> 2), dq = (lane & 3) * 2, cols = p.vdim + (EXP ? 1 : 0);
+  float S[2 * KS][4];                             // S^T: rows v0, v0 + 8; columns 8 j + dq, + 1
+  auto state_at = [&](int j, int i) -> float* {
+    const int64_t row = hbase + 8 * j + dq + (i & 1);
+    const int v = v0 + (i & 2) * 4;
+    return EXP && v == p.vdim ? p.n + row : p.S + row * p.vp + v;
+  };
+  auto in_state = [&](int j, int i) { return 8 * j + dq + (i & 1) < p.dim && v0 + (i & 2) * 4 < cols; };
+#pragma unroll
+  for (int j = 0; j < 2 * KS; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) S[j][i] = !fresh && in_state(j, i) ? *state_at(j, i) : 0.f;
+  float m = EXP ? p.m0[s * p.heads + h] * kLog2e : 0.f;
+  const bool keeps_m = EXP && blockIdx.x == 0 && warp == 0;
+
+  bool ok = true;
+  int c = 0;
+  for (; c < n_chunks; ++c) {
+    const int st = c % C::STAGES;
+    ok = mbar_wait(&full[st], (c / C::STAGES) & 1);
+    if (!__syncthreads_and(ok)) break;            // (uniform: every thread leaves together)
+    const uint8_t* base = smem + st * C::STAGE;
+    const uint4* k_r = reinterpret_cast<const uint4*>(base + lay.k);
+    const uint4* b_r = reinterpret_cast<const uint4*>(base + lay.b);
+    const float* extra = reinterpret_cast<const float*>(base + lay.extra);
+    const uint4 vw = reinterpret_cast<const uint4*>(base + C::SHARED)[warp * 32 + lane];
+    const uint32_t v[4] = {vw.x, vw.y, vw.z, vw.w};
+    float row_f[2][2], row_b[2][2], alpha = 1.f, beta = 1.f, m_end = 0.f;
+    if constexpr (EXP) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int t = n * 8 + dq + i;
+          const float from0 = extra[t] + m, local = extra[kChunk + t], mt = fmaxf(from0, local);
+          row_f[n][i] = p.q_scale * fast_exp2(from0 - mt);
+          row_b[n][i] = fast_exp2(local - mt);
+          if (keeps_m && lane < 4 && c * kChunk + t < n_tok) p.mt[static_cast<int64_t>(begin + c * kChunk + t) * p.heads + h] = mt * kLn2;
+        }
+      const float from0 = extra[kChunk - 1] + m, local = extra[2 * kChunk - 1];
+      m_end = fmaxf(from0, local);
+      alpha = fast_exp2(from0 - m_end); beta = fast_exp2(local - m_end);
+    }
+    float oa[2][4], ob[2][4], oc[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) oa[n][i] = ob[n][i] = oc[n][i] = 0.f;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {                 // V^T B^T
+      const uint4 b = b_r[n * 32 + lane];
+      mma_bf16_16816(oc[n], v, b.x, b.y);
+      mma_bf16_16816(oc[n], v, b.z, b.w);
+    }
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {             // S0^T Q^T
+      Split a;
+      split_tile(S[2 * ks], S[2 * ks + 1], a);
+      if constexpr (EXP) {
+        const uint2* q_r = reinterpret_cast<const uint2*>(base);
+        const uint2 q0 = q_r[(ks * 2) * 32 + lane], q1 = q_r[(ks * 2 + 1) * 32 + lane];
+        mma_bf16_16816(oa[0], a.hi, q0.x, q0.y); mma_bf16_16816(oa[1], a.hi, q1.x, q1.y);
+        mma_bf16_16816(ob[0], a.lo, q0.x, q0.y); mma_bf16_16816(ob[1], a.lo, q1.x, q1.y);
+      } else {
+        const uint4* q_r = reinterpret_cast<const uint4*>(base);
+        const uint4 q0 = q_r[(ks * 2) * 32 + lane], q1 = q_r[(ks * 2 + 1) * 32 + lane];
+        mma_bf16_16816(oa[0], a.hi, q0.x, q0.y); mma_bf16_16816(oa[1], a.hi, q1.x, q1.y);
+        mma_bf16_16816(ob[0], a.hi, q0.z, q0.w); mma_bf16_16816(ob[1], a.hi, q1.z, q1.w);
+        mma_bf16_16816(ob[0], a.lo, q0.x, q0.y); mma_bf16_16816(ob[1], a.lo, q1.x, q1.y);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 2 * KS; ++j) {            // S^T <- S^T decay + V^T K
+      const uint4 k = k_r[j * 32 + lane];
+      if constexpr (EXP) {
+        float d[4] = {0.f, 0.f, 0.f, 0.f};
+        mma_bf16_16816(d, v, k.x, k.y);
+        mma_bf16_16816(d, v, k.z, k.w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) S[j][i] = fmaf(beta, d[i], alpha * S[j][i]);
+      } else {
+        const float2 g = *reinterpret_cast<const float2*>(extra + 8 * j + dq);
+        S[j][0] *= g.x; S[j][1] *= g.y; S[j][2] *= g.x; S[j][3] *= g.y;
+        mma_bf16_16816(S[j], v, k.x, k.y);
+        mma_bf16_16816(S[j], v, k.z, k.w);
+      }
+    }
+    m = m_end;
+    __syncthreads();                              // the stage has been read
+    if (tid == 0 && c + C::STAGES < n_chunks) { fence_proxy_async(); fetch(c + C::STAGES); }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = c * kChunk + n * 8 + dq + (i & 1), col = v0 + (i & 2) * 4;
+        if (t >= n_tok) continue;
+        const int64_t th = static_cast<int64_t>(begin + t) * p.heads + h;
+        const float o = EXP ? fmaf(row_f[n][i & 1], oa[n][i] + ob[n][i], row_b[n][i & 1] * oc[n][i]) : (oa[n][i] + ob[n][i]) + oc[n][i];
+        if (col < p.vdim) p.o[th * p.vdim + col] = o;
+        else if (EXP && col == p.vdim) p.nq[th] = o;
+      }
+  }
+  if (c < n_chunks) {                             // a copy did not arrive in time: report it, let those in flight land, keep the old state
+    if (!ok) report(p.dev_status, kDevWaitTimeout, c);
+    for (int k = c; k < min(c + C::STAGES, n_chunks); ++k) mbar_wait(&full[k % C::STAGES], (k / C::STAGES) & 1, 1u << 16);
+    return;
+  }
+  if (slot < 0) return;
+  if (keeps_m && lane == 0) p.m[slot * p.heads + h] = m * kLn2;
+#pragma unroll
+  for (int j = 0; j < 2 * KS; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (in_state(j, i)) *state_at(j, i) = S[j][i];
+}
+
+template <bool EXP, int KS>
+static int launch_linear_chunks(const LinearParams& p, cudaStream_t st) {
+  constexpr int D32 = (16 * KS + 31) / 32 * 32;
+  const size_t smem = (EXP ? kChunk * (16 * KS + 2) : 3 * kChunk * (D32 + 4)) * sizeof(float) + static_cast<size_t>(p.vtp) * 16 * kChunk * 2;
+  if (smem > 200 * 1024) return kUnsupportedShape;
+  const int slots = p.tokens / kChunk + p.num_seqs;
+  struct PrepTag {};
+  auto prep = EXP ? &exp_chunk_prep<KS> : &decay_chunk_prep<KS>;
+  const int rc = opt_in_dynamic_smem<PrepTag>(reinterpret_cast<const void*>(prep), smem);
+  if (rc != kOk) return rc;
+  prep<<<dim3(slots, p.heads), 128, smem, st>>>(p);
+  if (cudaGetLastError() != cudaSuccess) return kLaunchFailed;
+  auto scan = [&](auto tag) -> int {
+    constexpr int WARPS = decltype(tag)::value;
+    using C = LinearScanCfg<EXP, KS, WARPS>;
+    struct ScanTag {};
+    const int r = opt_in_dynamic_smem<ScanTag>(reinterpret_cast<const void*>(&linear_chunk_scan<EXP, KS, WARPS>), C::SMEM);
+    if (r != kOk) return r;
+    linear_chunk_scan<EXP, KS, WARPS><<<dim3(p.vtp / WARPS, p.heads, p.num_seqs), WARPS * 32, C::SMEM, st>>>(p);
+    return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+  };
+  switch (linear_warps(p, EXP)) {
+    case 1: return scan(std::integral_constant<int, 1>{});
+    case 2: return scan(std::integral_constant<int, 2>{});
+    case 3: return scan(std::integral_constant<int, 3>{});
+    default: return scan(std::integral_constant<int, 4>{});
+  }
+}
+
+}  // namespace mvb

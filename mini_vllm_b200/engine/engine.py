@@ -38,6 +38,10 @@ class Engine:
         self.metrics = Metrics()
 
     def submit(self, tokens: list[int], sampling_params: SamplingParams) -> Request:
+        limit = getattr(getattr(self.config, "hf_config", None), "learned_positions", None)      # a position table has an end (the last token needs none)
+        if limit is not None and len(tokens) + sampling_params.max_tokens - 1 > limit:
+            raise ValueError(f"{len(tokens)} prompt tokens and {sampling_params.max_tokens} new ones need more than the model's "
+                             f"{limit} positions")
         req = Request(tokens, sampling_params)
         self.scheduler.submit(req)
         return req

@@ -77,8 +77,10 @@ class Executor:
         if not self.recurrent:
             config.num_state_slots = None
         self.attention_layers = [m for m in self.model.modules() if hasattr(m, "k_cache") and hasattr(m, "v_cache")]
+        self.latent_layers = [m for m in self.model.modules() if hasattr(m, "latent_cache")]     # (those with latents of their own)
         self.item_rows = 0                     # query-block size of the prefill kernel's work items for this model
-        for m in self.attention_layers[:1]:    # (a head layout the kernel does not take: no list, the plain grid)
+        for m in (self.attention_layers + self.latent_layers)[:1]:
+            # (a head layout the kernel does not take: no list, the plain grid)
             if m.head_dim in (128, 256) and config.hf_config.dtype == torch.bfloat16:
                 self.item_rows = ops.prefill_item_rows(m.num_heads, m.num_kv_heads, m.head_dim)
         self.h2d_bytes = 0                   # bytes uploaded by the packing path (for the bench's e2e line)
@@ -112,15 +114,17 @@ class Executor:
 
     def _init_kv_cache(self) -> None:
         """Pool ``[2, layers, blocks, block_size, kv_heads, head_dim]``; layer l's K is ``[0, l]`` (executor.py:31-60).
-        Attention layers of unequal shapes get a ``[2, blocks, ...]`` pool each, all of the same number of blocks."""
+        Attention layers of unequal shapes get a ``[2, blocks, ...]`` pool each, all of the same number of blocks; layers that cache
+        a latent instead of keys and values get ``[blocks, block_size, width]``, served by the same block tables."""
         cfg, hf = self.config, self.config.hf_config
         free, total = torch.cuda.mem_get_info()
         stats = torch.cuda.memory_stats()
         peak, current = stats["allocated_bytes.all.peak"], stats["allocated_bytes.all.current"]
         shapes = [(m.num_kv_heads, m.head_dim) for m in self.attention_layers]
-        block_bytes = 2 * self.block_size * sum(h * d for h, d in shapes) * hf.dtype.itemsize
+        per_token = 2 * sum(h * d for h, d in shapes) + sum(m.latent_width for m in self.latent_layers)
+        block_bytes = self.block_size * per_token * hf.dtype.itemsize
         room = int(total * cfg.gpu_memory_utilization - (total - free) - peak + current)
-        fit = room // block_bytes if shapes else cfg.kv_cache_num_blocks
+        fit = room // block_bytes if block_bytes else cfg.kv_cache_num_blocks
         if fit <= 0:
             raise RuntimeError("no memory left for the KV cache")
         cfg.kv_cache_num_blocks = min(fit, cfg.kv_cache_num_blocks)
@@ -135,6 +139,8 @@ class Executor:
         log.info("allocated %d KV blocks", cfg.kv_cache_num_blocks)
         for module, (k, v) in zip(self.attention_layers, layers):
             module.k_cache, module.v_cache = k, v
+        for module in self.latent_layers:
+            module.latent_cache = pool(cfg.kv_cache_num_blocks, self.block_size, module.latent_width)
 
     # ---- packing ---------------------------------------------------------------------------------
     @staticmethod
@@ -188,7 +194,7 @@ class Executor:
                       max_seqlen_q=int(q_len.max()), max_seqlen_k=int(seq_len.max()),
                       block_table=out["block_table"], status=self.status,
                       prefill_items=meta[meta.numel() - items.size:].view(-1, 2) if items.size else None,
-                      prefill_item_rows=self.item_rows, state_slots=state_slots)
+                      prefill_item_rows=self.item_rows, state_slots=state_slots, prompt_keys=int(seq_len.sum()))
         return out["input_ids"], ctx
 
     def _prefill_items(self, q_len: np.ndarray, seq_len: np.ndarray) -> np.ndarray:
@@ -224,7 +230,7 @@ class Executor:
                       max_seqlen_k=int(seq_len.max()), block_table=out["block_table"], num_decode=num_decode,
                       cache_seqlens=(cu_k[bp + 1:] - cu_k[bp:-1]).contiguous(), status=self.status,
                       prefill_items=meta[items_end - items.size:items_end].view(-1, 2) if items.size else None,
-                      prefill_item_rows=self.item_rows, state_slots=state_slots)
+                      prefill_item_rows=self.item_rows, state_slots=state_slots, prompt_keys=int(seq_len[:bp].sum()))
         if slots is None:
             return out["input_ids"], ctx
         return out["input_ids"], ctx, meta[meta.numel() - b:]
@@ -336,7 +342,8 @@ class Executor:
             ctx = Context(prefill=True, positions=out["positions"], cu_seqlens_q=out["cu_seqlens_q"],
                           cu_seqlens_k=out["cu_seqlens_k"], slot_mapping=out["slot_mapping"],
                           max_seqlen_q=int(q_len.max()), max_seqlen_k=int(seq_len.max()),
-                          block_table=out["block_table"], status=self.status, state_slots=state_slots)
+                          block_table=out["block_table"], status=self.status, state_slots=state_slots,
+                          prompt_keys=int(seq_len.sum()))
             input_ids = out["input_ids"]
         elif batch.type == Batch.MIXED:                # (its decode inputs come from Request.tokens: the caller has
             input_ids, ctx, slots_dev = self._build_mixed_input(reqs, batch.num_decode, slots)   # resolved them)

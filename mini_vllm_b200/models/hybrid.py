@@ -1,13 +1,14 @@
-"""Decoder assembled layer by layer from mixer branches (attention, selective scan, gated delta rule), with norms before
-and after each sublayer, an fp32 residual stream, and optional tanh caps on the logits.
+"""Decoder assembled layer by layer from mixer branches (attention, latent attention, selective scan, gated delta rule, gated linear
+attention, matrix-memory LSTM), a feed-forward of its own kind, and an fp32 residual of its own kind (``layers/residual.py``), with
+optional tanh caps on the logits.
 
 The step contract is ``DecoderLM``'s (``models/decoder.py``): ``forward(ctx, input_ids, positions, head)``, one row per
 sequence - or per entry of ``ctx.logit_rows`` - and the same loader, executor, KV pool, CUDA graphs and sampler.  Recurrent
 branches keep a row of state per sequence in slots that the scheduler hands out with the KV blocks; a sequence whose
 first token of a step has position 0 starts from zero, so a reused slot needs no clearing.
 
-Per sublayer the kernels are: input GEMM, branch kernels, output GEMM, and one kernel for [norm of the branch output +
-residual add + norm for the next sublayer].
+Per sublayer the kernels are: input GEMM, branch kernels, output GEMM, and one kernel for everything between the sublayer's output
+and the normalised input of the next one.
 """
 from __future__ import annotations
 
@@ -19,7 +20,7 @@ from torch import nn
 
 from .. import ops
 from ..executor.context import Context
-from .layers.branches import PackedMixer, pad8, pad_cols, pad_rows, weight
+from .layers.branches import PackedMixer, Weights, pad8, pad_cols, pad_rows, weight, weight_f32
 
 
 class ClampedGLU(nn.Module):
@@ -31,41 +32,59 @@ class ClampedGLU(nn.Module):
         self.gate_up, self.down = weight(2 * self.ip, width), weight(width, self.ip)
 
     @torch.no_grad()
-    def load(self, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> None:
-        self.gate_up.copy_(torch.cat([pad_rows(gate, self.ip), pad_rows(up, self.ip)]))
-        self.down.copy_(pad_cols(down, self.ip))
+    def load(self, w: Weights) -> None:
+        self.gate_up.copy_(torch.cat([pad_rows(w("gate"), self.ip), pad_rows(w("up"), self.ip)]))
+        self.down.copy_(pad_cols(w("down"), self.ip))
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         return F.linear(ops.clamped_glu(F.linear(h, self.gate_up), self.ip, self.limit, self.alpha), self.down)
 
 
-class HybridLayer(nn.Module):
-    """A mixer and, optionally, a feed-forward; each between a norm of its input and a norm of its output."""
+class PolyNormMLP(nn.Module):
+    """``down(a N(z) + b N(z^2) + c N(z^3) + e)`` with ``z = up(h)``, N over the row's root mean square, and four learned numbers."""
 
-    def __init__(self, width: int, mixer: PackedMixer, mlp: nn.Module | None):
+    def __init__(self, width: int, inter: int, eps: float):
+        super().__init__()
+        self.inter, self.ip, self.eps = inter, pad8(inter), eps
+        self.up, self.down, self.act = weight(self.ip, width), weight(width, self.ip), weight_f32(4)
+
+    @torch.no_grad()
+    def load(self, w: Weights) -> None:
+        self.up.copy_(pad_rows(w("up"), self.ip))
+        self.down.copy_(pad_cols(w("down"), self.ip))
+        self.act.copy_(w("act"))
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        return F.linear(ops.poly_norm(F.linear(h, self.up), self.inter, self.act, self.eps), self.down)
+
+
+class HybridLayer(nn.Module):
+    """A mixer and, optionally, a feed-forward, each with its connection to the residual stream."""
+
+    def __init__(self, stream: nn.Module, mixer: PackedMixer, mlp: nn.Module | None):
         super().__init__()
         self.mixer, self.mlp = mixer, mlp
-        for name in ("norm1", "norm1b") + (("norm2", "norm2b") if mlp is not None else ()):
-            self.register_parameter(name, nn.Parameter(torch.ones(width), requires_grad=False))
+        self.connections = nn.ModuleList([stream.connection() for _ in range(1 if mlp is None else 2)])
 
     def sublayers(self):
-        """(input norm, callable(ctx, h, positions), output norm) in order."""
-        yield self.norm1, self.mixer, self.norm1b
+        """(connection, callable(ctx, h, positions)) in order."""
+        yield self.connections[0], self.mixer
         if self.mlp is not None:
-            yield self.norm2, (lambda ctx, h, positions: self.mlp(h)), self.norm2b
+            yield self.connections[1], lambda ctx, h, positions: self.mlp(h)
 
 
 class HybridDecoder(nn.Module):
-    recurrent = False          # set by subclasses with recurrent branches: the scheduler hands out state slots
-
-    def __init__(self, cfg, layers: list[HybridLayer]):
+    def __init__(self, cfg, layers: list[HybridLayer], stream: nn.Module):
         super().__init__()
         self.config, self.eps = cfg, cfg.rms_norm_eps
         self.logit_cap = float(getattr(cfg, "logit_softcap", None) or 0.0)
         self.embed_tokens = weight(cfg.vocab_size, cfg.hidden_size)
+        self.stream = stream
         self.layers = nn.ModuleList(layers)
         self.norm = nn.Parameter(torch.ones(cfg.hidden_size), requires_grad=False)
         self.lm_head_weight = weight(cfg.vocab_size, cfg.hidden_size)
+        # with recurrent branches the scheduler hands out state slots
+        self.recurrent = any(b.state_specs(torch.float32) for layer in layers for b in layer.mixer.branches.values())
         self.residual_tap = None          # debugging aid: called with (layer index, residual stream) after each layer
 
     # ---- step ----------------------------------------------------------------------------------
@@ -81,19 +100,20 @@ class HybridDecoder(nn.Module):
 
     def _hidden_rows(self, ctx: Context, input_ids: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
         steps = [(i, *sub) for i, layer in enumerate(self.layers) for sub in layer.sublayers()]
-        x, h = ops.embed_norm(input_ids, self.embed_tokens, steps[0][1], self.eps, status=ctx.status)
+        x, h = self.stream.start(ctx, input_ids, positions, self.embed_tokens, steps[0][1])
         rows = None
         if ctx.prefill:
             rows = ctx.logit_rows if ctx.logit_rows is not None else ctx.cu_seqlens_q
-        for n, (i, _, run, out_norm) in enumerate(steps):
-            last = n == len(steps) - 1
+        for n, (i, connection, run) in enumerate(steps):
             y = run(ctx, h, positions)
+            last = n == len(steps) - 1
+            following = None if last else steps[n + 1][1]
             if last and self.residual_tap is None:
                 # the head reads a few rows: the closing add + final norm gather those themselves
-                return ops.residual_norm(x, y, self.norm, self.eps, y_weight=out_norm, row_ends=rows)
-            h = ops.residual_norm(x, y, self.norm if last else steps[n + 1][1], self.eps, y_weight=out_norm)
+                return self.stream.advance(x, y, connection, None, self.norm, rows)
+            h = self.stream.advance(x, y, connection, following, self.norm)
             if self.residual_tap is not None and (last or steps[n + 1][0] != i):
-                self.residual_tap(i, x)
+                self.residual_tap(i, self.stream.total(x))
         return h if rows is None else h[(rows[1:] - 1).long()]
 
     def logits(self, hidden_rows: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
@@ -141,13 +161,14 @@ class HybridDecoder(nn.Module):
         self.embed_tokens.copy_(w("embed"))
         self.norm.copy_(w("final.norm"))
         self.lm_head_weight.copy_(w("head"))
+        self.stream.load(w)
         for i, layer in enumerate(self.layers):
             p = f"l{i}."
             layer.mixer.load(self.mixer_prefixes(i), w)
-            layer.norm1.copy_(w(p + "norm1")); layer.norm1b.copy_(w(p + "norm1b"))
+            for q, connection in enumerate(layer.connections, 1):
+                connection.load(p, q, w)
             if layer.mlp is not None:
-                layer.norm2.copy_(w(p + "norm2")); layer.norm2b.copy_(w(p + "norm2b"))
-                layer.mlp.load(w(p + "mlp.gate"), w(p + "mlp.up"), w(p + "mlp.down"))
+                layer.mlp.load(lambda n, p=p: w(p + "mlp." + n))
         unknown = set(tensors) - used
         if unknown:
             raise KeyError(f"unrecognised parameter {sorted(unknown)[0]}")

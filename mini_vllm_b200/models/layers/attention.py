@@ -26,9 +26,8 @@ _workspaces: dict = {}
 _superseded: list = []      # outgrown buffers stay allocated: captured CUDA graphs keep writing through their pointers
 
 
-def _decode_workspace(device, max_seqs: int, num_heads: int, num_kv_heads: int, head_dim: int,
-                      window_left: int) -> torch.Tensor:
-    """One scratch buffer per (device, head shape, window); a larger one takes its place when a larger batch
+def decode_workspace_for(device, max_seqs: int, num_heads: int, num_kv_heads: int, head_dim: int, window_left) -> torch.Tensor:
+    """One scratch buffer per (device, head shape, window or kind of attention); a larger one takes its place when a larger batch
     arrives.  The smaller buffer is never freed: a graph captured while it was current has its address
     baked in, and a replay after the memory went back to the allocator would scribble over someone else."""
     key = (device, num_heads, num_kv_heads, head_dim, window_left)
@@ -43,6 +42,15 @@ def _decode_workspace(device, max_seqs: int, num_heads: int, num_kv_heads: int, 
         ws = ops.decode_workspace(max(max_seqs, 512), num_heads, head_dim, device)
         _workspaces[key] = ws
     return ws
+
+
+def prefill_items_for(ctx: Context, layer):
+    """The step's prefill work list, if the packing step built one for the layer's query-block size."""
+    if ctx.prefill_items is None:
+        return None
+    if layer._item_rows is None:
+        layer._item_rows = ops.prefill_item_rows(layer.num_heads, layer.num_kv_heads, layer.head_dim)
+    return ctx.prefill_items if ctx.prefill_item_rows == layer._item_rows else None
 
 
 class FlashAttention(nn.Module):
@@ -110,20 +118,12 @@ class FlashAttention(nn.Module):
                                   k_in_place=ctx.prefill and ctx.block_table is None, status=ctx.status)
         return self._attend(ctx, q, k, v)
 
-    def _items(self, ctx: Context):
-        """The step's prefill work list, if the packing step built one for this layer's query-block size."""
-        if ctx.prefill_items is None:
-            return None
-        if self._item_rows is None:
-            self._item_rows = ops.prefill_item_rows(self.num_heads, self.num_kv_heads, self.head_dim)
-        return ctx.prefill_items if ctx.prefill_item_rows == self._item_rows else None
-
     def _decode(self, ctx: Context, q: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
         wl = self.window_left
         key = (wl, self.num_heads, self.num_kv_heads, self.head_dim)
         ws = ctx.decode_plans.get(key)
         if ws is None:
-            ws = _decode_workspace(q.device, ctx.cache_seqlens.numel(), self.num_heads, self.num_kv_heads, self.head_dim, wl)
+            ws = decode_workspace_for(q.device, ctx.cache_seqlens.numel(), self.num_heads, self.num_kv_heads, self.head_dim, wl)
             ops.decode_plan(ctx.cache_seqlens, wl, self.num_heads, self.num_kv_heads, self.head_dim, ws,
                             block_table=table, block_size=self.k_cache.shape[1])
             ctx.decode_plans[key] = ws
@@ -132,7 +132,7 @@ class FlashAttention(nn.Module):
 
     def _prefill(self, ctx: Context, q, k, v, cu_q, cu_k, table, out=None) -> torch.Tensor:
         return ops.prefill_attn(q, k, v, cu_q, cu_k, ctx.max_seqlen_q, self.scaling, self.window_left, block_table=table,
-                                out=out, status=ctx.status, items=self._items(ctx), softcap=self.softcap,
+                                out=out, status=ctx.status, items=prefill_items_for(ctx, self), softcap=self.softcap,
                                 out_scale=self.out_scale)
 
     def _attend_mixed(self, ctx: Context, q: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:

@@ -1,6 +1,7 @@
 """Mixer branches for decoders whose layers are assembled from parts.
 
-A branch is one token mixer (attention, selective scan, gated delta rule) without its outer projections: it declares how
+A branch is one token mixer (attention, latent attention, selective scan, gated delta rule, gated linear attention, matrix-memory
+LSTM) without its outer projections: it declares how
 many rows it needs in the layer's packed input projection and how many columns it brings to the packed output
 projection, and works between the two.  ``PackedMixer`` puts any number of branches side by side on the same input: ONE
 input GEMM over the concatenated rows, the branches, ONE output GEMM over the concatenated columns, which also adds the
@@ -21,7 +22,7 @@ from torch import nn
 
 from ... import ops
 from ...executor.context import Context
-from .attention import FlashAttention
+from .attention import FlashAttention, decode_workspace_for, prefill_items_for
 from .rotary import RotaryEmbedding
 
 LOG2E = 1.0 / math.log(2.0)
@@ -211,6 +212,190 @@ class GatedDeltaBranch(Branch):
         ops.gated_delta(q, k, v, low[:, :h * self.dim], proj[:, c:c + h], low[:, self.hp:self.hp + h * self.vdim], self.exp_a,
                         self.dt_bias, self.norm_weight, out[:, :h * self.vdim].unflatten(1, (h, self.vdim)), self.delta_state,
                         ctx.state_slots, cu, positions, self.dim ** -0.5, self.eps, self.factor, status=ctx.status)
+
+
+class GatedLinearBranch(Branch):
+    """Linear attention with a decay per head and key channel, ``sigmoid(z)^(1/tau)`` with z from a low-rank pair, and a SiLU-gated
+    output norm."""
+
+    def __init__(self, heads: int, dim: int, vdim: int, tau: float, decay_rank: int, eps: float):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.tau, self.eps, self.decay_rank = heads, dim, vdim, tau, eps, decay_rank
+        self.kp, self.vp, self.ap = pad8(heads * dim), pad8(heads * vdim), pad8(decay_rank)
+        self.in_rows = 2 * self.kp + 2 * self.vp + self.ap                    # q | k | v | gate | decay
+        self.out_cols, self.out_used = self.vp, heads * vdim
+        self.decay_up = weight(self.kp, self.ap)
+        self.decay_bias, self.norm_weight = weight_f32(heads * dim), weight_f32(vdim)
+        self.memory = None
+
+    def state_specs(self, dtype):
+        return {"memory": ((self.heads, self.dim, -(-self.vdim // 4) * 4), torch.float32)}
+
+    def load(self, w: Weights):
+        self.decay_up.copy_(pad_cols(pad_rows(w("a2"), self.kp), self.ap))
+        self.decay_bias.copy_(w("a2.b").float().reshape(-1))
+        self.norm_weight.copy_(w("norm").float())
+        rows = [pad_rows(w(n), c) for n, c in (("q", self.kp), ("k", self.kp), ("v", self.vp), ("g", self.vp), ("a1", self.ap))]
+        return torch.cat(rows), pad_cols(w("o"), self.out_cols)
+
+    def forward(self, ctx, proj, out, positions):
+        q, k, v, gate, a = proj.split([self.kp, self.kp, self.vp, self.vp, self.ap], dim=1)
+        nk, nv = self.heads * self.dim, self.heads * self.vdim
+        decay = F.linear(a, self.decay_up)
+        q, k = (t[:, :nk].unflatten(1, (self.heads, self.dim)) for t in (q, k))
+        v, o = (t[:, :nv].unflatten(1, (self.heads, self.vdim)) for t in (v, out))
+        ops.gated_linear(q, k, v, decay[:, :nk], self.decay_bias, self.tau, gate[:, :nv], self.norm_weight, o, self.memory,
+                         ctx.state_slots, ragged(ctx), positions, self.dim ** -0.5, self.eps, status=ctx.status)
+
+
+class MatrixLSTMBranch(Branch):
+    """Matrix memory with exponential gates per head, a normaliser and a running maximum of the exponents, and a sigmoid-gated output
+    norm with a weight per head."""
+
+    def __init__(self, heads: int, dim: int, vdim: int, gate_cap: float, eps: float):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.cap, self.eps = heads, dim, vdim, gate_cap, eps
+        self.kp, self.vp, self.hp = pad8(heads * dim), pad8(heads * vdim), pad8(heads)
+        self.in_rows = 2 * self.kp + 2 * self.vp + 2 * self.hp                # q | k | v | output gate | input gate | forget gate
+        self.out_cols, self.out_used = self.vp, heads * vdim
+        self.input_bias, self.forget_bias, self.norm_weight = weight_f32(heads), weight_f32(heads), weight_f32(heads * vdim)
+        self.memory = self.normaliser = self.maximum = None
+
+    def state_specs(self, dtype):
+        return {"memory": ((self.heads, self.dim, -(-self.vdim // 4) * 4), torch.float32),
+                "normaliser": ((self.heads, self.dim), torch.float32), "maximum": ((self.heads,), torch.float32)}
+
+    def load(self, w: Weights):
+        self.input_bias.copy_(w("i.b").float())
+        self.forget_bias.copy_(w("f.b").float())
+        self.norm_weight.copy_(w("norm").float())
+        rows = [pad_rows(w(n), c) for n, c in (("q", self.kp), ("k", self.kp), ("v", self.vp), ("g", self.vp), ("i", self.hp), ("f", self.hp))]
+        return torch.cat(rows), pad_cols(w("o"), self.out_cols)
+
+    def forward(self, ctx, proj, out, positions):
+        q, k, v, gate, i, f = proj.split([self.kp, self.kp, self.vp, self.vp, self.hp, self.hp], dim=1)
+        nk, nv = self.heads * self.dim, self.heads * self.vdim
+        q, k = (t[:, :nk].unflatten(1, (self.heads, self.dim)) for t in (q, k))
+        v, o = (t[:, :nv].unflatten(1, (self.heads, self.vdim)) for t in (v, out))
+        states = None if self.memory is None else (self.memory, self.normaliser, self.maximum)
+        ops.mlstm(q, k, v, f[:, :self.heads], self.forget_bias, i[:, :self.heads], self.input_bias, self.cap, gate[:, :nv],
+                  self.norm_weight, o, states, ctx.state_slots, ragged(ctx), positions, self.dim ** -0.5, self.eps, status=ctx.status)
+
+
+class LatentAttentionBranch(Branch):
+    """Causal attention whose keys and values are projections of one cached latent per token, with a query latent and an output gate.
+
+    Two forms of the same product.  Prompts: keys and values of the whole context are computed from the latents (one GEMM) and go to
+    the prefill attention kernel, key and value sizes padded to a size it knows.  Decoding, and whatever that kernel does not take (fp32,
+    head sizes above 256): the key projection is applied to the query and the value projection to the attention's output, so that
+    attention itself runs over the latents, which all heads share.
+
+    ``source``: another latent branch, of an earlier layer, whose latents this one reads instead of making its own."""
+
+    def __init__(self, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, eps: float, dtype: torch.dtype,
+                 source: "LatentAttentionBranch | None" = None):
+        super().__init__()
+        self.num_heads = self.num_kv_heads = heads
+        self.scale, self.eps, self.q_rank, self.kv_rank = scale, eps, q_rank, kv_rank
+        self.__dict__["source"] = source                                      # (not a submodule of this one)
+        self.expands = dtype == torch.bfloat16 and max(dim, vdim) <= 256
+        self.head_dim = AttentionBranch.padded_size(dim, vdim, dtype) if self.expands else 0
+        self.dim, self.vdim = dim, vdim
+        self.dk, self.dv = (self.head_dim, self.head_dim) if self.expands else (pad8(dim), pad8(vdim))
+        self.qp = pad8(q_rank)
+        self.latent_width = pad8(kv_rank)
+        if dtype == torch.bfloat16:
+            self.latent_width = next((n for n in ops.LATENT_WIDTHS if n >= kv_rank), self.latent_width)
+        self.tensor_core_decode = dtype == torch.bfloat16 and self.latent_width in ops.LATENT_WIDTHS
+        if source is not None and source.kv_rank != kv_rank:
+            raise ValueError(f"latents of {source.kv_rank} values cannot serve a layer of kv_rank {kv_rank}")
+        own = self.latent_width if source is None else 0
+        self.in_sizes = [self.qp, own, heads * self.dv]                       # query latent | latent | gate
+        self.in_rows = sum(self.in_sizes)
+        self.out_cols = self.out_used = heads * self.dv
+        self.q_norm, self.q_up = weight(q_rank), weight(heads * self.dk, self.qp)
+        self.kv_up = weight(heads * (self.dk + self.dv), self.latent_width)   # keys of all heads, then values
+        if source is None:
+            self.kv_norm = weight(kv_rank)
+            self.latent_cache = torch.tensor([])                              # the executor's pool [blocks, block_size, latent_width]
+        self._item_rows = None
+
+    def load(self, w: Weights):
+        def heads_of(name: str, n: int, padded: int, cols: int) -> torch.Tensor:
+            src = w(name)
+            dst = src.new_zeros(self.num_heads, padded, cols)
+            dst[:, :n, :src.shape[1]] = src.view(self.num_heads, n, -1)
+            return dst.view(self.num_heads * padded, cols)
+        self.q_norm.copy_(w("dq.norm"))
+        self.q_up.copy_(heads_of("uq", self.dim, self.dk, self.qp))
+        self.kv_up.copy_(torch.cat([heads_of("uk", self.dim, self.dk, self.latent_width), heads_of("uv", self.vdim, self.dv, self.latent_width)]))
+        rows = [pad_rows(w("dq"), self.qp)]
+        if self.source is None:
+            self.kv_norm.copy_(w("dkv.norm"))
+            rows.append(pad_rows(w("dkv"), self.latent_width))
+        rows.append(heads_of("g", self.vdim, self.dv, w("g").shape[1]))
+        o = w("o")
+        cols = o.new_zeros(o.shape[0], self.num_heads, self.dv)
+        cols[:, :, :self.vdim] = o.view(o.shape[0], self.num_heads, self.vdim)
+        return torch.cat(rows), cols.view(o.shape[0], -1)
+
+    def forward(self, ctx, proj, out, positions):
+        dq, c, gate = proj.split(self.in_sizes, dim=1)
+        owner = self if self.source is None else self.source
+        cache = owner.latent_cache if owner.latent_cache.numel() else None
+        if self.source is None:
+            cq, c = ops.latent_norm(dq[:, :self.q_rank], self.q_norm, self.qp, c[:, :self.kv_rank], self.kv_norm, self.latent_width,
+                                    self.eps, cache, ctx.slot_mapping, status=ctx.status)
+            ctx.latents[owner] = c                                            # this step's rows, for layers that share them
+        else:
+            cq, _ = ops.latent_norm(dq[:, :self.q_rank], self.q_norm, self.qp, None, None, 0, self.eps, status=ctx.status)
+            c = ctx.latents[owner]
+        q = F.linear(cq, self.q_up).unflatten(1, (self.num_heads, self.dk))
+        o = torch.empty(q.shape[0], self.num_heads, self.dv, dtype=q.dtype, device=q.device)
+        if not self.expands or (not self.tensor_core_decode and (not ctx.prefill or ctx.num_decode)):
+            self._absorbed(ctx, q, c, cache, positions, o)
+        elif not ctx.prefill:
+            self._decode(ctx, q, cache, ctx.block_table, o)
+        else:
+            nd = ctx.num_decode
+            bp, tp = ctx.cu_seqlens_q.numel() - 1 - nd, q.shape[0] - nd
+            self._prompts(ctx, q[:tp], c, cache, ctx.cu_seqlens_q[:bp + 1], ctx.cu_seqlens_k[:bp + 1],
+                          None if ctx.block_table is None else ctx.block_table[:bp], o[:tp])
+            if nd:
+                self._decode(ctx, q[tp:], cache, ctx.block_table[bp:], o[tp:])
+        ops.gate_mul(o.flatten(1), gate, out)
+
+    def _prompts(self, ctx, q, c, cache, cu_q, cu_k, table, o) -> None:
+        if table is not None:                                                 # earlier tokens are in the cache
+            c = ops.gather_latents(cache, table, cu_k, ctx.prompt_keys, status=ctx.status)
+        kv = F.linear(c, self.kv_up).unflatten(1, (2 * self.num_heads, self.head_dim))
+        k, v = kv.split([self.num_heads, self.num_heads], dim=1)
+        ops.prefill_attn(q, k, v, cu_q, cu_k, ctx.max_seqlen_q, self.scale, -1, out=o, status=ctx.status, items=prefill_items_for(ctx, self))
+
+    def _up(self) -> tuple[torch.Tensor, torch.Tensor]:
+        """Key projection [heads, dk, latent] and value projection [heads, latent, dv] as views."""
+        k, v = self.kv_up.split([self.num_heads * self.dk, self.num_heads * self.dv])
+        return k.unflatten(0, (self.num_heads, self.dk)), v.unflatten(0, (self.num_heads, self.dv)).transpose(1, 2)
+
+    def _decode(self, ctx, q, cache, table, o) -> None:
+        uk, uv = self._up()
+        key = ("latent", self.num_heads, self.latent_width)
+        ws = ctx.decode_plans.get(key)
+        if ws is None:
+            ws = decode_workspace_for(q.device, ctx.cache_seqlens.numel(), self.num_heads, 1, self.latent_width, key)
+            ops.latent_decode_plan(ctx.cache_seqlens, table, cache.shape[1], self.num_heads, self.latent_width, ws)
+            ctx.decode_plans[key] = ws
+        mixed = ops.latent_decode(torch.bmm(q.transpose(0, 1), uk), cache, ctx.cache_seqlens, table, self.scale, ws, status=ctx.status)
+        torch.bmm(mixed, uv, out=o.transpose(0, 1))
+
+    def _absorbed(self, ctx, q, c, cache, positions, o) -> None:
+        uk, uv = self._up()
+        paged = ctx.block_table is not None
+        keys = cache.unsqueeze(2) if paged else c.unsqueeze(1)
+        mixed = ops.any_attn(torch.bmm(q.transpose(0, 1), uk).transpose(0, 1).contiguous(), keys, keys, positions, self.scale,
+                             cu_seqlens_q=ctx.cu_seqlens_q if ctx.prefill else None, cu_seqlens_k=ctx.cu_seqlens_k,
+                             block_table=ctx.block_table, cache_seqlens=None if ctx.prefill else ctx.cache_seqlens, status=ctx.status)
+        torch.bmm(mixed.transpose(0, 1), uv, out=o.transpose(0, 1))
 
 
 class PackedMixer(nn.Module):

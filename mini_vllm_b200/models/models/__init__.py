@@ -1,8 +1,10 @@
 from .fupupel import FupupelForCausalLM
 from .gemma3 import Gemma3ForCausalLM
 from .qwen3 import Qwen3ForCausalLM
+from .vebonex import VebonexForCausalLM
 
-_MODELS = {"Qwen3ForCausalLM": Qwen3ForCausalLM, "Gemma3ForCausalLM": Gemma3ForCausalLM, "Fupupel": FupupelForCausalLM}
+_MODELS = {"Qwen3ForCausalLM": Qwen3ForCausalLM, "Gemma3ForCausalLM": Gemma3ForCausalLM, "Fupupel": FupupelForCausalLM,
+           "Vebonex": VebonexForCausalLM}
 
 
 def get_model_class(architecture: str):

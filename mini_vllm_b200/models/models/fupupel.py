@@ -6,16 +6,16 @@ import torch
 
 from ..hybrid import ClampedGLU, HybridDecoder, HybridLayer
 from ..layers.branches import AttentionBranch, GatedDeltaBranch, PackedMixer, SelectiveScanBranch
+from ..layers.residual import SandwichStream
 from ..layers.rotary import RotaryEmbedding
 
 GLU_ALPHA = 1.702
 
 
 class FupupelForCausalLM(HybridDecoder):
-    recurrent = True
-
     def __init__(self, cfg):
         width, tables, layers = cfg.hidden_size, {}, []
+        stream = SandwichStream(width, cfg.rms_norm_eps)
 
         def rotary(dims: int, base: float, padded: int) -> RotaryEmbedding:
             key = (dims, float(base), padded)
@@ -45,8 +45,8 @@ class FupupelForCausalLM(HybridDecoder):
             if ff is not None and ff.get("kind", "dense") != "dense":
                 raise ValueError(f"unknown feed-forward kind {ff['kind']!r}")
             mlp = None if ff is None else ClampedGLU(width, ff["ff"], ff["limit"], GLU_ALPHA)
-            layers.append(HybridLayer(width, PackedMixer(width, branches), mlp))
-        super().__init__(cfg, layers)
+            layers.append(HybridLayer(stream, PackedMixer(width, branches), mlp))
+        super().__init__(cfg, layers, stream)
 
     def mixer_prefixes(self, index: int) -> dict[str, str]:
         p = f"l{index}.mix."

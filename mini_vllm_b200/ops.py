@@ -663,3 +663,209 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tens
     _cabi.check(rc, "mvb_gated_delta")
     LaunchCounter.add(3 if ragged else (2 if vdim > 128 else 1))
     return out
+
+
+def _linear_scratch(code: int, tokens: int, num_seqs: int, heads: int, dim: int, vdim: int, exp_gates: bool, ragged: bool, device):
+    n = _cabi.load().mvb_linear_attn_scratch_bytes(code, tokens, num_seqs, heads, dim, vdim, int(exp_gates), int(ragged))
+    return torch.empty(n, dtype=torch.uint8, device=device)
+
+
+def _linear_shapes(q, k, v, out):
+    for t, name in ((q, "q"), (k, "k"), (v, "v"), (out, "out")):
+        _heads_contiguous(t, name)
+    assert q.shape == k.shape and out.shape == v.shape and v.shape[:2] == q.shape[:2]
+    assert q.stride(0) == k.stride(0) == v.stride(0) or q.shape[0] <= 1
+    return (*q.shape, v.shape[2])
+
+
+def gated_linear(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, decay_bias: torch.Tensor, tau: float,
+                 gate: torch.Tensor, norm_weight: torch.Tensor, out: torch.Tensor, state: torch.Tensor | None,
+                 state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor, q_scale: float,
+                 eps: float, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Linear attention with a decay per key channel, ``sigmoid(decay + bias)^(1/tau)``, and its SiLU-gated output norm: q, k
+    [T, heads, dim], v and out [T, heads, vdim], raw ``decay`` [T, heads * dim], raw ``gate`` [T, heads * vdim]; ``state`` fp32
+    [slots, heads, dim, vdim padded to 4]."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v, decay=decay, gate=gate, out=out)
+    _same(torch.float32, decay_bias=decay_bias, norm_weight=norm_weight, state=state)
+    _need(positions, torch.int64, "positions")
+    tokens, heads, dim, vdim = _linear_shapes(q, k, v, out)
+    st, sl, n = _state_args(state, state_slots)
+    ragged = cu_seqlens_q is not None
+    num_seqs = cu_seqlens_q.numel() - 1 if ragged else tokens
+    scratch = _linear_scratch(code, tokens, num_seqs, heads, dim, vdim, False, ragged, q.device)
+    rc = _cabi.load().mvb_gated_linear(
+        code, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), decay.stride(0), _ptr(decay_bias), 1.0 / tau, _ptr(gate),
+        gate.stride(0), _ptr(norm_weight), _ptr(out), out.stride(0), st, sl, n, _ptr(cu_seqlens_q), _ptr(positions), num_seqs,
+        tokens, heads, dim, vdim, float(q_scale), float(eps), _ptr(scratch), scratch.numel(), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_gated_linear")
+    LaunchCounter.add(3 if ragged else 1)
+    return out
+
+
+def mlstm(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, forget: torch.Tensor, forget_bias: torch.Tensor, inp: torch.Tensor,
+          inp_bias: torch.Tensor, cap: float, gate: torch.Tensor, norm_weight: torch.Tensor, out: torch.Tensor,
+          states: tuple | None, state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor,
+          q_scale: float, eps: float, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Matrix memory with capped exponential gates, a normaliser and a running maximum, and its sigmoid-gated output norm: raw
+    ``forget`` and ``inp`` [T, heads], ``norm_weight`` [heads * vdim]; ``states`` = fp32 (memory [slots, heads, dim, vdim padded to 4],
+    normaliser [slots, heads, dim], maximum [slots, heads])."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v, forget=forget, inp=inp, gate=gate, out=out)
+    memory, normaliser, maximum = states or (None, None, None)
+    _same(torch.float32, forget_bias=forget_bias, inp_bias=inp_bias, norm_weight=norm_weight, memory=memory, normaliser=normaliser,
+          maximum=maximum)
+    _need(positions, torch.int64, "positions")
+    tokens, heads, dim, vdim = _linear_shapes(q, k, v, out)
+    st, sl, n = _state_args(memory, state_slots)
+    ragged = cu_seqlens_q is not None
+    num_seqs = cu_seqlens_q.numel() - 1 if ragged else tokens
+    scratch = _linear_scratch(code, tokens, num_seqs, heads, dim, vdim, True, ragged, q.device)
+    rc = _cabi.load().mvb_mlstm(
+        code, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(forget), forget.stride(0), _ptr(forget_bias), _ptr(inp), inp.stride(0),
+        _ptr(inp_bias), float(cap), _ptr(gate), gate.stride(0), _ptr(norm_weight), _ptr(out), out.stride(0), st,
+        _ptr(normaliser) if st else None, _ptr(maximum) if st else None, sl, n, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens,
+        heads, dim, vdim, float(q_scale), float(eps), _ptr(scratch), scratch.numel(), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_mlstm")
+    LaunchCounter.add(3 if ragged else 1)
+    return out
+
+
+def hyper_embed_norm(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos_table: torch.Tensor, streams: int,
+                     in_weights: torch.Tensor, weight: torch.Tensor, eps: float, groups: int,
+                     status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """(fp32 streams [T, streams, width], all ``table[ids] + pos_table[positions]``; the normalised input of the first sublayer)."""
+    code = _dtype_of(table, "table")
+    _need(ids, torch.int64, "ids"); _need(positions, torch.int64, "positions")
+    _same(table.dtype, weight=weight, pos_table=pos_table); _need(in_weights, torch.float32, "in_weights")
+    assert table.is_contiguous() and pos_table.is_contiguous() and pos_table.shape[1] == table.shape[1]
+    rows, width = ids.numel(), table.shape[1]
+    x = torch.empty(rows, streams, width, dtype=torch.float32, device=table.device)
+    h = torch.empty(rows, width, dtype=table.dtype, device=table.device)
+    rc = _cabi.load().mvb_hyper_embed_norm(
+        code, _ptr(ids), _ptr(positions), _ptr(table), table.shape[0], _ptr(pos_table), pos_table.shape[0], _ptr(x), _ptr(in_weights),
+        _ptr(weight), _ptr(h), rows, width, streams, groups, float(eps), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_hyper_embed_norm")
+    LaunchCounter.add(1)
+    return x, h
+
+
+def hyper_norm(x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out_weights: torch.Tensor, in_weights: torch.Tensor | None,
+               weight: torch.Tensor, eps: float, groups: int, row_ends: torch.Tensor | None = None) -> torch.Tensor:
+    """Streams ``x`` [T, streams, width] in place: ``x_t <- sum_s mix[s, t] x_s + out[t] y``; returns the grouped norm of
+    ``sum_s in[s] x_s`` (``in_weights`` None: of the plain sum) in y's dtype.  With ``row_ends`` only rows ``row_ends[1:] - 1`` are
+    produced and ``x`` is left as it is."""
+    code = _dtype_of(y, "y")
+    _need(x, torch.float32, "x"); _same(y.dtype, weight=weight); _same(torch.float32, mix=mix, out_weights=out_weights, in_weights=in_weights)
+    rows, streams, width = x.shape
+    assert x.is_contiguous() and y.shape == (rows, width) and y.stride(1) == 1 and mix.shape == (streams, streams) and mix.is_contiguous()
+    if row_ends is not None:
+        _need(row_ends, torch.int32, "row_ends")
+        rows = row_ends.numel() - 1
+    h = torch.empty(rows, width, dtype=y.dtype, device=x.device)
+    if rows == 0:
+        return h
+    rc = _cabi.load().mvb_hyper_norm(code, _ptr(x), _ptr(y), y.stride(0), _ptr(mix), _ptr(out_weights), _ptr(in_weights), _ptr(weight),
+                                     _ptr(h), _ptr(row_ends), rows, width, streams, groups, float(eps), _stream())
+    _cabi.check(rc, "mvb_hyper_norm")
+    LaunchCounter.add(1)
+    return h
+
+
+def poly_norm(z: torch.Tensor, cols: int, act: torch.Tensor, eps: float) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` over the first ``cols`` columns (N: over the row's root mean square, act = fp32 {a, b, c, e});
+    the columns behind them become 0."""
+    code = _dtype_of(z, "z")
+    _need(act, torch.float32, "act")
+    assert z.dim() == 2 and z.stride(1) == 1 and z.shape[1] >= cols and act.numel() == 4
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    rc = _cabi.load().mvb_poly_norm(code, _ptr(z), z.stride(0), _ptr(out), out.stride(0), z.shape[0], cols, z.shape[1], _ptr(act),
+                                    float(eps), _stream())
+    _cabi.check(rc, "mvb_poly_norm")
+    LaunchCounter.add(1)
+    return out
+
+
+LATENT_WIDTHS = (64, 128, 192, 256, 384, 512)      # cached row sizes of latent_decode
+
+
+def latent_norm(q: torch.Tensor, q_weight: torch.Tensor, q_pad: int, c: torch.Tensor | None, c_weight: torch.Tensor | None, c_pad: int,
+                eps: float, cache: torch.Tensor | None = None, slot_mapping: torch.Tensor | None = None,
+                status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """RMS norms of the query latent ``q`` and, unless None, of the key/value latent ``c``, each zero-padded to a width; ``c`` also goes
+    to its slots of ``cache`` [blocks, block_size, c_pad]."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, q_weight=q_weight, c=c, c_weight=c_weight, cache=cache)
+    tokens = q.shape[0]
+    assert q.stride(1) == 1 and q_weight.numel() == q.shape[1]
+    q_out = torch.empty(tokens, q_pad, dtype=q.dtype, device=q.device)
+    c_out, slots = None, 0
+    if c is not None:
+        assert c.stride(1) == 1 and c.shape[0] == tokens and c_weight.numel() == c.shape[1]
+        c_out = torch.empty(tokens, c_pad, dtype=q.dtype, device=q.device)
+        if cache is not None:
+            _need(slot_mapping, torch.int32, "slot_mapping")
+            assert cache.is_contiguous() and cache.shape[-1] == c_pad and slot_mapping.numel() == tokens
+            slots = cache.shape[0] * cache.shape[1]
+    rc = _cabi.load().mvb_latent_norm(
+        code, _ptr(q), q.stride(0), _ptr(q_weight), _ptr(q_out), q.shape[1], q_pad, _ptr(c), c.stride(0) if c is not None else 0,
+        _ptr(c_weight), _ptr(c_out), c.shape[1] if c is not None else 0, c_pad, _ptr(cache) if slots else None,
+        _ptr(slot_mapping) if slots else None, slots, tokens, float(eps), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_latent_norm")
+    LaunchCounter.add(1)
+    return q_out, c_out
+
+
+def gather_latents(cache: torch.Tensor, block_table: torch.Tensor, cu_seqlens_k: torch.Tensor, rows: int,
+                   status: torch.Tensor | None = None) -> torch.Tensor:
+    """The contexts of a ragged step ([blocks, block_size, width] pool, lengths in ``cu_seqlens_k``, ``rows`` in all) as dense rows."""
+    _need(block_table, torch.int32, "block_table"); _need(cu_seqlens_k, torch.int32, "cu_seqlens_k")
+    assert cache.is_cuda and cache.is_contiguous() and block_table.stride(1) == 1
+    out = torch.empty(rows, cache.shape[-1], dtype=cache.dtype, device=cache.device)
+    rc = _cabi.load().mvb_gather_latents(
+        _ptr(cache), cache.shape[0] * cache.shape[1], cache.shape[-1] * cache.element_size(), _ptr(block_table), block_table.stride(0),
+        block_table.shape[1], cache.shape[1], _ptr(cu_seqlens_k), cu_seqlens_k.numel() - 1, rows, _ptr(out), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_gather_latents")
+    LaunchCounter.add(1)
+    return out
+
+
+def gate_mul(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out = o * sigmoid(gate)``; 2-D, free row strides."""
+    code = _dtype_of(o, "o")
+    _same(o.dtype, gate=gate, out=out)
+    assert o.shape == gate.shape == out.shape and o.stride(1) == gate.stride(1) == out.stride(1) == 1
+    rc = _cabi.load().mvb_gate_mul(code, _ptr(o), o.stride(0), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0), o.shape[0], o.shape[1],
+                                   _stream())
+    _cabi.check(rc, "mvb_gate_mul")
+    LaunchCounter.add(1)
+    return out
+
+
+def latent_decode_plan(cache_seqlens: torch.Tensor, block_table: torch.Tensor, block_size: int, heads: int, width: int,
+                       workspace: torch.Tensor) -> None:
+    _need(cache_seqlens, torch.int32, "cache_seqlens"); _need(block_table, torch.int32, "block_table")
+    assert block_table.stride(1) == 1 and block_table.shape[0] >= cache_seqlens.numel()
+    rc = _cabi.load().mvb_latent_decode_plan(_ptr(cache_seqlens), _ptr(block_table), block_table.stride(0), block_size,
+                                             cache_seqlens.numel(), heads, width, _ptr(workspace), workspace.numel(), _stream())
+    _cabi.check(rc, "mvb_latent_decode_plan")
+    LaunchCounter.add(1)
+
+
+def latent_decode(q: torch.Tensor, cache: torch.Tensor, cache_seqlens: torch.Tensor, block_table: torch.Tensor, scale: float,
+                  workspace: torch.Tensor, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Absorbed decode attention: q [heads, B, width] (queries already in the latent's space) over ``cache`` [blocks, block_size, width];
+    returns [heads, B, width].  The plan for ``cache_seqlens`` must already be in ``workspace``."""
+    _need(q, torch.bfloat16, "q"); _need(cache, torch.bfloat16, "cache")
+    _need(cache_seqlens, torch.int32, "cache_seqlens"); _need(block_table, torch.int32, "block_table")
+    heads, b, width = q.shape
+    nblk, bs, w2 = cache.shape
+    assert w2 == width and cache.is_contiguous() and q.stride(2) == 1 and block_table.stride(1) == 1 and cache_seqlens.numel() >= b
+    out = torch.empty(heads, b, width, dtype=q.dtype, device=q.device)
+    rc = _cabi.load().mvb_latent_decode(
+        _ptr(q), q.stride(1), q.stride(0), _ptr(cache), nblk, bs, _ptr(cache_seqlens), _ptr(block_table), block_table.stride(0),
+        block_table.shape[1], b, heads, width, float(scale), _ptr(out), out.stride(1), out.stride(0), _ptr(workspace), workspace.numel(),
+        _ptr(status), _stream())
+    _cabi.check(rc, "mvb_latent_decode")
+    LaunchCounter.add(1)
+    return out
