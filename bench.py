@@ -611,56 +611,70 @@ def fupupel_bench_shape(size: str, window: int = 1024):
     return fupupel_shape([scan if i % 2 == 0 else both for i in range(layers)], width, 32768)
 
 
-def fupupel_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
-    """Prefill (8 prompts of 2048 tokens) and decode (32 and 256 sequences) through ``Engine.generate`` with random weights,
-    beside Qwen3 layers of the same width, heads, feed-forward and count."""
+def engine_throughput(models) -> dict:
+    """Prefill (8 prompts of 2048 tokens) and decode (32 and 256 sequences) through ``Engine.generate`` with random weights, for each
+    (name, model description)."""
     from mini_vllm_b200.engine.engine import Engine
     out = {}
-    for size in sizes:
-        width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
-        twin = qwen3_shape(num_hidden_layers=layers, hidden_size=width, intermediate_size=ff, num_attention_heads=heads,
-                           num_key_value_heads=kv, vocab_size=32768)
-        for name, hf in (("fupupel", fupupel_bench_shape(size)), ("qwen3", twin)):
-            eng = Engine(Config(hf_config=hf, kv_cache_num_blocks=1024, max_num_batched_seqs=256, max_graph_batch_size=256,
-                                max_num_batched_tokens=16384, gpu_memory_utilization=0.85, seed=0))
-            params = sum(p.numel() for p in eng.executor.model.parameters())
-            job = lambda n, length, new: (eng.generate([[(7 * i + j) % 32768 for j in range(length)] for i in range(n)],
-                                                       SamplingParams(max_tokens=new, ignore_eos=True), use_tqdm=False),
-                                          eng.last_job_device_ms)[1]
-            med = lambda *a: statistics.median(job(*a) for _ in range(3))
-            job(8, 2048, 1)
-            row = {"parameters": params, "prefill_tok_s": round(8 * 2048 / med(8, 2048, 1) * 1e3)}
-            for n in (32, 256):
-                job(n, 512, 2)
-                row[f"decode{n}_step_ms"] = round((med(n, 512, 65) - med(n, 512, 1)) / 64, 4)
-                row[f"decode{n}_tok_s"] = round(n / row[f"decode{n}_step_ms"] * 1e3)
-            out[f"{size}_{name}"] = row
-            del eng
-            torch.cuda.empty_cache()
+    for name, hf in models:
+        eng = Engine(Config(hf_config=hf, kv_cache_num_blocks=1024, max_num_batched_seqs=256, max_graph_batch_size=256,
+                            max_num_batched_tokens=16384, gpu_memory_utilization=0.85, seed=0))
+        params = sum(p.numel() for p in eng.executor.model.parameters())
+        job = lambda n, length, new: (eng.generate([[(7 * i + j) % 32768 for j in range(length)] for i in range(n)],
+                                                   SamplingParams(max_tokens=new, ignore_eos=True), use_tqdm=False),
+                                      eng.last_job_device_ms)[1]
+        med = lambda *a: statistics.median(job(*a) for _ in range(3))
+        job(8, 2048, 1)
+        row = {"parameters": params, "prefill_tok_s": round(8 * 2048 / med(8, 2048, 1) * 1e3)}
+        for n in (32, 256):
+            job(n, 512, 2)
+            row[f"decode{n}_step_ms"] = round((med(n, 512, 65) - med(n, 512, 1)) / 64, 4)
+            row[f"decode{n}_tok_s"] = round(n / row[f"decode{n}_step_ms"] * 1e3)
+        out[name] = row
+        del eng
+        torch.cuda.empty_cache()
     return out
+
+
+def qwen3_twin(size: str):
+    width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
+    return qwen3_shape(num_hidden_layers=layers, hidden_size=width, intermediate_size=ff, num_attention_heads=heads,
+                       num_key_value_heads=kv, vocab_size=32768)
+
+
+def fupupel_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
+    """Beside Qwen3 layers of the same width, heads, feed-forward and count."""
+    return engine_throughput((f"{size}_{name}", hf) for size in sizes
+                             for name, hf in (("fupupel", fupupel_bench_shape(size)), ("qwen3", qwen3_twin(size))))
+
+
+class Legs:
+    """Kernels against their rooflines: each leg is timed from a CUDA graph over ``nbuf`` launches on buffers of their own."""
+
+    def __init__(self, dev, peaks):
+        self.peaks, self.rows = peaks, {}
+        self.sms, self.ghz = torch.cuda.get_device_properties(dev).multi_processor_count, 1.9
+
+    def __call__(self, name, call, nbuf, byts=None, flops=None, mufu=None, fp32=None):
+        ms = graph_time_ms(lambda: [call(i) for i in range(nbuf)], nbuf)
+        row = {"us": round(ms * 1e3, 2)}
+        if byts:
+            row.update({"GB/s": round(byts / ms / 1e6, 1), "frac_of_measured_hbm": round(byts / ms / 1e6 / self.peaks["hbm_gbs"], 4)})
+        if flops:
+            row.update({"TFLOP/s": round(flops / ms / 1e9, 1), "frac_of_measured_bf16": round(flops / ms / 1e9 / self.peaks["bf16_tflops"], 4)})
+        if mufu:
+            row["frac_of_special_function_rate"] = round(mufu / (self.sms * 16 * self.ghz * 1e9) / (ms * 1e-3), 4)
+        if fp32:
+            row["frac_of_fp32_fma_rate"] = round(fp32 / (self.sms * 128 * self.ghz * 1e9) / (ms * 1e-3), 4)
+        self.rows[name] = row
 
 
 def fupupel_kernel_legs(dev, peaks) -> dict:
     """Each kernel of the design against its roofline, next to the like kernel of the existing models where there is one.
     16 heads of 128 (8 KV heads), width 2048, scan of 4096 channels x 16 states, 8192 prefill tokens, 256 decode rows."""
     from mini_vllm_b200 import ops
-    out, bf = {}, torch.bfloat16
-    sms, ghz = torch.cuda.get_device_properties(dev).multi_processor_count, 1.9
+    bf, leg = torch.bfloat16, Legs(dev, peaks)
     rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
-
-    def leg(name, call, nbuf, byts=None, flops=None, mufu=None, fp32=None):
-        ms = graph_time_ms(lambda: [call(i) for i in range(nbuf)], nbuf)
-        row = {"us": round(ms * 1e3, 2)}
-        if byts:
-            row.update({"GB/s": round(byts / ms / 1e6, 1), "frac_of_measured_hbm": round(byts / ms / 1e6 / peaks["hbm_gbs"], 4)})
-        if flops:
-            row.update({"TFLOP/s": round(flops / ms / 1e9, 1), "frac_of_measured_bf16": round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)})
-        if mufu:
-            row["frac_of_special_function_rate"] = round(mufu / (sms * 16 * ghz * 1e9) / (ms * 1e-3), 4)
-        if fp32:
-            row["frac_of_fp32_fma_rate"] = round(fp32 / (sms * 128 * ghz * 1e9) / (ms * 1e-3), 4)
-        out[name] = row
-
     heads, kv, d, width, ff, window = 16, 8, 128, 2048, 6144, 1024
     for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
         tokens = sum(lens)
@@ -736,7 +750,109 @@ def fupupel_kernel_legs(dev, peaks) -> dict:
     x16 = rnd(b, width)
     leg("add_rmsnorm_branch_norm_256", lambda i: ops.add_rmsnorm(x16, y16, w, 1e-6, True, y_weight=w), 8, byts=b * width * 8)
     leg("residual_norm_f32_256", lambda i: ops.residual_norm(x32, y16, w, 1e-6, y_weight=w), 8, byts=b * width * 12)
-    return out
+    return leg.rows
+
+
+# ---- Vebonex: beside the models above, and the kernels of its own ---------------------------------------------
+def vebonex_bench_shape(size: str):
+    """Layers in turn: matrix LSTM, gated linear attention, latent attention, latent attention on the latents of the one before; heads of
+    128 everywhere; a feed-forward of as many weights as the gated one of the other models."""
+    from mini_vllm_b200.config import vebonex_shape
+    width, heads, _, ff, layers = FUPUPEL_SIZES[size]
+    mlp = {"kind": "dense", "ff": ff * 3 // 2}
+    head = {"heads": heads, "dim": 128, "vdim": 128}
+    latent = {**head, "kv_rank": 512, "q_rank": width * 3 // 4, "scale": 128 ** -0.5}
+    turn = lambda i: [("mlstm", {**head, "gate_cap": 15.0}), ("gla", {**head, "tau": 16.0, "decay_rank": 16}), ("latent_attention", latent),
+                      ("latent_attention", {**latent, "kv_from": i - 1})][i % 4]
+    return vebonex_shape([{"type": turn(i)[0], "mixer": turn(i)[1], "mlp": mlp} for i in range(layers)], width, 32768, streams=4, groups=8)
+
+
+def vebonex_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
+    """Beside Fupupel, the closest design there is, and Qwen3 layers of the same width, heads, feed-forward and count."""
+    return engine_throughput((f"{size}_{name}", hf) for size in sizes
+                             for name, hf in (("vebonex", vebonex_bench_shape(size)), ("fupupel", fupupel_bench_shape(size)), ("qwen3", qwen3_twin(size))))
+
+
+def vebonex_kernel_legs(dev, peaks) -> dict:
+    """Each kernel of the design against its roofline, next to the like kernel of the other models.  16 heads of 128, width 2048, latent
+    of 512, 4 streams, 8192 prefill tokens, 256 decode rows."""
+    from mini_vllm_b200 import ops
+    bf, leg = torch.bfloat16, Legs(dev, peaks)
+    rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
+    heads, d, width, ff, latent, streams, tokens = 16, 128, 2048, 9216, 512, 4, 8192
+    hd, scale, eps = heads * d, d ** -0.5, 1e-6
+    ones = torch.ones(hd, device=dev)
+    qd, kd, vd, gate, od = (rnd(tokens, heads, d) for _ in range(5))
+    raw_a, raw_b, raw_c = rnd(tokens, hd), rnd(tokens, heads), rnd(tokens, heads)
+    ea, db, hb = torch.rand(heads, device=dev) * 8 + 1, torch.full((hd,), -4.0, device=dev), torch.full((heads,), 4.0, device=dev)
+
+    def recurrent(tag, rows, cu, pos, slots, nbuf):
+        states = [(torch.randn(slots.numel(), heads, d, d, device=dev) * 0.01, torch.zeros(slots.numel(), heads, d, device=dev),
+                   torch.zeros(slots.numel(), heads, device=dev)) for _ in range(nbuf)]
+        q, k, v, o, g, a, b, c = qd[:rows], kd[:rows], vd[:rows], od[:rows], gate[:rows].flatten(1), raw_a[:rows], raw_b[:rows], raw_c[:rows]
+        work = {"byts": rows * heads * d * d * 8} if cu is None else {"byts": rows * hd * 6 * 2, "fp32": rows * heads * d * d * 2}
+        leg(f"gated_delta_{tag}", lambda i: ops.gated_delta(q, k, v, a, b, g, ea, db, ones[:d], o, states[i][0], slots, cu, pos, scale, eps), nbuf, **work)
+        leg(f"gated_linear_{tag}", lambda i: ops.gated_linear(q, k, v, a, db, 16.0, g, ones[:d], o, states[i][0], slots, cu, pos, scale, eps), nbuf, **work)
+        if cu is not None:
+            work["byts"] = rows * hd * 5 * 2
+        leg(f"mlstm_{tag}", lambda i: ops.mlstm(q, k, v, b, hb, c, hb, 15.0, g, ones, o, states[i], slots, cu, pos, scale, eps), nbuf, **work)
+
+    w16 = torch.ones(width, device=dev, dtype=bf)
+    for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        pos = torch.cat([torch.arange(n, device=dev) for n in lens])
+        recurrent(tag, tokens, cu, pos, torch.arange(len(lens), dtype=torch.int32, device=dev), 1)
+        k8, v8, kv = rnd(tokens, heads // 2, d), rnd(tokens, heads // 2, d), rnd(tokens, 2 * heads, d)
+        pairs = sum(n * (n + 1) // 2 for n in lens)
+        leg(f"prefill_attn_{tag}", lambda i: ops.prefill_attn(qd, k8, v8, cu, cu, max(lens), scale), 2, flops=4 * hd * pairs)
+        leg(f"prefill_attn_of_latents_{tag}", lambda i: ops.prefill_attn(qd, kv[:, :heads], kv[:, heads:], cu, cu, max(lens), scale), 2, flops=4 * hd * pairs)
+    xs32, ys = [torch.randn(tokens, width, device=dev) for _ in range(3)], [rnd(tokens, width) for _ in range(3)]
+    leg("residual_norm_8192", lambda i: ops.residual_norm(xs32[i], ys[i], w16, eps, y_weight=w16), 3, byts=tokens * width * 12)
+    x4 = [torch.randn(tokens, streams, width, device=dev) for _ in range(2)]
+    mix, sw = torch.eye(streams, device=dev), torch.full((streams,), 0.25, device=dev)
+    leg("hyper_norm_8192", lambda i: ops.hyper_norm(x4[i], ys[i], mix, sw, sw, w16, eps, 8), 2, byts=tokens * width * (8 * streams + 4))
+    del x4, xs32
+    z, act = [rnd(tokens, ff) for _ in range(2)], torch.tensor([0.5, 0.4, 0.3, 0.1], device=dev)
+    leg("act_mul_8192", lambda i: ops.act_mul(z[i], ff // 2, False), 2, byts=tokens * ff * 3)
+    leg("poly_norm_8192", lambda i: ops.poly_norm(z[i], ff, act, eps), 2, byts=tokens * ff * 4)
+    del z
+    proj = [rnd(tokens, 1536 + latent + hd) for _ in range(3)]
+    pool, slots = torch.zeros(tokens // 256, 256, latent, device=dev, dtype=bf), torch.arange(tokens, dtype=torch.int32, device=dev)
+    lw = torch.ones(1536, device=dev, dtype=bf)
+    leg("latent_norm_8192", lambda i: ops.latent_norm(proj[i][:, :1536], lw, 1536, proj[i][:, 1536:2048], lw[:latent], latent, eps, pool, slots), 3,
+        byts=tokens * (1536 * 2 + latent * 3) * 2)
+    leg("gate_mul_8192", lambda i: ops.gate_mul(od.flatten(1), proj[i][:, 2048:], ys[i]), 3, byts=tokens * hd * 6)
+    # decode: 256 sequences
+    b = 256
+    pos, slots = torch.full((b,), 1199, device=dev), torch.arange(b, dtype=torch.int32, device=dev)
+    recurrent(f"decode{b}", b, None, pos, slots, 2)
+    x4 = [torch.randn(b, streams, width, device=dev) for _ in range(24)]
+    xs32 = [torch.randn(b, width, device=dev) for _ in range(64)]
+    leg(f"residual_norm_{b}", lambda i: ops.residual_norm(xs32[i], ys[0][:b], w16, eps, y_weight=w16), 64, byts=b * width * 12)
+    leg(f"hyper_norm_{b}", lambda i: ops.hyper_norm(x4[i], ys[0][:b], mix, sw, sw, w16, eps, 8), 24, byts=b * width * (8 * streams + 4))
+    zs = [rnd(b, ff) for _ in range(32)]
+    leg(f"act_mul_{b}", lambda i: ops.act_mul(zs[i], ff // 2, False), 32, byts=b * ff * 3)
+    leg(f"poly_norm_{b}", lambda i: ops.poly_norm(zs[i], ff, act, eps), 32, byts=b * ff * 4)
+    del x4, xs32, zs
+    for n in (1200, 4096):
+        per = -(-n // 256)
+        lens = torch.full((b,), n, dtype=torch.int32, device=dev)
+        bt = torch.arange(b * per, dtype=torch.int32, device=dev).view(b, per)
+        pools = torch.randn(2, b * per, 256, heads // 2, d, device=dev, dtype=bf)
+        ws = ops.decode_workspace(b, heads, d, dev)
+        ops.decode_plan(lens, -1, heads, heads // 2, d, ws, block_table=bt, block_size=256)
+        leg(f"decode_attn_{b}x{n}", lambda i: ops.decode_attn(qd[:b], pools[0], pools[1], lens, bt, scale, -1, ws), 1, byts=b * n * hd * 2)
+        del pools
+        for h in (16, 32):
+            ws = ops.decode_workspace(b, h, latent, dev)
+            ops.latent_decode_plan(lens, bt, 256, h, latent, ws)
+            lat, ql = rnd(b * per, 256, latent), rnd(h, b, latent)
+            leg(f"latent_decode_{h}heads_{b}x{n}", lambda i: ops.latent_decode(ql, lat, lens, bt, scale, ws), 1, byts=b * n * latent * 2)
+            del lat
+    # the projections around it, as the batched products they are
+    up, qh = rnd(heads, d, latent), rnd(b, heads, d)
+    leg(f"absorb_queries_{b}", lambda i: torch.bmm(qh.transpose(0, 1), up), 8, byts=(heads * d * latent + b * heads * (d + latent)) * 2)
+    return leg.rows
 
 
 # ---- CPU leg: the oracle restatement of the reference path on the host cores ------------------------
@@ -855,6 +971,8 @@ def main():
     ap.add_argument("--fupupel", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
                     help="the Fupupel design with random weights: prefill and decode throughput beside Qwen3 layers of equal "
                          "size, and its kernels against their rooflines beside the like kernels")
+    ap.add_argument("--vebonex", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
+                    help="the same for the Vebonex design, beside Fupupel and Qwen3")
     ap.add_argument("--engine-steps", type=int, default=0,
                     help="profiling aid: prefill + N decode steps of the workload without CUDA graphs, then exit")
     args = ap.parse_args()
@@ -884,6 +1002,15 @@ def main():
         if args.fupupel in ("all", "engine"):
             line["engine"] = fupupel_throughput()
         print(json.dumps({"fupupel": line}))
+        return
+    if args.vebonex:
+        torch.cuda.set_device(0)
+        line = {}
+        if args.vebonex in ("all", "kernels"):
+            line["kernels"] = vebonex_kernel_legs(torch.device("cuda", 0), measured_peaks()[0])
+        if args.vebonex in ("all", "engine"):
+            line["engine"] = vebonex_throughput()
+        print(json.dumps({"vebonex": line}))
         return
     if args.kernel_legs:
         peaks, _ = measured_peaks()

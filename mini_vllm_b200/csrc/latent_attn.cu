@@ -9,11 +9,14 @@
 //                           cache is loaded once for all of them: the roofline is HBM, sum_b context(b) * width * 2 bytes
 //   gate_mul_kernel         o * sigmoid(gate)
 //
-// latent_decode_kernel: persistent CTAs over the tile ranges of decode_plan.cuh, 8 warps, a tile = 64 tokens x width in 128-byte-swizzled
-// shared memory, brought by TMA through the block table, NST tiles deep.  Per tile, three CTA barriers:
-//   scores   S[heads x 64] = Q' C^T     warp = 16 tokens x half the width (mma.sync, heads in M, both halves meet in shared memory)
+// latent_decode_kernel: persistent CTAs over the tile ranges of decode_plan.cuh.  A tile = 32 tokens x width in 128-byte-swizzled shared
+// memory, brought by TMA through the block table, up to six tiles deep.  Two groups of eight warps take the tiles in turn, so that one
+// group's barriers and latencies lie under the other's arithmetic; each keeps its own running softmax, and they meet at the end of a
+// sequence.  Per tile and group, three barriers of 256 threads:
+//   scores   S[heads x 32] = Q' C^T     warp = 16 tokens x a quarter of the width (mma.sync, heads in M); the quarters meet in shared memory
 //   softmax  a few threads per head, running maximum and sum in registers, P as bf16 through shared memory
 //   output   O[heads x width] += P C    warp = an eighth of the width (C again, as transposed fragments), O in registers
+// A stage is filled again by the group that has just read it, so the groups never wait for each other inside a sequence.
 // A sequence that is split between CTAs is merged by the CTA that arrives last, as in decode_attn.cu; nothing waits on another CTA.
 #include "chunk_common.cuh"
 #include "decode_plan.cuh"
@@ -142,19 +145,20 @@ static int launch_gate(const void* o, int64_t os, const void* g, int64_t gs, voi
 }
 
 // ---- decode -----------------------------------------------------------------------------------------------------
-constexpr int kLatentTile = 64;
+constexpr int kLatentTile = 32;
 
 template <int RH, int MT>                       // width = 64 RH, 16 MT heads per CTA
 struct LatentCfg {
   static constexpr int W = 64 * RH, HEADS = 16 * MT, TOK = kLatentTile;
-  static constexpr int HALF = TOK * 128, STAGE = RH * HALF;             // 64 tokens x 64 columns
+  static constexpr int HALF = TOK * 128, STAGE = RH * HALF;             // 32 tokens x 64 columns
   static constexpr int QROW = W * 2 + 16, SROW = TOK + 4, PROW = TOK * 2 + 16;
-  static constexpr int Q = HEADS * QROW, SB = 2 * HEADS * SROW * 4, P = HEADS * PROW, ROWS = 3 * HEADS * 4;
-  static constexpr int FIXED = Q + SB + P + ROWS + 64;
+  static constexpr int Q = HEADS * QROW, SB = 4 * HEADS * SROW * 4, P = HEADS * PROW, ROWS = 3 * HEADS * 4;     // (the last three per group)
+  static constexpr int FIXED = Q + 2 * (SB + P + ROWS) + 64;
   static constexpr int FIT = (226 * 1024 - 1024 - FIXED) / STAGE;
-  static constexpr int NST = FIT > 4 ? 4 : FIT;
+  static constexpr int NST = FIT > 6 ? 6 : FIT;
   static constexpr int SMEM = 1024 + NST * STAGE + FIXED;
-  static_assert(NST >= 2, "two stages at least");
+  static_assert(NST >= 3, "a tile per group and one in flight at least");
+  static_assert(HEADS * (W / 2) * 4 <= 2 * SB, "half of O fits the score buffers");
 };
 
 struct LatentDecodeParams {
@@ -174,32 +178,46 @@ struct LatentDecodeParams {
 
 struct SeqSpan { int b, tp0, tp1, n; };          // a sequence, its tile range, its length
 
+__device__ __forceinline__ void group_sync(int group) { asm volatile("barrier.cta.sync.aligned %0, 256;" ::"r"(group + 1) : "memory"); }
+__device__ __forceinline__ bool group_all(int group, bool ok) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.u32 q, %1, 0;\n\t"
+      "barrier.cta.red.and.aligned.pred p, %2, 256, q;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(r) : "r"(static_cast<uint32_t>(ok)), "r"(group + 1) : "memory");
+  return r != 0;
+}
+
 template <int RH, int MT>
-__global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDecodeParams p) {
+__global__ void __launch_bounds__(512, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDecodeParams p) {
   using C = LatentCfg<RH, MT>;
   constexpr int TOK = C::TOK, NST = C::NST, W = C::W, HEADS = C::HEADS;
   constexpr uint32_t FULL = 0xffffffffu;
   extern __shared__ uint8_t smem_raw[];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c = blockIdx.x;
+  const int tid = threadIdx.x, group = tid >> 8, gt = tid & 255, warp = gt >> 5, lane = tid & 31, c = blockIdx.x;
   const int head0 = blockIdx.y * HEADS, nheads = min(HEADS, p.heads - head0);
   const CtaDesc desc = p.descs[c];
   auto zero_empty_rows = [&]() {
     for (int b = c; b < p.num_seqs; b += gridDim.x)
       if (p.cache_seqlens[b] <= 0)
-        for (int e = tid; e < nheads * W; e += 256)
+        for (int e = tid; e < nheads * W; e += 512)
           p.out[b * p.out_stride + (head0 + e / W) * p.out_head_stride + e % W] = __float2bfloat16_rn(0.f);
   };
   if (desc.t0 >= desc.t1) { zero_empty_rows(); return; }
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  const uint32_t q_base = base + NST * C::STAGE, p_base = q_base + C::Q + C::SB;
   uint8_t* q_s = base_ptr + NST * C::STAGE;
-  float* s_s = reinterpret_cast<float*>(q_s + C::Q);                    // [2][HEADS][SROW]
-  uint8_t* p_s = q_s + C::Q + C::SB;                                    // [HEADS][PROW bytes]
-  float* alpha_s = reinterpret_cast<float*>(p_s + C::P);                // [HEADS]; behind it the final l and m
-  float *l_s = alpha_s + HEADS, *m_s = l_s + HEADS;
-  uint64_t* full = reinterpret_cast<uint64_t*>(m_s + HEADS);
+  float* scores = reinterpret_cast<float*>(q_s + C::Q);                 // [group][quarter][HEADS][SROW]; also O and weights in a merge
+  uint8_t* p_all = q_s + C::Q + 2 * C::SB;                              // [group][HEADS][PROW bytes]
+  float* rows_s = reinterpret_cast<float*>(p_all + 2 * C::P);           // [group][alpha | l | m][HEADS]
+  uint64_t* full = reinterpret_cast<uint64_t*>(rows_s + 6 * HEADS);
+  float* s_s = scores + group * (C::SB / 4);
+  uint8_t* p_s = p_all + group * C::P;
+  float *alpha_s = rows_s + group * 3 * HEADS, *l_s = alpha_s + HEADS, *m_s = l_s + HEADS;
+  const uint32_t q_base = smem_u32(q_s), p_base = smem_u32(p_s);
   if (tid == 0) {
     tma_prefetch_desc(&map);
     for (int i = 0; i < NST; ++i) mbar_init(&full[i], 1);
@@ -207,18 +225,19 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
   }
   __syncthreads();
 
-  // ---- producer: warp 0, the same tile walk as the consumer, up to NST tiles ahead ----
+  // ---- producer: warp 0 of a group; tiles are counted from desc.t0, tile i lives in stage i % NST ----
+  const int total = desc.t1 - desc.t0;
   SeqSpan fs{desc.b, desc.tp0, desc.tp1, desc.n}, cs = fs;
   auto next_seq = [&](SeqSpan& v) {
     ++v.b; v.tp0 = p.tile_prefix[v.b]; v.tp1 = p.tile_prefix[v.b + 1]; v.n = p.cache_seqlens[v.b];
   };
-  int ft = desc.t0, nfetch = 0, blk_base = -1, blk_reg = -1, blk_n = 0;
+  int blk_base = -1, blk_reg = -1, blk_n = 0, fetched = -1;
   if (desc.blk0 >= 0) { blk_base = (desc.t0 - desc.tp0) * TOK / p.block_size; blk_reg = desc.blk0; blk_n = 1; }
-  auto fetch_next = [&]() {                                             // warp 0, all lanes
-    if (ft >= desc.t1) return;
-    while (ft >= fs.tp1 && fs.b + 1 < p.num_seqs) { next_seq(fs); blk_base = -1; blk_n = 0; }
-    const int token0 = (ft - fs.tp0) * TOK, bi = token0 / p.block_size;
-    ++ft;
+  auto fetch = [&](int i) {                                             // all lanes; i only grows
+    if (i >= total) return;
+    const int t = desc.t0 + i;
+    while (t >= fs.tp1 && fs.b + 1 < p.num_seqs) { next_seq(fs); blk_base = -1; blk_n = 0; }
+    const int token0 = (t - fs.tp0) * TOK, bi = token0 / p.block_size;
     if (blk_base < 0 || bi < blk_base || bi >= blk_base + blk_n) {
       blk_base = bi; blk_n = 32;
       const int col = bi + lane;
@@ -229,33 +248,40 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
     if (blk >= 0 && blk < p.num_blocks) slot0 = blk * p.block_size + (token0 - bi * p.block_size);
     else if (lane == 0) report(p.dev_status, kDevBadBlock, fs.b);
     if (lane == 0) {
-      const int st = nfetch % NST;
+      const int st = i % NST;
       fence_proxy_async();
       mbar_arrive_expect_tx(&full[st], C::STAGE);
 #pragma unroll
       for (int h = 0; h < RH; ++h) tma_load_3d(base_ptr + st * C::STAGE + h * C::HALF, &map, &full[st], h * 64, 0, slot0);
     }
-    ++nfetch;
+    fetched = i;
   };
-  if (warp == 0)
-    for (int i = 0; i < NST - 1; ++i) fetch_next();
+  if (group == 0 && warp == 0)
+    for (int i = 0; i < NST; ++i) fetch(i);
 
   const int first_b = cs.b;
-  int t = desc.t0, ncomp = 0;
+  int seg = 0, i = group;                                               // first tile of the segment; this group's next tile
   bool dead = false;
-  const int tg = warp & 3, kh = warp >> 2;                              // scores: 16-token group, half of the width
+  const int tg = warp & 1, kq = warp >> 1;                              // scores: 16-token group, quarter of the width
   constexpr int TPR = 256 / HEADS, TPT = TOK / TPR;                     // softmax: threads per head, tokens per thread
-  const int srow = tid / TPR, ssub = tid % TPR;
-  while (t < desc.t1 && !dead) {
-    while (t >= cs.tp1 && cs.b + 1 < p.num_seqs) next_seq(cs);
-    const int seg_end = min(desc.t1, cs.tp1), b = cs.b;
-    const bool whole = t == cs.tp0 && seg_end == cs.tp1;
+  const int srow = gt / TPR, ssub = gt % TPR, mi = lane >> 3;
+  while (seg < total) {
+    while (desc.t0 + seg >= cs.tp1 && cs.b + 1 < p.num_seqs) next_seq(cs);
+    const int seg_end = min(desc.t1, cs.tp1) - desc.t0, b = cs.b;
+    const bool whole = desc.t0 + seg == cs.tp0 && desc.t0 + seg_end == cs.tp1;
     __syncthreads();                                                    // the queries of the sequence before have been read
-    for (int e = tid; e < HEADS * (W / 8); e += 256) {
+    for (int e = tid; e < HEADS * (W / 8); e += 512) {
       const int h = e / (W / 8), v = e % (W / 8);
       uint4 x = make_uint4(0u, 0u, 0u, 0u);
       if (h < nheads) x = *reinterpret_cast<const uint4*>(p.q + b * p.q_stride + (head0 + h) * p.q_head_stride + v * 8);
       *reinterpret_cast<uint4*>(q_s + h * C::QROW + v * 16) = x;
+    }
+    __syncthreads();
+    const uint32_t qrow = q_base + ((lane & 7) + (mi & 1) * 8) * C::QROW + (lane >> 4) * 16 + kq * RH * 32;
+    uint32_t qa[MT == 1 ? RH : 1][4];                                   // one head tile: its query fragments stay in registers
+    if constexpr (MT == 1) {
+#pragma unroll
+      for (int k = 0; k < RH; ++k) ldmatrix_x4(qa[k], qrow + k * 32);
     }
     float o[MT][RH][4];
 #pragma unroll
@@ -264,24 +290,24 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
       for (int n = 0; n < RH; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
     float m_run = -INFINITY, l_run = 0.f;
 
-    for (; t < seg_end; ++t) {
-      const int st = ncomp % NST;
-      const bool ok = mbar_wait(&full[st], (ncomp / NST) & 1);
-      if (!__syncthreads_and(ok)) {                                     // (also: everyone is done with the tile before)
-        if (!ok) report(p.dev_status, kDevWaitTimeout, ncomp);
+    for (; i < seg_end; i += 2) {
+      if (dead) continue;
+      const int st = i % NST;
+      const bool ok = mbar_wait(&full[st], (i / NST) & 1);
+      if (!group_all(group, ok)) {                                      // (also: the group is done with its tile before)
+        if (!ok) report(p.dev_status, kDevWaitTimeout, i);
         dead = true;
-        break;
+        continue;
       }
-      ++ncomp;
-      if (warp == 0) fetch_next();
+      if (warp == 0 && i >= 2) fetch(i - 2 + NST);                      // into the stage that tile has left
       const uint32_t stage = base + st * C::STAGE;
-      const int token0 = (t - cs.tp0) * TOK, valid = cs.n - token0;
+      const int token0 = (desc.t0 + i - cs.tp0) * TOK, valid = cs.n - token0;
       if (valid < TOK) {                                                // rows behind the end may hold anything: zero them
-        for (int e = tid; e < (TOK - valid) * RH * 8; e += 256) {
+        for (int e = gt; e < (TOK - valid) * RH * 8; e += 256) {
           const int r = valid + e / (RH * 8), k = e % (RH * 8);
           *reinterpret_cast<uint4*>(base_ptr + st * C::STAGE + (k >> 3) * C::HALF + r * 128 + (k & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
-        __syncthreads();
+        group_sync(group);
       }
       {                                                                 // scores
         float s[MT][2][4];
@@ -289,114 +315,151 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
         for (int m = 0; m < MT; ++m)
 #pragma unroll
           for (int n = 0; n < 2; ++n) s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f;
-        const int mi = lane >> 3, tok = tg * 16 + (lane & 7) + (mi >> 1) * 8;
+        const int tok = tg * 16 + (lane & 7) + (mi >> 1) * 8;
         const uint32_t trow = stage + tok * 128;
-        const uint32_t qrow = q_base + ((lane & 7) + (mi & 1) * 8) * C::QROW + (lane >> 4) * 16;
 #pragma unroll
-        for (int k = 0; k < RH * 2; ++k) {
-          const int ks = kh * RH * 2 + k, chunk = ks * 2 + (mi & 1);
+        for (int k = 0; k < RH; ++k) {
+          const int chunk = (kq * RH + k) * 2 + (mi & 1);
           uint32_t cb[4];
           ldmatrix_x4(cb, trow + (chunk >> 3) * C::HALF + (((chunk & 7) ^ (tok & 7)) << 4));
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
-            uint32_t a[4];
-            ldmatrix_x4(a, qrow + m * 16 * C::QROW + ks * 32);
-            mma_bf16_16816(s[m][0], a, cb[0], cb[1]);
-            mma_bf16_16816(s[m][1], a, cb[2], cb[3]);
+            if constexpr (MT == 1) {
+              mma_bf16_16816(s[0][0], qa[k], cb[0], cb[1]);
+              mma_bf16_16816(s[0][1], qa[k], cb[2], cb[3]);
+            } else {
+              uint32_t a[4];
+              ldmatrix_x4(a, qrow + m * 16 * C::QROW + k * 32);
+              mma_bf16_16816(s[m][0], a, cb[0], cb[1]);
+              mma_bf16_16816(s[m][1], a, cb[2], cb[3]);
+            }
           }
         }
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
           for (int n = 0; n < 2; ++n) {
-            float* d = s_s + (kh * HEADS + m * 16 + (lane >> 2)) * C::SROW + tg * 16 + n * 8 + (lane & 3) * 2;
+            float* d = s_s + (kq * HEADS + m * 16 + (lane >> 2)) * C::SROW + tg * 16 + n * 8 + (lane & 3) * 2;
             *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
             *reinterpret_cast<float2*>(d + 8 * C::SROW) = make_float2(s[m][n][2], s[m][n][3]);
           }
       }
-      __syncthreads();
+      group_sync(group);
       {                                                                 // softmax
         float x[TPT], top = -INFINITY;
         const float* r0 = s_s + srow * C::SROW + ssub * TPT;
-        const float* r1 = r0 + HEADS * C::SROW;
 #pragma unroll
-        for (int i = 0; i < TPT; i += 4) {
-          const float4 a = *reinterpret_cast<const float4*>(r0 + i), d = *reinterpret_cast<const float4*>(r1 + i);
-          x[i] = a.x + d.x; x[i + 1] = a.y + d.y; x[i + 2] = a.z + d.z; x[i + 3] = a.w + d.w;
+        for (int j = 0; j < TPT; j += 2) {
+          float2 a = *reinterpret_cast<const float2*>(r0 + j);
+#pragma unroll
+          for (int k = 1; k < 4; ++k) {
+            const float2 d = *reinterpret_cast<const float2*>(r0 + k * HEADS * C::SROW + j);
+            a.x += d.x; a.y += d.y;
+          }
+          x[j] = a.x; x[j + 1] = a.y;
         }
 #pragma unroll
-        for (int i = 0; i < TPT; ++i) {
-          x[i] = ssub * TPT + i < valid ? x[i] * p.scale_log2 : -INFINITY;
-          top = fmaxf(top, x[i]);
+        for (int j = 0; j < TPT; ++j) {
+          x[j] = ssub * TPT + j < valid ? x[j] * p.scale_log2 : -INFINITY;
+          top = fmaxf(top, x[j]);
         }
 #pragma unroll
         for (int off = 1; off < TPR; off <<= 1) top = fmaxf(top, __shfl_xor_sync(FULL, top, off));
         const float m_new = fmaxf(m_run, top), alpha = fast_exp2(m_run - m_new);      // (a tile has a visible token: m_new is finite)
         float sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < TPT; ++i) { x[i] = fast_exp2(x[i] - m_new); sum += x[i]; }
+        for (int j = 0; j < TPT; ++j) { x[j] = fast_exp2(x[j] - m_new); sum += x[j]; }
 #pragma unroll
         for (int off = 1; off < TPR; off <<= 1) sum += __shfl_xor_sync(FULL, sum, off);
         l_run = l_run * alpha + sum;
         m_run = m_new;
 #pragma unroll
-        for (int i = 0; i < TPT; i += 4)
-          *reinterpret_cast<uint2*>(p_s + srow * C::PROW + (ssub * TPT + i) * 2) = make_uint2(pack_bf16(x[i], x[i + 1]), pack_bf16(x[i + 2], x[i + 3]));
+        for (int j = 0; j < TPT; j += 2)
+          *reinterpret_cast<uint32_t*>(p_s + srow * C::PROW + (ssub * TPT + j) * 2) = pack_bf16(x[j], x[j + 1]);
         if (ssub == 0) alpha_s[srow] = alpha;
       }
-      __syncthreads();
+      group_sync(group);
       {                                                                 // output
-        uint32_t pa[MT][4][4];
-        const uint32_t prow = p_base + ((lane & 7) + ((lane >> 3) & 1) * 8) * C::PROW + (lane >> 4) * 16;
+        uint32_t pa[MT][2][4];
+        const uint32_t prow = p_base + ((lane & 7) + (mi & 1) * 8) * C::PROW + (lane >> 4) * 16;
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           const float a0 = alpha_s[m * 16 + (lane >> 2)], a1 = alpha_s[m * 16 + (lane >> 2) + 8];
 #pragma unroll
+          for (int k = 0; k < 2; ++k) ldmatrix_x4(pa[m][k], prow + m * 16 * C::PROW + k * 32);
+#pragma unroll
           for (int n = 0; n < RH; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
-#pragma unroll
-          for (int k = 0; k < 4; ++k) ldmatrix_x4(pa[m][k], prow + m * 16 * C::PROW + k * 32);
         }
+        const uint32_t trow = stage + lane * 128;                       // a lane addresses its token: two 16-token steps
 #pragma unroll
-        for (int k = 0; k < 4; k += 2) {
-          const int tok = k * 16 + lane;                                // 32 tokens: two 16-token steps
-          const uint32_t trow = stage + tok * 128;
+        for (int n = 0; n < RH; ++n) {
+          const int chunk = warp * RH + n;
+          uint32_t cb[4];
+          ldmatrix_x4_trans(cb, trow + (chunk >> 3) * C::HALF + (((chunk & 7) ^ (lane & 7)) << 4));
 #pragma unroll
-          for (int n = 0; n < RH; ++n) {
-            const int chunk = warp * RH + n;
-            uint32_t cb[4];
-            ldmatrix_x4_trans(cb, trow + (chunk >> 3) * C::HALF + (((chunk & 7) ^ (tok & 7)) << 4));
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-              mma_bf16_16816(o[m][n], pa[m][k], cb[0], cb[1]);
-              mma_bf16_16816(o[m][n], pa[m][k + 1], cb[2], cb[3]);
-            }
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16_16816(o[m][n], pa[m][0], cb[0], cb[1]);
+            mma_bf16_16816(o[m][n], pa[m][1], cb[2], cb[3]);
           }
         }
       }
     }
-    if (dead) break;
-    // ---- end of the segment: output, or a partial result ----
+    // ---- end of the segment: the groups meet (half of the columns at a time), then output or a partial result ----
     if (ssub == 0) { l_s[srow] = l_run; m_s[srow] = m_run; }
     __syncthreads();
     const int part = b == first_b ? 0 : 1;
+    auto row_weights = [&](int h, float& w0, float& w1, float& m, float& l) {          // of the groups' O in the result
+      const float m0 = rows_s[2 * HEADS + h], m1 = rows_s[5 * HEADS + h];
+      m = fmaxf(m0, m1);
+      w0 = m0 == -INFINITY ? 0.f : fast_exp2(m0 - m);
+      w1 = m1 == -INFINITY ? 0.f : fast_exp2(m1 - m);
+      l = rows_s[HEADS + h] * w0 + rows_s[4 * HEADS + h] * w1;
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      w0 *= inv; w1 *= inv;
+    };
+#pragma unroll 1
+    for (int half = 0; half < 2; ++half) {
+      const int wl = warp - half * 4;
+      const bool mine = wl >= 0 && wl < 4;
+      if (group == 1 && mine) {
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+        for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int h = m * 16 + (lane >> 2) + r * 8;
-        if (h >= nheads) continue;
-        const float inv = l_s[h] > 0.f ? 1.f / l_s[h] : 0.f;
+          for (int r = 0; r < 2; ++r)
 #pragma unroll
-        for (int n = 0; n < RH; ++n) {
-          const int col = (warp * RH + n) * 8 + (lane & 3) * 2;
-          const float x = o[m][n][2 * r] * inv, y = o[m][n][2 * r + 1] * inv;
-          if (whole) *reinterpret_cast<uint32_t*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) = pack_bf16(x, y);
-          else *reinterpret_cast<float2*>(p.part_o + ((static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + h) * W + col) = make_float2(x, y);
-        }
+            for (int n = 0; n < RH; ++n)
+              *reinterpret_cast<float2*>(scores + (m * 16 + (lane >> 2) + r * 8) * (W / 2) + (wl * RH + n) * 8 + (lane & 3) * 2) =
+                  make_float2(o[m][n][2 * r], o[m][n][2 * r + 1]);
       }
+      __syncthreads();
+      if (group == 0 && mine) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const int h = m * 16 + (lane >> 2) + r * 8;
+            if (h >= nheads) continue;
+            float w0, w1, mm, ll;
+            row_weights(h, w0, w1, mm, ll);
+#pragma unroll
+            for (int n = 0; n < RH; ++n) {
+              const float2 other = *reinterpret_cast<const float2*>(scores + h * (W / 2) + (wl * RH + n) * 8 + (lane & 3) * 2);
+              const int col = (warp * RH + n) * 8 + (lane & 3) * 2;
+              const float x = o[m][n][2 * r] * w0 + other.x * w1, y = o[m][n][2 * r + 1] * w0 + other.y * w1;
+              if (whole) *reinterpret_cast<uint32_t*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) = pack_bf16(x, y);
+              else *reinterpret_cast<float2*>(p.part_o + ((static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + h) * W + col) = make_float2(x, y);
+            }
+          }
+      }
+      __syncthreads();
+    }
     if (!whole) {
       __shared__ int is_last;
-      if (tid < nheads) p.part_lse[(static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + tid] = m_s[tid] + log2f(l_s[tid]);
+      if (tid < nheads) {
+        float w0, w1, m, l;
+        row_weights(tid, w0, w1, m, l);
+        p.part_lse[(static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + tid] = l > 0.f ? m + log2f(l) : -INFINITY;
+      }
       const int per = desc.per, c1 = cs.tp0 / per, c2 = (cs.tp1 - 1) / per, nparts = c2 - c1 + 1;
       // the CTA barrier orders every thread's partial stores before thread 0's release; the last arriver's acquire plus its CTA
       // barrier order them before every merging thread's loads
@@ -414,36 +477,34 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
         auto part_index = [&](int j, int h) -> int64_t {
           return ((static_cast<int64_t>(c1 + j) * 2 + (j > 0 || first_is_head ? 0 : 1)) * p.heads) + head0 + h;
         };
-        constexpr int PC = 32;                                          // parts weighted per pass, in the score buffer
-        for (int e = tid; e < nheads; e += 256) {
-          float top = -INFINITY;
+        constexpr int PC = 32;                                          // parts weighted per pass, in the score buffers
+        float *top_s = rows_s, *inv_s = rows_s + HEADS;
+        for (int e = tid; e < nheads; e += 512) {
+          float top = -INFINITY, sum = 0.f;
           for (int j = 0; j < nparts; ++j) top = fmaxf(top, __ldcg(p.part_lse + part_index(j, e)));
-          m_s[e] = top;
-          l_s[e] = 0.f;
+          for (int j = 0; j < nparts; ++j) sum += top == -INFINITY ? 0.f : fast_exp2(__ldcg(p.part_lse + part_index(j, e)) - top);
+          top_s[e] = top;
+          inv_s[e] = sum > 0.f ? 1.f / sum : 0.f;
         }
         __syncthreads();
-        for (int e = tid; e < nheads; e += 256) {
-          float sum = 0.f;
-          for (int j = 0; j < nparts; ++j) sum += fast_exp2(__ldcg(p.part_lse + part_index(j, e)) - m_s[e]);
-          l_s[e] = 1.f / sum;
-        }
-        __syncthreads();
-        constexpr int ITEMS = (HEADS * W / 4 + 255) / 256;
+        constexpr int ITEMS = (HEADS * W / 4 + 511) / 512;
         float4 acc[ITEMS];
 #pragma unroll
         for (int k = 0; k < ITEMS; ++k) acc[k] = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int p0 = 0; p0 < nparts; p0 += PC) {
           const int pn = min(PC, nparts - p0);
-          for (int e = tid; e < pn * nheads; e += 256)
-            s_s[e] = fast_exp2(__ldcg(p.part_lse + part_index(p0 + e / nheads, e % nheads)) - m_s[e % nheads]) * l_s[e % nheads];
+          for (int e = tid; e < pn * nheads; e += 512) {
+            const int h = e % nheads;
+            scores[e] = inv_s[h] == 0.f ? 0.f : fast_exp2(__ldcg(p.part_lse + part_index(p0 + e / nheads, h)) - top_s[h]) * inv_s[h];
+          }
           __syncthreads();
 #pragma unroll
           for (int k = 0; k < ITEMS; ++k) {
-            const int it = tid + k * 256, h = it * 4 / W, col = it * 4 % W;
+            const int it = tid + k * 512, h = it * 4 / W, col = it * 4 % W;
             if (h >= nheads) continue;
 #pragma unroll 4
             for (int j = 0; j < pn; ++j) {
-              const float w = s_s[j * nheads + h];
+              const float w = scores[j * nheads + h];
               const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + part_index(p0 + j, h) * W + col));
               acc[k].x = fmaf(w, v.x, acc[k].x); acc[k].y = fmaf(w, v.y, acc[k].y);
               acc[k].z = fmaf(w, v.z, acc[k].z); acc[k].w = fmaf(w, v.w, acc[k].w);
@@ -453,16 +514,17 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const __grid_cons
         }
 #pragma unroll
         for (int k = 0; k < ITEMS; ++k) {
-          const int it = tid + k * 256, h = it * 4 / W, col = it * 4 % W;
+          const int it = tid + k * 512, h = it * 4 / W, col = it * 4 % W;
           if (h < nheads)
             *reinterpret_cast<uint2*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) =
                 make_uint2(pack_bf16(acc[k].x, acc[k].y), pack_bf16(acc[k].z, acc[k].w));
         }
       }
     }
+    seg = seg_end;
   }
   if (dead && warp == 0) {                                              // a wait gave up: let the copies in flight land, within bounds
-    for (int i = ncomp; i < nfetch; ++i) mbar_wait(&full[i % NST], (i / NST) & 1, 1u << 16);
+    for (int k = max(0, fetched - NST + 1); k <= fetched; ++k) mbar_wait(&full[k % NST], (k / NST) & 1, 1u << 16);
   }
   zero_empty_rows();
 }
@@ -473,7 +535,7 @@ static int launch_latent_decode(const CUtensorMap& map, const LatentDecodeParams
   struct Tag {};
   const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&latent_decode_kernel<RH, MT>), C::SMEM);
   if (rc != kOk) return rc;
-  latent_decode_kernel<RH, MT><<<dim3(num_ctas, (p.heads + C::HEADS - 1) / C::HEADS), 256, C::SMEM, st>>>(map, p);
+  latent_decode_kernel<RH, MT><<<dim3(num_ctas, (p.heads + C::HEADS - 1) / C::HEADS), 512, C::SMEM, st>>>(map, p);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 template <int RH>

@@ -40,7 +40,7 @@ def _need(t: torch.Tensor, dtype, name: str) -> None:
 
 
 def _heads_contiguous(t: torch.Tensor, name: str) -> None:
-    if t.dim() != 3 or t.stride(2) != 1 or t.stride(1) != t.shape[2]:
+    if t.dim() != 3 or t.stride(2) != 1 or (t.shape[1] != 1 and t.stride(1) != t.shape[2]):
         raise ValueError(f"{name} must be [tokens, heads, head_dim] with contiguous heads")
 
 

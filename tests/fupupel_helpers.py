@@ -2,7 +2,6 @@
 from __future__ import annotations
 
 import copy
-import json
 
 import torch
 
@@ -76,18 +75,3 @@ def tensors(cfg: dict, seed: int = 0, ranks=(6, 10)) -> dict[str, torch.Tensor]:
                     p + "a1": rn(ranks[0], width), p + "a2": rn(r["heads"] * r["dim"], ranks[0]), p + "g1": rn(ranks[1], width),
                     p + "g2": rn(r["heads"] * r["vdim"], ranks[1]), p + "o": rn(width, r["heads"] * r["vdim"])})
     return {k: v.to(torch.bfloat16).contiguous() for k, v in out.items()}
-
-
-def write_checkpoint(path, cfg: dict, weights: dict) -> str:
-    from safetensors.torch import save_file
-    path.mkdir(parents=True, exist_ok=True)
-    (path / "config.json").write_text(json.dumps(cfg))
-    save_file(weights, str(path / "model.safetensors"))
-    return str(path)
-
-
-def row_errors(got: torch.Tensor, want: torch.Tensor) -> torch.Tensor:
-    """Per row: RMS difference with the mean taken off, relative to the RMS of all wanted logits."""
-    d = got.double().cpu() - want.double()
-    d = d - d.mean(-1, keepdim=True)
-    return d.pow(2).mean(-1).sqrt() / want.double().pow(2).mean().sqrt()

@@ -13,7 +13,8 @@ from mini_vllm_b200.kvcache.state_slots import StateSlots
 from mini_vllm_b200.scheduler.batch import Batch
 from mini_vllm_b200.scheduler.scheduler import Scheduler
 from oracle import fupupel as plain
-from tests.fupupel_helpers import CONFIGS, both_layer, config, scan_layer, tensors, write_checkpoint
+from tests.fupupel_helpers import CONFIGS, both_layer, config, scan_layer, tensors
+from tests.replay_helpers import write_checkpoint
 from tests.test_host_engine_loop import StandInExecutor, make_engine
 
 

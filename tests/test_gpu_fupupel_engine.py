@@ -8,7 +8,8 @@ import torch
 
 from mini_vllm_b200.config import Config, SamplingParams
 from oracle.fupupel import OracleFupupel
-from tests.fupupel_helpers import CONFIGS, both_layer, config, row_errors, scan_layer, tensors, write_checkpoint
+from tests.fupupel_helpers import CONFIGS, both_layer, config, scan_layer, tensors
+from tests.replay_helpers import assert_tokens, feed, make_engine, portions, row_errors, write_checkpoint
 
 pytestmark = pytest.mark.gpu
 BF, F32 = torch.bfloat16, torch.float32
@@ -29,12 +30,6 @@ def reference(name):
     return cfg, w, prompts, [model.forward(p) for p in prompts]
 
 
-def make_engine(path, dtype, blocks=12, slots=4, seqs=4, **extra):
-    from mini_vllm_b200.engine.engine import Engine
-    return Engine(Config(model=path, dtype=dtype, kv_cache_num_blocks=blocks, kv_cache_block_size=128, max_model_len=1024,
-                         max_num_batched_seqs=seqs, num_state_slots=slots, gpu_memory_utilization=0.5, **extra))
-
-
 @pytest.fixture(scope="module", params=[(n, d) for n in CONFIGS for d in (BF, F32)], ids=lambda p: f"{p[0]}-{str(p[1])[6:]}")
 def served(request, cuda, tmp_path_factory):
     name, dtype = request.param
@@ -43,38 +38,6 @@ def served(request, cuda, tmp_path_factory):
     yield eng, dtype, ref
     del eng
     torch.cuda.empty_cache()
-
-
-def feed(eng, prompts, plan):
-    """Runs a plan - steps of (prompt index, number of tokens) - and returns each prompt's logits; a prompt fed to its end
-    gives its memory back at once."""
-    from mini_vllm_b200.engine.request import Request
-    live, at, got = {}, {}, {}
-    for step in plan:
-        entries = []
-        for i, n in step:
-            lo = at.get(i, 0)
-            at[i] = lo + n
-            entries.append((live.setdefault(i, Request([])), prompts[i][lo:lo + n], list(range(n))))
-        out, row = eng.replay_step(entries).cpu(), 0
-        for i, n in step:
-            got.setdefault(i, []).append(out[row:row + n])
-            row += n
-            if at[i] == len(prompts[i]):
-                eng.release(live.pop(i))
-                at.pop(i)
-    eng.executor.check_device_status()
-    bm = eng.scheduler.block_manager
-    if not live:                                                     # everything was given back
-        assert bm.num_free_blocks == bm.capacity and bm.state_slots.num_free == bm.state_slots.capacity
-    return {i: torch.cat(v) for i, v in got.items()}
-
-
-def portions(n, sizes):
-    out = []
-    while sum(out) < n:
-        out.append(min(sizes[len(out) % len(sizes)], n - sum(out)))
-    return out
 
 
 def check(got, want, dtype):
@@ -187,18 +150,6 @@ def greedy_case(n, seed, lens, new):
     prompts = [[rnd.randrange(70) for _ in range(rnd.choice(lens))] for _ in range(n)]
     model = OracleFupupel(w, cfg)
     return cfg, w, prompts, [model.greedy(p, new) for p in prompts]
-
-
-def assert_tokens(got, want, margin):
-    """Equal until the oracle's own two best logits come closer than rounding can keep apart."""
-    compared = 0
-    for toks, (ref, margins) in zip(got, want):
-        for t, r, m in zip(toks, ref, margins):
-            if m < margin:
-                break
-            assert t == r
-            compared += 1
-    return compared
 
 
 @pytest.mark.parametrize("dtype,margin", [(F32, 1e-3), (BF, 0.5)])
