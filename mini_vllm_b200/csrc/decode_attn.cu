@@ -35,6 +35,8 @@
 
 namespace mvb {
 
+constexpr int kMergeTiles = 4;        // what a partial + arrival + merge costs a CTA, in 64 KB tiles of streaming
+
 template <int D, int HPC>
 struct DecodeCfg {
   static constexpr int NW = (D == 128) ? 8 : 4;       // warps per CTA
@@ -534,7 +536,7 @@ static int decode_plan_impl(const int32_t* cache_seqlens, const int32_t* block_t
   int num_ctas = sm_count();
   if (num_ctas > kMaxCtas) num_ctas = kMaxCtas;
   decode_plan_kernel<<<1, kPlanThreads, 0, static_cast<cudaStream_t>(stream)>>>(
-      cache_seqlens, num_seqs, window_left, cta_tokens_for(num_kv_heads, head_dim), num_ctas,
+      cache_seqlens, num_seqs, window_left, cta_tokens_for(num_kv_heads, head_dim), kMergeTiles, num_ctas,
       num_seqs * num_q_heads, block_table, table_stride, block_size, reinterpret_cast<DecodeHeader*>(ws),
       reinterpret_cast<CtaDesc*>(ws + l.descs), reinterpret_cast<int32_t*>(ws + l.tile_prefix));
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;

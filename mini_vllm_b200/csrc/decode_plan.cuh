@@ -11,7 +11,6 @@ constexpr int kMaxCtas = 160;          // workspace is sized for this many persi
 constexpr int kPlanThreads = 256;
 constexpr int kMinTilesPerCta = 2;
 constexpr int kMaxPartsPerSeq = 32;   // target bound on the partials one sequence is split into
-constexpr int kMergeTiles = 4;        // what a partial + arrival + merge costs a CTA, in 64 KB tiles of streaming
 
 struct DecodeHeader {                  // first 32 bytes of the workspace (device memory)
   int32_t total_tiles, per_cta, num_ctas, cta_tokens, num_seqs, window_left, aligned, pad1;
@@ -50,7 +49,7 @@ __device__ __forceinline__ int visible_start(int n, int window_left) {
 }
 
 static __global__ void __launch_bounds__(kPlanThreads) decode_plan_kernel(const int32_t* __restrict__ cache_seqlens,
-                                                                   int num_seqs, int window_left, int cta_tokens,
+                                                                   int num_seqs, int window_left, int cta_tokens, int merge_tiles,
                                                                    int num_ctas, int num_counters,
                                                                    const int32_t* __restrict__ block_table,
                                                                    int64_t table_stride, int block_size,
@@ -97,7 +96,7 @@ static __global__ void __launch_bounds__(kPlanThreads) decode_plan_kernel(const 
   for (int c = threadIdx.x; c < num_ctas; c += kPlanThreads)
     atomicMax(&max_load_s, aligned_start(c + 1) - aligned_start(c));
   __syncthreads();
-  const bool aligned = total > 0 && max_load_s <= per + kMergeTiles;
+  const bool aligned = total > 0 && max_load_s <= per + merge_tiles;
   if (threadIdx.x == 0) {
     hdr->total_tiles = total; hdr->per_cta = per; hdr->num_ctas = num_ctas; hdr->cta_tokens = cta_tokens;
     hdr->num_seqs = num_seqs; hdr->window_left = window_left; hdr->aligned = aligned ? 1 : 0; hdr->pad1 = 0;

@@ -9,14 +9,14 @@
 //                           cache is loaded once for all of them: the roofline is HBM, sum_b context(b) * width * 2 bytes
 //   gate_mul_kernel         o * sigmoid(gate)
 //
-// latent_decode_kernel: persistent CTAs over the tile ranges of decode_plan.cuh.  A tile = 32 tokens x width in 128-byte-swizzled shared
-// memory, brought by TMA through the block table, up to six tiles deep.  Two groups of eight warps take the tiles in turn, so that one
-// group's barriers and latencies lie under the other's arithmetic; each keeps its own running softmax, and they meet at the end of a
-// sequence.  Per tile and group, three barriers of 256 threads:
-//   scores   S[heads x 32] = Q' C^T     warp = 16 tokens x a quarter of the width (mma.sync, heads in M); the quarters meet in shared memory
+// latent_decode_kernel: persistent CTAs over the tile ranges of decode_plan.cuh, eight working warps and one that fetches.  A tile = 64
+// tokens x width in two halves of 32 tokens, 128-byte-swizzled in shared memory; a half is one TMA copy through the block table (its
+// tensor map has the 64-column blocks of a row as a dimension), and the ring holds NH of them.  Per tile, three barriers of the
+// working warps:
+//   scores   S[heads x 64] = Q' C^T     warp = 32 tokens x a quarter of the width (mma.sync, heads in M; the queries stay in registers);
+//                                       the quarters meet in shared memory
 //   softmax  a few threads per head, running maximum and sum in registers, P as bf16 through shared memory
 //   output   O[heads x width] += P C    warp = an eighth of the width (C again, as transposed fragments), O in registers
-// A stage is filled again by the group that has just read it, so the groups never wait for each other inside a sequence.
 // A sequence that is split between CTAs is merged by the CTA that arrives last, as in decode_attn.cu; nothing waits on another CTA.
 #include "chunk_common.cuh"
 #include "decode_plan.cuh"
@@ -145,20 +145,22 @@ static int launch_gate(const void* o, int64_t os, const void* g, int64_t gs, voi
 }
 
 // ---- decode -----------------------------------------------------------------------------------------------------
-constexpr int kLatentTile = 32;
+constexpr int kLatentTile = 64, kLatentHalf = 32;
+constexpr int kLatentMergeTiles = 12;           // what a partial + arrival + merge costs a CTA, in tiles of streaming (decode_plan.cuh)
 
-template <int RH, int MT>                       // width = 64 RH, 16 MT heads per CTA
+constexpr int kLatentHeads = 16;                // heads per CTA
+
+template <int RH>                               // width = 64 RH
 struct LatentCfg {
-  static constexpr int W = 64 * RH, HEADS = 16 * MT, TOK = kLatentTile;
-  static constexpr int HALF = TOK * 128, STAGE = RH * HALF;             // 32 tokens x 64 columns
-  static constexpr int QROW = W * 2 + 16, SROW = TOK + 4, PROW = TOK * 2 + 16;
-  static constexpr int Q = HEADS * QROW, SB = 4 * HEADS * SROW * 4, P = HEADS * PROW, ROWS = 3 * HEADS * 4;     // (the last three per group)
-  static constexpr int FIXED = Q + 2 * (SB + P + ROWS) + 64;
-  static constexpr int FIT = (226 * 1024 - 1024 - FIXED) / STAGE;
-  static constexpr int NST = FIT > 6 ? 6 : FIT;
-  static constexpr int SMEM = 1024 + NST * STAGE + FIXED;
-  static_assert(NST >= 3, "a tile per group and one in flight at least");
-  static_assert(HEADS * (W / 2) * 4 <= 2 * SB, "half of O fits the score buffers");
+  static constexpr int W = 64 * RH, HEADS = kLatentHeads, TOK = kLatentTile;
+  static constexpr int COLS = kLatentHalf * 128, HALF = RH * COLS;      // 32 tokens x 64 columns; 32 tokens
+  static constexpr int SROW = TOK + 4, PROW = TOK * 2 + 16;
+  static constexpr int SB = 4 * HEADS * SROW * 4, P = HEADS * PROW, ROWS = 3 * HEADS * 4;
+  static constexpr int FIXED = SB + P + ROWS + 128;                     // (eight full and eight empty barriers at most)
+  static constexpr int FIT = (226 * 1024 - 1024 - FIXED) / HALF;
+  static constexpr int NH = FIT > 8 ? 8 : FIT;
+  static constexpr int SMEM = 1024 + NH * HALF + FIXED;
+  static_assert(NH >= 5, "a tile in use and more than one in flight");
 };
 
 struct LatentDecodeParams {
@@ -178,185 +180,173 @@ struct LatentDecodeParams {
 
 struct SeqSpan { int b, tp0, tp1, n; };          // a sequence, its tile range, its length
 
-__device__ __forceinline__ void group_sync(int group) { asm volatile("barrier.cta.sync.aligned %0, 256;" ::"r"(group + 1) : "memory"); }
-__device__ __forceinline__ bool group_all(int group, bool ok) {
+// barriers of the working warps
+__device__ __forceinline__ void workers_sync() { asm volatile("barrier.cta.sync.aligned 1, 256;" ::: "memory"); }
+__device__ __forceinline__ bool workers_all(bool ok) {
   uint32_t r;
   asm volatile(
       "{\n\t.reg .pred p, q;\n\t"
       "setp.ne.u32 q, %1, 0;\n\t"
-      "barrier.cta.red.and.aligned.pred p, %2, 256, q;\n\t"
+      "barrier.cta.red.and.aligned.pred p, 1, 256, q;\n\t"
       "selp.u32 %0, 1, 0, p;\n\t}"
-      : "=r"(r) : "r"(static_cast<uint32_t>(ok)), "r"(group + 1) : "memory");
+      : "=r"(r) : "r"(static_cast<uint32_t>(ok)) : "memory");
   return r != 0;
 }
 
-template <int RH, int MT>
-__global__ void __launch_bounds__(512, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDecodeParams p) {
-  using C = LatentCfg<RH, MT>;
-  constexpr int TOK = C::TOK, NST = C::NST, W = C::W, HEADS = C::HEADS;
+template <int RH>
+__global__ void __launch_bounds__(288, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDecodeParams p) {
+  using C = LatentCfg<RH>;
+  constexpr int TOK = C::TOK, NH = C::NH, W = C::W, HEADS = C::HEADS;
   constexpr uint32_t FULL = 0xffffffffu;
   extern __shared__ uint8_t smem_raw[];
-  const int tid = threadIdx.x, group = tid >> 8, gt = tid & 255, warp = gt >> 5, lane = tid & 31, c = blockIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c = blockIdx.x;
   const int head0 = blockIdx.y * HEADS, nheads = min(HEADS, p.heads - head0);
   const CtaDesc desc = p.descs[c];
-  auto zero_empty_rows = [&]() {
+  auto zero_empty_rows = [&]() {                                        // one warp
     for (int b = c; b < p.num_seqs; b += gridDim.x)
       if (p.cache_seqlens[b] <= 0)
-        for (int e = tid; e < nheads * W; e += 512)
+        for (int e = lane; e < nheads * W; e += 32)
           p.out[b * p.out_stride + (head0 + e / W) * p.out_head_stride + e % W] = __float2bfloat16_rn(0.f);
   };
-  if (desc.t0 >= desc.t1) { zero_empty_rows(); return; }
+  if (desc.t0 >= desc.t1) {
+    if (warp == 0) zero_empty_rows();
+    return;
+  }
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  uint8_t* q_s = base_ptr + NST * C::STAGE;
-  float* scores = reinterpret_cast<float*>(q_s + C::Q);                 // [group][quarter][HEADS][SROW]; also O and weights in a merge
-  uint8_t* p_all = q_s + C::Q + 2 * C::SB;                              // [group][HEADS][PROW bytes]
-  float* rows_s = reinterpret_cast<float*>(p_all + 2 * C::P);           // [group][alpha | l | m][HEADS]
-  uint64_t* full = reinterpret_cast<uint64_t*>(rows_s + 6 * HEADS);
-  float* s_s = scores + group * (C::SB / 4);
-  uint8_t* p_s = p_all + group * C::P;
-  float *alpha_s = rows_s + group * 3 * HEADS, *l_s = alpha_s + HEADS, *m_s = l_s + HEADS;
-  const uint32_t q_base = smem_u32(q_s), p_base = smem_u32(p_s);
+  float* s_s = reinterpret_cast<float*>(base_ptr + NH * C::HALF);       // [quarter][HEADS][SROW]; weights of the parts in a merge
+  uint8_t* p_s = base_ptr + NH * C::HALF + C::SB;                       // [HEADS][PROW bytes]
+  float* alpha_s = reinterpret_cast<float*>(p_s + C::P);                // [HEADS]; behind it the final l and m
+  float *l_s = alpha_s + HEADS, *m_s = l_s + HEADS;
+  uint64_t *full = reinterpret_cast<uint64_t*>(m_s + HEADS), *empty = full + 8;
+  const uint32_t p_base = smem_u32(p_s);
   if (tid == 0) {
     tma_prefetch_desc(&map);
-    for (int i = 0; i < NST; ++i) mbar_init(&full[i], 1);
+    for (int i = 0; i < NH; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); }
     fence_mbar_init();
   }
   __syncthreads();
 
-  // ---- producer: warp 0 of a group; tiles are counted from desc.t0, tile i lives in stage i % NST ----
-  const int total = desc.t1 - desc.t0;
-  SeqSpan fs{desc.b, desc.tp0, desc.tp1, desc.n}, cs = fs;
+  SeqSpan cs{desc.b, desc.tp0, desc.tp1, desc.n};
   auto next_seq = [&](SeqSpan& v) {
     ++v.b; v.tp0 = p.tile_prefix[v.b]; v.tp1 = p.tile_prefix[v.b + 1]; v.n = p.cache_seqlens[v.b];
   };
-  int blk_base = -1, blk_reg = -1, blk_n = 0, fetched = -1;
-  if (desc.blk0 >= 0) { blk_base = (desc.t0 - desc.tp0) * TOK / p.block_size; blk_reg = desc.blk0; blk_n = 1; }
-  auto fetch = [&](int i) {                                             // all lanes; i only grows
-    if (i >= total) return;
-    const int t = desc.t0 + i;
-    while (t >= fs.tp1 && fs.b + 1 < p.num_seqs) { next_seq(fs); blk_base = -1; blk_n = 0; }
-    const int token0 = (t - fs.tp0) * TOK, bi = token0 / p.block_size;
-    if (blk_base < 0 || bi < blk_base || bi >= blk_base + blk_n) {
-      blk_base = bi; blk_n = 32;
-      const int col = bi + lane;
-      blk_reg = col < p.table_width ? p.block_table[fs.b * p.table_stride + col] : -1;
+  // ---- the fetching warp: halves are counted from desc.t0, half i lives in place i % NH ----
+  const int total = 2 * (desc.t1 - desc.t0);
+  if (warp == 8) {
+    int blk_base = -1, blk_reg = -1, blk_n = 0, i = 0;
+    if (desc.blk0 >= 0) { blk_base = (desc.t0 - desc.tp0) * TOK / p.block_size; blk_reg = desc.blk0; blk_n = 1; }
+    for (; i < total; ++i) {
+      const int t = desc.t0 + (i >> 1);
+      while (t >= cs.tp1 && cs.b + 1 < p.num_seqs) { next_seq(cs); blk_base = -1; blk_n = 0; }
+      const int token0 = (t - cs.tp0) * TOK + (i & 1) * kLatentHalf, bi = token0 / p.block_size;
+      if (blk_base < 0 || bi < blk_base || bi >= blk_base + blk_n) {
+        blk_base = bi; blk_n = 32;
+        const int col = bi + lane;
+        blk_reg = col < p.table_width ? p.block_table[cs.b * p.table_stride + col] : -1;
+      }
+      const int blk = __shfl_sync(FULL, blk_reg, bi - blk_base), st = i % NH;
+      int slot0 = -kLatentHalf;                                         // out of range: TMA fills zeros
+      if (blk >= 0 && blk < p.num_blocks) slot0 = blk * p.block_size + (token0 - bi * p.block_size);
+      else if (lane == 0) report(p.dev_status, kDevBadBlock, cs.b);
+      if (i >= NH && !__all_sync(FULL, mbar_wait(&empty[st], (i / NH - 1) & 1))) {      // the working warps have given up
+        if (lane == 0) report(p.dev_status, kDevWaitTimeout, i);
+        break;
+      }
+      if (lane == 0) {
+        mbar_arrive_expect_tx(&full[st], C::HALF);
+        tma_load_3d(base_ptr + st * C::HALF, &map, &full[st], 0, slot0, 0);
+      }
     }
-    const int blk = __shfl_sync(FULL, blk_reg, bi - blk_base);
-    int slot0 = -TOK;                                                   // out of range: TMA fills zeros
-    if (blk >= 0 && blk < p.num_blocks) slot0 = blk * p.block_size + (token0 - bi * p.block_size);
-    else if (lane == 0) report(p.dev_status, kDevBadBlock, fs.b);
-    if (lane == 0) {
-      const int st = i % NST;
-      fence_proxy_async();
-      mbar_arrive_expect_tx(&full[st], C::STAGE);
-#pragma unroll
-      for (int h = 0; h < RH; ++h) tma_load_3d(base_ptr + st * C::STAGE + h * C::HALF, &map, &full[st], h * 64, 0, slot0);
-    }
-    fetched = i;
-  };
-  if (group == 0 && warp == 0)
-    for (int i = 0; i < NST; ++i) fetch(i);
+    if (i < total)                                                      // let the copies in flight land, within bounds
+      for (int k = max(0, i - NH); k < i; ++k) mbar_wait(&full[k % NH], (k / NH) & 1, 1u << 16);
+    zero_empty_rows();
+    return;
+  }
 
   const int first_b = cs.b;
-  int seg = 0, i = group;                                               // first tile of the segment; this group's next tile
-  bool dead = false;
-  const int tg = warp & 1, kq = warp >> 1;                              // scores: 16-token group, quarter of the width
+  int t = 0;                                                            // tile, from desc.t0
+  bool ok = true;
+  const int tg = warp & 1, kq = warp >> 1, mi = lane >> 3;              // scores: half of the tile, quarter of the width
   constexpr int TPR = 256 / HEADS, TPT = TOK / TPR;                     // softmax: threads per head, tokens per thread
-  const int srow = gt / TPR, ssub = gt % TPR, mi = lane >> 3;
-  while (seg < total) {
-    while (desc.t0 + seg >= cs.tp1 && cs.b + 1 < p.num_seqs) next_seq(cs);
+  const int srow = tid / TPR, ssub = tid % TPR, ntiles = total / 2;
+  while (t < ntiles && ok) {
+    while (desc.t0 + t >= cs.tp1 && cs.b + 1 < p.num_seqs) next_seq(cs);
     const int seg_end = min(desc.t1, cs.tp1) - desc.t0, b = cs.b;
-    const bool whole = desc.t0 + seg == cs.tp0 && desc.t0 + seg_end == cs.tp1;
-    __syncthreads();                                                    // the queries of the sequence before have been read
-    for (int e = tid; e < HEADS * (W / 8); e += 512) {
-      const int h = e / (W / 8), v = e % (W / 8);
-      uint4 x = make_uint4(0u, 0u, 0u, 0u);
-      if (h < nheads) x = *reinterpret_cast<const uint4*>(p.q + b * p.q_stride + (head0 + h) * p.q_head_stride + v * 8);
-      *reinterpret_cast<uint4*>(q_s + h * C::QROW + v * 16) = x;
+    const bool whole = desc.t0 + t == cs.tp0 && desc.t0 + seg_end == cs.tp1;
+    uint32_t qa[RH][4];                                             // this warp's quarter of the queries, as first operand
+    {
+      const __nv_bfloat16* q = p.q + b * p.q_stride + static_cast<int64_t>(head0) * p.q_head_stride + kq * RH * 16 + (lane & 3) * 2;
+#pragma unroll
+      for (int k = 0; k < RH; ++k)
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          const int h = (lane >> 2) + (r & 1) * 8;
+          qa[k][r] = h < nheads ? *reinterpret_cast<const uint32_t*>(q + h * p.q_head_stride + k * 16 + (r >> 1) * 8) : 0u;
+        }
     }
-    __syncthreads();
-    const uint32_t qrow = q_base + ((lane & 7) + (mi & 1) * 8) * C::QROW + (lane >> 4) * 16 + kq * RH * 32;
-    uint32_t qa[MT == 1 ? RH : 1][4];                                   // one head tile: its query fragments stay in registers
-    if constexpr (MT == 1) {
+    float o[RH][4];
 #pragma unroll
-      for (int k = 0; k < RH; ++k) ldmatrix_x4(qa[k], qrow + k * 32);
-    }
-    float o[MT][RH][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int n = 0; n < RH; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
+    for (int n = 0; n < RH; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m_run = -INFINITY, l_run = 0.f;
-
-    for (; i < seg_end; i += 2) {
-      if (dead) continue;
-      const int st = i % NST;
-      const bool ok = mbar_wait(&full[st], (i / NST) & 1);
-      if (!group_all(group, ok)) {                                      // (also: the group is done with its tile before)
-        if (!ok) report(p.dev_status, kDevWaitTimeout, i);
-        dead = true;
-        continue;
+    // scores of tile u into s_s; false: its half did not arrive
+    auto scores = [&](int u) -> bool {
+      const int i = 2 * u + tg;
+      const bool here = mbar_wait(&full[i % NH], (i / NH) & 1);
+      const uint32_t half = base + (i % NH) * C::HALF;
+      float s[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+      const int tok = (lane & 7) + (mi >> 1) * 8;
+      const uint32_t trow = half + tok * 128;
+#pragma unroll
+      for (int k = 0; k < RH; ++k) {
+        const int chunk = (kq * RH + k) * 2 + (mi & 1);
+        const uint32_t at = trow + (chunk >> 3) * C::COLS + (((chunk & 7) ^ (tok & 7)) << 4);
+        uint32_t c0[4], c1[4];
+        ldmatrix_x4(c0, at);
+        ldmatrix_x4(c1, at + 16 * 128);
+        mma_bf16_16816(s[0], qa[k], c0[0], c0[1]);
+        mma_bf16_16816(s[1], qa[k], c0[2], c0[3]);
+        mma_bf16_16816(s[2], qa[k], c1[0], c1[1]);
+        mma_bf16_16816(s[3], qa[k], c1[2], c1[3]);
       }
-      if (warp == 0 && i >= 2) fetch(i - 2 + NST);                      // into the stage that tile has left
-      const uint32_t stage = base + st * C::STAGE;
-      const int token0 = (desc.t0 + i - cs.tp0) * TOK, valid = cs.n - token0;
-      if (valid < TOK) {                                                // rows behind the end may hold anything: zero them
-        for (int e = gt; e < (TOK - valid) * RH * 8; e += 256) {
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        float* d = s_s + (kq * HEADS + (lane >> 2)) * C::SROW + tg * 32 + n * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(d) = make_float2(s[n][0], s[n][1]);
+        *reinterpret_cast<float2*>(d + 8 * C::SROW) = make_float2(s[n][2], s[n][3]);
+      }
+      return here;
+    };
+    for (; t < seg_end; ++t) {
+      const bool here = scores(t);
+      ok = workers_all(here);
+      if (!ok) {
+        if (!here) report(p.dev_status, kDevWaitTimeout, t);
+        break;
+      }
+      const int valid = cs.n - (desc.t0 + t - cs.tp0) * TOK;
+      if (valid < TOK) {                                                // rows behind the end may hold anything: zero them for P C
+        for (int e = tid; e < (TOK - valid) * RH * 8; e += 256) {
           const int r = valid + e / (RH * 8), k = e % (RH * 8);
-          *reinterpret_cast<uint4*>(base_ptr + st * C::STAGE + (k >> 3) * C::HALF + r * 128 + (k & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+          *reinterpret_cast<uint4*>(base_ptr + (2 * t + (r >> 5)) % NH * C::HALF + (k >> 3) * C::COLS + (r & 31) * 128 + (k & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
-        group_sync(group);
+        fence_proxy_async();                                            // (a copy will go over them)
       }
-      {                                                                 // scores
-        float s[MT][2][4];
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int n = 0; n < 2; ++n) s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f;
-        const int tok = tg * 16 + (lane & 7) + (mi >> 1) * 8;
-        const uint32_t trow = stage + tok * 128;
-#pragma unroll
-        for (int k = 0; k < RH; ++k) {
-          const int chunk = (kq * RH + k) * 2 + (mi & 1);
-          uint32_t cb[4];
-          ldmatrix_x4(cb, trow + (chunk >> 3) * C::HALF + (((chunk & 7) ^ (tok & 7)) << 4));
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            if constexpr (MT == 1) {
-              mma_bf16_16816(s[0][0], qa[k], cb[0], cb[1]);
-              mma_bf16_16816(s[0][1], qa[k], cb[2], cb[3]);
-            } else {
-              uint32_t a[4];
-              ldmatrix_x4(a, qrow + m * 16 * C::QROW + k * 32);
-              mma_bf16_16816(s[m][0], a, cb[0], cb[1]);
-              mma_bf16_16816(s[m][1], a, cb[2], cb[3]);
-            }
-          }
-        }
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            float* d = s_s + (kq * HEADS + m * 16 + (lane >> 2)) * C::SROW + tg * 16 + n * 8 + (lane & 3) * 2;
-            *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
-            *reinterpret_cast<float2*>(d + 8 * C::SROW) = make_float2(s[m][n][2], s[m][n][3]);
-          }
-      }
-      group_sync(group);
       {                                                                 // softmax
         float x[TPT], top = -INFINITY;
         const float* r0 = s_s + srow * C::SROW + ssub * TPT;
 #pragma unroll
-        for (int j = 0; j < TPT; j += 2) {
-          float2 a = *reinterpret_cast<const float2*>(r0 + j);
+        for (int j = 0; j < TPT; j += 4) {
+          float4 a = *reinterpret_cast<const float4*>(r0 + j);
 #pragma unroll
           for (int k = 1; k < 4; ++k) {
-            const float2 d = *reinterpret_cast<const float2*>(r0 + k * HEADS * C::SROW + j);
-            a.x += d.x; a.y += d.y;
+            const float4 d = *reinterpret_cast<const float4*>(r0 + k * HEADS * C::SROW + j);
+            a.x += d.x; a.y += d.y; a.z += d.z; a.w += d.w;
           }
-          x[j] = a.x; x[j + 1] = a.y;
+          x[j] = a.x; x[j + 1] = a.y; x[j + 2] = a.z; x[j + 3] = a.w;
         }
 #pragma unroll
         for (int j = 0; j < TPT; ++j) {
@@ -369,101 +359,65 @@ __global__ void __launch_bounds__(512, 1) latent_decode_kernel(const __grid_cons
         float sum = 0.f;
 #pragma unroll
         for (int j = 0; j < TPT; ++j) { x[j] = fast_exp2(x[j] - m_new); sum += x[j]; }
-#pragma unroll
-        for (int off = 1; off < TPR; off <<= 1) sum += __shfl_xor_sync(FULL, sum, off);
-        l_run = l_run * alpha + sum;
+        l_run = l_run * alpha + sum;                                    // (of this thread's tokens; the row meets at the end)
         m_run = m_new;
 #pragma unroll
-        for (int j = 0; j < TPT; j += 2)
-          *reinterpret_cast<uint32_t*>(p_s + srow * C::PROW + (ssub * TPT + j) * 2) = pack_bf16(x[j], x[j + 1]);
+        for (int j = 0; j < TPT; j += 4)
+          *reinterpret_cast<uint2*>(p_s + srow * C::PROW + (ssub * TPT + j) * 2) = make_uint2(pack_bf16(x[j], x[j + 1]), pack_bf16(x[j + 2], x[j + 3]));
         if (ssub == 0) alpha_s[srow] = alpha;
       }
-      group_sync(group);
+      workers_sync();
       {                                                                 // output
-        uint32_t pa[MT][2][4];
         const uint32_t prow = p_base + ((lane & 7) + (mi & 1) * 8) * C::PROW + (lane >> 4) * 16;
+        const float a0 = alpha_s[lane >> 2], a1 = alpha_s[(lane >> 2) + 8];
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          const float a0 = alpha_s[m * 16 + (lane >> 2)], a1 = alpha_s[m * 16 + (lane >> 2) + 8];
+        for (int n = 0; n < RH; ++n) { o[n][0] *= a0; o[n][1] *= a0; o[n][2] *= a1; o[n][3] *= a1; }
 #pragma unroll
-          for (int k = 0; k < 2; ++k) ldmatrix_x4(pa[m][k], prow + m * 16 * C::PROW + k * 32);
+        for (int k = 0; k < 2; ++k) {
+          uint32_t pa[2][4];
+          ldmatrix_x4(pa[0], prow + k * 64);
+          ldmatrix_x4(pa[1], prow + k * 64 + 32);
+          const uint32_t trow = base + (2 * t + k) % NH * C::HALF + lane * 128;        // a lane addresses its token: two 16-token steps
 #pragma unroll
-          for (int n = 0; n < RH; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
-        }
-        const uint32_t trow = stage + lane * 128;                       // a lane addresses its token: two 16-token steps
-#pragma unroll
-        for (int n = 0; n < RH; ++n) {
-          const int chunk = warp * RH + n;
-          uint32_t cb[4];
-          ldmatrix_x4_trans(cb, trow + (chunk >> 3) * C::HALF + (((chunk & 7) ^ (lane & 7)) << 4));
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            mma_bf16_16816(o[m][n], pa[m][0], cb[0], cb[1]);
-            mma_bf16_16816(o[m][n], pa[m][1], cb[2], cb[3]);
+          for (int n = 0; n < RH; ++n) {
+            const int chunk = warp * RH + n;
+            uint32_t cb[4];
+            ldmatrix_x4_trans(cb, trow + (chunk >> 3) * C::COLS + (((chunk & 7) ^ (lane & 7)) << 4));
+            mma_bf16_16816(o[n], pa[0], cb[0], cb[1]);
+            mma_bf16_16816(o[n], pa[1], cb[2], cb[3]);
           }
         }
       }
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(&empty[2 * t % NH]); mbar_arrive(&empty[(2 * t + 1) % NH]); }
     }
-    // ---- end of the segment: the groups meet (half of the columns at a time), then output or a partial result ----
+    if (!ok) break;
+    // ---- end of the segment: output, or a partial result ----
+#pragma unroll
+    for (int off = 1; off < TPR; off <<= 1) l_run += __shfl_xor_sync(FULL, l_run, off);
     if (ssub == 0) { l_s[srow] = l_run; m_s[srow] = m_run; }
-    __syncthreads();
+    workers_sync();
     const int part = b == first_b ? 0 : 1;
-    auto row_weights = [&](int h, float& w0, float& w1, float& m, float& l) {          // of the groups' O in the result
-      const float m0 = rows_s[2 * HEADS + h], m1 = rows_s[5 * HEADS + h];
-      m = fmaxf(m0, m1);
-      w0 = m0 == -INFINITY ? 0.f : fast_exp2(m0 - m);
-      w1 = m1 == -INFINITY ? 0.f : fast_exp2(m1 - m);
-      l = rows_s[HEADS + h] * w0 + rows_s[4 * HEADS + h] * w1;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      w0 *= inv; w1 *= inv;
-    };
-#pragma unroll 1
-    for (int half = 0; half < 2; ++half) {
-      const int wl = warp - half * 4;
-      const bool mine = wl >= 0 && wl < 4;
-      if (group == 1 && mine) {
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+    for (int r = 0; r < 2; ++r) {
+      const int h = (lane >> 2) + r * 8;
+      if (h >= nheads) continue;
+      const float inv = l_s[h] > 0.f ? 1.f / l_s[h] : 0.f;
 #pragma unroll
-          for (int r = 0; r < 2; ++r)
-#pragma unroll
-            for (int n = 0; n < RH; ++n)
-              *reinterpret_cast<float2*>(scores + (m * 16 + (lane >> 2) + r * 8) * (W / 2) + (wl * RH + n) * 8 + (lane & 3) * 2) =
-                  make_float2(o[m][n][2 * r], o[m][n][2 * r + 1]);
+      for (int n = 0; n < RH; ++n) {
+        const int col = (warp * RH + n) * 8 + (lane & 3) * 2;
+        const float x = o[n][2 * r] * inv, y = o[n][2 * r + 1] * inv;
+        if (whole) *reinterpret_cast<uint32_t*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) = pack_bf16(x, y);
+        else *reinterpret_cast<float2*>(p.part_o + ((static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + h) * W + col) = make_float2(x, y);
       }
-      __syncthreads();
-      if (group == 0 && mine) {
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int h = m * 16 + (lane >> 2) + r * 8;
-            if (h >= nheads) continue;
-            float w0, w1, mm, ll;
-            row_weights(h, w0, w1, mm, ll);
-#pragma unroll
-            for (int n = 0; n < RH; ++n) {
-              const float2 other = *reinterpret_cast<const float2*>(scores + h * (W / 2) + (wl * RH + n) * 8 + (lane & 3) * 2);
-              const int col = (warp * RH + n) * 8 + (lane & 3) * 2;
-              const float x = o[m][n][2 * r] * w0 + other.x * w1, y = o[m][n][2 * r + 1] * w0 + other.y * w1;
-              if (whole) *reinterpret_cast<uint32_t*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) = pack_bf16(x, y);
-              else *reinterpret_cast<float2*>(p.part_o + ((static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + h) * W + col) = make_float2(x, y);
-            }
-          }
-      }
-      __syncthreads();
     }
     if (!whole) {
       __shared__ int is_last;
-      if (tid < nheads) {
-        float w0, w1, m, l;
-        row_weights(tid, w0, w1, m, l);
-        p.part_lse[(static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + tid] = l > 0.f ? m + log2f(l) : -INFINITY;
-      }
+      if (tid < nheads) p.part_lse[(static_cast<int64_t>(c) * 2 + part) * p.heads + head0 + tid] = m_s[tid] + log2f(l_s[tid]);
       const int per = desc.per, c1 = cs.tp0 / per, c2 = (cs.tp1 - 1) / per, nparts = c2 - c1 + 1;
       // the CTA barrier orders every thread's partial stores before thread 0's release; the last arriver's acquire plus its CTA
       // barrier order them before every merging thread's loads
-      __syncthreads();
+      workers_sync();
       if (tid == 0) {
         int32_t* cnt = p.arrivals + static_cast<int64_t>(b) * gridDim.y + blockIdx.y;
         int prev;
@@ -471,76 +425,78 @@ __global__ void __launch_bounds__(512, 1) latent_decode_kernel(const __grid_cons
         is_last = prev == nparts - 1;
         if (is_last) *cnt = 0;                                          // re-arm for the next launch
       }
-      __syncthreads();
+      workers_sync();
       if (is_last) {
         const bool first_is_head = cs.tp0 % per == 0;                   // does CTA c1's range start at this sequence?
         auto part_index = [&](int j, int h) -> int64_t {
           return ((static_cast<int64_t>(c1 + j) * 2 + (j > 0 || first_is_head ? 0 : 1)) * p.heads) + head0 + h;
         };
-        constexpr int PC = 32;                                          // parts weighted per pass, in the score buffers
-        float *top_s = rows_s, *inv_s = rows_s + HEADS;
-        for (int e = tid; e < nheads; e += 512) {
+        static_assert((kMaxPartsPerSeq + 2) * HEADS <= C::SB / 4, "a weight per part and head fits the score buffer");
+        for (int e = tid; e < nparts * nheads; e += 256) s_s[e] = __ldcg(p.part_lse + part_index(e / nheads, e % nheads));
+        workers_sync();
+        if (tid < nheads) {
           float top = -INFINITY, sum = 0.f;
-          for (int j = 0; j < nparts; ++j) top = fmaxf(top, __ldcg(p.part_lse + part_index(j, e)));
-          for (int j = 0; j < nparts; ++j) sum += top == -INFINITY ? 0.f : fast_exp2(__ldcg(p.part_lse + part_index(j, e)) - top);
-          top_s[e] = top;
-          inv_s[e] = sum > 0.f ? 1.f / sum : 0.f;
+          for (int j = 0; j < nparts; ++j) top = fmaxf(top, s_s[j * nheads + tid]);
+          for (int j = 0; j < nparts; ++j) { const float w = fast_exp2(s_s[j * nheads + tid] - top); s_s[j * nheads + tid] = w; sum += w; }
+          l_s[tid] = 1.f / sum;
         }
-        __syncthreads();
-        constexpr int ITEMS = (HEADS * W / 4 + 511) / 512;
-        float4 acc[ITEMS];
+        workers_sync();
+        constexpr int ITEMS = (HEADS * W / 4 + 255) / 256, GROUP = ITEMS < 8 ? ITEMS : 8;
+#pragma unroll 1
+        for (int k0 = 0; k0 < ITEMS; k0 += GROUP) {
+          float4 acc[GROUP];
 #pragma unroll
-        for (int k = 0; k < ITEMS; ++k) acc[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int p0 = 0; p0 < nparts; p0 += PC) {
-          const int pn = min(PC, nparts - p0);
-          for (int e = tid; e < pn * nheads; e += 512) {
-            const int h = e % nheads;
-            scores[e] = inv_s[h] == 0.f ? 0.f : fast_exp2(__ldcg(p.part_lse + part_index(p0 + e / nheads, h)) - top_s[h]) * inv_s[h];
-          }
-          __syncthreads();
+          for (int k = 0; k < GROUP; ++k) acc[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+          for (int j = 0; j < nparts; ++j) {                            // a part's loads are independent: they pipeline
+            const float* src = p.part_o + part_index(j, 0) * W;
 #pragma unroll
-          for (int k = 0; k < ITEMS; ++k) {
-            const int it = tid + k * 512, h = it * 4 / W, col = it * 4 % W;
-            if (h >= nheads) continue;
-#pragma unroll 4
-            for (int j = 0; j < pn; ++j) {
-              const float w = scores[j * nheads + h];
-              const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + part_index(p0 + j, h) * W + col));
+            for (int k = 0; k < GROUP; ++k) {
+              const int e = (tid + (k0 + k) * 256) * 4, h = e / W;
+              if (h >= nheads) continue;
+              const float w = s_s[j * nheads + h];
+              const float4 v = __ldcg(reinterpret_cast<const float4*>(src + e));
               acc[k].x = fmaf(w, v.x, acc[k].x); acc[k].y = fmaf(w, v.y, acc[k].y);
               acc[k].z = fmaf(w, v.z, acc[k].z); acc[k].w = fmaf(w, v.w, acc[k].w);
             }
           }
-          __syncthreads();
-        }
 #pragma unroll
-        for (int k = 0; k < ITEMS; ++k) {
-          const int it = tid + k * 512, h = it * 4 / W, col = it * 4 % W;
-          if (h < nheads)
-            *reinterpret_cast<uint2*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + col) =
-                make_uint2(pack_bf16(acc[k].x, acc[k].y), pack_bf16(acc[k].z, acc[k].w));
+          for (int k = 0; k < GROUP; ++k) {
+            const int e = (tid + (k0 + k) * 256) * 4, h = e / W;
+            if (h >= nheads) continue;
+            const float w = l_s[h];
+            *reinterpret_cast<uint2*>(p.out + b * p.out_stride + (head0 + h) * p.out_head_stride + e % W) =
+                make_uint2(pack_bf16(acc[k].x * w, acc[k].y * w), pack_bf16(acc[k].z * w, acc[k].w * w));
+          }
         }
       }
     }
-    seg = seg_end;
+    workers_sync();                                                    // l, m and the score buffer are about to be written again
   }
-  if (dead && warp == 0) {                                              // a wait gave up: let the copies in flight land, within bounds
-    for (int k = max(0, fetched - NST + 1); k <= fetched; ++k) mbar_wait(&full[k % NST], (k / NST) & 1, 1u << 16);
-  }
-  zero_empty_rows();
 }
 
-template <int RH, int MT>
+static int head_groups(int heads) { return (heads + kLatentHeads - 1) / kLatentHeads; }
+
+template <int RH>
 static int launch_latent_decode(const CUtensorMap& map, const LatentDecodeParams& p, int num_ctas, cudaStream_t st) {
-  using C = LatentCfg<RH, MT>;
+  using C = LatentCfg<RH>;
   struct Tag {};
-  const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&latent_decode_kernel<RH, MT>), C::SMEM);
+  const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&latent_decode_kernel<RH>), C::SMEM);
   if (rc != kOk) return rc;
-  latent_decode_kernel<RH, MT><<<dim3(num_ctas, (p.heads + C::HEADS - 1) / C::HEADS), 512, C::SMEM, st>>>(map, p);
+  latent_decode_kernel<RH><<<dim3(num_ctas, head_groups(p.heads)), 288, C::SMEM, st>>>(map, p);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
-template <int RH>
-static int launch_latent_width(const CUtensorMap& map, const LatentDecodeParams& p, int num_ctas, cudaStream_t st) {
-  return p.heads <= 16 ? launch_latent_decode<RH, 1>(map, p, num_ctas, st) : launch_latent_decode<RH, 2>(map, p, num_ctas, st);
+// the pool as [64-column blocks, slots, 64 columns], so that one box is 32 tokens with all their columns, block after block
+static int make_latent_map(CUtensorMap* map, const void* base, int64_t rows, int width) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (fn == nullptr) return kNoDriverEntry;
+  const cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(rows), static_cast<cuuint64_t>(width / 64)};
+  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(width) * 2, 128};
+  const cuuint32_t box[3] = {64, kLatentHalf, static_cast<cuuint32_t>(width / 64)}, estr[3] = {1, 1, 1};
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? kOk : kTensorMapFailed;
 }
 
 static bool latent_width_ok(int width) {                                 // the instances there are
@@ -549,7 +505,11 @@ static bool latent_width_ok(int width) {                                 // the 
   return false;
 }
 
-static int plan_ctas() { return sm_count() < kMaxCtas ? sm_count() : kMaxCtas; }
+// the groups of heads share the SMs, so that all of them stream the same ranges at the same time and meet in L2
+static int latent_ctas(int heads) {
+  const int n = (sm_count() < kMaxCtas ? sm_count() : kMaxCtas) / head_groups(heads);
+  return n > 1 ? n : 1;
+}
 
 }  // namespace mvb
 
@@ -602,7 +562,7 @@ extern "C" int mvb_latent_decode_plan(const int32_t* cache_seqlens, const int32_
   if (workspace_bytes < l.total || !is_aligned(workspace, 256)) return kInvalidArgument;
   uint8_t* ws = static_cast<uint8_t*>(workspace);
   decode_plan_kernel<<<1, kPlanThreads, 0, static_cast<cudaStream_t>(stream)>>>(
-      cache_seqlens, num_seqs, -1, kLatentTile, plan_ctas(), num_seqs * num_heads, block_table, table_stride, block_size,
+      cache_seqlens, num_seqs, -1, kLatentTile, kLatentMergeTiles, latent_ctas(num_heads), num_seqs * num_heads, block_table, table_stride, block_size,
       reinterpret_cast<DecodeHeader*>(ws), reinterpret_cast<CtaDesc*>(ws + l.descs), reinterpret_cast<int32_t*>(ws + l.tile_prefix));
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
@@ -620,7 +580,7 @@ extern "C" int mvb_latent_decode(const void* q, int64_t q_row_stride, int64_t q_
   const DecodeLayout l = decode_layout(num_seqs, num_heads, width);
   if (workspace_bytes < l.total || !is_aligned(workspace, 256)) return kInvalidArgument;
   CUtensorMap map;
-  const int rc = make_kv_tensor_map(&map, cache, num_blocks * block_size, 1, width, width, kLatentTile);
+  const int rc = make_latent_map(&map, cache, num_blocks * block_size, width);
   if (rc != kOk) return rc;
   uint8_t* ws = static_cast<uint8_t*>(workspace);
   LatentDecodeParams p{};
@@ -635,13 +595,13 @@ extern "C" int mvb_latent_decode(const void* q, int64_t q_row_stride, int64_t q_
   p.arrivals = reinterpret_cast<int32_t*>(ws + l.tile_prefix) + num_seqs + 1;
   p.dev_status = dev_status;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int n = plan_ctas();
+  const int n = latent_ctas(num_heads);
   switch (width / 64) {
-    case 1: return launch_latent_width<1>(map, p, n, st);
-    case 2: return launch_latent_width<2>(map, p, n, st);
-    case 3: return launch_latent_width<3>(map, p, n, st);
-    case 4: return launch_latent_width<4>(map, p, n, st);
-    case 6: return launch_latent_width<6>(map, p, n, st);
-    default: return launch_latent_width<8>(map, p, n, st);
+    case 1: return launch_latent_decode<1>(map, p, n, st);
+    case 2: return launch_latent_decode<2>(map, p, n, st);
+    case 3: return launch_latent_decode<3>(map, p, n, st);
+    case 4: return launch_latent_decode<4>(map, p, n, st);
+    case 6: return launch_latent_decode<6>(map, p, n, st);
+    default: return launch_latent_decode<8>(map, p, n, st);
   }
 }

@@ -1,13 +1,13 @@
 // Linear attention with decay over chunks of 16 tokens on the tensor cores (ragged steps with bf16 activations).
 //
-// Channel decay: with log-decays summed inside a chunk, G_t = sum_{s <= t} log a_s (per key channel), and the chunk's initial S0:
-//   o_t = (q_t e^{G_t}) S0 + sum_{s <= t} B_ts v_s          B_ts = sum_d q_t k_s e^{G_t - G_s}
-//   S  <- e^{G_16} S0 + sum_s (k_s e^{G_16 - G_s}) v_s^T
+// Channel decay: with A_ts = a_{s+1} .. a_t (per key channel) inside a chunk, and the chunk's initial S0:
+//   o_t = (q_t A_t0) S0 + sum_{s <= t} B_ts v_s             B_ts = sum_d q_t k_s A_ts
+//   S  <- A_{16,0} S0 + sum_s (k_s A_{16,s}) v_s^T
 // Exponential gates: F_t = sum_{s <= t} f_s (a scalar per head), M_t = max_{s <= t} (F_t - F_s + i_s), m_t = max(F_t + m_0, M_t):
 //   o_t = e^{F_t + m_0 - m_t} q_t S0 + e^{M_t - m_t} sum_{s <= t} B_ts v_s          B_ts = (q_t . k_s) e^{F_t - F_s + i_s - M_t}
 //   S  <- e^{F_16 + m_0 - m_16} S0 + e^{M_16 - m_16} sum_s (k_s e^{F_16 - F_s + i_s - M_16}) v_s^T
 // B, M and the scaled keys do not depend on what came before the chunk; only the row factors do, through the one scalar m_0.
-// All exponents are <= 0, whatever the gates are.  The normaliser n is column vdim of S, with value 1.
+// All factors are <= 1, whatever the gates are.  The normaliser n is column vdim of S, with value 1.
 //
 // The prep kernels (parallel over chunks and heads) leave one contiguous record per (chunk, head) with everything the recurrence
 // needs, already in the register order of mma.sync operands.  linear_chunk_scan (sequential over the chunks of a sequence, parallel
@@ -119,8 +119,8 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const L
   extern __shared__ __align__(16) float sm[];
   float* q_s = sm;                               // [16][ROW]
   float* k_s = q_s + kChunk * ROW;
-  float* g_s = k_s + kChunk * ROW;               // log2 of the decay, then its running sum
-  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(g_s + kChunk * ROW);
+  float* a_s = k_s + kChunk * ROW;               // decay factors
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(a_s + kChunk * ROW);
   __shared__ float bm[kChunk][kChunk + 1];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const ChunkSite c = chunk_site(p, blockIdx.x);
@@ -157,36 +157,45 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const L
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
         const int d = i * 32 + lane, x = t * ROW + d;
-        g_s[x] = t < c.n && d < p.dim ? to_log2 * log_sigmoid_of<__nv_bfloat16>(ra[m][i] + bias[i]) : 0.f;
+        a_s[x] = t < c.n && d < p.dim ? fast_exp2(to_log2 * log_sigmoid_of<__nv_bfloat16>(ra[m][i] + bias[i])) : 1.f;
         q_s[x] = rq[m][i] * p.q_scale;
         k_s[x] = rk[m][i];
       }
     }
   }
   __syncthreads();
-  for (int d = tid; d < D32; d += 128) {
-    float run = 0.f;
+  // B below and on the diagonal: a warp takes every fourth column s and walks down the rows with w = k_s a_{s+1} .. a_t in registers,
+  // two rows at a time
+  {
+    float w[4][NI];
 #pragma unroll
-    for (int t = 0; t < kChunk; ++t) { run += g_s[t * ROW + d]; g_s[t * ROW + d] = run; }
-  }
-  __syncthreads();
-  // B below and on the diagonal: a warp takes every fourth row, eight columns at a time (those past the diagonal are not stored)
-  for (int t = warp; t < kChunk; t += 4) {
-    float q[NI], g[NI];
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
-    for (int i = 0; i < NI; ++i) { const int x = t * ROW + i * 32 + lane; q[i] = q_s[x]; g[i] = g_s[x]; }
+      for (int i = 0; i < NI; ++i) w[j][i] = 0.f;
 #pragma unroll 1
-    for (int s0 = 0; s0 <= t; s0 += 8) {
+    for (int t0 = 0; t0 < kChunk; t0 += 2) {
       float v[8];
 #pragma unroll
-      for (int m = 0; m < 8; ++m) {
-        float b = 0.f;
+      for (int r = 0; r < 2; ++r) {
+        const int t = t0 + r, x = t * ROW + lane;
+        float q[NI], a[NI];
 #pragma unroll
-        for (int i = 0; i < NI; ++i) {
-          const int x = (s0 + m) * ROW + i * 32 + lane;
-          b = fmaf(q[i], k_s[x] * fast_exp2(fminf(g[i] - g_s[x], 0.f)), b);
+        for (int i = 0; i < NI; ++i) { q[i] = q_s[x + i * 32]; a[i] = a_s[x + i * 32]; }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int col = warp + 4 * j;          // (the same for the whole warp)
+          if (col == t) {
+#pragma unroll
+            for (int i = 0; i < NI; ++i) w[j][i] = k_s[x + i * 32];
+          } else if (col < t) {
+#pragma unroll
+            for (int i = 0; i < NI; ++i) w[j][i] *= a[i];
+          }
+          float b = 0.f;
+#pragma unroll
+          for (int i = 0; i < NI; ++i) b = fmaf(q[i], w[j][i], b);
+          v[r * 4 + j] = b;
         }
-        v[m] = b;
       }
       // halving exchanges leave lane groups of four with one sum each
       const bool up16 = lane & 16, up8 = lane & 8, up4 = lane & 4;
@@ -206,21 +215,26 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const L
       }
       v[0] += __shfl_xor_sync(0xffffffffu, v[0], 2);
       v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
-      const int sc = s0 + (up16 ? 4 : 0) + (up8 ? 2 : 0) + (up4 ? 1 : 0);
-      if ((lane & 3) == 0 && sc <= t) bm[t][sc] = v[0];
+      if ((lane & 3) == 0) bm[t0 + (up16 ? 1 : 0)][warp + (up8 ? 8 : 0) + (up4 ? 4 : 0)] = v[0];      // (above the diagonal: not read)
     }
   }
   __syncthreads();
   if (warp == 0) write_triangle([&](int t, int s) { return bm[t][s]; }, lane, rec + lay.b);
-  for (int d = tid; d < D32; d += 128) {         // a thread owns a key channel: q e^G and k e^{G_16 - G} in place
-    const float g_end = g_s[(kChunk - 1) * ROW + d];
+  for (int d = tid; d < D32; d += 128) {         // a thread owns a key channel: q times the decay so far, k times what is still to come
+    float a[kChunk], run = 1.f;
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      const float g = g_s[t * ROW + d];
-      q_s[t * ROW + d] *= fast_exp2(g);
-      k_s[t * ROW + d] *= fast_exp2(g_end - g);
+      a[t] = a_s[t * ROW + d];
+      run *= a[t];
+      q_s[t * ROW + d] *= run;
     }
-    if (d < 16 * KS) reinterpret_cast<float*>(rec + lay.extra)[d] = fast_exp2(g_end);
+    if (d < 16 * KS) reinterpret_cast<float*>(rec + lay.extra)[d] = run;
+    run = 1.f;
+#pragma unroll
+    for (int t = kChunk - 1; t >= 0; --t) {
+      k_s[t * ROW + d] *= run;
+      run *= a[t];
+    }
   }
   __syncthreads();
   for (int i = tid; i < KS * 64; i += 128) {
@@ -322,24 +336,30 @@ __global__ void __launch_bounds__(128) exp_chunk_prep(const LinearParams p) {
 }
 
 // ---- the recurrence over chunks ------------------------------------------------------------------------------
-template <bool EXP, int KS, int WARPS>
+// SPLIT warps share a 16-column tile: each keeps the state of its part of the key channels, and the first adds their outputs up one
+// chunk later than they are left in shared memory
+template <bool EXP, int KS, int WARPS, int SPLIT>
 struct LinearScanCfg {
   static constexpr int STAGES = 3;
   static constexpr int SHARED = KS * (EXP ? 512 : 1024) + KS * 1024 + 1024 + (EXP ? 128 : KS * 64);
-  static constexpr int STAGE = SHARED + WARPS * 512;           // common part + a tile of values per warp
-  static constexpr int SMEM = STAGES * STAGE + 64;
-  static_assert(STAGE % 16 == 0, "stages start at multiples of 16 bytes");
+  static constexpr int STAGE = SHARED + WARPS * 512;           // common part + a tile of values per tile
+  static constexpr int SUMS = 2 * WARPS * (SPLIT - 1) * 1024;
+  static constexpr int SMEM = STAGES * STAGE + SUMS + 64;
+  static_assert(STAGE % 16 == 0 && KS % SPLIT == 0, "stages start at multiples of 16 bytes; parts are equal");
 };
 
-template <bool EXP, int KS, int WARPS>
-__global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearParams p) {
-  using C = LinearScanCfg<EXP, KS, WARPS>;
+template <bool EXP, int KS, int WARPS, int SPLIT>
+__global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const LinearParams p) {
+  using C = LinearScanCfg<EXP, KS, WARPS, SPLIT>;
+  constexpr int KP = KS / SPLIT;
   extern __shared__ __align__(128) uint8_t smem[];
-  uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::STAGES * C::STAGE);
-  const int s = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* sums = reinterpret_cast<float*>(smem + C::STAGES * C::STAGE);
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::STAGES * C::STAGE + C::SUMS);
+  const int s = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+  const int tile = (tid >> 5) % WARPS, part = (tid >> 5) / WARPS;
   const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin;
   if (n_tok <= 0) return;
-  const int n_chunks = (n_tok + kChunk - 1) / kChunk, vt = blockIdx.x * WARPS + warp;
+  const int n_chunks = (n_tok + kChunk - 1) / kChunk, vt = blockIdx.x * WARPS + tile;
   const LinearLayout lay = linear_layout(KS, p.vtp, EXP);
   const uint8_t* rec = p.records + (static_cast<int64_t>(chunk_base(begin, s)) * p.heads + h) * lay.total;
   const int64_t rec_step = static_cast<int64_t>(p.heads) * lay.total;
@@ -361,20 +381,20 @@ __global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearPara
 
   const int64_t slot = linear_slot(p, s), hbase = (slot * p.heads + h) * static_cast<int64_t>(p.dim);
   const bool fresh = slot < 0 || p.positions[begin] == 0;
-  const int v0 = vt * 16 + (lane >> 2), dq = (lane & 3) * 2, cols = p.vdim + (EXP ? 1 : 0);
-  float S[2 * KS][4];                             // S^T: rows v0, v0 + 8; columns 8 j + dq, + 1
+  const int v0 = vt * 16 + (lane >> 2), dq = (lane & 3) * 2, d0 = part * KP * 16 + dq, cols = p.vdim + (EXP ? 1 : 0);
+  float S[2 * KP][4];                             // S^T: rows v0, v0 + 8; columns 8 j + d0, + 1
   auto state_at = [&](int j, int i) -> float* {
-    const int64_t row = hbase + 8 * j + dq + (i & 1);
+    const int64_t row = hbase + 8 * j + d0 + (i & 1);
     const int v = v0 + (i & 2) * 4;
     return EXP && v == p.vdim ? p.n + row : p.S + row * p.vp + v;
   };
-  auto in_state = [&](int j, int i) { return 8 * j + dq + (i & 1) < p.dim && v0 + (i & 2) * 4 < cols; };
+  auto in_state = [&](int j, int i) { return 8 * j + d0 + (i & 1) < p.dim && v0 + (i & 2) * 4 < cols; };
 #pragma unroll
-  for (int j = 0; j < 2 * KS; ++j)
+  for (int j = 0; j < 2 * KP; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) S[j][i] = !fresh && in_state(j, i) ? *state_at(j, i) : 0.f;
   float m = EXP ? p.m0[s * p.heads + h] * kLog2e : 0.f;
-  const bool keeps_m = EXP && blockIdx.x == 0 && warp == 0;
+  const bool keeps_m = EXP && blockIdx.x == 0 && tile == 0 && part == 0;
 
   bool ok = true;
   int c = 0;
@@ -383,23 +403,24 @@ __global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearPara
     ok = mbar_wait(&full[st], (c / C::STAGES) & 1);
     if (!__syncthreads_and(ok)) break;            // (uniform: every thread leaves together)
     const uint8_t* base = smem + st * C::STAGE;
-    const uint4* k_r = reinterpret_cast<const uint4*>(base + lay.k);
-    const uint4* b_r = reinterpret_cast<const uint4*>(base + lay.b);
+    const uint4* k_r = reinterpret_cast<const uint4*>(base + lay.k) + part * KP * 64;
     const float* extra = reinterpret_cast<const float*>(base + lay.extra);
-    const uint4 vw = reinterpret_cast<const uint4*>(base + C::SHARED)[warp * 32 + lane];
+    const uint4 vw = reinterpret_cast<const uint4*>(base + C::SHARED)[tile * 32 + lane];
     const uint32_t v[4] = {vw.x, vw.y, vw.z, vw.w};
     float row_f[2][2], row_b[2][2], alpha = 1.f, beta = 1.f, m_end = 0.f;
     if constexpr (EXP) {
+      if (SPLIT == 1 || part == 0) {
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const int t = n * 8 + dq + i;
-          const float from0 = extra[t] + m, local = extra[kChunk + t], mt = fmaxf(from0, local);
-          row_f[n][i] = p.q_scale * fast_exp2(from0 - mt);
-          row_b[n][i] = fast_exp2(local - mt);
-          if (keeps_m && lane < 4 && c * kChunk + t < n_tok) p.mt[static_cast<int64_t>(begin + c * kChunk + t) * p.heads + h] = mt * kLn2;
-        }
+          for (int i = 0; i < 2; ++i) {
+            const int t = n * 8 + dq + i;
+            const float from0 = extra[t] + m, local = extra[kChunk + t], mt = fmaxf(from0, local);
+            row_f[n][i] = p.q_scale * fast_exp2(from0 - mt);
+            row_b[n][i] = fast_exp2(local - mt);
+            if (keeps_m && lane < 4 && c * kChunk + t < n_tok) p.mt[static_cast<int64_t>(begin + c * kChunk + t) * p.heads + h] = mt * kLn2;
+          }
+      }
       const float from0 = extra[kChunk - 1] + m, local = extra[2 * kChunk - 1];
       m_end = fmaxf(from0, local);
       alpha = fast_exp2(from0 - m_end); beta = fast_exp2(local - m_end);
@@ -409,31 +430,35 @@ __global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearPara
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) oa[n][i] = ob[n][i] = oc[n][i] = 0.f;
+    if (SPLIT == 1 || part == 0) {                // V^T B^T
+      const uint4* b_r = reinterpret_cast<const uint4*>(base + lay.b);
 #pragma unroll
-    for (int n = 0; n < 2; ++n) {                 // V^T B^T
-      const uint4 b = b_r[n * 32 + lane];
-      mma_bf16_16816(oc[n], v, b.x, b.y);
-      mma_bf16_16816(oc[n], v, b.z, b.w);
+      for (int n = 0; n < 2; ++n) {
+        const uint4 b = b_r[n * 32 + lane];
+        mma_bf16_16816(oc[n], v, b.x, b.y);
+        mma_bf16_16816(oc[n], v, b.z, b.w);
+      }
     }
 #pragma unroll
-    for (int ks = 0; ks < KS; ++ks) {             // S0^T Q^T
+    for (int ks = 0; ks < KP; ++ks) {             // S0^T Q^T
       Split a;
       split_tile(S[2 * ks], S[2 * ks + 1], a);
+      const int at = (part * KP + ks) * 64 + lane;
       if constexpr (EXP) {
         const uint2* q_r = reinterpret_cast<const uint2*>(base);
-        const uint2 q0 = q_r[(ks * 2) * 32 + lane], q1 = q_r[(ks * 2 + 1) * 32 + lane];
+        const uint2 q0 = q_r[at], q1 = q_r[at + 32];
         mma_bf16_16816(oa[0], a.hi, q0.x, q0.y); mma_bf16_16816(oa[1], a.hi, q1.x, q1.y);
         mma_bf16_16816(ob[0], a.lo, q0.x, q0.y); mma_bf16_16816(ob[1], a.lo, q1.x, q1.y);
       } else {
         const uint4* q_r = reinterpret_cast<const uint4*>(base);
-        const uint4 q0 = q_r[(ks * 2) * 32 + lane], q1 = q_r[(ks * 2 + 1) * 32 + lane];
+        const uint4 q0 = q_r[at], q1 = q_r[at + 32];
         mma_bf16_16816(oa[0], a.hi, q0.x, q0.y); mma_bf16_16816(oa[1], a.hi, q1.x, q1.y);
         mma_bf16_16816(ob[0], a.hi, q0.z, q0.w); mma_bf16_16816(ob[1], a.hi, q1.z, q1.w);
         mma_bf16_16816(ob[0], a.lo, q0.x, q0.y); mma_bf16_16816(ob[1], a.lo, q1.x, q1.y);
       }
     }
 #pragma unroll
-    for (int j = 0; j < 2 * KS; ++j) {            // S^T <- S^T decay + V^T K
+    for (int j = 0; j < 2 * KP; ++j) {            // S^T <- S^T decay + V^T K
       const uint4 k = k_r[j * 32 + lane];
       if constexpr (EXP) {
         float d[4] = {0.f, 0.f, 0.f, 0.f};
@@ -442,26 +467,42 @@ __global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearPara
 #pragma unroll
         for (int i = 0; i < 4; ++i) S[j][i] = fmaf(beta, d[i], alpha * S[j][i]);
       } else {
-        const float2 g = *reinterpret_cast<const float2*>(extra + 8 * j + dq);
+        const float2 g = *reinterpret_cast<const float2*>(extra + 8 * j + d0);
         S[j][0] *= g.x; S[j][1] *= g.y; S[j][2] *= g.x; S[j][3] *= g.y;
         mma_bf16_16816(S[j], v, k.x, k.y);
         mma_bf16_16816(S[j], v, k.z, k.w);
       }
     }
     m = m_end;
-    __syncthreads();                              // the stage has been read
-    if (tid == 0 && c + C::STAGES < n_chunks) { fence_proxy_async(); fetch(c + C::STAGES); }
+    float4* mine = reinterpret_cast<float4*>(sums) + (((c & 1) * WARPS + tile) * (SPLIT - 1)) * 64 + lane;
+    if (SPLIT > 1 && part > 0) {
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+      for (int n = 0; n < 2; ++n)
+        mine[((part - 1) * 2 + n) * 32] = make_float4(oa[n][0] + ob[n][0], oa[n][1] + ob[n][1], oa[n][2] + ob[n][2], oa[n][3] + ob[n][3]);
+    }
+    __syncthreads();                              // the stage has been read, the sums are there
+    if (tid == 0 && c + C::STAGES < n_chunks) { fence_proxy_async(); fetch(c + C::STAGES); }
+    if (SPLIT > 1 && part > 0) continue;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      float sum[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) sum[i] = oa[n][i] + ob[n][i];
+#pragma unroll
+      for (int k = 0; k < SPLIT - 1; ++k) {
+        const float4 x = mine[(k * 2 + n) * 32];
+        sum[0] += x.x; sum[1] += x.y; sum[2] += x.z; sum[3] += x.w;
+      }
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = c * kChunk + n * 8 + dq + (i & 1), col = v0 + (i & 2) * 4;
         if (t >= n_tok) continue;
         const int64_t th = static_cast<int64_t>(begin + t) * p.heads + h;
-        const float o = EXP ? fmaf(row_f[n][i & 1], oa[n][i] + ob[n][i], row_b[n][i & 1] * oc[n][i]) : (oa[n][i] + ob[n][i]) + oc[n][i];
+        const float o = EXP ? fmaf(row_f[n][i & 1], sum[i], row_b[n][i & 1] * oc[n][i]) : sum[i] + oc[n][i];
         if (col < p.vdim) p.o[th * p.vdim + col] = o;
         else if (EXP && col == p.vdim) p.nq[th] = o;
       }
+    }
   }
   if (c < n_chunks) {                             // a copy did not arrive in time: report it, let those in flight land, keep the old state
     if (!ok) report(p.dev_status, kDevWaitTimeout, c);
@@ -471,7 +512,7 @@ __global__ void __launch_bounds__(WARPS * 32) linear_chunk_scan(const LinearPara
   if (slot < 0) return;
   if (keeps_m && lane == 0) p.m[slot * p.heads + h] = m * kLn2;
 #pragma unroll
-  for (int j = 0; j < 2 * KS; ++j)
+  for (int j = 0; j < 2 * KP; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i)
       if (in_state(j, i)) *state_at(j, i) = S[j][i];
@@ -489,20 +530,24 @@ static int launch_linear_chunks(const LinearParams& p, cudaStream_t st) {
   if (rc != kOk) return rc;
   prep<<<dim3(slots, p.heads), 128, smem, st>>>(p);
   if (cudaGetLastError() != cudaSuccess) return kLaunchFailed;
-  auto scan = [&](auto tag) -> int {
-    constexpr int WARPS = decltype(tag)::value;
-    using C = LinearScanCfg<EXP, KS, WARPS>;
+  auto scan = [&](auto tiles, auto parts) -> int {
+    constexpr int WARPS = decltype(tiles)::value, SPLIT = decltype(parts)::value;
+    using C = LinearScanCfg<EXP, KS, WARPS, SPLIT>;
     struct ScanTag {};
-    const int r = opt_in_dynamic_smem<ScanTag>(reinterpret_cast<const void*>(&linear_chunk_scan<EXP, KS, WARPS>), C::SMEM);
+    auto kernel = &linear_chunk_scan<EXP, KS, WARPS, SPLIT>;
+    const int r = opt_in_dynamic_smem<ScanTag>(reinterpret_cast<const void*>(kernel), C::SMEM);
     if (r != kOk) return r;
-    linear_chunk_scan<EXP, KS, WARPS><<<dim3(p.vtp / WARPS, p.heads, p.num_seqs), WARPS * 32, C::SMEM, st>>>(p);
+    kernel<<<dim3(p.vtp / WARPS, p.heads, p.num_seqs), WARPS * SPLIT * 32, C::SMEM, st>>>(p);
     return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
   };
+  using One = std::integral_constant<int, 1>; using Two = std::integral_constant<int, 2>;
+  using Three = std::integral_constant<int, 3>; using Four = std::integral_constant<int, 4>;
+  using Parts = std::conditional_t<KS % 2 == 0 && KS >= 4, Two, One>;
   switch (linear_warps(p, EXP)) {
-    case 1: return scan(std::integral_constant<int, 1>{});
-    case 2: return scan(std::integral_constant<int, 2>{});
-    case 3: return scan(std::integral_constant<int, 3>{});
-    default: return scan(std::integral_constant<int, 4>{});
+    case 1: return scan(One{}, std::conditional_t<KS % 4 == 0, Four, Parts>{});
+    case 2: return scan(Two{}, Parts{});
+    case 3: return scan(Three{}, Parts{});
+    default: return scan(Four{}, Parts{});
   }
 }
 
