@@ -5,7 +5,7 @@
 //   exponential gates (EXP = true) m' = max(f + m, i);  S <- e^{f + m - m'} S + e^{i - m'} k v^T;  n likewise with k alone;
 //       o = S^T q / (max(|n . q|, e^{-m'}) + 1e-6);  i = cap tanh((raw_i + bias_i) / cap), f = log sigmoid(cap tanh((raw_f + bias_f) / cap))
 //
-// and then o / rms(o) * w * gate function (head_norm.cuh).  Columns of S never mix; n is a column of S whose value is 1.
+// and then o / rms(o) * w * gate function (head_norm.cuh).  Columns of S never mix; n is one more column, whose value is 1.
 // State slots: S [slots, heads, dim, vp] fp32, vp = vdim rounded up to 4; n [slots, heads, dim]; m [slots, heads].
 //
 // One token per sequence (linear_step_kernel): a CTA per (sequence, head); a thread holds RPT rows x 4 columns of S in registers,
@@ -401,7 +401,7 @@ static int run_linear(LinearParams& p, int dtype, bool exp_gates, void* scratch,
   if (p.tokens == 0 || p.num_seqs == 0) return kOk;
   p.vp = (p.vdim + 3) / 4 * 4;
   p.dp = linear_row_pad(p.dim);
-  p.vtp = linear_tiles(p, exp_gates);
+  p.vtp = linear_tiles(p);
   if (p.cu != nullptr) {
     if (!scratch || scratch_bytes < carve_linear_scratch(p, dtype, exp_gates, nullptr) * sizeof(float)) return kInvalidArgument;
     carve_linear_scratch(p, dtype, exp_gates, static_cast<float*>(scratch));
@@ -420,7 +420,7 @@ extern "C" size_t mvb_linear_attn_scratch_bytes(int dtype, int num_tokens, int n
   LinearParams p{};
   p.tokens = num_tokens; p.num_seqs = num_seqs; p.heads = heads; p.dim = dim; p.vdim = vdim;
   p.dp = linear_row_pad(dim);
-  p.vtp = linear_tiles(p, exp_gates != 0);
+  p.vtp = linear_tiles(p);
   return carve_linear_scratch(p, dtype, exp_gates != 0, nullptr) * sizeof(float);
 }
 

@@ -5,14 +5,15 @@
 //   S  <- A_{16,0} S0 + sum_s (k_s A_{16,s}) v_s^T
 // Exponential gates: F_t = sum_{s <= t} f_s (a scalar per head), M_t = max_{s <= t} (F_t - F_s + i_s), m_t = max(F_t + m_0, M_t):
 //   o_t = e^{F_t + m_0 - m_t} q_t S0 + e^{M_t - m_t} sum_{s <= t} B_ts v_s          B_ts = (q_t . k_s) e^{F_t - F_s + i_s - M_t}
-//   S  <- e^{F_16 + m_0 - m_16} S0 + e^{M_16 - m_16} sum_s (k_s e^{F_16 - F_s + i_s - M_16}) v_s^T
+//   S  <- e^{F_16 + m_0 - m_16} S0 + e^{M_16 - m_16} sum_s (k_s e^{F_16 - F_s + i_s - M_16}) v_s^T,    n likewise with v = 1
 // B, M and the scaled keys do not depend on what came before the chunk; only the row factors do, through the one scalar m_0.
-// All factors are <= 1, whatever the gates are.  The normaliser n is column vdim of S, with value 1.
+// All factors are <= 1, whatever the gates are.
 //
 // The prep kernels (parallel over chunks and heads) leave one contiguous record per (chunk, head) with everything the recurrence
 // needs, already in the register order of mma.sync operands.  linear_chunk_scan (sequential over the chunks of a sequence, parallel
 // over heads and 16-column tiles) keeps S^T in the fp32 accumulator registers of one warp per 16 columns, whose fragments are operand
-// fragments of the next product as they stand; records arrive by bulk copies, three chunks ahead.
+// fragments of the next product as they stand; records arrive by bulk copies, several chunks ahead.  With exponential gates one more warp
+// carries the normaliser and the maximum, in plain fp32.
 // v (and, with exponential gates, q) is a bf16 projection and enters exactly; every other operand enters as bf16 high + low part:
 // 16 significant bits per factor with fp32 accumulation.  The state itself is never rounded below fp32.
 #pragma once
@@ -21,20 +22,20 @@
 namespace mvb {
 
 struct LinearLayout {             // bytes inside a record
-  int k, b, extra, v, total;      // q at 0; extra: decay of the chunk per key channel, or F and M of its tokens
+  int k, b, extra, v, total;      // q at 0; extra: decay of the chunk per key channel, or F, M, row sums of B, and sums of scaled keys
 };
 __host__ __device__ inline LinearLayout linear_layout(int ks, int vtp, bool exp_gates) {
   LinearLayout l;
   l.k = ks * (exp_gates ? 512 : 1024);
   l.b = l.k + ks * 1024;
   l.extra = l.b + 1024;
-  l.v = l.extra + (exp_gates ? 128 : ks * 64);
+  l.v = l.extra + (exp_gates ? 192 : 0) + ks * 64;
   l.total = l.v + vtp * 512;
   return l;
 }
 
-static inline int linear_warps(const LinearParams& p, bool exp_gates) {      // 16-column tiles per CTA
-  const int tiles = (p.vdim + (exp_gates ? 1 : 0) + 15) / 16;
+static inline int linear_warps(const LinearParams& p) {       // 16-column tiles per CTA
+  const int tiles = (p.vdim + 15) / 16;
   // few (sequence, head) pairs: one warp per CTA, so that they spread over the SMs
   if (static_cast<int64_t>(tiles) * p.heads * p.num_seqs <= sm_count() * 2) return 1;
   int best = 4;
@@ -42,8 +43,8 @@ static inline int linear_warps(const LinearParams& p, bool exp_gates) {      // 
     if ((tiles + w - 1) / w * w < (tiles + best - 1) / best * best) best = w;
   return tiles == 1 ? 1 : best;
 }
-static inline int linear_tiles(const LinearParams& p, bool exp_gates) {
-  const int tiles = (p.vdim + (exp_gates ? 1 : 0) + 15) / 16, w = linear_warps(p, exp_gates);
+static inline int linear_tiles(const LinearParams& p) {
+  const int tiles = (p.vdim + 15) / 16, w = linear_warps(p);
   return (tiles + w - 1) / w * w;
 }
 
@@ -60,8 +61,8 @@ __device__ __forceinline__ ChunkSite chunk_site(const LinearParams& p, int slot)
 
 __device__ __forceinline__ float bf_at(const void* base, int64_t i) { return __bfloat162float(static_cast<const __nv_bfloat16*>(base)[i]); }
 
-// v of a chunk as [16][cols] bf16 in shared memory: zeros behind the tokens and columns there are, ones in column `one`
-__device__ __forceinline__ void stage_values(const LinearParams& p, const ChunkSite& c, int h, int cols, int one, __nv_bfloat16* v_s) {
+// v of a chunk as [16][cols] bf16 in shared memory: zeros behind the tokens and columns there are
+__device__ __forceinline__ void stage_values(const LinearParams& p, const ChunkSite& c, int h, int cols, __nv_bfloat16* v_s) {
   const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(p.v) + c.row * p.qkv_stride + static_cast<int64_t>(h) * p.vdim;
   if (p.vdim % 8 == 0 && p.qkv_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(p.v) & 15) == 0) {
     const int vec = cols / 8;
@@ -69,13 +70,12 @@ __device__ __forceinline__ void stage_values(const LinearParams& p, const ChunkS
       const int t = e / vec, col = (e % vec) * 8;
       uint4 w = make_uint4(0u, 0u, 0u, 0u);
       if (t < c.n && col < p.vdim) w = *reinterpret_cast<const uint4*>(v + t * p.qkv_stride + col);
-      if (t < c.n && col == one) w.x = 0x3f80u;               // (one = vdim is a multiple of 8 here)
       *reinterpret_cast<uint4*>(v_s + t * cols + col) = w;
     }
   } else {
     for (int e = threadIdx.x; e < kChunk * cols; e += blockDim.x) {
       const int t = e / cols, col = e % cols;
-      v_s[e] = t < c.n && col < p.vdim ? v[t * p.qkv_stride + col] : __float2bfloat16_rn(t < c.n && col == one ? 1.f : 0.f);
+      v_s[e] = t < c.n && col < p.vdim ? v[t * p.qkv_stride + col] : __float2bfloat16_rn(0.f);
     }
   }
 }
@@ -114,7 +114,7 @@ __device__ __forceinline__ void write_keys(const float* k_s, int row, int ks, ui
 
 // ---- channel decay ----------------------------------------------------------------------------------------
 template <int KS>
-__global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const LinearParams p) {
+__global__ void __launch_bounds__(128, KS <= 8 ? 7 : 3) decay_chunk_prep(const LinearParams p) {
   constexpr int D32 = (16 * KS + 31) / 32 * 32, ROW = D32 + 4, NI = D32 / 32;
   extern __shared__ __align__(16) float sm[];
   float* q_s = sm;                               // [16][ROW]
@@ -129,12 +129,12 @@ __global__ void __launch_bounds__(128, KS <= 8 ? 4 : 2) decay_chunk_prep(const L
   uint8_t* rec = p.records + (static_cast<int64_t>(blockIdx.x) * p.heads + h) * lay.total;
 
   // a warp takes every fourth token; the raw operands of U tokens are requested before any is worked on
-  constexpr int U = NI <= 4 ? 4 : 2;
+  constexpr int U = 2;
   const float to_log2 = p.inv_tau * kLog2e;
   float bias[NI];
 #pragma unroll
   for (int i = 0; i < NI; ++i) bias[i] = i * 32 + lane < p.dim ? p.decay_bias[h * p.dim + i * 32 + lane] : 0.f;
-  stage_values(p, c, h, p.vtp * 16, -1, v_s);
+  stage_values(p, c, h, p.vtp * 16, v_s);
 #pragma unroll 1
   for (int tb = warp; tb < kChunk; tb += 4 * U) {
     float rq[U][NI], rk[U][NI], ra[U][NI];
@@ -257,14 +257,14 @@ __global__ void __launch_bounds__(128) exp_chunk_prep(const LinearParams p) {
   extern __shared__ __align__(16) float sm[];
   float* k_s = sm;                               // [16][ROW], scaled
   __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(k_s + kChunk * ROW);
-  __shared__ float part[4][kChunk][kChunk + 1], e_s[kChunk], top_s[kChunk];
+  __shared__ float part[4][kChunk][kChunk + 1], bm[kChunk][kChunk + 1], e_s[kChunk], top_s[kChunk];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const ChunkSite c = chunk_site(p, blockIdx.x);
   if (c.n <= 0) return;
   const LinearLayout lay = linear_layout(KS, p.vtp, true);
   uint8_t* rec = p.records + (static_cast<int64_t>(blockIdx.x) * p.heads + h) * lay.total;
   if (tid == 0 && c.row == p.cu[c.seq]) stash_maximum(p, c.seq, h);
-  stage_values(p, c, h, p.vtp * 16, p.vdim, v_s);
+  stage_values(p, c, h, p.vtp * 16, v_s);
   // gates, every warp for itself (lanes 0..15): F, the running maximum of i - F, and with them M, all in log2 units
   float f = 0.f, i = -INFINITY;
   if (lane < c.n) {
@@ -326,11 +326,28 @@ __global__ void __launch_bounds__(128) exp_chunk_prep(const LinearParams p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) part[warp][(lane >> 2) + (j >> 1) * 8][n * 8 + (lane & 3) * 2 + (j & 1)] = acc[n][j];
   __syncthreads();
-  if (warp == 0)
-    write_triangle([&](int t, int s) {
-      const float dot = (part[0][t][s] + part[1][t][s]) + (part[2][t][s] + part[3][t][s]);
-      return dot * p.q_scale * fast_exp2(e_s[s] - top_s[t]);
-    }, lane, rec + lay.b);
+#pragma unroll
+  for (int x = tid; x < kChunk * kChunk; x += 128) {
+    const int t = x / kChunk, s = x % kChunk;
+    const float dot = (part[0][t][s] + part[1][t][s]) + (part[2][t][s] + part[3][t][s]);
+    bm[t][s] = s <= t ? dot * p.q_scale * fast_exp2(e_s[s] - top_s[t]) : 0.f;
+  }
+  float* extra = reinterpret_cast<float*>(rec + lay.extra);
+  for (int d = tid; d < DP; d += 128) {
+    float sum = 0.f;
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) sum += k_s[t * ROW + d];
+    extra[3 * kChunk + d] = sum;
+  }
+  __syncthreads();
+  if (warp == 0) {
+    write_triangle([&](int t, int s) { return bm[t][s]; }, lane, rec + lay.b);
+  } else if (warp == 1 && lane < kChunk) {
+    float sum = 0.f;
+#pragma unroll
+    for (int s = 0; s < kChunk; ++s) sum += bm[lane][s];
+    extra[2 * kChunk + lane] = sum;
+  }
   write_keys(k_s, ROW, KS, rec + lay.k);
   write_values(v_s, p.vtp * 16, rec + lay.v);
 }
@@ -340,21 +357,25 @@ __global__ void __launch_bounds__(128) exp_chunk_prep(const LinearParams p) {
 // chunk later than they are left in shared memory
 template <bool EXP, int KS, int WARPS, int SPLIT>
 struct LinearScanCfg {
-  static constexpr int STAGES = 3;
-  static constexpr int SHARED = KS * (EXP ? 512 : 1024) + KS * 1024 + 1024 + (EXP ? 128 : KS * 64);
+  static constexpr int SHARED = KS * (EXP ? 512 : 1024) + KS * 1024 + 1024 + (EXP ? 192 : 0) + KS * 64;
+  static constexpr int THREADS = (WARPS * SPLIT + (EXP ? 1 : 0)) * 32;
   static constexpr int STAGE = SHARED + WARPS * 512;           // common part + a tile of values per tile
   static constexpr int SUMS = 2 * WARPS * (SPLIT - 1) * 1024;
-  static constexpr int SMEM = STAGES * STAGE + SUMS + 64;
+  // deep enough for the latency of a record: two CTAs per SM, or one where a CTA is a single tile (few heads and sequences)
+  static constexpr int FIT = ((WARPS == 1 ? 200 : 100) * 1024 - SUMS) / STAGE;
+  static constexpr int STAGES = FIT < 3 ? 3 : FIT > 10 ? 10 : FIT;
+  static constexpr int SMEM = STAGES * STAGE + SUMS + STAGES * 8;
   static_assert(STAGE % 16 == 0 && KS % SPLIT == 0, "stages start at multiples of 16 bytes; parts are equal");
 };
 
 template <bool EXP, int KS, int WARPS, int SPLIT>
-__global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const LinearParams p) {
+__global__ void __launch_bounds__(LinearScanCfg<EXP, KS, WARPS, SPLIT>::THREADS) linear_chunk_scan(const LinearParams p) {
   using C = LinearScanCfg<EXP, KS, WARPS, SPLIT>;
   constexpr int KP = KS / SPLIT;
   extern __shared__ __align__(128) uint8_t smem[];
   float* sums = reinterpret_cast<float*>(smem + C::STAGES * C::STAGE);
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::STAGES * C::STAGE + C::SUMS);
+  __shared__ int dead_s;                          // a copy did not arrive: nobody waits any more, nothing is kept
   const int s = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
   const int tile = (tid >> 5) % WARPS, part = (tid >> 5) / WARPS;
   const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin;
@@ -365,6 +386,7 @@ __global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const Li
   const int64_t rec_step = static_cast<int64_t>(p.heads) * lay.total;
   if (tid == 0) {
     for (int i = 0; i < C::STAGES; ++i) mbar_init(&full[i], 1);
+    dead_s = 0;
     fence_mbar_init();
   }
   __syncthreads();
@@ -381,28 +403,86 @@ __global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const Li
 
   const int64_t slot = linear_slot(p, s), hbase = (slot * p.heads + h) * static_cast<int64_t>(p.dim);
   const bool fresh = slot < 0 || p.positions[begin] == 0;
-  const int v0 = vt * 16 + (lane >> 2), dq = (lane & 3) * 2, d0 = part * KP * 16 + dq, cols = p.vdim + (EXP ? 1 : 0);
+  const int v0 = vt * 16 + (lane >> 2), dq = (lane & 3) * 2, d0 = part * KP * 16 + dq;
+  const bool normaliser = EXP && part == SPLIT;   // the warp behind the tiles
   float S[2 * KP][4];                             // S^T: rows v0, v0 + 8; columns 8 j + d0, + 1
-  auto state_at = [&](int j, int i) -> float* {
-    const int64_t row = hbase + 8 * j + d0 + (i & 1);
-    const int v = v0 + (i & 2) * 4;
-    return EXP && v == p.vdim ? p.n + row : p.S + row * p.vp + v;
+  auto state_at = [&](int j, int i) { return p.S + (hbase + 8 * j + d0 + (i & 1)) * p.vp + v0 + (i & 2) * 4; };
+  auto in_state = [&](int j, int i) { return 8 * j + d0 + (i & 1) < p.dim && v0 + (i & 2) * 4 < p.vdim; };
+  float m = EXP ? p.m0[s * p.heads + h] * kLog2e : 0.f;
+  volatile int* dead = &dead_s;
+  auto arrived = [&](int c) {
+    if (!*dead && !mbar_wait(&full[c % C::STAGES], (c / C::STAGES) & 1)) {
+      *dead = 1;
+      report(p.dev_status, kDevWaitTimeout, c);
+    }
+    __syncwarp();
   };
-  auto in_state = [&](int j, int i) { return 8 * j + d0 + (i & 1) < p.dim && v0 + (i & 2) * 4 < cols; };
+  if (normaliser) {
+    // n at the channels of this lane's query fragments: 16 ks + dq, + 1, + 8, + 9.  The CTA of the first columns has it; the others'
+    // warp keeps step with the barriers
+    const bool works = blockIdx.x == 0;
+    auto channel = [&](int ks, int i) { return ks * 16 + dq + (i & 1) + (i & 2) * 4; };
+    float n[KS][4];
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) n[ks][i] = works && !fresh && channel(ks, i) < p.dim ? p.n[hbase + channel(ks, i)] : 0.f;
+    for (int c = 0; c < n_chunks; ++c) {
+      if (works) {
+        arrived(c);
+        const uint8_t* base = smem + c % C::STAGES * C::STAGE;
+        const float* extra = reinterpret_cast<const float*>(base + lay.extra);
+        const uint2* q_r = reinterpret_cast<const uint2*>(base);
+        const float from0 = extra[kChunk - 1] + m, local = extra[2 * kChunk - 1], m_end = fmaxf(from0, local);
+        const float alpha = fast_exp2(from0 - m_end), beta = fast_exp2(local - m_end);
+        float dot[2] = {0.f, 0.f};                // tokens lane / 4 and lane / 4 + 8
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const uint2 q = q_r[(ks * 2 + r) * 32 + lane];
+            dot[r] = fmaf(bf16_lo(q.x), n[ks][0], dot[r]); dot[r] = fmaf(bf16_hi(q.x), n[ks][1], dot[r]);
+            dot[r] = fmaf(bf16_lo(q.y), n[ks][2], dot[r]); dot[r] = fmaf(bf16_hi(q.y), n[ks][3], dot[r]);
+          }
+          const float* sum = extra + 3 * kChunk + ks * 16 + dq;
+          const float2 lo = *reinterpret_cast<const float2*>(sum), hi = *reinterpret_cast<const float2*>(sum + 8);
+          n[ks][0] = fmaf(beta, lo.x, alpha * n[ks][0]); n[ks][1] = fmaf(beta, lo.y, alpha * n[ks][1]);
+          n[ks][2] = fmaf(beta, hi.x, alpha * n[ks][2]); n[ks][3] = fmaf(beta, hi.y, alpha * n[ks][3]);
+        }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], 1);
+          dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], 2);
+          const int t = r * 8 + (lane >> 2);
+          if ((lane & 3) == 0 && c * kChunk + t < n_tok) {
+            const int64_t th = static_cast<int64_t>(begin + c * kChunk + t) * p.heads + h;
+            const float f0 = extra[t] + m, loc = extra[kChunk + t], mt = fmaxf(f0, loc);
+            p.mt[th] = mt * kLn2;
+            p.nq[th] = fmaf(p.q_scale * fast_exp2(f0 - mt), dot[r], fast_exp2(loc - mt) * extra[2 * kChunk + t]);
+          }
+        }
+        m = m_end;
+      }
+      __syncthreads();
+    }
+    if (works && slot >= 0 && !*dead) {
+      if (lane == 0) p.m[slot * p.heads + h] = m * kLn2;
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (lane < 4 && channel(ks, i) < p.dim) p.n[hbase + channel(ks, i)] = n[ks][i];
+    }
+    return;
+  }
 #pragma unroll
   for (int j = 0; j < 2 * KP; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) S[j][i] = !fresh && in_state(j, i) ? *state_at(j, i) : 0.f;
-  float m = EXP ? p.m0[s * p.heads + h] * kLog2e : 0.f;
-  const bool keeps_m = EXP && blockIdx.x == 0 && tile == 0 && part == 0;
 
-  bool ok = true;
-  int c = 0;
-  for (; c < n_chunks; ++c) {
-    const int st = c % C::STAGES;
-    ok = mbar_wait(&full[st], (c / C::STAGES) & 1);
-    if (!__syncthreads_and(ok)) break;            // (uniform: every thread leaves together)
-    const uint8_t* base = smem + st * C::STAGE;
+  for (int c = 0; c < n_chunks; ++c) {
+    arrived(c);
+    const uint8_t* base = smem + c % C::STAGES * C::STAGE;
     const uint4* k_r = reinterpret_cast<const uint4*>(base + lay.k) + part * KP * 64;
     const float* extra = reinterpret_cast<const float*>(base + lay.extra);
     const uint4 vw = reinterpret_cast<const uint4*>(base + C::SHARED)[tile * 32 + lane];
@@ -418,7 +498,6 @@ __global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const Li
             const float from0 = extra[t] + m, local = extra[kChunk + t], mt = fmaxf(from0, local);
             row_f[n][i] = p.q_scale * fast_exp2(from0 - mt);
             row_b[n][i] = fast_exp2(local - mt);
-            if (keeps_m && lane < 4 && c * kChunk + t < n_tok) p.mt[static_cast<int64_t>(begin + c * kChunk + t) * p.heads + h] = mt * kLn2;
           }
       }
       const float from0 = extra[kChunk - 1] + m, local = extra[2 * kChunk - 1];
@@ -500,17 +579,14 @@ __global__ void __launch_bounds__(WARPS * SPLIT * 32) linear_chunk_scan(const Li
         const int64_t th = static_cast<int64_t>(begin + t) * p.heads + h;
         const float o = EXP ? fmaf(row_f[n][i & 1], sum[i], row_b[n][i & 1] * oc[n][i]) : sum[i] + oc[n][i];
         if (col < p.vdim) p.o[th * p.vdim + col] = o;
-        else if (EXP && col == p.vdim) p.nq[th] = o;
       }
     }
   }
-  if (c < n_chunks) {                             // a copy did not arrive in time: report it, let those in flight land, keep the old state
-    if (!ok) report(p.dev_status, kDevWaitTimeout, c);
-    for (int k = c; k < min(c + C::STAGES, n_chunks); ++k) mbar_wait(&full[k % C::STAGES], (k / C::STAGES) & 1, 1u << 16);
+  if (*dead) {                                    // let the copies in flight land, within bounds; keep the old state
+    for (int k = max(0, n_chunks - C::STAGES); k < n_chunks; ++k) mbar_wait(&full[k % C::STAGES], (k / C::STAGES) & 1, 1u << 16);
     return;
   }
   if (slot < 0) return;
-  if (keeps_m && lane == 0) p.m[slot * p.heads + h] = m * kLn2;
 #pragma unroll
   for (int j = 0; j < 2 * KP; ++j)
 #pragma unroll
@@ -537,13 +613,13 @@ static int launch_linear_chunks(const LinearParams& p, cudaStream_t st) {
     auto kernel = &linear_chunk_scan<EXP, KS, WARPS, SPLIT>;
     const int r = opt_in_dynamic_smem<ScanTag>(reinterpret_cast<const void*>(kernel), C::SMEM);
     if (r != kOk) return r;
-    kernel<<<dim3(p.vtp / WARPS, p.heads, p.num_seqs), WARPS * SPLIT * 32, C::SMEM, st>>>(p);
+    kernel<<<dim3(p.vtp / WARPS, p.heads, p.num_seqs), C::THREADS, C::SMEM, st>>>(p);
     return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
   };
   using One = std::integral_constant<int, 1>; using Two = std::integral_constant<int, 2>;
   using Three = std::integral_constant<int, 3>; using Four = std::integral_constant<int, 4>;
   using Parts = std::conditional_t<KS % 2 == 0 && KS >= 4, Two, One>;
-  switch (linear_warps(p, EXP)) {
+  switch (linear_warps(p)) {
     case 1: return scan(One{}, std::conditional_t<KS % 4 == 0, Four, Parts>{});
     case 2: return scan(Two{}, Parts{});
     case 3: return scan(Three{}, Parts{});
