@@ -331,6 +331,37 @@ int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_ca
                            size_t workspace_bytes, float softcap, float out_scale, int32_t* dev_status, void* stream);
 
 /*
+ * What attention may have beyond a window and a cap; every field is optional (NULL / 0).
+ *   sinks [num_q_heads]   a score per head that takes its part of the softmax and brings no value: not scaled, no bias, counted once
+ *   slopes [num_q_heads]  slope * (query position - key position) is taken off a scaled score
+ *   head_gate             [tokens, num_q_heads] in the activations' type: a head's output is multiplied by sigmoid(gate)
+ *   keep_first            with a window: keys at positions below it stay visible
+ * The _ext entry points are the ones above with it (no score cap beside it, except in mvb_any_attn_ext).  A plan for kept first tokens
+ * comes from mvb_decode_plan_ext with the same keep_first.
+ */
+typedef struct {
+  const float* sinks;
+  const float* slopes;
+  const void* head_gate;
+  int64_t head_gate_row_stride;
+  int keep_first;
+} mvb_attn_extras;
+int mvb_prefill_attn_ext(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* v, int64_t v_row_stride,
+                         int64_t kv_rows, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const int32_t* block_table,
+                         int64_t table_stride, int block_size, int num_seqs, int total_q, int max_seqlen_q, int num_q_heads,
+                         int num_kv_heads, int head_dim, float scale, int window_left, void* out, int64_t out_row_stride,
+                         const int32_t* items, int num_items, float out_scale, const mvb_attn_extras* extras, int32_t* dev_status,
+                         void* stream);
+int mvb_decode_plan_ext(const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int block_size, int num_seqs,
+                        int window_left, int keep_first, int num_q_heads, int num_kv_heads, int head_dim, void* workspace,
+                        size_t workspace_bytes, void* stream);
+int mvb_decode_attn_ext(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache, int64_t num_blocks, int block_size,
+                        const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
+                        int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left, void* out, int64_t out_row_stride,
+                        void* workspace, size_t workspace_bytes, float out_scale, const mvb_attn_extras* extras, int32_t* dev_status,
+                        void* stream);
+
+/*
  * The entry points below take dtype 0 (activations, weights and K/V in bf16) or 1 (fp32); the arithmetic between loads and
  * stores is fp32 in both.  A "ragged step" has cu_seqlens_q [num_seqs + 1]; with cu_seqlens_q == NULL every sequence
  * brings one token and row t is sequence t.  positions [num_tokens] are absolute; a sequence whose first token of the
@@ -341,6 +372,9 @@ int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_ca
  *   tensor-core kernels do not take.  block_table == NULL: dense K/V rows cu_seqlens_k[s] + j (row strides); else a pool of
  *   kv_rows slots (k_row_stride = v_row_stride = num_kv_heads * head_dim).  cache_seqlens (optional): rows of length 0 give 0.
  * mvb_rope_kv_write_f32: mvb_rope_kv_write for fp32 activations and pools.
+ * mvb_rope_norm_kv_write: the same in either dtype, with a norm behind the rotation: norm_dim > 0 divides every q and k head by
+ *   sqrt(mean(x^2) + eps), the mean over norm_dim coordinates (what a head is padded with is zero).  cos_sin == NULL: no rotation;
+ *   num_kv_heads == 0: q alone (k, v and the caches may be NULL).
  */
 int mvb_any_attn(int dtype, const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* v,
                  int64_t v_row_stride, int64_t kv_rows, const int32_t* block_table, int64_t table_stride, int table_width,
@@ -348,6 +382,16 @@ int mvb_any_attn(int dtype, const void* q, int64_t q_row_stride, const void* k, 
                  const int32_t* cache_seqlens, int num_seqs, int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
                  float scale, int window_left, float softcap, float out_scale, void* out, int64_t out_row_stride,
                  int32_t* dev_status, void* stream);
+int mvb_any_attn_ext(int dtype, const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* v,
+                     int64_t v_row_stride, int64_t kv_rows, const int32_t* block_table, int64_t table_stride, int table_width,
+                     int block_size, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const int64_t* positions,
+                     const int32_t* cache_seqlens, int num_seqs, int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                     float scale, int window_left, float softcap, float out_scale, const mvb_attn_extras* extras, void* out,
+                     int64_t out_row_stride, int32_t* dev_status, void* stream);
+int mvb_rope_norm_kv_write(int dtype, void* q, int64_t q_row_stride, void* k, int64_t k_row_stride, const void* v, int64_t v_row_stride,
+                           const int64_t* positions, const float* cos_sin, int64_t max_pos, const int32_t* slot_mapping, void* k_cache,
+                           void* v_cache, int64_t num_slots, int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                           int k_in_place, int norm_dim, float eps, int32_t* dev_status, void* stream);
 int mvb_rope_kv_write_f32(float* q, int64_t q_row_stride, float* k, int64_t k_row_stride, const float* v,
                           int64_t v_row_stride, const int64_t* positions, const float* cos_sin, int64_t max_pos,
                           const int32_t* slot_mapping, float* k_cache, float* v_cache, int64_t num_slots, int num_tokens,
@@ -358,8 +402,11 @@ int mvb_rope_kv_write_f32(float* q, int64_t q_row_stride, float* k, int64_t k_ro
  * mvb_residual_norm: x += (y_weight ? rmsnorm(y, y_weight) : y) in place; out = rmsnorm(x, weight).  row_ends != NULL: output
  *   row r is computed from source row row_ends[r + 1] - 1 and x is left as it is.
  * mvb_embed_norm: x[r] = table[ids[r]]; out = rmsnorm(x, weight).
- * mvb_clamped_glu: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1) on a packed
- *   [rows, 2 * intermediate] projection.
+ * mvb_residual_norm_pair, mvb_embed_norm_pair: for layers whose two sublayers read the same stream through norms of their own: out =
+ *   rmsnorm(x, weight), out2 = rmsnorm(x, weight2) (both optional together).  The looked-up row is multiplied by scale; the stream of
+ *   row r also gets extra[extra_index[r, j]], j < num_extra (rows of routed experts), added in that order.
+ * mvb_glu: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + offset) on a packed
+ *   [rows, 2 * intermediate] projection, times sigmoid(row_gate[row]) where there is one.  mvb_clamped_glu: offset 1.
  * mvb_cap_logits: out = cap tanh(in / cap) (cap == 0: a copy), each side bf16 or fp32.
  * mvb_argmax_f32: the greedy token of fp32 logits (lowest column wins ties); scatter_* as for mvb_sample.
  */
@@ -369,6 +416,14 @@ int mvb_residual_norm(int dtype, float* x, const void* y, int64_t y_row_stride, 
                       void* out, const int32_t* row_ends, int rows, int width, float eps, void* stream);
 int mvb_embed_norm(int dtype, const int64_t* ids, const void* table, int64_t vocab, float* x, const void* weight, void* out,
                    int rows, int width, float eps, int32_t* dev_status, void* stream);
+int mvb_residual_norm_pair(int dtype, float* x, const void* y, int64_t y_row_stride, const void* extra, int64_t extra_row_stride,
+                           int64_t extra_rows, const int32_t* extra_index, int num_extra, const void* weight, void* out,
+                           const void* weight2, void* out2, const int32_t* row_ends, int rows, int width, float eps, int32_t* dev_status,
+                           void* stream);
+int mvb_embed_norm_pair(int dtype, const int64_t* ids, const void* table, int64_t vocab, float scale, float* x, const void* weight,
+                        void* out, const void* weight2, void* out2, int rows, int width, float eps, int32_t* dev_status, void* stream);
+int mvb_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows, int intermediate,
+            float limit, float alpha, float offset, const void* row_gate, int64_t gate_row_stride, void* stream);
 int mvb_clamped_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows,
                     int intermediate, float limit, float alpha, void* stream);
 int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_stride, void* out, int64_t out_row_stride,
@@ -376,6 +431,8 @@ int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_s
 
 /*
  * Recurrent mixers with per-sequence state slots.
+ * mvb_short_conv: mvb_short_conv_silu with the SiLU optional, and the last `copies` channels written a second time, right behind the
+ *   others.
  * mvb_short_conv_silu: out[t, c] = silu(bias[c] + sum_j weight[j, c] u[t - j, c]), j < taps <= 32; inputs from before the
  *   step come from state [num_slots, taps - 1, channels] (dtype; oldest input first), which is then brought up to date.
  * mvb_selective_scan: S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n, out_c = (sum_n S[c, n] C_n + D_c u_c) silu(z_c),
@@ -387,6 +444,10 @@ int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_s
  *   [tokens, kv_heads, dim], v [tokens, heads, vdim] share one row stride; dim <= 256.  state [num_slots, heads, dim,
  *   vdim rounded up to 4] fp32.  scratch: mvb_gated_delta_scratch_bytes(...) bytes.
  */
+int mvb_short_conv(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias, void* out,
+                   int64_t out_row_stride, void* state, const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q,
+                   const int64_t* positions, int num_seqs, int num_tokens, int channels, int taps, int silu, int copies,
+                   int32_t* dev_status, void* stream);
 int mvb_short_conv_silu(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias, void* out,
                         int64_t out_row_stride, void* state, const int32_t* state_slots, int64_t num_slots,
                         const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int channels,
@@ -473,6 +534,28 @@ int mvb_latent_decode(const void* q, int64_t q_row_stride, int64_t q_head_stride
                       const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
                       int num_heads, int width, float scale, void* out, int64_t out_row_stride, int64_t out_head_stride, void* workspace,
                       size_t workspace_bytes, int32_t* dev_status, void* stream);
+
+/*
+ * Mixture of experts.  Group sizes stay on the device.
+ * mvb_moe_route: the `top` largest of fp32 logits [num_tokens, num_experts <= 1024] per token (ids, and weights = sigmoid(logit)), each
+ *   row's number among its expert's (ranks), every expert's first row in sorted order (offsets [num_experts + 1]), and row tiles
+ *   (expert, first row, rows, 0) of at most block_rows rows; their number is tile_offsets[num_experts].  counters [num_experts + 1] must
+ *   be zero and is left zero.  max_tiles >= num_tokens * top / block_rows + min(num_experts, num_tokens * top).
+ * mvb_moe_gather: rows of h in sorted order; slots [num_tokens, top] and row_weights [num_tokens * top] come with it.
+ * mvb_moe_gemm: per expert, out rows = weight [num_experts, m, k] times x rows; gated: weight [num_experts, 2, m, k] (gate, up) and
+ *   y = g sigmoid(alpha g) (u + offset), g = min(w gate, limit), u = clamp(w up, -limit, limit), w = row_weights (NULL: 1).  block_rows
+ *   32, 64 or 128 (fp32: 64, w_row_stride = k), as in the tiles.
+ */
+int mvb_moe_route(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int top, int block_rows, int max_tiles,
+                  int32_t* counters, int32_t* ids, float* weights, int32_t* ranks, int32_t* offsets, int32_t* tile_offsets,
+                  int32_t* tiles, void* stream);
+int mvb_moe_gather(int dtype, const void* h, int64_t h_row_stride, const int32_t* ids, const float* weights, const int32_t* ranks,
+                   const int32_t* offsets, void* out, int64_t out_row_stride, int32_t* slots, float* row_weights, int num_tokens, int top,
+                   int width, void* stream);
+int mvb_moe_gemm(int dtype, const void* x, int64_t x_row_stride, int64_t num_rows, const void* weight, int64_t w_row_stride,
+                 int num_experts, int m, int k, int gated, float limit, float alpha, float offset, const float* row_weights,
+                 const int32_t* num_tiles, const int32_t* tiles, int max_tiles, int block_rows, void* out, int64_t out_row_stride,
+                 int32_t* dev_status, void* stream);
 
 #ifdef __cplusplus
 }

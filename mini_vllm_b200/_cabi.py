@@ -11,6 +11,12 @@ _LIB_PATH = Path(__file__).resolve().parent / "libmini_vllm_b200.so"
 
 i32, i64, f32, u64, vp, sz = C.c_int, C.c_int64, C.c_float, C.c_uint64, C.c_void_p, C.c_size_t
 
+
+class AttnExtras(C.Structure):
+    """``mvb_attn_extras``"""
+    _fields_ = [("sinks", vp), ("slopes", vp), ("head_gate", vp), ("head_gate_row_stride", i64), ("keep_first", i32)]
+
+
 # name -> (restype, argtypes); mirrors include/mini_vllm_b200.h exactly
 SIGNATURES = {
     "mvb_abi_version": (i32, []),
@@ -73,6 +79,22 @@ SIGNATURES = {
     "mvb_latent_decode_plan": (i32, [vp, vp, i64, i32, i32, i32, i32, vp, sz, vp]),
     "mvb_latent_decode": (i32, [vp, i64, i64, vp, i64, i32, vp, vp, i64, i32, i32, i32, i32, f32, vp, i64, i64, vp, sz, vp,
                                 vp]),
+    "mvb_prefill_attn_ext": (i32, [vp, i64, vp, i64, vp, i64, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, f32,
+                                   i32, vp, i64, vp, i32, f32, vp, vp, vp]),
+    "mvb_decode_plan_ext": (i32, [vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, vp, sz, vp]),
+    "mvb_decode_attn_ext": (i32, [vp, i64, vp, vp, i64, i32, vp, vp, i64, i32, i32, i32, i32, i32, f32, i32, vp, i64, vp, sz,
+                                  f32, vp, vp, vp]),
+    "mvb_any_attn_ext": (i32, [i32, vp, i64, vp, i64, vp, i64, i64, vp, i64, i32, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32,
+                               f32, i32, f32, f32, vp, vp, i64, vp, vp]),
+    "mvb_rope_norm_kv_write": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32,
+                                     i32, f32, vp, vp]),
+    "mvb_residual_norm_pair": (i32, [i32, vp, vp, i64, vp, i64, i64, vp, i32, vp, vp, vp, vp, vp, i32, i32, f32, vp, vp]),
+    "mvb_embed_norm_pair": (i32, [i32, vp, vp, i64, f32, vp, vp, vp, vp, vp, i32, i32, f32, vp, vp]),
+    "mvb_glu": (i32, [i32, vp, i64, vp, i64, i32, i32, f32, f32, f32, vp, i64, vp]),
+    "mvb_short_conv": (i32, [i32, vp, i64, vp, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp]),
+    "mvb_moe_route": (i32, [vp, i64, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp]),
+    "mvb_moe_gather": (i32, [i32, vp, i64, vp, vp, vp, vp, vp, i64, vp, vp, i32, i32, i32, vp]),
+    "mvb_moe_gemm": (i32, [i32, vp, i64, i64, vp, i64, i32, i32, i32, i32, f32, f32, f32, vp, vp, vp, i32, i32, vp, i64, vp, vp]),
 }
 
 _lib = None

@@ -148,3 +148,12 @@ def vebonex_shape(layers: list[dict], width: int, vocab: int, streams: int = 4, 
     from .native import vebonex_config
     return vebonex_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": groups}, "streams": streams,
                            "max_positions": max_positions}, None, dtype)
+
+
+def sunulorn_shape(layers: list[dict], width: int, vocab: int, embedding_scale: float | None = None, eps: float = 1e-6,
+                   max_position_embeddings: int = 32768, dtype: torch.dtype = torch.bfloat16) -> SimpleNamespace:
+    """A Sunulorn description without a checkpoint; ``layers`` as in its config.json."""
+    from .native import sunulorn_config
+    return sunulorn_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
+                            "embedding": {"scale": width ** 0.5 if embedding_scale is None else embedding_scale}}, None, dtype,
+                           max_position_embeddings)

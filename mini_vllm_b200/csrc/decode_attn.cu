@@ -75,6 +75,12 @@ struct DecodeParams {
   float cap_in, cap_log2;       // score cap c > 0: s -> c tanh(s scale / c), in log2 units; cap_log2 = 0: none
   float out_scale;
   int window_left;
+  // form 2; any of them may be nullptr / 0 (see mvb_attn_extras)
+  const float* sinks;
+  const float* slopes;
+  const __nv_bfloat16* head_gate;
+  int64_t gate_stride;
+  int keep_first;
   const DecodeHeader* hdr;
   const CtaDesc* descs;
   const int32_t* tile_prefix;
@@ -85,7 +91,7 @@ struct DecodeParams {
 };
 
 struct SeqView {
-  int b, tp0, tp1, n, start, start_al;
+  int b, tp0, tp1, n, start, skip;
 };
 
 template <int CT>
@@ -95,15 +101,18 @@ __device__ __forceinline__ void load_seq(SeqView& s, int b, const DecodeParams& 
   s.tp1 = p.tile_prefix[b + 1];
   s.n = p.cache_seqlens[b];
   s.start = visible_start(s.n, p.window_left);
-  s.start_al = s.start / CT * CT;
+  s.skip = skipped_tiles(s.start, p.keep_first, CT);
 }
 
-// CAP: scores pass c tanh(s / c) before the softmax.
-template <int D, int HPC, bool CAP>
+// FORM 1: scores pass c tanh(s / c) before the softmax.  2: sinks, a bias by distance, kept first tokens, head gates.  A sink is one
+// more part of a sequence when its parts are put together.
+template <int D, int HPC, int FORM>
 __global__ void __launch_bounds__(DecodeCfg<D, HPC>::NW * 32, 1)
 decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                    const DecodeParams p) {
   using C = DecodeCfg<D, HPC>;
+  constexpr bool CAP = FORM == 1, EXT = FORM == 2;
+  constexpr float kLog2e = 1.4426950408889634f;
   constexpr int NW = C::NW, CT = C::CT, NST = C::NSTAGES;
   constexpr uint32_t FULL = 0xffffffffu;
   extern __shared__ uint8_t smem_raw[];
@@ -155,14 +164,20 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
   auto seq_from_desc = [&](SeqView& v) {
     v.b = desc.b; v.tp0 = desc.tp0; v.tp1 = desc.tp1; v.n = desc.n;
     v.start = visible_start(v.n, p.window_left);
-    v.start_al = v.start / CT * CT;
+    v.skip = skipped_tiles(v.start, p.keep_first, CT);
+  };
+  const int keep = EXT ? p.keep_first : 0;
+  // first token of this warp's part of tile t, and whether all of it is out of sight
+  auto first_token = [&](const SeqView& v, int t) -> int { return tile_token(t - v.tp0, v.skip, keep, CT) + sub * 16; };
+  auto unseen = [&](const SeqView& v, int token0) -> bool {
+    return token0 >= v.n || (token0 + 16 <= v.start && (!EXT || token0 >= keep));
   };
   SeqView fs;
   seq_from_desc(fs);
   // lane i caches the block id of table column blk_base + i (blk_n valid lanes); seeded from the plan
   int ft = t0, nfetch = 0, blk_base = -1, blk_reg = -1, blk_n = 0;
   if (desc.blk0 >= 0) {
-    blk_base = (fs.start_al + (t0 - fs.tp0) * CT) / p.block_size;
+    blk_base = tile_token(t0 - fs.tp0, fs.skip, keep, CT) / p.block_size;
     blk_reg = desc.blk0;
     blk_n = 1;
   }
@@ -170,9 +185,9 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
     while (true) {
       if (ft >= t1) return false;
       while (ft >= fs.tp1 && fs.b + 1 < p.num_seqs) { load_seq<CT>(fs, fs.b + 1, p); blk_base = -1; blk_n = 0; }
-      const int token0 = fs.start_al + (ft - fs.tp0) * CT + sub * 16;
+      const int token0 = first_token(fs, ft);
       ++ft;
-      if (token0 >= fs.n || token0 + 16 <= fs.start) continue;
+      if (unseen(fs, token0)) continue;
       const int bi = token0 / p.block_size;
       if (blk_base < 0 || bi < blk_base || bi >= blk_base + blk_n) {
         blk_base = bi;
@@ -235,10 +250,18 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
 #pragma unroll
     for (int mt = 0; mt < D / 16; ++mt) { o[mt][0] = o[mt][1] = o[mt][2] = o[mt][3] = 0.f; }
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+    float slope_a = 0.f, slope_b = 0.f;                      // of this lane's two heads
+    if constexpr (EXT) {
+      if (p.slopes != nullptr) {
+        const int ha = (lane & 3) * 2;
+        if (ha < G) slope_a = p.slopes[kvh * G + ha] * kLog2e;
+        if (ha + 1 < G) slope_b = p.slopes[kvh * G + ha + 1] * kLog2e;
+      }
+    }
 
     for (; t < seg_end; ++t) {
-      const int token0 = cs.start_al + (t - cs.tp0) * CT + sub * 16;
-      if (token0 >= cs.n || token0 + 16 <= cs.start) continue;
+      const int token0 = first_token(cs, t);
+      if (unseen(cs, token0)) continue;
       if (dead) continue;
       fetch_next();
       const int st = ncomp % NST;
@@ -280,15 +303,16 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
         }
       }
       const int j0 = token0 + (lane >> 2), j1 = j0 + 8;
-      const bool v0 = j0 < cs.n && j0 >= cs.start, v1 = j1 < cs.n && j1 >= cs.start;
-      auto score = [&](float s) -> float {
-        if constexpr (CAP) return fmaf(-2.f * p.cap_log2, fast_rcp(1.f + fast_exp2(s * p.cap_in)), p.cap_log2);
+      const bool v0 = j0 < cs.n && (j0 >= cs.start || j0 < keep), v1 = j1 < cs.n && (j1 >= cs.start || j1 < keep);
+      auto score = [&](float s, float slope, int j) -> float {
+        if constexpr (EXT) return fmaf(s, p.scale_log2, slope * static_cast<float>(j - (cs.n - 1)));
+        else if constexpr (CAP) return fmaf(-2.f * p.cap_log2, fast_rcp(1.f + fast_exp2(s * p.cap_in)), p.cap_log2);
         else return s * p.scale_log2;
       };
-      const float x0 = v0 ? score(s0[0] + s1[0]) : -INFINITY;
-      const float x1 = v0 ? score(s0[1] + s1[1]) : -INFINITY;
-      const float x2 = v1 ? score(s0[2] + s1[2]) : -INFINITY;
-      const float x3 = v1 ? score(s0[3] + s1[3]) : -INFINITY;
+      const float x0 = v0 ? score(s0[0] + s1[0], slope_a, j0) : -INFINITY;
+      const float x1 = v0 ? score(s0[1] + s1[1], slope_b, j0) : -INFINITY;
+      const float x2 = v1 ? score(s0[2] + s1[2], slope_a, j1) : -INFINITY;
+      const float x3 = v1 ? score(s0[3] + s1[3], slope_b, j1) : -INFINITY;
       float ta = fmaxf(x0, x2), tb = fmaxf(x1, x3);
 #pragma unroll
       for (int off = 4; off < 32; off <<= 1) {
@@ -350,6 +374,16 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
     __nv_bfloat16* __restrict__ outp = p.out;
     const int heads = HPC * G;                               // query heads of this CTA
     const int items = heads * D / 4;                         // 4-dim groups to produce
+    auto sink_of = [&](int qh) -> float { return EXT && p.sinks != nullptr ? p.sinks[qh] * kLog2e : -INFINITY; };
+    auto out_factor = [&](int qh) -> float {                 // factor of a finished head
+      if constexpr (EXT) {
+        if (p.head_gate != nullptr) {
+          const float z = __bfloat162float(p.head_gate[b * p.gate_stride + qh]);
+          return p.out_scale * fast_rcp(1.f + fast_exp2(z * -kLog2e));
+        }
+      }
+      return p.out_scale;
+    };
     {
       const int slot = (b == first_b) ? 0 : 1;
       for (int it = threadIdx.x; it < items; it += NW * 32) {
@@ -368,13 +402,15 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
           L += f[D + 1] * w;
           acc.x += v.x * w; acc.y += v.y * w; acc.z += v.z * w; acc.w += v.w * w;
         }
-        const float inv = L > 0.f ? 1.f / L : 0.f;
-        acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
         const int qh = blockIdx.y * heads + h;
+        const float share = EXT && whole ? fast_exp2(sink_of(qh) - M) : 0.f;      // the sink's part (no keys at all: M = -inf, L = 0)
+        const float inv = L > 0.f ? 1.f / (L + share) : 0.f;
+        acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
         if (whole) {
+          const float f = out_factor(qh);
           uint2 w2;
-          w2.x = pack_bf16(acc.x * p.out_scale, acc.y * p.out_scale);
-          w2.y = pack_bf16(acc.z * p.out_scale, acc.w * p.out_scale);
+          w2.x = pack_bf16(acc.x * f, acc.y * f);
+          w2.y = pack_bf16(acc.z * f, acc.w * f);
           *reinterpret_cast<uint2*>(outp + b * p.out_stride + static_cast<int64_t>(qh) * D + dim) = w2;
         } else {
           const int64_t pi = (static_cast<int64_t>(c) * 2 + slot) * p.hq + qh;
@@ -455,7 +491,12 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
           const int it = threadIdx.x + k * NW * 32;
           if (it < items) {
             const int h = (it * 4) / D, dim = (it * 4) % D, qh = blockIdx.y * heads + h;
-            const float inv = wsum[k] > 0.f ? p.out_scale / wsum[k] : 0.f;
+            float total = wsum[k];
+            if constexpr (EXT) {
+              const int enc = m_enc[h];
+              total += fast_exp2(sink_of(qh) - __int_as_float(enc >= 0 ? enc : enc ^ 0x7fffffff));
+            }
+            const float inv = wsum[k] > 0.f ? out_factor(qh) / total : 0.f;
             uint2 w2;
             w2.x = pack_bf16(acc[k].x * inv, acc[k].y * inv); w2.y = pack_bf16(acc[k].z * inv, acc[k].w * inv);
             *reinterpret_cast<uint2*>(outp + b * p.out_stride + static_cast<int64_t>(qh) * D + dim) = w2;
@@ -474,7 +515,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_const
 }
 
 template <int D, int HPC>
-static int launch_decode(const CUtensorMap& km, const CUtensorMap& vm, const DecodeParams& p, int hkv, int num_ctas,
+static int launch_decode(const CUtensorMap& km, const CUtensorMap& vm, const DecodeParams& p, bool extended, int hkv, int num_ctas,
                          cudaStream_t stream) {
   using C = DecodeCfg<D, HPC>;
   const size_t smem = 1024 + static_cast<size_t>(C::NW) * C::NSTAGES * C::STAGE_BYTES +
@@ -482,14 +523,15 @@ static int launch_decode(const CUtensorMap& km, const CUtensorMap& vm, const Dec
                       static_cast<size_t>(C::NW) * p.group * C::FIN_STRIDE * sizeof(float);
   if (smem + 64 > 227 * 1024) return kUnsupportedShape;       // static shared memory counts too
   auto launch = [&](auto tag) -> int {
-    constexpr bool CAP = decltype(tag)::value;
+    constexpr int FORM = decltype(tag)::value;
     struct Tag {};
-    const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&decode_attn_kernel<D, HPC, CAP>), smem);
+    const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(&decode_attn_kernel<D, HPC, FORM>), smem);
     if (rc != kOk) return rc;
-    decode_attn_kernel<D, HPC, CAP><<<dim3(num_ctas, hkv / HPC), C::NW * 32, smem, stream>>>(km, vm, p);
+    decode_attn_kernel<D, HPC, FORM><<<dim3(num_ctas, hkv / HPC), C::NW * 32, smem, stream>>>(km, vm, p);
     return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
   };
-  return p.cap_log2 > 0.f ? launch(std::true_type{}) : launch(std::false_type{});
+  if (extended) return launch(std::integral_constant<int, 2>{});
+  return p.cap_log2 > 0.f ? launch(std::integral_constant<int, 1>{}) : launch(std::integral_constant<int, 0>{});
 }
 
 }  // namespace mvb
@@ -525,10 +567,10 @@ static int decode_check_args(const void* q, int64_t q_row_stride, const void* k_
 }
 
 static int decode_plan_impl(const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride,
-                            int block_size, int num_seqs, int window_left, int num_q_heads, int num_kv_heads,
+                            int block_size, int num_seqs, int window_left, int keep_first, int num_q_heads, int num_kv_heads,
                             int head_dim, void* workspace, size_t workspace_bytes, void* stream) {
   using namespace mvb;
-  if (!cache_seqlens || !workspace || num_seqs <= 0) return kInvalidArgument;
+  if (!cache_seqlens || !workspace || num_seqs <= 0 || keep_first < 0) return kInvalidArgument;
   if (!decode_shape_ok(num_q_heads, num_kv_heads, head_dim)) return kUnsupportedShape;
   const DecodeLayout l = decode_layout(num_seqs, num_q_heads, head_dim);
   if (workspace_bytes < l.total || !is_aligned(workspace, 256)) return kInvalidArgument;
@@ -536,7 +578,7 @@ static int decode_plan_impl(const int32_t* cache_seqlens, const int32_t* block_t
   int num_ctas = sm_count();
   if (num_ctas > kMaxCtas) num_ctas = kMaxCtas;
   decode_plan_kernel<<<1, kPlanThreads, 0, static_cast<cudaStream_t>(stream)>>>(
-      cache_seqlens, num_seqs, window_left, cta_tokens_for(num_kv_heads, head_dim), kMergeTiles, num_ctas,
+      cache_seqlens, num_seqs, window_left, window_left >= 0 ? keep_first : 0, cta_tokens_for(num_kv_heads, head_dim), kMergeTiles, num_ctas,
       num_seqs * num_q_heads, block_table, table_stride, block_size, reinterpret_cast<DecodeHeader*>(ws),
       reinterpret_cast<CtaDesc*>(ws + l.descs), reinterpret_cast<int32_t*>(ws + l.tile_prefix));
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
@@ -545,7 +587,7 @@ static int decode_plan_impl(const int32_t* cache_seqlens, const int32_t* block_t
 extern "C" int mvb_decode_plan(const int32_t* cache_seqlens, int num_seqs, int window_left, int num_q_heads,
                                int num_kv_heads, int head_dim, void* workspace, size_t workspace_bytes,
                                void* stream) {
-  return decode_plan_impl(cache_seqlens, nullptr, 0, 0, num_seqs, window_left, num_q_heads, num_kv_heads, head_dim,
+  return decode_plan_impl(cache_seqlens, nullptr, 0, 0, num_seqs, window_left, 0, num_q_heads, num_kv_heads, head_dim,
                           workspace, workspace_bytes, stream);
 }
 
@@ -554,18 +596,26 @@ extern "C" int mvb_decode_plan_with_table(const int32_t* cache_seqlens, const in
                                           int num_q_heads, int num_kv_heads, int head_dim, void* workspace,
                                           size_t workspace_bytes, void* stream) {
   if (!block_table || block_size <= 0 || table_stride <= 0) return mvb::kInvalidArgument;
-  return decode_plan_impl(cache_seqlens, block_table, table_stride, block_size, num_seqs, window_left, num_q_heads,
+  return decode_plan_impl(cache_seqlens, block_table, table_stride, block_size, num_seqs, window_left, 0, num_q_heads,
                           num_kv_heads, head_dim, workspace, workspace_bytes, stream);
 }
 
-extern "C" int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
-                                      int64_t num_blocks, int block_size, const int32_t* cache_seqlens,
-                                      const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
-                                      int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left,
-                                      void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
-                                      float softcap, float out_scale, int32_t* dev_status, void* stream) {
+extern "C" int mvb_decode_plan_ext(const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride, int block_size,
+                                   int num_seqs, int window_left, int keep_first, int num_q_heads, int num_kv_heads, int head_dim,
+                                   void* workspace, size_t workspace_bytes, void* stream) {
+  if (!block_table || block_size <= 0 || table_stride <= 0) return mvb::kInvalidArgument;
+  return decode_plan_impl(cache_seqlens, block_table, table_stride, block_size, num_seqs, window_left, keep_first, num_q_heads,
+                          num_kv_heads, head_dim, workspace, workspace_bytes, stream);
+}
+
+static int decode_attn_impl(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
+                            int64_t num_blocks, int block_size, const int32_t* cache_seqlens, const int32_t* block_table,
+                            int64_t table_stride, int table_width, int num_seqs, int num_q_heads, int num_kv_heads, int head_dim,
+                            float scale, int window_left, void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                            float softcap, float out_scale, const mvb_attn_extras* extras, int32_t* dev_status, void* stream) {
   using namespace mvb;
   if (!workspace || !(softcap >= 0.f)) return kInvalidArgument;
+  if (extras != nullptr && (extras->keep_first < 0 || softcap > 0.f)) return kUnsupportedShape;
   int rc = decode_check_args(q, q_row_stride, k_cache, v_cache, num_blocks, block_size, cache_seqlens, block_table,
                              table_stride, table_width, num_seqs, num_q_heads, num_kv_heads, head_dim, out,
                              out_row_stride);
@@ -594,6 +644,12 @@ extern "C" int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const
   p.cap_log2 = softcap * kLog2e;
   p.out_scale = out_scale;
   p.window_left = window_left;
+  p.sinks = p.slopes = nullptr; p.head_gate = nullptr; p.gate_stride = 0; p.keep_first = 0;
+  if (extras != nullptr) {
+    p.sinks = extras->sinks; p.slopes = extras->slopes;
+    p.head_gate = static_cast<const __nv_bfloat16*>(extras->head_gate); p.gate_stride = extras->head_gate_row_stride;
+    p.keep_first = window_left >= 0 ? extras->keep_first : 0;
+  }
   p.hdr = reinterpret_cast<const DecodeHeader*>(ws);
   p.descs = reinterpret_cast<const CtaDesc*>(ws + l.descs);
   p.tile_prefix = reinterpret_cast<const int32_t*>(ws + l.tile_prefix);
@@ -608,16 +664,38 @@ extern "C" int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const
   const int hpc = heads_per_cta(num_kv_heads, head_dim);
   rc = kUnsupportedShape;
   if (head_dim == 128) {
-    if (hpc == 8) rc = launch_decode<128, 8>(km, vm, p, num_kv_heads, num_ctas, st);
-    else if (hpc == 4) rc = launch_decode<128, 4>(km, vm, p, num_kv_heads, num_ctas, st);
-    else if (hpc == 2) rc = launch_decode<128, 2>(km, vm, p, num_kv_heads, num_ctas, st);
-    else if (hpc == 1) rc = launch_decode<128, 1>(km, vm, p, num_kv_heads, num_ctas, st);
+    if (hpc == 8) rc = launch_decode<128, 8>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
+    else if (hpc == 4) rc = launch_decode<128, 4>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
+    else if (hpc == 2) rc = launch_decode<128, 2>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
+    else if (hpc == 1) rc = launch_decode<128, 1>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
   } else {
-    if (hpc == 4) rc = launch_decode<256, 4>(km, vm, p, num_kv_heads, num_ctas, st);
-    else if (hpc == 2) rc = launch_decode<256, 2>(km, vm, p, num_kv_heads, num_ctas, st);
-    else if (hpc == 1) rc = launch_decode<256, 1>(km, vm, p, num_kv_heads, num_ctas, st);
+    if (hpc == 4) rc = launch_decode<256, 4>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
+    else if (hpc == 2) rc = launch_decode<256, 2>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
+    else if (hpc == 1) rc = launch_decode<256, 1>(km, vm, p, extras != nullptr, num_kv_heads, num_ctas, st);
   }
   return rc;
+}
+
+extern "C" int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,
+                                      int64_t num_blocks, int block_size, const int32_t* cache_seqlens,
+                                      const int32_t* block_table, int64_t table_stride, int table_width, int num_seqs,
+                                      int num_q_heads, int num_kv_heads, int head_dim, float scale, int window_left,
+                                      void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                                      float softcap, float out_scale, int32_t* dev_status, void* stream) {
+  return decode_attn_impl(q, q_row_stride, k_cache, v_cache, num_blocks, block_size, cache_seqlens, block_table, table_stride,
+                          table_width, num_seqs, num_q_heads, num_kv_heads, head_dim, scale, window_left, out, out_row_stride,
+                          workspace, workspace_bytes, softcap, out_scale, nullptr, dev_status, stream);
+}
+
+extern "C" int mvb_decode_attn_ext(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache, int64_t num_blocks,
+                                   int block_size, const int32_t* cache_seqlens, const int32_t* block_table, int64_t table_stride,
+                                   int table_width, int num_seqs, int num_q_heads, int num_kv_heads, int head_dim, float scale,
+                                   int window_left, void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                                   float out_scale, const mvb_attn_extras* extras, int32_t* dev_status, void* stream) {
+  if (extras == nullptr) return mvb::kInvalidArgument;
+  return decode_attn_impl(q, q_row_stride, k_cache, v_cache, num_blocks, block_size, cache_seqlens, block_table, table_stride,
+                          table_width, num_seqs, num_q_heads, num_kv_heads, head_dim, scale, window_left, out, out_row_stride,
+                          workspace, workspace_bytes, 0.f, out_scale, extras, dev_status, stream);
 }
 
 extern "C" int mvb_decode_attn(const void* q, int64_t q_row_stride, const void* k_cache, const void* v_cache,

@@ -48,8 +48,18 @@ __device__ __forceinline__ int visible_start(int n, int window_left) {
   return window_left >= 0 ? max(0, n - 1 - window_left) : 0;
 }
 
+// A window with kept first tokens: a sequence's tiles are numbered without the gap between the kept ones and the window's.
+// tiles left out, and the token a tile starts with
+__device__ __forceinline__ int skipped_tiles(int start, int keep_first, int cta_tokens) {
+  return max(0, start / cta_tokens - (keep_first + cta_tokens - 1) / cta_tokens);
+}
+__device__ __forceinline__ int tile_token(int tile, int skip, int keep_first, int cta_tokens) {
+  return (tile < (keep_first + cta_tokens - 1) / cta_tokens ? tile : tile + skip) * cta_tokens;
+}
+
 static __global__ void __launch_bounds__(kPlanThreads) decode_plan_kernel(const int32_t* __restrict__ cache_seqlens,
-                                                                   int num_seqs, int window_left, int cta_tokens, int merge_tiles,
+                                                                   int num_seqs, int window_left, int keep_first, int cta_tokens,
+                                                                   int merge_tiles,
                                                                    int num_ctas, int num_counters,
                                                                    const int32_t* __restrict__ block_table,
                                                                    int64_t table_stride, int block_size,
@@ -63,8 +73,7 @@ static __global__ void __launch_bounds__(kPlanThreads) decode_plan_kernel(const 
       [&](int b) {
         const int n = cache_seqlens[b];
         if (n <= 0) return 0;
-        const int start_al = visible_start(n, window_left) / cta_tokens * cta_tokens;
-        const int tiles = (n - start_al + cta_tokens - 1) / cta_tokens;
+        const int tiles = (n + cta_tokens - 1) / cta_tokens - skipped_tiles(visible_start(n, window_left), keep_first, cta_tokens);
         atomicMax(&max_tiles_s, tiles);
         return tiles;
       },
@@ -112,8 +121,8 @@ static __global__ void __launch_bounds__(kPlanThreads) decode_plan_kernel(const 
       const int lo = seq_of_tile(d.t0);
       d.b = lo; d.tp0 = tile_prefix[lo]; d.tp1 = tile_prefix[lo + 1]; d.n = cache_seqlens[lo];
       if (block_table != nullptr) {      // spare the attention kernel one dependent load before its first TMA
-        const int start_al = visible_start(d.n, window_left) / cta_tokens * cta_tokens;
-        const int token0 = start_al + (static_cast<int>(t) - d.tp0) * cta_tokens;
+        const int skip = skipped_tiles(visible_start(d.n, window_left), keep_first, cta_tokens);
+        const int token0 = tile_token(static_cast<int>(t) - d.tp0, skip, keep_first, cta_tokens);
         d.blk0 = block_table[lo * table_stride + token0 / block_size];
       }
     }

@@ -562,7 +562,7 @@ extern "C" int mvb_latent_decode_plan(const int32_t* cache_seqlens, const int32_
   if (workspace_bytes < l.total || !is_aligned(workspace, 256)) return kInvalidArgument;
   uint8_t* ws = static_cast<uint8_t*>(workspace);
   decode_plan_kernel<<<1, kPlanThreads, 0, static_cast<cudaStream_t>(stream)>>>(
-      cache_seqlens, num_seqs, -1, kLatentTile, kLatentMergeTiles, latent_ctas(num_heads), num_seqs * num_heads, block_table, table_stride, block_size,
+      cache_seqlens, num_seqs, -1, 0, kLatentTile, kLatentMergeTiles, latent_ctas(num_heads), num_seqs * num_heads, block_table, table_stride, block_size,
       reinterpret_cast<DecodeHeader*>(ws), reinterpret_cast<CtaDesc*>(ws + l.descs), reinterpret_cast<int32_t*>(ws + l.tile_prefix));
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }

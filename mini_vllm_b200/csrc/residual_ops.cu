@@ -22,6 +22,12 @@ struct NormParams {
   const int32_t* row_ends;      // nullptr, or: output row r comes from source row row_ends[r + 1] - 1 and x is left alone
   int width;
   float eps;
+  // the form with two norms of the same stream (PAIR): a factor of the looked-up row, further rows to add (row `row` of the stream
+  // gets extra[extra_index[row, j]], j < num_extra), and a second weight and output (nullptr: none)
+  float table_scale;
+  const void* extra; const int32_t* extra_index; int num_extra; int64_t extra_stride, extra_rows;
+  const void* weight2;
+  void* out2;
   int* dev_status;
 };
 
@@ -39,7 +45,7 @@ __device__ __forceinline__ float row_sum(float v, float* scratch) {
   return s;
 }
 
-template <class T, int V, int ITEMS>
+template <class T, int V, int ITEMS, bool PAIR>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p) {
   __shared__ float scratch[32];
   const int out_row = blockIdx.x;
@@ -64,6 +70,31 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p)
     if (i >= nvec) continue;
     load_vec<T, V>(yrow + i * V, v[k]);
     if (p.ids == nullptr) load_f32<V>(xrow + i * V, res[k]);
+    if constexpr (PAIR) {
+      if (p.ids != nullptr) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[k][j] *= p.table_scale;
+      }
+    }
+  }
+  if constexpr (PAIR) {
+    for (int e = 0; e < p.num_extra; ++e) {
+      const int32_t r = p.extra_index[static_cast<int64_t>(row) * p.num_extra + e];
+      if (r < 0 || r >= p.extra_rows) {
+        if (threadIdx.x == 0) report(p.dev_status, kDevBadPosition, row);
+        continue;
+      }
+      const T* erow = static_cast<const T*>(p.extra) + r * p.extra_stride;
+#pragma unroll
+      for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x + k * nt;
+        if (i >= nvec) continue;
+        float a[V];
+        load_vec<T, V>(erow + i * V, a);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[k][j] += a[j];
+      }
+    }
   }
   if (p.y_weight != nullptr) {
 #pragma unroll
@@ -107,10 +138,18 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p)
 #pragma unroll
     for (int j = 0; j < V; ++j) w[j] = v[k][j] * r * w[j];
     store_vec<T, V>(orow + i * V, w);
+    if constexpr (PAIR) {
+      if (p.weight2 != nullptr) {
+        load_vec<T, V>(static_cast<const T*>(p.weight2) + i * V, w);
+#pragma unroll
+        for (int j = 0; j < V; ++j) w[j] = v[k][j] * r * w[j];
+        store_vec<T, V>(static_cast<T*>(p.out2) + static_cast<int64_t>(out_row) * p.width + i * V, w);
+      }
+    }
   }
 }
 
-template <class T, int V>
+template <class T, int V, bool PAIR>
 static int launch_norm_v(const NormParams& p, int rows, cudaStream_t st) {
   const int nvec = p.width / V;
   // about four vectors in flight per thread for wide rows, a whole warp at least for narrow ones
@@ -118,25 +157,28 @@ static int launch_norm_v(const NormParams& p, int rows, cudaStream_t st) {
   while (items < 8 && (nvec + items - 1) / items > 1024) items *= 2;
   const int nt = ((nvec + items - 1) / items + 31) / 32 * 32;
   if (nt > 1024) return kUnsupportedShape;
-  if (items == 1) residual_norm_kernel<T, V, 1><<<rows, nt, 0, st>>>(p);
-  else if (items == 2) residual_norm_kernel<T, V, 2><<<rows, nt, 0, st>>>(p);
-  else if (items == 4) residual_norm_kernel<T, V, 4><<<rows, nt, 0, st>>>(p);
-  else residual_norm_kernel<T, V, 8><<<rows, nt, 0, st>>>(p);
+  if (items == 1) residual_norm_kernel<T, V, 1, PAIR><<<rows, nt, 0, st>>>(p);
+  else if (items == 2) residual_norm_kernel<T, V, 2, PAIR><<<rows, nt, 0, st>>>(p);
+  else if (items == 4) residual_norm_kernel<T, V, 4, PAIR><<<rows, nt, 0, st>>>(p);
+  else residual_norm_kernel<T, V, 8, PAIR><<<rows, nt, 0, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
-template <class T>
+template <class T, bool PAIR = false>
 static int launch_norm(const NormParams& p, int rows, cudaStream_t st) {
   constexpr int V = kVec<T>;
   const bool vec = p.width % V == 0 && p.width % 4 == 0 && p.y_stride % V == 0 && is_aligned(p.x, 16) && is_aligned(p.y, 16) &&
-                   is_aligned(p.y_weight, 16) && is_aligned(p.weight, 16) && is_aligned(p.out, 16);
-  return vec ? launch_norm_v<T, V>(p, rows, st) : launch_norm_v<T, 1>(p, rows, st);
+                   is_aligned(p.y_weight, 16) && is_aligned(p.weight, 16) && is_aligned(p.out, 16) &&
+                   p.extra_stride % V == 0 && is_aligned(p.extra, 16) && is_aligned(p.weight2, 16) && is_aligned(p.out2, 16);
+  return vec ? launch_norm_v<T, V, PAIR>(p, rows, st) : launch_norm_v<T, 1, PAIR>(p, rows, st);
 }
 
-// out = g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+// out = g sigmoid(alpha g) (u + offset) with g = min(gate, limit), u = clamp(up, -limit, limit), times sigmoid(row_gate) of the row
+// (alpha 1, offset 0, limit infinite: the SiLU-gated unit)
 template <class T, int V>
 __global__ void __launch_bounds__(128) clamped_glu_kernel(const T* __restrict__ gate_up, int64_t in_stride, T* __restrict__ out,
-                                                          int64_t out_stride, int rows, int inter, float limit, float alpha) {
+                                                          int64_t out_stride, int rows, int inter, float limit, float alpha,
+                                                          float offset, const T* __restrict__ row_gate, int64_t gate_stride) {
   const int c = (blockIdx.x * 128 + threadIdx.x) * V;
   if (c >= inter) return;
   const float k = -alpha * 1.4426950408889634f;
@@ -145,27 +187,30 @@ __global__ void __launch_bounds__(128) clamped_glu_kernel(const T* __restrict__ 
     float g[V], u[V];
     load_vec<T, V>(r, g);
     load_vec<T, V>(r + inter, u);
+    const float f = row_gate != nullptr ? sigmoid_f(to_f(row_gate[t * gate_stride])) : 1.f;
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       const float gi = fminf(g[i], limit), ui = fminf(fmaxf(u[i], -limit), limit);
       // gi -> -inf: exp2 -> inf, the reciprocal -> 0 and the product with the finite gi -> 0
-      g[i] = gi * fast_rcp(1.f + fast_exp2(k * gi)) * (ui + 1.f);
+      g[i] = gi * fast_rcp(1.f + fast_exp2(k * gi)) * (ui + offset) * f;
     }
     store_vec<T, V>(out + t * out_stride + c, g);
   }
 }
 
 template <class T>
-static int launch_glu(const void* gu, int64_t is, void* out, int64_t os, int rows, int inter, float limit, float alpha,
-                      cudaStream_t st) {
+static int launch_glu(const void* gu, int64_t is, void* out, int64_t os, int rows, int inter, float limit, float alpha, float offset,
+                      const void* row_gate, int64_t gate_stride, cudaStream_t st) {
   constexpr int V = kVec<T>;
   const bool vec = inter % V == 0 && is % V == 0 && os % V == 0 && is_aligned(gu, 16) && is_aligned(out, 16);
   const int v = vec ? V : 1, bx = (inter + 128 * v - 1) / (128 * v);
   int by = rows, cap = (sm_count() * 16 + bx - 1) / bx;
   if (by > cap) by = cap;
   if (by > 65535) by = 65535;
-  if (vec) clamped_glu_kernel<T, V><<<dim3(bx, by), 128, 0, st>>>(static_cast<const T*>(gu), is, static_cast<T*>(out), os, rows, inter, limit, alpha);
-  else clamped_glu_kernel<T, 1><<<dim3(bx, by), 128, 0, st>>>(static_cast<const T*>(gu), is, static_cast<T*>(out), os, rows, inter, limit, alpha);
+  auto tg = static_cast<const T*>(gu), tr = static_cast<const T*>(row_gate);
+  auto to = static_cast<T*>(out);
+  if (vec) clamped_glu_kernel<T, V><<<dim3(bx, by), 128, 0, st>>>(tg, is, to, os, rows, inter, limit, alpha, offset, tr, gate_stride);
+  else clamped_glu_kernel<T, 1><<<dim3(bx, by), 128, 0, st>>>(tg, is, to, os, rows, inter, limit, alpha, offset, tr, gate_stride);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
@@ -223,7 +268,7 @@ extern "C" int mvb_residual_norm(int dtype, float* x, const void* y, int64_t y_r
   using namespace mvb;
   if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
   if (rows == 0) return kOk;
-  const NormParams p{x, y, y_row_stride, nullptr, 0, y_weight, weight, out, row_ends, width, eps, nullptr};
+  const NormParams p{x, y, y_row_stride, nullptr, 0, y_weight, weight, out, row_ends, width, eps, 1.f, nullptr, nullptr, 0, 0, 0, nullptr, nullptr, nullptr};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
 }
@@ -234,19 +279,56 @@ extern "C" int mvb_embed_norm(int dtype, const int64_t* ids, const void* table, 
   if (!ids || !table || !x || !weight || !out || rows < 0 || width <= 0 || vocab <= 0 || (dtype != kBf16 && dtype != kF32))
     return kInvalidArgument;
   if (rows == 0) return kOk;
-  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, dev_status};
+  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, 1.f, nullptr, nullptr, 0, 0, 0, nullptr,
+                     nullptr, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
 }
 
-extern "C" int mvb_clamped_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride,
-                               int rows, int intermediate, float limit, float alpha, void* stream) {
+extern "C" int mvb_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows,
+                       int intermediate, float limit, float alpha, float offset, const void* row_gate, int64_t gate_row_stride,
+                       void* stream) {
   using namespace mvb;
   if (!gate_up || !out || rows < 0 || intermediate <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
   if (rows == 0) return kOk;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return dtype == kBf16 ? launch_glu<__nv_bfloat16>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, st)
-                        : launch_glu<float>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, st);
+  return dtype == kBf16 ? launch_glu<__nv_bfloat16>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, offset,
+                                                    row_gate, gate_row_stride, st)
+                        : launch_glu<float>(gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, offset,
+                                            row_gate, gate_row_stride, st);
+}
+
+extern "C" int mvb_clamped_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride,
+                               int rows, int intermediate, float limit, float alpha, void* stream) {
+  return mvb_glu(dtype, gate_up, in_row_stride, out, out_row_stride, rows, intermediate, limit, alpha, 1.f, nullptr, 0, stream);
+}
+
+extern "C" int mvb_embed_norm_pair(int dtype, const int64_t* ids, const void* table, int64_t vocab, float scale, float* x,
+                                   const void* weight, void* out, const void* weight2, void* out2, int rows, int width, float eps,
+                                   int32_t* dev_status, void* stream) {
+  using namespace mvb;
+  if (!ids || !table || !x || !weight || !out || rows < 0 || width <= 0 || vocab <= 0 || (dtype != kBf16 && dtype != kF32))
+    return kInvalidArgument;
+  if ((weight2 == nullptr) != (out2 == nullptr)) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, scale, nullptr, nullptr, 0, 0, 0, weight2, out2,
+                     dev_status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_norm<__nv_bfloat16, true>(p, rows, st) : launch_norm<float, true>(p, rows, st);
+}
+
+extern "C" int mvb_residual_norm_pair(int dtype, float* x, const void* y, int64_t y_row_stride, const void* extra,
+                                      int64_t extra_row_stride, int64_t extra_rows, const int32_t* extra_index, int num_extra,
+                                      const void* weight, void* out, const void* weight2, void* out2, const int32_t* row_ends, int rows,
+                                      int width, float eps, int32_t* dev_status, void* stream) {
+  using namespace mvb;
+  if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
+  if ((weight2 == nullptr) != (out2 == nullptr) || num_extra < 0 || (num_extra > 0 && (!extra || !extra_index))) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  const NormParams p{x, y, y_row_stride, nullptr, 0, nullptr, weight, out, row_ends, width, eps, 1.f, extra, extra_index, num_extra,
+                     extra_row_stride, extra_rows, weight2, out2, dev_status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_norm<__nv_bfloat16, true>(p, rows, st) : launch_norm<float, true>(p, rows, st);
 }
 
 extern "C" int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_stride, void* out,

@@ -10,6 +10,7 @@
 #include "common.cuh"
 #include "host_util.cuh"
 #include "mini_vllm_b200.h"
+#include "rope_any.cuh"
 
 #include <type_traits>
 
@@ -76,17 +77,22 @@ __device__ __forceinline__ void rotate8(uint4& lo, uint4& hi, const float* cs, c
 // (y = x * rsqrt(mean(x^2) + eps) * w, or * (1 + w) for Gemma), rounded to bf16 as the separate norm kernel
 // would, then rotated.  The D/16 lanes of a head row are consecutive lanes of an aligned group, so the sum of
 // squares is a shuffle reduction inside the group.
+//
+// NORM == 2 has the norm behind the rotation and no weight: rotation keeps a head's length, so the sum of squares is the same, and
+// 1 / rms multiplies the angle's cosine and sine; one rounding, at the end.  The mean runs over norm_dim coordinates (the head's own
+// size; what it is padded with is zero).
 struct NormRopeParams {
   RopeParams r;
   const __nv_bfloat16* q_weight;
   const __nv_bfloat16* k_weight;
   float eps;
   int unit_offset;
+  int norm_dim;
 };
 
 // PPH fixes the chunk pairs per head at compile time (8: head_dim 128, 16: head_dim 256; 0: read it from the
 // parameters), which turns the task -> (head, chunk) divisions of every group into shifts.
-template <int ITEMS, bool NORM, int PPH>
+template <int ITEMS, int NORM, int PPH>
 __global__ void __launch_bounds__(256, 3) rope_kv_kernel(const NormRopeParams np) {
   const RopeParams& p = np.r;
   const int pph = PPH ? PPH : p.d / 16;                      // chunk pairs per head
@@ -155,6 +161,7 @@ __global__ void __launch_bounds__(256, 3) rope_kv_kernel(const NormRopeParams np
     const int head = is_rope ? task / pph : 0;
     const int c = is_rope ? task - head * pph : 0;
     const bool is_q = head < p.hq;
+    float rstd2 = 1.f;
     if (NORM) {
       float ss = 0.f;
       if (is_rope) {
@@ -168,7 +175,9 @@ __global__ void __launch_bounds__(256, 3) rope_kv_kernel(const NormRopeParams np
       }
       // every lane of the warp takes part; a head's lanes form an aligned group of pph
       for (int off = 1; off < pph; off <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-      if (is_rope && (is_q || slot >= 0 || p.k_in_place)) {
+      if constexpr (NORM == 2) {
+        rstd2 = 1.f / sqrtf(ss / static_cast<float>(np.norm_dim) + np.eps);
+      } else if (is_rope && (is_q || slot >= 0 || p.k_in_place)) {
         const float rstd = rsqrtf(ss / static_cast<float>(d) + np.eps);
         const __nv_bfloat16* w = is_q ? np.q_weight : np.k_weight;
         const uint4 wl = *reinterpret_cast<const uint4*>(w + c * 8);
@@ -195,7 +204,14 @@ __global__ void __launch_bounds__(256, 3) rope_kv_kernel(const NormRopeParams np
     if (is_q && !rotate && !NORM) continue;                  // plain store_kvcache leaves q alone
     if (rotate && pos_ok) {
       if (!same_chunk) load_table(c);
-      rotate8<!NORM>(lo[j], hi[j], cs, sn);
+      if constexpr (NORM == 2) {
+        float cn[8], sm[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { cn[i] = cs[i] * rstd2; sm[i] = sn[i] * rstd2; }
+        rotate8<false>(lo[j], hi[j], cn, sm);
+      } else {
+        rotate8<!NORM>(lo[j], hi[j], cs, sn);
+      }
     }
     __nv_bfloat16* row = is_q ? p.q + t * p.q_stride + head * d : p.k + t * p.k_stride + (head - p.hq) * d;
     if ((is_q || p.k_in_place) && (rotate || NORM)) {
@@ -210,7 +226,7 @@ __global__ void __launch_bounds__(256, 3) rope_kv_kernel(const NormRopeParams np
   }
 }
 
-template <bool NORM>
+template <int NORM>
 static int launch_rope(const NormRopeParams& np, cudaStream_t stream) {
   const RopeParams& p = np.r;
   const int64_t tasks = static_cast<int64_t>(p.hq + p.hkv) * (p.d / 16) + static_cast<int64_t>(p.hkv) * p.d / 8;
@@ -237,6 +253,23 @@ static int launch_rope(const NormRopeParams& np, cudaStream_t stream) {
 }
 
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
+
+int rope_norm_bf16(const RopeAnyParams& a, cudaStream_t st) {
+  const int pph = a.d / 16;
+  const bool vec = a.q_stride % 8 == 0 && a.k_stride % 8 == 0 && a.v_stride % 8 == 0 && aligned16(a.q) && aligned16(a.k) &&
+                   aligned16(a.v) && aligned16(a.k_cache) && aligned16(a.v_cache) && aligned16(a.cos_sin);
+  if (a.d % 16 != 0 || pph > 32 || (pph & (pph - 1)) != 0 || a.cos_sin == nullptr || !vec) return kUnsupportedShape;
+  NormRopeParams np;
+  RopeParams& p = np.r;
+  p.q = static_cast<__nv_bfloat16*>(a.q); p.k = static_cast<__nv_bfloat16*>(a.k); p.v = static_cast<const __nv_bfloat16*>(a.v);
+  p.q_stride = a.q_stride; p.k_stride = a.k_stride; p.v_stride = a.v_stride;
+  p.positions = a.positions; p.cos_sin = a.cos_sin; p.max_pos = a.max_pos; p.slot_mapping = a.slot_mapping;
+  p.k_cache = static_cast<__nv_bfloat16*>(a.k_cache); p.v_cache = static_cast<__nv_bfloat16*>(a.v_cache);
+  p.num_slots = a.num_slots; p.num_tokens = a.tokens; p.hq = a.hq; p.hkv = a.hkv; p.d = a.d; p.k_in_place = a.k_in_place;
+  p.dev_status = a.dev_status;
+  np.q_weight = np.k_weight = nullptr; np.eps = a.eps; np.unit_offset = 0; np.norm_dim = a.norm_dim;
+  return a.norm_dim > 0 ? launch_rope<2>(np, st) : launch_rope<0>(np, st);
+}
 
 }  // namespace mvb
 
@@ -271,8 +304,8 @@ extern "C" int mvb_rope_kv_write(void* q, int64_t q_row_stride, void* k, int64_t
   p.dev_status = dev_status;
   NormRopeParams np;
   np.r = p;
-  np.q_weight = np.k_weight = nullptr; np.eps = 0.f; np.unit_offset = 0;
-  return launch_rope<false>(np, static_cast<cudaStream_t>(stream));
+  np.q_weight = np.k_weight = nullptr; np.eps = 0.f; np.unit_offset = 0; np.norm_dim = 0;
+  return launch_rope<0>(np, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int mvb_qk_norm_rope_kv_write(void* q, int64_t q_row_stride, void* k, int64_t k_row_stride, const void* v,
@@ -308,6 +341,6 @@ extern "C" int mvb_qk_norm_rope_kv_write(void* q, int64_t q_row_stride, void* k,
   p.dev_status = dev_status;
   np.q_weight = static_cast<const __nv_bfloat16*>(q_weight);
   np.k_weight = static_cast<const __nv_bfloat16*>(k_weight);
-  np.eps = eps; np.unit_offset = unit_offset;
-  return launch_rope<true>(np, static_cast<cudaStream_t>(stream));
+  np.eps = eps; np.unit_offset = unit_offset; np.norm_dim = head_dim;
+  return launch_rope<1>(np, static_cast<cudaStream_t>(stream));
 }

@@ -1,6 +1,8 @@
-// Depthwise causal convolution over a few taps, with bias and SiLU, on a packed ragged batch with carried inputs.
+// Depthwise causal convolution over a few taps, with bias and, where asked, SiLU, on a packed ragged batch with carried inputs.
 //
 //   out[t, c] = silu(bias[c] + sum_j w[j, c] u[t - j, c])
+//
+// The last `copies` channels may also be written a second time, behind the others (for a mixer that rotates one copy in place).
 //
 // The taps - 1 inputs in front of a step's tokens come from the sequence's state slot ([slots, taps - 1, channels], row
 // taps - 1 - d = the input d tokens before the step), zeros before the start of the sequence; afterwards the slot holds the
@@ -41,6 +43,7 @@ struct ConvParams {
   const int32_t* cu;             // [num_seqs + 1] or nullptr
   const int64_t* positions;      // [tokens]
   int num_seqs, tokens, channels, taps;
+  int silu, copies;
   int* dev_status;
 };
 
@@ -114,8 +117,10 @@ __global__ void __launch_bounds__(128, TAPS <= 4 ? 7 : 1) short_conv_kernel(cons
 #pragma unroll
           for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], hist[j][i], acc[i]);
 #pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] = acc[i] * fast_rcp(1.f + fast_exp2(acc[i] * -1.4426950408889634f));
+        for (int i = 0; i < V; ++i)
+          if (p.silu) acc[i] = acc[i] * fast_rcp(1.f + fast_exp2(acc[i] * -1.4426950408889634f));
         put<T, V>(out + (t + m) * p.out_stride, acc);
+        if (c >= C - p.copies) put<T, V>(out + (t + m) * p.out_stride + p.copies, acc);
         if (p.cu == nullptr) {                               // the slot's rows are this thread's alone
           const int64_t slot = conv_slot(p, s);
           if (slot >= 0) {
@@ -171,7 +176,7 @@ static int launch_conv_t(const ConvParams& p, cudaStream_t st) {
 template <class T>
 static int launch_conv(const ConvParams& p, cudaStream_t st) {
   constexpr int V = 4;                                       // (8 bf16 would double the registers and halve the warps)
-  const bool vec = p.channels % V == 0 && p.u_stride % V == 0 && p.out_stride % V == 0 && is_aligned(p.u, 16) &&
+  const bool vec = p.channels % V == 0 && p.copies % V == 0 && p.u_stride % V == 0 && p.out_stride % V == 0 && is_aligned(p.u, 16) &&
                    is_aligned(p.out, 16) && is_aligned(p.state, 16) && is_aligned(p.w, 16) && is_aligned(p.bias, 16);
   if (p.taps <= 4) return vec ? launch_conv_t<T, V, 4>(p, st) : launch_conv_t<T, 1, 4>(p, st);
   if (p.taps <= 8) return vec ? launch_conv_t<T, V, 8>(p, st) : launch_conv_t<T, 1, 8>(p, st);
@@ -181,18 +186,26 @@ static int launch_conv(const ConvParams& p, cudaStream_t st) {
 
 }  // namespace mvb
 
-extern "C" int mvb_short_conv_silu(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias,
+extern "C" int mvb_short_conv(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias,
                                    void* out, int64_t out_row_stride, void* state, const int32_t* state_slots,
                                    int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs,
-                                   int num_tokens, int channels, int taps, int32_t* dev_status, void* stream) {
+                                   int num_tokens, int channels, int taps, int silu, int copies, int32_t* dev_status, void* stream) {
   using namespace mvb;
-  if (!u || !weight || !out || !positions || num_seqs < 0 || num_tokens < 0 || channels <= 0 || taps <= 0) return kInvalidArgument;
+  if (!u || !weight || !out || !positions || num_seqs < 0 || num_tokens < 0 || channels <= 0 || taps <= 0 || copies < 0 || copies > channels) return kInvalidArgument;
   if (state != nullptr && (state_slots == nullptr || num_slots <= 0)) return kInvalidArgument;
   if (cu_seqlens_q == nullptr && num_seqs != num_tokens) return kInvalidArgument;
   if (dtype != kBf16 && dtype != kF32) return kInvalidArgument;
   if (num_tokens == 0 || num_seqs == 0) return kOk;
   const ConvParams p{u, u_row_stride, weight, bias, out, out_row_stride, taps > 1 ? state : nullptr, state_slots, num_slots,
-                     cu_seqlens_q, positions, num_seqs, num_tokens, channels, taps, dev_status};
+                     cu_seqlens_q, positions, num_seqs, num_tokens, channels, taps, silu, copies, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_conv<__nv_bfloat16>(p, st) : launch_conv<float>(p, st);
+}
+
+extern "C" int mvb_short_conv_silu(int dtype, const void* u, int64_t u_row_stride, const void* weight, const void* bias,
+                                   void* out, int64_t out_row_stride, void* state, const int32_t* state_slots,
+                                   int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs,
+                                   int num_tokens, int channels, int taps, int32_t* dev_status, void* stream) {
+  return mvb_short_conv(dtype, u, u_row_stride, weight, bias, out, out_row_stride, state, state_slots, num_slots, cu_seqlens_q, positions,
+                        num_seqs, num_tokens, channels, taps, 1, 0, dev_status, stream);
 }

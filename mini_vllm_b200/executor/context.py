@@ -45,10 +45,10 @@ class Context:
     # token of every sequence, i.e. cu_seqlens_q itself)
     logit_rows: Optional[torch.Tensor] = None
 
-    # extension (latent attention): the context tokens of the step's prompts in all; the step's own latents by the layer that made
-    # them, for later layers that share them
+    # extension: the context tokens of the step's prompts in all (latent attention); the step's own latents, or keys and values, by the
+    # layer that made them, for later layers that share them
     prompt_keys: int = 0
-    latents: dict = field(default_factory=dict, repr=False, compare=False)
+    shared: dict = field(default_factory=dict, repr=False, compare=False)
 
     # filled by the attention layer on first use within this forward pass
     decode_plans: dict = field(default_factory=dict, repr=False, compare=False)

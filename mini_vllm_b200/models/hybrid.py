@@ -8,7 +8,8 @@ branches keep a row of state per sequence in slots that the scheduler hands out 
 first token of a step has position 0 starts from zero, so a reused slot needs no clearing.
 
 Per sublayer the kernels are: input GEMM, branch kernels, output GEMM, and one kernel for everything between the sublayer's output
-and the normalised input of the next one.
+and the normalised input of the next one.  A layer has its mixer and its feed-forward one after the other (``HybridLayer``) or side by
+side as one sublayer (``ParallelLayer``).
 """
 from __future__ import annotations
 
@@ -73,8 +74,40 @@ class HybridLayer(nn.Module):
             yield self.connections[1], lambda ctx, h, positions: self.mlp(h)
 
 
+    @torch.no_grad()
+    def load(self, prefix: str, mixer_prefixes: dict[str, str], w: Weights) -> None:
+        self.mixer.load(mixer_prefixes, w)
+        for q, connection in enumerate(self.connections, 1):
+            connection.load(prefix, q, w)
+        if self.mlp is not None:
+            self.mlp.load(lambda n: w(prefix + "mlp." + n))
+
+
+class ParallelLayer(nn.Module):
+    """A mixer and, optionally, a feed-forward beside it: one sublayer over two norms of the same stream (``ParallelStream``).  The
+    feed-forward is part of the mixer's packed output projection; routed experts' rows are added where the stream is brought up to date."""
+
+    def __init__(self, stream: nn.Module, mixer: PackedMixer):
+        super().__init__()
+        self.mixer = mixer
+        self.connections = nn.ModuleList([stream.connection(1 if mixer.feed is None else 2)])
+
+    def run(self, ctx: Context, h: tuple, positions: torch.Tensor):
+        h_mix, h_feed = h
+        y = self.mixer(ctx, h_mix, positions, h_feed)
+        return y, None if self.mixer.feed is None else self.mixer.feed.routed(h_feed, ctx.status)
+
+    def sublayers(self):
+        yield self.connections[0], self.run
+
+    @torch.no_grad()
+    def load(self, prefix: str, mixer_prefixes: dict[str, str], w: Weights) -> None:
+        self.mixer.load(mixer_prefixes, w, prefix + "mlp.")
+        self.connections[0].load(prefix, 1, w)
+
+
 class HybridDecoder(nn.Module):
-    def __init__(self, cfg, layers: list[HybridLayer], stream: nn.Module):
+    def __init__(self, cfg, layers: list[HybridLayer | ParallelLayer], stream: nn.Module):
         super().__init__()
         self.config, self.eps = cfg, cfg.rms_norm_eps
         self.logit_cap = float(getattr(cfg, "logit_softcap", None) or 0.0)
@@ -163,12 +196,7 @@ class HybridDecoder(nn.Module):
         self.lm_head_weight.copy_(w("head"))
         self.stream.load(w)
         for i, layer in enumerate(self.layers):
-            p = f"l{i}."
-            layer.mixer.load(self.mixer_prefixes(i), w)
-            for q, connection in enumerate(layer.connections, 1):
-                connection.load(p, q, w)
-            if layer.mlp is not None:
-                layer.mlp.load(lambda n, p=p: w(p + "mlp." + n))
+            layer.load(f"l{i}.", self.mixer_prefixes(i), w)
         unknown = set(tensors) - used
         if unknown:
             raise KeyError(f"unrecognised parameter {sorted(unknown)[0]}")

@@ -58,6 +58,7 @@ class Branch(nn.Module):
     in_rows: int        # rows of the packed input projection, a multiple of 8
     out_cols: int       # columns of the packed output projection, a multiple of 8
     out_used: int       # of these, the ones the branch writes (the rest stay zero)
+    in_bias = out_bias = False          # whether the branch's projections have biases
 
     def state_specs(self, dtype: torch.dtype) -> dict[str, tuple[tuple[int, ...], torch.dtype]]:
         return {}
@@ -66,12 +67,33 @@ class Branch(nn.Module):
         """Load the branch's own parameters; returns its input rows [in_rows, width] and output columns [width, out_cols]."""
         raise NotImplementedError
 
+    def load_biases(self, w: Weights) -> tuple[torch.Tensor | None, torch.Tensor | None]:
+        """Bias of the input rows [in_rows] and of the output [width]; None where the branch has none."""
+        return None, None
+
     def forward(self, ctx: Context, proj: torch.Tensor, out: torch.Tensor, positions: torch.Tensor) -> None:
         raise NotImplementedError
 
 
+def alibi_slopes(heads: int) -> torch.Tensor:
+    """2^(-8 (h + 1) / heads): what a distance bias takes off a score per token, head by head."""
+    return torch.exp2(-8.0 * torch.arange(1, heads + 1, dtype=torch.float64, device="cpu") / heads).float()
+
+
 class AttentionBranch(Branch):
     """Grouped-query attention with rotation, optional window and score cap, and a value size of its own.
+
+    Options, each independent of the others:
+
+    * ``interleaved``: the rotated pairs are (2i, 2i + 1) instead of (i, i + dims/2); ``rotary`` None: no rotation
+    * ``taps``: a causal convolution over time on the channels of q and k, in front of the rotation (its inputs are per-sequence state)
+    * ``keys_are_values``: v is k in front of the rotation (``vdim`` = ``dim``)
+    * ``norm_eps``: q and k are divided by their root mean square behind the rotation
+    * ``in_bias``, ``out_bias``: the projections have biases (the gate's has none)
+    * ``keep_first``: first tokens that the window never drops
+    * ``sink``: "zero" or "learned" - a score per head in the softmax's denominator; ``slopes``: a bias by distance, per head
+    * ``gate``: "value" or "head" - the sigmoid of a projection multiplies every value of the output, or a head's
+    * ``source``: an earlier layer's branch whose keys and values this one reads instead of making its own
 
     The kernels know one head size, so q/k heads (``dim``) and v heads (``vdim``) are both padded to it inside the packed
     projections: zero rows cost nothing but projection width, leave every score unchanged and give zero output columns
@@ -79,15 +101,43 @@ class AttentionBranch(Branch):
     permutation common to q and k, which no score sees - so the kernel that pairs the halves of a head serves any
     ``rot_dims``; the coordinates that are not rotated fill the other pairs and get angle 0."""
 
-    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rotary: RotaryEmbedding, rot_dims: int,
-                 padded: int, window: int | None = None, softcap: float | None = None, factor: float = 1.0):
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rotary: RotaryEmbedding | None, rot_dims: int,
+                 padded: int, window: int | None = None, softcap: float | None = None, factor: float = 1.0, interleaved: bool = False,
+                 taps: int = 0, keys_are_values: bool = False, norm_eps: float | None = None, in_bias: bool = False,
+                 out_bias: bool = False, keep_first: int = 0, sink: str | None = None, slopes: torch.Tensor | None = None,
+                 gate: str | None = None, source: "AttentionBranch | None" = None):
         super().__init__()
+        if keys_are_values and vdim != dim:
+            raise ValueError(f"values that are the keys have their size, not {vdim} beside {dim}")
+        if source is not None and (source.kv_heads, source.dim, source.vdim, source.d) != (kv_heads, dim, vdim, padded):
+            raise ValueError(f"keys and values of {source.kv_heads} heads of {source.dim} and {source.vdim} cannot serve a layer with "
+                             f"{kv_heads} of {dim} and {vdim}")
+        if source is not None and taps:
+            raise ValueError("a layer that borrows its keys has no convolution")
         self.heads, self.kv_heads, self.dim, self.vdim, self.d, self.rot_dims = heads, kv_heads, dim, vdim, padded, rot_dims
-        self.rotary = rotary
+        self.rotary, self.interleaved, self.keys_are_values, self.gate, self.sink = rotary, interleaved, keys_are_values, gate, sink
+        self.norm = None if norm_eps is None else (dim, norm_eps)
+        self.in_bias, self.out_bias, self.borrows = in_bias, out_bias, source is not None
         self.attn = FlashAttention(heads, padded, scale, kv_heads, (-1 if window is None else window - 1, -1),
-                                   softcap=softcap or 0.0, out_scale=factor)
-        self.in_rows = (heads + 2 * kv_heads) * padded
+                                   softcap=softcap or 0.0, out_scale=factor, keep_first=keep_first,
+                                   source=None if source is None else source.attn)
+        if sink is not None:
+            self.attn.sinks = weight_f32(heads)
+        if slopes is not None:
+            self.attn.slopes = nn.Parameter(slopes.to(torch.empty(0).device), requires_grad=False)
+        self.made = [] if self.borrows else ["k"] if keys_are_values else ["k", "v"]
+        self.qk = (heads + (0 if self.borrows else kv_heads)) * padded
+        self.gate_rows = {None: 0, "value": heads * padded, "head": pad8(heads)}[gate]
+        self.in_sizes = [heads * padded] + [kv_heads * padded] * len(self.made) + [self.gate_rows]
+        self.in_rows = sum(self.in_sizes)
         self.out_cols = self.out_used = heads * padded
+        self.taps = taps
+        if taps:
+            self.conv_weight = weight(taps, self.qk)
+            self.conv_state = None
+
+    def state_specs(self, dtype):
+        return {"conv_state": ((self.taps - 1, self.qk), dtype)} if self.taps > 1 else {}
 
     @staticmethod
     def padded_size(dim: int, vdim: int, dtype: torch.dtype) -> int:
@@ -100,26 +150,63 @@ class AttentionBranch(Branch):
         """Where coordinate i of a q/k head goes inside the padded head."""
         half, r = self.d // 2, self.rot_dims // 2
         free = [j for j in range(self.d) if not (j < r or half <= j < half + r)]
-        place = list(range(r)) + [half + i for i in range(r)] + free[:self.dim - 2 * r]
-        return torch.tensor(place, dtype=torch.long)
+        low, high = list(range(r)), [half + i for i in range(r)]
+        turned = [j for pair in zip(low, high) for j in pair] if self.interleaved else low + high
+        return torch.tensor(turned + free[:self.dim - 2 * r], dtype=torch.long)
+
+    def _place(self, name: str) -> torch.Tensor:
+        """Where coordinate i of a head of ``name`` goes; values keep their order unless they are the keys."""
+        return torch.arange(self.vdim) if name == "v" and not self.keys_are_values else self._layout()
+
+    def _heads(self, src: torch.Tensor, name: str, n: int) -> torch.Tensor:
+        """``src`` [n * size, ...] with every head laid out in ``d`` rows."""
+        place = self._place(name).to(src.device)
+        dst = src.new_zeros(n, self.d, *src.shape[1:])
+        dst[:, place] = src.view(n, place.numel(), *src.shape[1:])
+        return dst.flatten(0, 1)
 
     def load(self, w: Weights):
-        rows = []
-        place = self._layout()
-        for name, n, used in (("q", self.heads, self.dim), ("k", self.kv_heads, self.dim), ("v", self.kv_heads, self.vdim)):
-            src = w(name)
-            dst = src.new_zeros(n, self.d, src.shape[1])
-            dst[:, place.to(src.device) if name != "v" else slice(0, used)] = src.view(n, used, -1)
-            rows.append(dst.view(n * self.d, -1))
+        rows = [self._heads(w("q"), "q", self.heads)] + [self._heads(w(n), n, self.kv_heads) for n in self.made]
+        if self.taps:
+            conv = [self._heads(w(n + ".conv"), n, c) for n, c in (("q", self.heads), ("k", self.kv_heads))]
+            self.conv_weight.copy_(torch.cat(conv).flip(1).T)
+        if self.gate == "value":
+            rows.append(self._heads(w("g"), "v", self.heads))
+        elif self.gate == "head":
+            rows.append(pad_rows(w("g"), self.gate_rows))
+        if self.sink == "learned":
+            self.attn.sinks.copy_(w("sink").float().reshape(-1))
         o = w("o")
+        place = self._place("v").to(o.device)
         cols = o.new_zeros(o.shape[0], self.heads, self.d)
-        cols[:, :, :self.vdim] = o.view(o.shape[0], self.heads, self.vdim)
+        cols[:, :, place] = o.view(o.shape[0], self.heads, self.vdim)
         return torch.cat(rows), cols.view(o.shape[0], -1)
+
+    def load_biases(self, w: Weights):
+        rows = None
+        if self.in_bias:
+            parts = [self._heads(w("q.b"), "q", self.heads)] + [self._heads(w(n + ".b"), n, self.kv_heads) for n in self.made]
+            rows = F.pad(torch.cat(parts), (0, self.gate_rows))
+        return rows, w("o.b") if self.out_bias else None
 
     def forward(self, ctx, proj, out, positions):
         h, g, d = self.heads, self.kv_heads, self.d
-        q, k, v = (t.unflatten(1, (-1, d)) for t in proj.split([h * d, g * d, g * d], dim=1))
-        self.attn.forward_fused(ctx, q, k, v, positions, self.rotary.cos_sin_cache, out=out.unflatten(1, (h, d)))
+        q, *made, gate = proj.split(self.in_sizes, dim=1)
+        if self.taps:
+            turned = ops.short_conv(proj[:, :self.qk], self.conv_weight, None, self.conv_state, ctx.state_slots, ragged(ctx), positions,
+                                    copies=g * d if self.keys_are_values else 0, status=ctx.status)
+            q, *rest = turned.split([h * d] + [g * d] * (2 if self.keys_are_values else 1), dim=1)
+            made = rest if self.keys_are_values else [rest[0], made[1]]
+        elif self.keys_are_values:
+            made = [made[0], made[0].clone()]                                 # (the rotation works in place)
+        q, *kv = (t.unflatten(1, (-1, d)) for t in (q, *made))
+        k, v = kv or (None, None)
+        o = out.unflatten(1, (h, d))
+        mixed = torch.empty(o.shape, dtype=o.dtype, device=o.device) if self.gate == "value" else o
+        self.attn.forward_fused(ctx, q, k, v, positions, None if self.rotary is None else self.rotary.cos_sin_cache, out=mixed,
+                                head_gate=gate[:, :h] if self.gate == "head" else None, norm=self.norm)
+        if self.gate == "value":
+            ops.gate_mul(mixed.flatten(1), gate, out)
 
 
 class SelectiveScanBranch(Branch):
@@ -346,10 +433,10 @@ class LatentAttentionBranch(Branch):
         if self.source is None:
             cq, c = ops.latent_norm(dq[:, :self.q_rank], self.q_norm, self.qp, c[:, :self.kv_rank], self.kv_norm, self.latent_width,
                                     self.eps, cache, ctx.slot_mapping, status=ctx.status)
-            ctx.latents[owner] = c                                            # this step's rows, for layers that share them
+            ctx.shared[owner] = c                                            # this step's rows, for layers that share them
         else:
             cq, _ = ops.latent_norm(dq[:, :self.q_rank], self.q_norm, self.qp, None, None, 0, self.eps, status=ctx.status)
-            c = ctx.latents[owner]
+            c = ctx.shared[owner]
         q = F.linear(cq, self.q_up).unflatten(1, (self.num_heads, self.dk))
         o = torch.empty(q.shape[0], self.num_heads, self.dv, dtype=q.dtype, device=q.device)
         if not self.expands or (not self.tensor_core_decode and (not ctx.prefill or ctx.num_decode)):
@@ -399,26 +486,44 @@ class LatentAttentionBranch(Branch):
 
 
 class PackedMixer(nn.Module):
-    """Branches side by side on one input; their outputs meet in one output projection."""
+    """Branches side by side on one input; their outputs meet in one output projection.
 
-    def __init__(self, width: int, branches: dict[str, Branch]):
+    ``feed``: a feed-forward (``feedforward.py``) beside the branches, on an input of its own, whose down projection is part of the
+    same output projection."""
+
+    def __init__(self, width: int, branches: dict[str, Branch], feed: nn.Module | None = None):
         super().__init__()
-        self.branches = nn.ModuleDict(branches)
+        self.branches, self.feed = nn.ModuleDict(branches), feed
         self.in_sizes = [b.in_rows for b in branches.values()]
-        self.out_sizes = [b.out_cols for b in branches.values()]
+        self.out_sizes = [b.out_cols for b in branches.values()] + ([] if feed is None else [feed.out_cols])
         self.in_proj, self.out_proj = weight(sum(self.in_sizes), width), weight(width, sum(self.out_sizes))
+        self.in_bias = weight(sum(self.in_sizes)) if any(b.in_bias for b in branches.values()) else None
+        self.out_bias = weight(width) if any(b.out_bias for b in branches.values()) else None
         self.dense_out = all(b.out_used == b.out_cols for b in branches.values())
 
     @torch.no_grad()
-    def load(self, prefixes: dict[str, str], w: Weights) -> None:
-        parts = [b.load(lambda n, p=prefixes[key]: w(p + n)) for key, b in self.branches.items()]
+    def load(self, prefixes: dict[str, str], w: Weights, feed_prefix: str = "") -> None:
+        named = [(b, lambda n, p=prefixes[key]: w(p + n)) for key, b in self.branches.items()]
+        parts = [b.load(of) for b, of in named]
+        cols = [p[1] for p in parts]
+        if self.feed is not None:
+            down = self.feed.load(lambda n: w(feed_prefix + n))
+            cols += [] if down is None else [down]
         self.in_proj.copy_(torch.cat([p[0] for p in parts]))
-        self.out_proj.copy_(torch.cat([p[1] for p in parts], dim=1))
+        self.out_proj.copy_(torch.cat(cols, dim=1))
+        biases = [b.load_biases(of) for b, of in named]
+        if self.in_bias is not None:
+            self.in_bias.copy_(torch.cat([self.in_bias.new_zeros(n) if b[0] is None else b[0] for n, b in zip(self.in_sizes, biases)]))
+        if self.out_bias is not None:
+            self.out_bias.copy_(sum(b[1].float() for b in biases if b[1] is not None))
 
-    def forward(self, ctx: Context, h: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
-        proj = F.linear(h, self.in_proj)
+    def forward(self, ctx: Context, h: torch.Tensor, positions: torch.Tensor, h_feed: torch.Tensor | None = None) -> torch.Tensor:
+        proj = F.linear(h, self.in_proj, self.in_bias)
         make = torch.empty if self.dense_out else torch.zeros     # columns nobody writes meet zero weights and must be finite
         y = make(h.shape[0], self.out_proj.shape[1], dtype=h.dtype, device=h.device)
-        for b, pi, yi in zip(self.branches.values(), proj.split(self.in_sizes, dim=1), y.split(self.out_sizes, dim=1)):
+        cols = y.split(self.out_sizes, dim=1)
+        for b, pi, yi in zip(self.branches.values(), proj.split(self.in_sizes, dim=1), cols):
             b(ctx, pi, yi, positions)
-        return F.linear(y, self.out_proj)
+        if self.feed is not None:
+            self.feed.write(h_feed, cols[-1])
+        return F.linear(y, self.out_proj, self.out_bias)

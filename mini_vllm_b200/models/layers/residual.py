@@ -6,7 +6,8 @@ per sublayer:
 
 * ``SandwichStream``: one fp32 stream, a norm in front of and behind every sublayer;
 * ``HyperStream``: several fp32 streams.  A sublayer reads a weighted sum of them; afterwards every stream becomes a weighted sum of all
-  old ones plus its own multiple of the output.  Norms in equal consecutive groups, learned positions added to the embedding.
+  old ones plus its own multiple of the output.  Norms in equal consecutive groups, learned positions added to the embedding;
+* ``ParallelStream``: one fp32 stream, from which a mixer and a feed-forward side by side read through norms of their own.
 """
 from __future__ import annotations
 
@@ -96,3 +97,46 @@ class HyperStream(nn.Module):
     @staticmethod
     def total(x: torch.Tensor) -> torch.Tensor:
         return x.sum(1)
+
+
+class ParallelConnection(nn.Module):
+    def __init__(self, width: int, norms: int):
+        super().__init__()
+        self.norm, self.feed_norm = gain(width), gain(width) if norms > 1 else None
+
+    @torch.no_grad()
+    def load(self, prefix: str, index: int, w: Weights) -> None:
+        self.norm.copy_(w(f"{prefix}norm{index}"))
+        if self.feed_norm is not None:
+            self.feed_norm.copy_(w(f"{prefix}norm{index + 1}"))
+
+
+class ParallelStream(nn.Module):
+    """A sublayer's input is a pair of normalised rows (the second None without a feed-forward); its output what one GEMM adds up, with the
+    rows of routed experts beside it, if there are any."""
+
+    def __init__(self, width: int, eps: float, embedding_scale: float = 1.0):
+        super().__init__()
+        self.width, self.eps, self.embedding_scale = width, eps, embedding_scale
+
+    def connection(self, norms: int = 2) -> nn.Module:
+        return ParallelConnection(self.width, norms)
+
+    def load(self, w: Weights) -> None:
+        pass
+
+    def start(self, ctx, ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, first: ParallelConnection):
+        x, h, h_feed = ops.embed_norm_pair(ids, table, self.embedding_scale, first.norm, first.feed_norm, self.eps, status=ctx.status)
+        return x, (h, h_feed)
+
+    def advance(self, x: torch.Tensor, y, done: ParallelConnection, following: ParallelConnection | None, final_norm: torch.Tensor,
+                rows: torch.Tensor | None = None):
+        summed, routed = y
+        norm, feed_norm = (final_norm, None) if following is None else (following.norm, following.feed_norm)
+        extra, index = routed or (None, None)
+        h = ops.residual_norm_pair(x, summed, norm, feed_norm, self.eps, extra, index, row_ends=rows)
+        return h[0] if following is None else h
+
+    @staticmethod
+    def total(x: torch.Tensor) -> torch.Tensor:
+        return x

@@ -5,6 +5,9 @@ raises on a non-zero status.  Nothing here computes on the host.
 """
 from __future__ import annotations
 
+import ctypes
+from dataclasses import dataclass, replace
+
 import torch
 
 from . import _cabi
@@ -42,6 +45,34 @@ def _need(t: torch.Tensor, dtype, name: str) -> None:
 def _heads_contiguous(t: torch.Tensor, name: str) -> None:
     if t.dim() != 3 or t.stride(2) != 1 or (t.shape[1] != 1 and t.stride(1) != t.shape[2]):
         raise ValueError(f"{name} must be [tokens, heads, head_dim] with contiguous heads")
+
+
+@dataclass(frozen=True)
+class AttnExtras:
+    """What attention may have beyond a window and a cap: ``sinks`` (fp32 [heads], a score that takes its part of the softmax and brings
+    no value), ``slopes`` (fp32 [heads], taken off a score per token of distance), ``head_gate`` ([tokens, heads], a head's output is
+    multiplied by the sigmoid), ``keep_first`` (with a window: these first tokens stay visible)."""
+    sinks: torch.Tensor | None = None
+    slopes: torch.Tensor | None = None
+    head_gate: torch.Tensor | None = None
+    keep_first: int = 0
+
+    def rows(self, start: int, end: int) -> "AttnExtras":
+        """The same for a part of the step's tokens."""
+        return self if self.head_gate is None else replace(self, head_gate=self.head_gate[start:end])
+
+    def struct(self, q: torch.Tensor):
+        """The C argument for queries ``q`` [tokens, heads, size]."""
+        for t, name in ((self.sinks, "sinks"), (self.slopes, "slopes")):
+            if t is not None:
+                _need(t, torch.float32, name)
+                assert t.numel() == q.shape[1] and t.is_contiguous()
+        gate = self.head_gate
+        if gate is not None:
+            _need(gate, q.dtype, "head_gate")
+            assert gate.shape == q.shape[:2] and gate.stride(1) == 1
+        return ctypes.byref(_cabi.AttnExtras(_ptr(self.sinks), _ptr(self.slopes), _ptr(gate), 0 if gate is None else gate.stride(0),
+                                             int(self.keep_first)))
 
 
 def new_status(device) -> torch.Tensor:
@@ -197,17 +228,19 @@ def decode_workspace(max_seqs: int, num_q_heads: int, head_dim: int, device) -> 
 
 def decode_plan(cache_seqlens: torch.Tensor, window_left: int, num_q_heads: int, num_kv_heads: int,
                 head_dim: int, workspace: torch.Tensor, block_table: torch.Tensor | None = None,
-                block_size: int = 0) -> None:
+                block_size: int = 0, keep_first: int = 0) -> None:
     """Plan the split of one decode step.  With ``block_table`` (the one the attention calls will get)
-    the plan also records each CTA's first block id, sparing every layer a dependent load."""
+    the plan also records each CTA's first block id, sparing every layer a dependent load.  ``keep_first`` (needs the table): as
+    in the attention's ``AttnExtras``."""
     _need(cache_seqlens, torch.int32, "cache_seqlens")
     if block_table is not None:
         _need(block_table, torch.int32, "block_table")
         assert block_table.stride(1) == 1 and block_table.shape[0] >= cache_seqlens.numel() and block_size > 0
-        rc = _cabi.load().mvb_decode_plan_with_table(
+        rc = _cabi.load().mvb_decode_plan_ext(
             _ptr(cache_seqlens), _ptr(block_table), block_table.stride(0), block_size, cache_seqlens.numel(),
-            window_left, num_q_heads, num_kv_heads, head_dim, _ptr(workspace), workspace.numel(), _stream())
+            window_left, int(keep_first), num_q_heads, num_kv_heads, head_dim, _ptr(workspace), workspace.numel(), _stream())
     else:
+        assert keep_first == 0
         rc = _cabi.load().mvb_decode_plan(_ptr(cache_seqlens), cache_seqlens.numel(), window_left, num_q_heads,
                                           num_kv_heads, head_dim, _ptr(workspace), workspace.numel(), _stream())
     _cabi.check(rc, "mvb_decode_plan")
@@ -217,7 +250,7 @@ def decode_plan(cache_seqlens: torch.Tensor, window_left: int, num_q_heads: int,
 def decode_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cache_seqlens: torch.Tensor,
                 block_table: torch.Tensor, scale: float, window_left: int, workspace: torch.Tensor,
                 out: torch.Tensor | None = None, status: torch.Tensor | None = None, softcap: float = 0.0,
-                out_scale: float = 1.0) -> torch.Tensor:
+                out_scale: float = 1.0, extras: AttnExtras | None = None) -> torch.Tensor:
     """q [B,Hq,D]; the plan for (cache_seqlens, window_left) must already be in ``workspace``.  ``softcap`` > 0: scores
     pass ``softcap * tanh(score / softcap)``; ``out_scale`` multiplies the output."""
     _need(q, torch.bfloat16, "q"); _heads_contiguous(q, "q")
@@ -229,10 +262,14 @@ def decode_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, c
     assert cache_seqlens.numel() >= B
     if out is None:
         out = torch.empty(B, hq, d, dtype=torch.bfloat16, device=q.device)
-    rc = _cabi.load().mvb_decode_attn_capped(
-        _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), nblk, bs, _ptr(cache_seqlens), _ptr(block_table),
-        block_table.stride(0), block_table.shape[1], B, hq, hkv, d, float(scale), window_left, _ptr(out),
-        out.stride(0), _ptr(workspace), workspace.numel(), float(softcap), float(out_scale), _ptr(status), _stream())
+    args = (_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), nblk, bs, _ptr(cache_seqlens), _ptr(block_table),
+            block_table.stride(0), block_table.shape[1], B, hq, hkv, d, float(scale), window_left, _ptr(out),
+            out.stride(0), _ptr(workspace), workspace.numel())
+    if extras is None:
+        rc = _cabi.load().mvb_decode_attn_capped(*args, float(softcap), float(out_scale), _ptr(status), _stream())
+    else:
+        assert softcap == 0
+        rc = _cabi.load().mvb_decode_attn_ext(*args, float(out_scale), extras.struct(q), _ptr(status), _stream())
     _cabi.check(rc, "mvb_decode_attn_capped")
     LaunchCounter.add(1)
     return out
@@ -292,7 +329,7 @@ def prefill_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q
                  cu_seqlens_k: torch.Tensor, max_seqlen_q: int, scale: float, window_left: int = -1,
                  block_table: torch.Tensor | None = None, out: torch.Tensor | None = None,
                  status: torch.Tensor | None = None, items: torch.Tensor | None = None, softcap: float = 0.0,
-                 out_scale: float = 1.0) -> torch.Tensor:
+                 out_scale: float = 1.0, extras: AttnExtras | None = None) -> torch.Tensor:
     """q [Tq,Hq,D]; k/v dense [Tk,Hkv,D] (block_table None) or the paged pool [blocks,bs,Hkv,D].
 
     ``items`` (int32 [n, 2] on the device, from ``build_prefill_items``) gives the launch its work as a list of
@@ -315,11 +352,14 @@ def prefill_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q
     if use:
         _need(items, torch.int32, "items")
         assert items.dim() == 2 and items.shape[1] == 2 and items.is_contiguous()
-    rc = _cabi.load().mvb_prefill_attn_capped(
-        _ptr(q), q.stride(0), _ptr(k), k_stride, _ptr(v), v_stride, kv_rows, _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
-        _ptr(block_table), tstride, bs, cu_seqlens_q.numel() - 1, Tq, int(max_seqlen_q), hq, hkv, d, float(scale),
-        window_left, _ptr(out), out.stride(0), _ptr(items) if use else None, items.shape[0] if use else 0,
-        float(softcap), float(out_scale), _ptr(status), _stream())
+    args = (_ptr(q), q.stride(0), _ptr(k), k_stride, _ptr(v), v_stride, kv_rows, _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
+            _ptr(block_table), tstride, bs, cu_seqlens_q.numel() - 1, Tq, int(max_seqlen_q), hq, hkv, d, float(scale),
+            window_left, _ptr(out), out.stride(0), _ptr(items) if use else None, items.shape[0] if use else 0)
+    if extras is None:
+        rc = _cabi.load().mvb_prefill_attn_capped(*args, float(softcap), float(out_scale), _ptr(status), _stream())
+    else:
+        assert softcap == 0
+        rc = _cabi.load().mvb_prefill_attn_ext(*args, float(out_scale), extras.struct(q), _ptr(status), _stream())
     _cabi.check(rc, "mvb_prefill_attn_capped")
     LaunchCounter.add(1)
     return out
@@ -446,7 +486,8 @@ def _same(dtype, **tensors) -> None:
 def any_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: torch.Tensor, scale: float,
              window_left: int = -1, cu_seqlens_q: torch.Tensor | None = None, cu_seqlens_k: torch.Tensor | None = None,
              block_table: torch.Tensor | None = None, cache_seqlens: torch.Tensor | None = None, softcap: float = 0.0,
-             out_scale: float = 1.0, out: torch.Tensor | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
+             out_scale: float = 1.0, out: torch.Tensor | None = None, status: torch.Tensor | None = None,
+             extras: AttnExtras | None = None) -> torch.Tensor:
     """Attention of any head size, group size and dtype (one warp per token and head).  k/v are the paged pool with a
     ``block_table``, else dense rows; without ``cu_seqlens_q`` every row is a sequence of its own."""
     code = _dtype_of(q, "q")
@@ -466,11 +507,12 @@ def any_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: torch
     num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
     if out is None:
         out = torch.empty(tokens, hq, d, dtype=q.dtype, device=q.device)
-    rc = _cabi.load().mvb_any_attn(
+    rc = _cabi.load().mvb_any_attn_ext(
         code, _ptr(q), q.stride(0), _ptr(k), ks, _ptr(v), vs, kv_rows, _ptr(block_table), tstride, width, bs,
         _ptr(cu_seqlens_q), _ptr(cu_seqlens_k), _ptr(positions), _ptr(cache_seqlens), num_seqs, tokens, hq, hkv, d,
-        float(scale), window_left, float(softcap), float(out_scale), _ptr(out), out.stride(0), _ptr(status), _stream())
-    _cabi.check(rc, "mvb_any_attn")
+        float(scale), window_left, float(softcap), float(out_scale), None if extras is None else extras.struct(q), _ptr(out),
+        out.stride(0), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_any_attn_ext")
     LaunchCounter.add(1)
     return out
 
@@ -497,6 +539,40 @@ def rope_kv_write_f32(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positio
         _ptr(v_cache) if slot_mapping is not None else None, num_slots, tokens, q.shape[1], hkv, d, 1 if k_in_place else 0,
         _ptr(status), _stream())
     _cabi.check(rc, "mvb_rope_kv_write_f32")
+    LaunchCounter.add(1)
+
+
+def rope_norm_kv_write(q: torch.Tensor, k: torch.Tensor | None, v: torch.Tensor | None, positions: torch.Tensor,
+                       cos_sin: torch.Tensor | None, slot_mapping: torch.Tensor | None, k_cache: torch.Tensor | None,
+                       v_cache: torch.Tensor | None, k_in_place: bool = True, norm_dim: int = 0, eps: float = 0.0,
+                       status: torch.Tensor | None = None) -> None:
+    """Rotates q (in place) and k, divides every head by the root mean square of its ``norm_dim`` used coordinates (0: no norm), and
+    writes k and v to their cache slots.  ``cos_sin`` None: no rotation; ``k`` None: q alone.  Either dtype, any even head size."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v)
+    _same(torch.float32, cos_sin=cos_sin)
+    _need(positions, torch.int64, "positions")
+    for t, n in ((q, "q"), (k, "k"), (v, "v")):
+        if t is not None:
+            _heads_contiguous(t, n)
+    tokens, hq, d = q.shape
+    hkv, num_slots = 0 if k is None else k.shape[1], 0
+    assert k is None or (v is not None and k.shape == v.shape == (tokens, hkv, d))
+    assert cos_sin is None or (cos_sin.is_contiguous() and cos_sin.shape[1] == d)
+    if k is None:
+        slot_mapping = None
+    if slot_mapping is not None:
+        _need(slot_mapping, torch.int32, "slot_mapping")
+        _same(q.dtype, k_cache=k_cache, v_cache=v_cache)
+        assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[-2:] == (hkv, d)
+        num_slots = k_cache.shape[0] * k_cache.shape[1]
+    cached = slot_mapping is not None
+    rc = _cabi.load().mvb_rope_norm_kv_write(
+        code, _ptr(q), q.stride(0), _ptr(k), 0 if k is None else k.stride(0), _ptr(v), 0 if v is None else v.stride(0), _ptr(positions),
+        _ptr(cos_sin), 0 if cos_sin is None else cos_sin.shape[0], _ptr(slot_mapping), _ptr(k_cache) if cached else None,
+        _ptr(v_cache) if cached else None, num_slots, tokens, hq, hkv, d, 1 if k_in_place else 0, int(norm_dim), float(eps), _ptr(status),
+        _stream())
+    _cabi.check(rc, "mvb_rope_norm_kv_write")
     LaunchCounter.add(1)
 
 
@@ -537,17 +613,76 @@ def embed_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps
     return x, out
 
 
-def clamped_glu(gate_up: torch.Tensor, intermediate: int, limit: float, alpha: float) -> torch.Tensor:
-    """``g sigmoid(alpha g) (u + 1)``, ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, packed ``[gate | up]``."""
+def residual_norm_pair(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, weight2: torch.Tensor | None, eps: float,
+                       extra: torch.Tensor | None = None, extra_index: torch.Tensor | None = None,
+                       row_ends: torch.Tensor | None = None,
+                       status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """``x += y`` in place, and ``extra[extra_index[row, j]]`` for every j; returns the norms of x with ``weight`` and ``weight2`` (None:
+    None) in y's dtype.  ``row_ends`` as in ``residual_norm``."""
+    code = _dtype_of(y, "y")
+    _need(x, torch.float32, "x"); _same(y.dtype, weight=weight, weight2=weight2, extra=extra)
+    assert x.dim() == 2 and x.is_contiguous() and y.shape == x.shape and y.stride(1) == 1
+    rows, width = x.shape
+    if row_ends is not None:
+        _need(row_ends, torch.int32, "row_ends")
+        rows = row_ends.numel() - 1
+    count = 0
+    if extra is not None:
+        _need(extra_index, torch.int32, "extra_index")
+        count = extra_index.shape[1]
+        assert extra_index.shape[0] == x.shape[0] and extra_index.is_contiguous() and extra.shape[1] >= width and extra.stride(1) == 1
+    out = torch.empty(rows, width, dtype=y.dtype, device=x.device)
+    out2 = None if weight2 is None else torch.empty_like(out)
+    if rows == 0:
+        return out, out2
+    rc = _cabi.load().mvb_residual_norm_pair(
+        code, _ptr(x), _ptr(y), y.stride(0), _ptr(extra), 0 if extra is None else extra.stride(0), 0 if extra is None else extra.shape[0],
+        _ptr(extra_index), count, _ptr(weight), _ptr(out), _ptr(weight2), _ptr(out2), _ptr(row_ends), rows, width, float(eps), _ptr(status),
+        _stream())
+    _cabi.check(rc, "mvb_residual_norm_pair")
+    LaunchCounter.add(1)
+    return out, out2
+
+
+def embed_norm_pair(ids: torch.Tensor, table: torch.Tensor, scale: float, weight: torch.Tensor, weight2: torch.Tensor | None, eps: float,
+                    status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor | None]:
+    """(fp32 residual stream ``scale * table[ids]``, its norms with ``weight`` and ``weight2`` in the table's dtype)."""
+    code = _dtype_of(table, "table")
+    _need(ids, torch.int64, "ids"); _same(table.dtype, weight=weight, weight2=weight2)
+    assert table.is_contiguous() and ids.dim() == 1 and ids.is_contiguous()
+    rows, width = ids.numel(), table.shape[1]
+    x = torch.empty(rows, width, dtype=torch.float32, device=table.device)
+    out = torch.empty(rows, width, dtype=table.dtype, device=table.device)
+    out2 = None if weight2 is None else torch.empty_like(out)
+    rc = _cabi.load().mvb_embed_norm_pair(code, _ptr(ids), _ptr(table), table.shape[0], float(scale), _ptr(x), _ptr(weight), _ptr(out),
+                                          _ptr(weight2), _ptr(out2), rows, width, float(eps), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_embed_norm_pair")
+    LaunchCounter.add(1)
+    return x, out, out2
+
+
+def glu(gate_up: torch.Tensor, intermediate: int, limit: float = float("inf"), alpha: float = 1.0, offset: float = 0.0,
+        row_gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``g sigmoid(alpha g) (u + offset)``, ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, packed ``[gate | up]``; times
+    ``sigmoid(row_gate)`` ([rows], any stride) of the row.  The defaults are the SiLU-gated unit."""
     code = _dtype_of(gate_up, "gate_up")
     assert gate_up.dim() == 2 and gate_up.stride(1) == 1 and gate_up.shape[1] == 2 * intermediate
     rows = gate_up.shape[0]
-    out = torch.empty(rows, intermediate, dtype=gate_up.dtype, device=gate_up.device)
-    rc = _cabi.load().mvb_clamped_glu(code, _ptr(gate_up), gate_up.stride(0), _ptr(out), out.stride(0), rows, intermediate,
-                                      float(limit), float(alpha), _stream())
-    _cabi.check(rc, "mvb_clamped_glu")
+    _same(gate_up.dtype, row_gate=row_gate, out=out)
+    assert row_gate is None or row_gate.shape == (rows,)
+    if out is None:
+        out = torch.empty(rows, intermediate, dtype=gate_up.dtype, device=gate_up.device)
+    assert out.shape == (rows, intermediate) and out.stride(1) == 1
+    rc = _cabi.load().mvb_glu(code, _ptr(gate_up), gate_up.stride(0), _ptr(out), out.stride(0), rows, intermediate, float(limit),
+                              float(alpha), float(offset), _ptr(row_gate), 0 if row_gate is None else row_gate.stride(0), _stream())
+    _cabi.check(rc, "mvb_glu")
     LaunchCounter.add(1)
     return out
+
+
+def clamped_glu(gate_up: torch.Tensor, intermediate: int, limit: float, alpha: float) -> torch.Tensor:
+    """``glu`` with one added to the clamped up projection."""
+    return glu(gate_up, intermediate, limit, alpha, 1.0)
 
 
 def cap_logits(logits: torch.Tensor, cap: float, out_dtype: torch.dtype) -> torch.Tensor:
@@ -589,8 +724,15 @@ def _state_args(state: torch.Tensor | None, slots: torch.Tensor | None):
 def short_conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor | None,
                     state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor,
                     status: torch.Tensor | None = None) -> torch.Tensor:
-    """Causal depthwise convolution + SiLU.  ``u`` [T, C] (free row stride), ``weight`` [taps, C] (row j weighs the input j
-    tokens back), ``state`` [slots, taps - 1, C]."""
+    """``short_conv`` with SiLU behind it."""
+    return short_conv(u, weight, bias, state, state_slots, cu_seqlens_q, positions, silu=True, status=status)
+
+
+def short_conv(u: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor | None,
+               state_slots: torch.Tensor | None, cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor, silu: bool = False,
+               copies: int = 0, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal depthwise convolution, optionally with SiLU.  ``u`` [T, C] (free row stride), ``weight`` [taps, C] (row j weighs the
+    input j tokens back), ``state`` [slots, taps - 1, C].  [T, C + copies]: the last ``copies`` channels come a second time."""
     code = _dtype_of(u, "u")
     _same(u.dtype, weight=weight, bias=bias, state=state)
     _need(positions, torch.int64, "positions")
@@ -598,13 +740,13 @@ def short_conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | 
     taps = weight.shape[0]
     assert u.stride(1) == 1 and weight.is_contiguous() and weight.shape[1] == channels
     assert state is None or state.shape[1:] == (taps - 1, channels)
-    out = torch.empty(tokens, channels, dtype=u.dtype, device=u.device)
+    out = torch.empty(tokens, channels + copies, dtype=u.dtype, device=u.device)
     st, sl, n = _state_args(state, state_slots)
     num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
-    rc = _cabi.load().mvb_short_conv_silu(code, _ptr(u), u.stride(0), _ptr(weight), _ptr(bias), _ptr(out), out.stride(0), st, sl,
-                                          n, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, channels, taps,
-                                          _ptr(status), _stream())
-    _cabi.check(rc, "mvb_short_conv_silu")
+    rc = _cabi.load().mvb_short_conv(code, _ptr(u), u.stride(0), _ptr(weight), _ptr(bias), _ptr(out), out.stride(0), st, sl,
+                                     n, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, channels, taps, 1 if silu else 0,
+                                     int(copies), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_short_conv")
     LaunchCounter.add(2 if cu_seqlens_q is not None and st is not None and taps > 1 else 1)
     return out
 
@@ -867,5 +1009,69 @@ def latent_decode(q: torch.Tensor, cache: torch.Tensor, cache_seqlens: torch.Ten
         block_table.shape[1], b, heads, width, float(scale), _ptr(out), out.stride(1), out.stride(0), _ptr(workspace), workspace.numel(),
         _ptr(status), _stream())
     _cabi.check(rc, "mvb_latent_decode")
+    LaunchCounter.add(1)
+    return out
+
+
+# ---- mixture of experts -----------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class ExpertRows:
+    """A step's tokens sorted by expert, as the grouped products need them; every number stays on the device."""
+    slots: torch.Tensor           # int32 [T, top]: the sorted row of a token's j-th expert
+    weights: torch.Tensor         # fp32 [T * top], in sorted order
+    tiles: torch.Tensor           # int32 [max tiles, 4]
+    num_tiles: torch.Tensor       # int32 [1]
+    block_rows: int
+    experts: int
+
+
+def moe_block_rows(rows: int, experts: int, dtype: torch.dtype) -> int:
+    """Rows of a tile of the grouped products, by how many an expert gets on average."""
+    if dtype == torch.float32:
+        return 64
+    return 128 if rows >= 96 * experts else 64 if rows >= 40 * experts else 32
+
+
+def moe_sort(h: torch.Tensor, logits: torch.Tensor, top: int, counters: torch.Tensor) -> tuple[torch.Tensor, ExpertRows]:
+    """Picks each token's ``top`` experts by the fp32 ``logits`` [T, E] (weight: the sigmoid) and gathers the rows of ``h`` expert by
+    expert.  ``counters``: int32 [E + 1], zero, left zero."""
+    code = _dtype_of(h, "h")
+    _need(logits, torch.float32, "logits"); _need(counters, torch.int32, "counters")
+    (tokens, width), experts, dev, lib = h.shape, logits.shape[1], h.device, _cabi.load()
+    assert h.stride(1) == 1 and logits.shape[0] == tokens and logits.stride(1) == 1 and counters.numel() > experts
+    rows = tokens * top
+    block_rows = moe_block_rows(rows, experts, h.dtype)
+    max_tiles = rows // block_rows + min(rows, experts)
+    ints = torch.empty(3, rows, dtype=torch.int32, device=dev)           # expert, rank, slot
+    picked = torch.empty(2, rows, dtype=torch.float32, device=dev)       # weights by token, by sorted row
+    offsets = torch.empty(2, experts + 1, dtype=torch.int32, device=dev)
+    tiles = torch.empty(max_tiles, 4, dtype=torch.int32, device=dev)
+    rc = lib.mvb_moe_route(_ptr(logits), logits.stride(0), tokens, experts, top, block_rows, max_tiles, _ptr(counters), _ptr(ints[0]),
+                           _ptr(picked[0]), _ptr(ints[1]), _ptr(offsets[0]), _ptr(offsets[1]), _ptr(tiles), _stream())
+    _cabi.check(rc, "mvb_moe_route")
+    x = torch.empty(rows, -(-width // 8) * 8, dtype=h.dtype, device=dev)[:, :width]
+    rc = lib.mvb_moe_gather(code, _ptr(h), h.stride(0), _ptr(ints[0]), _ptr(picked[0]), _ptr(ints[1]), _ptr(offsets[0]), _ptr(x),
+                            x.stride(0), _ptr(ints[2]), _ptr(picked[1]), tokens, top, width, _stream())
+    _cabi.check(rc, "mvb_moe_gather")
+    LaunchCounter.add(2)
+    return x, ExpertRows(ints[2].view(tokens, top), picked[1], tiles, offsets[1, experts:], block_rows, experts)
+
+
+def moe_gemm(x: torch.Tensor, weight: torch.Tensor, rows: ExpertRows, k: int,
+             gated: tuple[float, float, float] | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Each expert's product over its sorted rows: ``weight`` [E, m, K] or, ``gated`` = (limit, alpha, offset), [E, 2, m, K] with the
+    gated unit behind it and the token's weight on the expert's input.  K >= k is what a weight row is padded to."""
+    code = _dtype_of(x, "x")
+    _same(x.dtype, weight=weight)
+    m = weight.shape[-2]
+    assert weight.is_contiguous() and weight.shape[0] == rows.experts and weight.dim() == (3 if gated is None else 4)
+    assert x.stride(1) == 1 and x.shape[1] >= k and weight.shape[-1] >= k
+    out = torch.empty(x.shape[0], -(-m // 8) * 8, dtype=x.dtype, device=x.device)[:, :m]
+    limit, alpha, offset = gated or (0.0, 0.0, 0.0)
+    rc = _cabi.load().mvb_moe_gemm(
+        code, _ptr(x), x.stride(0), x.shape[0], _ptr(weight), weight.shape[-1], rows.experts, m, k, 0 if gated is None else 1, float(limit),
+        float(alpha), float(offset), None if gated is None else _ptr(rows.weights), _ptr(rows.num_tiles), _ptr(rows.tiles),
+        rows.tiles.shape[0], rows.block_rows, _ptr(out), out.stride(0), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_moe_gemm")
     LaunchCounter.add(1)
     return out
