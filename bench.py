@@ -855,6 +855,130 @@ def vebonex_kernel_legs(dev, peaks) -> dict:
     return leg.rows
 
 
+# ---- Sunulorn: beside Qwen3 layers of as many active weights, and the kernels of its own ------------------------
+SUNULORN_EXPERTS, SUNULORN_TOP = 16, 2
+
+
+def sunulorn_bench_shape(size: str, window: int = 1024, keep: int = 64):
+    """Layers in turn: convolved keys + dense, window + experts, distance bias + dense, the same on borrowed keys + experts.  A token meets
+    as many feed-forward weights in every layer: two experts of a quarter and a shared one of half the dense size."""
+    from mini_vllm_b200.config import sunulorn_shape
+    width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
+    head = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": SUNULORN_EXPERTS, "top": SUNULORN_TOP},
+           "shared": {"ff": ff // 2, "limit": 7.0}}
+    turn = lambda i: [("attention", {**head, "conv": 4, "rot": {"dims": 64, "base": 1e6}}, dense),
+                      ("attention_2", {**head, "rot": {"dims": 128, "base": 1e6}, "mask": {"size": window, "keep_first": keep}}, moe),
+                      ("attention_3", head, dense), ("attention_3", {**head, "kv_from": i - 1}, moe)][i % 4]
+    return sunulorn_shape([dict(zip(("type", "mixer", "mlp"), turn(i))) for i in range(layers)], width, 32768)
+
+
+def sunulorn_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
+    return engine_throughput((f"{size}_{name}", hf) for size in sizes
+                             for name, hf in (("sunulorn", sunulorn_bench_shape(size)), ("qwen3", qwen3_twin(size))))
+
+
+def sunulorn_kernel_legs(dev, peaks) -> dict:
+    """Each kernel of the design against its roofline, next to the like kernel of the other models.  16 heads of 128 (8 KV heads), width
+    2048, 16 experts of 1536 with 2 per token, 8192 prefill tokens, 32 and 256 decode rows."""
+    from mini_vllm_b200 import ops
+    from mini_vllm_b200.models.layers.branches import alibi_slopes
+    from mini_vllm_b200.models.layers.rotary import build_cos_sin_cache
+    bf, leg = torch.bfloat16, Legs(dev, peaks)
+    rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
+    heads, kv, d, width, ff, tokens, window, keep, eps = 16, 8, 128, 2048, 6144, 8192, 1024, 64, 1e-6
+    sinks, slopes, scale = torch.zeros(heads, device=dev), alibi_slopes(heads).to(dev), d ** -0.5
+    gate = rnd(tokens, heads)
+    forms = {"plain": (-1, None), "sink": (-1, ops.AttnExtras(sinks=sinks)),
+             "distance_sink_gate": (-1, ops.AttnExtras(sinks=sinks, slopes=slopes, head_gate=gate)),
+             "window": (window - 1, None), "window_kept": (window - 1, ops.AttnExtras(keep_first=keep))}
+    q, k, v = rnd(tokens, heads, d), rnd(tokens, kv, d), rnd(tokens, kv, d)
+    for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        for name, (wl, ex) in forms.items():
+            kept = keep if ex is not None and ex.keep_first else 0
+            seen = lambda i: i + 1 if wl < 0 else min(i + 1, wl + 1) + min(kept, max(i - wl, 0))
+            leg(f"prefill_attn_{name}_{tag}", lambda i: ops.prefill_attn(q, k, v, cu, cu, max(lens), scale, wl, extras=ex), 4,
+                flops=4 * heads * d * sum(sum(seen(i) for i in range(n)) for n in lens))
+    # between projection and attention
+    proj = [rnd(tokens, (heads + 2 * kv) * d) for _ in range(4)]
+    cut = lambda x: tuple(t.unflatten(1, (-1, d)) for t in x.split([heads * d, kv * d, kv * d], dim=1))
+    pools = [torch.zeros(2, tokens // 256 + 2, 256, kv, d, device=dev, dtype=bf) for _ in range(4)]
+    table, ones = build_cos_sin_cache(128, 8192, 1e6, head_dim=128).to(dev), torch.ones(d, device=dev, dtype=bf)
+    for rows in (tokens, 256):
+        pos, slots = torch.arange(rows, device=dev), torch.randperm(rows, device=dev).to(torch.int32)
+        byts = rows * (heads + 2 * kv) * d * 2 * 2
+        part = lambda i: cut(proj[i][:rows])
+        leg(f"rope_kv_write_{rows}", lambda i: ops.rope_kv_write(*part(i), pos, table, slots, *pools[i], k_in_place=False), 4, byts=byts)
+        leg(f"qk_norm_rope_kv_write_{rows}", lambda i: ops.qk_norm_rope_kv_write(*part(i), ones, ones, eps, False, pos, table, slots, *pools[i],
+                                                                               k_in_place=False), 4, byts=byts)
+        leg(f"rope_norm_kv_write_{rows}", lambda i: ops.rope_norm_kv_write(*part(i), pos, table, slots, *pools[i], k_in_place=False, norm_dim=d,
+                                                                         eps=eps), 4, byts=byts)
+        qk = (heads + kv) * d
+        cu = None if rows == 256 else torch.tensor([0, rows], dtype=torch.int32, device=dev)
+        w4, state = rnd(4, qk), torch.zeros(256, 3, qk, device=dev, dtype=bf)
+        sl = torch.arange(256 if cu is None else 1, dtype=torch.int32, device=dev)
+        more = rows * qk * 2 * 6 if cu is None else 0
+        leg(f"short_conv_silu_{rows}", lambda i: ops.short_conv_silu(proj[i][:rows, :qk], w4, None, state, sl, cu, pos), 4, byts=rows * qk * 4 + more)
+        leg(f"short_conv_copied_keys_{rows}", lambda i: ops.short_conv(proj[i][:rows, :qk], w4, None, state, sl, cu, pos, copies=kv * d), 4,
+            byts=rows * (2 * qk + kv * d) * 2 + more)
+    del pools
+    o2 = [rnd(tokens, heads * d) for _ in range(3)]
+    leg("gate_mul_8192", lambda i: ops.gate_mul(q.flatten(1), proj[i][:, :heads * d], o2[i]), 3, byts=tokens * heads * d * 6)
+    del proj, o2
+    # norms and gated units
+    for rows, n in ((tokens, 3), (256, 48)):
+        xs, ys, w = [torch.randn(rows, width, device=dev) for _ in range(n)], [rnd(rows, width) for _ in range(n)], torch.ones(width, device=dev, dtype=bf)
+        extra, index = rnd(rows * 2, width), torch.randperm(rows * 2, device=dev).view(rows, 2).to(torch.int32)
+        leg(f"residual_norm_{rows}", lambda i: ops.residual_norm(xs[i], ys[i], w, eps, y_weight=w), n, byts=rows * width * 12)
+        leg(f"residual_norm_pair_{rows}", lambda i: ops.residual_norm_pair(xs[i], ys[i], w, w, eps), n, byts=rows * width * 14)
+        leg(f"residual_norm_pair_experts_{rows}", lambda i: ops.residual_norm_pair(xs[i], ys[i], w, w, eps, extra, index), n, byts=rows * width * 18)
+        del xs, ys
+        m = 2 if rows == tokens else 32
+        gu = [rnd(rows, 2 * ff) for _ in range(m)]
+        leg(f"act_mul_{rows}", lambda i: ops.act_mul(gu[i], ff, False), m, byts=rows * ff * 6)
+        leg(f"glu_{rows}", lambda i: ops.glu(gu[i], ff), m, byts=rows * ff * 6)
+        leg(f"glu_clamped_row_gate_{rows}", lambda i: ops.glu(gu[i], ff, 7.0, 1.702, 1.0, row_gate=gu[i][:, 0]), m, byts=rows * ff * 6)
+        del gu
+    # experts beside a dense product of as many operations
+    E, top, inter = SUNULORN_EXPERTS, SUNULORN_TOP, ff // 4
+    for rows in (tokens, 256, 32):
+        nbuf = 2 if rows == tokens else 4
+        up, down = [rnd(E, 2, inter, width, scale=width ** -0.5) for _ in range(nbuf)], [rnd(E, width, inter, scale=inter ** -0.5) for _ in range(nbuf)]
+        h, counters = rnd(rows, width), torch.zeros(E + 1, dtype=torch.int32, device=dev)
+        logits = torch.randn(rows, E, device=dev)
+        leg(f"moe_route_and_gather_{rows}", lambda i: ops.moe_sort(h, logits, top, counters), 4, byts=rows * (1 + top) * width * 2)
+        x, er = ops.moe_sort(h, logits, top, counters)
+        y = ops.moe_gemm(x, up[0], er, width, gated=(7.0, 1.702, 1.0))
+        used = len(set(torch.topk(logits, top).indices.flatten().tolist()))
+        work = lambda m, k: ({"flops": 2 * rows * top * m * k} if rows == tokens else {"byts": (used * m * k + rows * top * (m + k)) * 2})
+        leg(f"moe_gemm_gated_{rows}", lambda i: ops.moe_gemm(x, up[i], er, width, gated=(7.0, 1.702, 1.0)), nbuf, **work(2 * inter, width))
+        leg(f"moe_gemm_down_{rows}", lambda i: ops.moe_gemm(y, down[i], er, inter), nbuf, **work(width, inter))
+        # dense: as many operations for a prompt, as many weights for decoding
+        xr, wide = (rows * top, 2 * inter) if rows == tokens else (rows * top // E if rows > E else 1, used * 2 * inter)
+        wd, xd = [rnd(wide, width, scale=width ** -0.5) for _ in range(nbuf)], rnd(xr, width)
+        leg(f"dense_gemm_up_{rows}", lambda i: torch.nn.functional.linear(xd, wd[i]), nbuf,
+            **({"flops": 2 * xr * wide * width} if rows == tokens else {"byts": (wide * width + xr * (wide + width)) * 2}))
+        del up, down, wd
+    # decode attention
+    b = 256
+    for n in (1200, 4096):
+        per = -(-n // 256)
+        lens, bt = torch.full((b,), n, dtype=torch.int32, device=dev), torch.arange(b * per, dtype=torch.int32, device=dev).view(b, per)
+        pool = torch.randn(2, b * per, 256, kv, d, device=dev, dtype=bf)
+        ws = ops.decode_workspace(b, heads, d, dev)
+        for name, (wl, ex) in forms.items():
+            ex = None if ex is None else ex.rows(0, b)
+            kept = 0 if ex is None else ex.keep_first
+            ops.decode_plan(lens, wl, heads, kv, d, ws, block_table=bt, block_size=256, keep_first=kept)
+            seen = n if wl < 0 else min(n, wl + 1) + min(kept, max(n - wl - 1, 0))
+            leg(f"decode_attn_{name}_{b}x{n}", lambda i: ops.decode_attn(q[:b], pool[0], pool[1], lens, bt, scale, wl, ws, extras=ex), 1,
+                byts=b * seen * kv * d * 4)
+        del pool
+    return leg.rows
+
+
 # ---- CPU leg: the oracle restatement of the reference path on the host cores ------------------------
 class CpuReference:
     """The oracle model (restatement of the reference's PyTorch path, pinned to the reference's own engine loop by
@@ -973,6 +1097,8 @@ def main():
                          "size, and its kernels against their rooflines beside the like kernels")
     ap.add_argument("--vebonex", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
                     help="the same for the Vebonex design, beside Fupupel and Qwen3")
+    ap.add_argument("--sunulorn", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
+                    help="the same for the Sunulorn design, beside Qwen3")
     ap.add_argument("--engine-steps", type=int, default=0,
                     help="profiling aid: prefill + N decode steps of the workload without CUDA graphs, then exit")
     args = ap.parse_args()
@@ -1011,6 +1137,15 @@ def main():
         if args.vebonex in ("all", "engine"):
             line["engine"] = vebonex_throughput()
         print(json.dumps({"vebonex": line}))
+        return
+    if args.sunulorn:
+        torch.cuda.set_device(0)
+        line = {}
+        if args.sunulorn in ("all", "kernels"):
+            line["kernels"] = sunulorn_kernel_legs(torch.device("cuda", 0), measured_peaks()[0])
+        if args.sunulorn in ("all", "engine"):
+            line["engine"] = sunulorn_throughput()
+        print(json.dumps({"sunulorn": line}))
         return
     if args.kernel_legs:
         peaks, _ = measured_peaks()

@@ -108,31 +108,41 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RoutePar
   if (tid == 0) p.counters[p.experts] = 0;
 }
 
+// A warp per token and part of its row: read once, written to every expert's place.
+constexpr int kGatherPart = 128;                             // 16-byte vectors of a row that a warp takes
+
 template <class T>
 __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ h, int64_t h_stride, const int32_t* __restrict__ ids,
                                                          const float* __restrict__ weights, const int32_t* __restrict__ ranks,
                                                          const int32_t* __restrict__ offsets, T* __restrict__ out, int64_t out_stride,
-                                                         int32_t* __restrict__ slots, float* __restrict__ row_weights, int rows, int top,
-                                                         int width, int vec) {
-  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (r >= rows) return;
-  const int slot = offsets[ids[r]] + ranks[r];
-  if (lane == 0) { slots[r] = slot; row_weights[slot] = weights[r]; }
-  const T* src = h + static_cast<int64_t>(r / top) * h_stride;
-  T* dst = out + static_cast<int64_t>(slot) * out_stride;
+                                                         int32_t* __restrict__ slots, float* __restrict__ row_weights, int tokens, int top,
+                                                         int width, int parts, int vec) {
+  const int w = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = w / parts, part = w % parts;
+  if (t >= tokens) return;
+  const int64_t at = static_cast<int64_t>(t) * top;
+  constexpr int V = kVec<T>, N = kGatherPart / 32;
+  const T* src = h + t * h_stride;
+  const int first = part * kGatherPart, last = min(first + kGatherPart, width / V);
+  uint4 row[N];
   if (vec) {
-    constexpr int V = kVec<T>;
-    const uint4* s4 = reinterpret_cast<const uint4*>(src);
-    uint4* d4 = reinterpret_cast<uint4*>(dst);
-    const int n = width / V;
-    int i = lane;
-    for (; i + 96 < n; i += 128) {
-      const uint4 a = s4[i], b = s4[i + 32], c = s4[i + 64], d = s4[i + 96];
-      d4[i] = a; d4[i + 32] = b; d4[i + 64] = c; d4[i + 96] = d;
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (first + i * 32 + lane < last) row[i] = reinterpret_cast<const uint4*>(src)[first + i * 32 + lane];
+  }
+  for (int j0 = 0; j0 < top; j0 += 32) {
+    const int n = min(32, top - j0);
+    const int slot = lane < n ? offsets[ids[at + j0 + lane]] + ranks[at + j0 + lane] : 0;
+    if (part == 0 && lane < n) { slots[at + j0 + lane] = slot; row_weights[slot] = weights[at + j0 + lane]; }
+    for (int j = 0; j < n; ++j) {
+      T* dst = out + static_cast<int64_t>(__shfl_sync(0xffffffffu, slot, j)) * out_stride;
+      if (vec) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+          if (first + i * 32 + lane < last) reinterpret_cast<uint4*>(dst)[first + i * 32 + lane] = row[i];
+      } else {
+        for (int i = lane; i < width; i += 32) dst[i] = src[i];
+      }
     }
-    for (; i < n; i += 32) d4[i] = s4[i];
-  } else {
-    for (int i = lane; i < width; i += 32) dst[i] = src[i];
   }
 }
 
@@ -406,7 +416,7 @@ extern "C" int mvb_moe_route(const float* logits, int64_t logits_row_stride, int
                       tile_offsets, reinterpret_cast<int4*>(tiles)};
   const int warps = kRouteThreads / 32;
   int grid = (num_tokens + warps - 1) / warps;
-  if (grid > 2 * sm_count()) grid = 2 * sm_count();
+  if (grid > 4 * sm_count()) grid = 4 * sm_count();
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (num_experts <= 32) moe_route_kernel<1><<<grid, kRouteThreads, 0, st>>>(p);
   else if (num_experts <= 64) moe_route_kernel<2><<<grid, kRouteThreads, 0, st>>>(p);
@@ -424,16 +434,20 @@ extern "C" int mvb_moe_gather(int dtype, const void* h, int64_t h_row_stride, co
       (dtype != kBf16 && dtype != kF32))
     return kInvalidArgument;
   if (num_tokens == 0) return kOk;
-  const int rows = num_tokens * top, v = dtype == kBf16 ? 8 : 4;
+  const int v = dtype == kBf16 ? 8 : 4;
   const int vec = width % v == 0 && h_row_stride % v == 0 && out_row_stride % v == 0 && is_aligned(h, 16) && is_aligned(out, 16);
+  const int parts = vec ? (width / v + kGatherPart - 1) / kGatherPart : 1;
+  const int64_t blocks = (static_cast<int64_t>(num_tokens) * parts + 7) / 8;
+  if (blocks > 0x7fffffffLL / 8) return kUnsupportedShape;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const unsigned grid = (rows + 7) / 8;
+  const unsigned grid = static_cast<unsigned>(blocks);
   if (dtype == kBf16)
     moe_gather_kernel<<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(h), h_row_stride, ids, weights, ranks, offsets,
-                                            static_cast<__nv_bfloat16*>(out), out_row_stride, slots, row_weights, rows, top, width, vec);
+                                            static_cast<__nv_bfloat16*>(out), out_row_stride, slots, row_weights, num_tokens, top, width,
+                                            parts, vec);
   else
     moe_gather_kernel<<<grid, 256, 0, st>>>(static_cast<const float*>(h), h_row_stride, ids, weights, ranks, offsets,
-                                            static_cast<float*>(out), out_row_stride, slots, row_weights, rows, top, width, vec);
+                                            static_cast<float*>(out), out_row_stride, slots, row_weights, num_tokens, top, width, parts, vec);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 

@@ -1029,7 +1029,7 @@ def moe_block_rows(rows: int, experts: int, dtype: torch.dtype) -> int:
     """Rows of a tile of the grouped products, by how many an expert gets on average."""
     if dtype == torch.float32:
         return 64
-    return 128 if rows >= 96 * experts else 64 if rows >= 40 * experts else 32
+    return 128 if rows >= 40 * experts else 64 if rows >= 16 * experts else 32
 
 
 def moe_sort(h: torch.Tensor, logits: torch.Tensor, top: int, counters: torch.Tensor) -> tuple[torch.Tensor, ExpertRows]:

@@ -124,7 +124,7 @@ def test_random_weights_have_the_checkpoint_s_names():
 
 
 def test_tiles_grow_with_the_rows_per_expert():
-    assert [ops.moe_block_rows(r, 8, torch.bfloat16) for r in (8, 256, 320, 768, 60000)] == [32, 32, 64, 128, 128]
+    assert [ops.moe_block_rows(r, 8, torch.bfloat16) for r in (8, 120, 128, 320, 60000)] == [32, 32, 64, 128, 128]
     assert ops.moe_block_rows(60000, 8, torch.float32) == 64
 
 
