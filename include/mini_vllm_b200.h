@@ -332,7 +332,7 @@ int mvb_decode_attn_capped(const void* q, int64_t q_row_stride, const void* k_ca
 
 /*
  * What attention may have beyond a window and a cap; every field is optional (NULL / 0).
- *   sinks [num_q_heads]   a score per head that takes its part of the softmax and brings no value: not scaled, no bias, counted once
+ *   sinks [num_q_heads]   one more logit per head, as it is, in the softmax's denominator only
  *   slopes [num_q_heads]  slope * (query position - key position) is taken off a scaled score
  *   head_gate             [tokens, num_q_heads] in the activations' type: a head's output is multiplied by sigmoid(gate)
  *   keep_first            with a window: keys at positions below it stay visible
