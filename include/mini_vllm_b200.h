@@ -407,6 +407,9 @@ int mvb_rope_kv_write_f32(float* q, int64_t q_row_stride, float* k, int64_t k_ro
  *   row r also gets extra[extra_index[r, j]], j < num_extra (rows of routed experts), added in that order.
  * mvb_glu: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + offset) on a packed
  *   [rows, 2 * intermediate] projection, times sigmoid(row_gate[row]) where there is one.  mvb_clamped_glu: offset 1.
+ * mvb_residual_norm_pair_ext: the stream of row r also gets own_weights[r] (fp32; NULL: nothing) times row r of `own`, and an extra
+ *   index of -1 adds nothing.
+ * mvb_xielu: act[0] z^2 + z / 2 for z > 0, act[1] (e^z - 1 - z) + z / 2 for z <= 0 (act: fp32, on the device).
  * mvb_cap_logits: out = cap tanh(in / cap) (cap == 0: a copy), each side bf16 or fp32.
  * mvb_argmax_f32: the greedy token of fp32 logits (lowest column wins ties); scatter_* as for mvb_sample.
  */
@@ -420,6 +423,12 @@ int mvb_residual_norm_pair(int dtype, float* x, const void* y, int64_t y_row_str
                            int64_t extra_rows, const int32_t* extra_index, int num_extra, const void* weight, void* out,
                            const void* weight2, void* out2, const int32_t* row_ends, int rows, int width, float eps, int32_t* dev_status,
                            void* stream);
+int mvb_residual_norm_pair_ext(int dtype, float* x, const void* y, int64_t y_row_stride, const void* extra, int64_t extra_row_stride,
+                               int64_t extra_rows, const int32_t* extra_index, int num_extra, const void* own, int64_t own_row_stride,
+                               const float* own_weights, const void* weight, void* out, const void* weight2, void* out2,
+                               const int32_t* row_ends, int rows, int width, float eps, int32_t* dev_status, void* stream);
+int mvb_xielu(int dtype, const void* in, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows, int cols, const float* act,
+              void* stream);
 int mvb_embed_norm_pair(int dtype, const int64_t* ids, const void* table, int64_t vocab, float scale, float* x, const void* weight,
                         void* out, const void* weight2, void* out2, int rows, int width, float eps, int32_t* dev_status, void* stream);
 int mvb_glu(int dtype, const void* gate_up, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows, int intermediate,
@@ -541,14 +550,22 @@ int mvb_latent_decode(const void* q, int64_t q_row_stride, int64_t q_head_stride
  *   row's number among its expert's (ranks), every expert's first row in sorted order (offsets [num_experts + 1]), and row tiles
  *   (expert, first row, rows, 0) of at most block_rows rows; their number is tile_offsets[num_experts].  counters [num_experts + 1] must
  *   be zero and is left zero.  max_tiles >= num_tokens * top / block_rows + min(num_experts, num_tokens * top).
- * mvb_moe_gather: rows of h in sorted order; slots [num_tokens, top] and row_weights [num_tokens * top] come with it.
+ * mvb_moe_route_ext: scores are the softmax over all num_experts + num_identity outputs (softmax != 0) or sigmoids; the choice is by score
+ *   + correction [outputs] (NULL: the score), the weight is the score times weight_scale.  The outputs behind the experts are identity
+ *   experts: rank -1, no row; their weights are added up per token in identity_weights [num_tokens].
+ * mvb_moe_gather: rows of h in sorted order (none, and slot -1, for a rank of -1); slots [num_tokens, top] and row_weights [num_tokens * top] come with it.
  * mvb_moe_gemm: per expert, out rows = weight [num_experts, m, k] times x rows; gated: weight [num_experts, 2, m, k] (gate, up) and
- *   y = g sigmoid(alpha g) (u + offset), g = min(w gate, limit), u = clamp(w up, -limit, limit), w = row_weights (NULL: 1).  block_rows
+ *   y = g sigmoid(alpha g) (u + offset), g = min(w gate, limit), u = clamp(w up, -limit, limit), w = row_weights (NULL: 1); gated == 2: w multiplies y instead
+ *   of gate and up.  block_rows
  *   32, 64 or 128 (fp32: 64, w_row_stride = k), as in the tiles.
  */
 int mvb_moe_route(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int top, int block_rows, int max_tiles,
                   int32_t* counters, int32_t* ids, float* weights, int32_t* ranks, int32_t* offsets, int32_t* tile_offsets,
                   int32_t* tiles, void* stream);
+int mvb_moe_route_ext(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int num_identity, int top, int softmax,
+                      const float* correction, float weight_scale, int block_rows, int max_tiles, int32_t* counters, int32_t* ids,
+                      float* weights, int32_t* ranks, int32_t* offsets, int32_t* tile_offsets, int32_t* tiles, float* identity_weights,
+                      void* stream);
 int mvb_moe_gather(int dtype, const void* h, int64_t h_row_stride, const int32_t* ids, const float* weights, const int32_t* ranks,
                    const int32_t* offsets, void* out, int64_t out_row_stride, int32_t* slots, float* row_weights, int num_tokens, int top,
                    int width, void* stream);
@@ -556,6 +573,28 @@ int mvb_moe_gemm(int dtype, const void* x, int64_t x_row_stride, int64_t num_row
                  int num_experts, int m, int k, int gated, float limit, float alpha, float offset, const float* row_weights,
                  const int32_t* num_tiles, const int32_t* tiles, int max_tiles, int block_rows, void* out, int64_t out_row_stride,
                  int32_t* dev_status, void* stream);
+
+/*
+ * mvb_state_space: per head, S <- e^(a dt) S + dt B x^T, y = S^T C + D x, dt = softplus(raw + dt_bias); head h uses the B and C of group
+ *   h / (heads / groups).  x [num_tokens, heads, vdim], b and c [num_tokens, groups, num_states <= 256] with one row stride; fp32
+ *   dt_bias, a_log2e (= a log2(e), a <= 0) and d [heads]; state fp32 [num_slots, heads, num_states, vdim rounded up to 4].
+ * mvb_gated_group_norm: out = u / rms(u) * weight with u = y silu(z), the root mean square over each of `groups` equal consecutive parts
+ *   of a row of `width`.
+ * mvb_row_norm_rope_kv_write: q and k are divided by the root mean square of their whole row (q_dim, k_dim used coordinates) and
+ *   multiplied by q_weight, k_weight [heads * head_dim] (both NULL: neither), then rotated (cos_sin NULL: not); v is divided by the root mean square of each
+ *   head's v_dim used coordinates (0: not).  q in place; k and v to their cache slots and, with kv_in_place, in place too.
+ */
+int mvb_state_space(int dtype, const void* x, const void* b, const void* c, int64_t xbc_row_stride, const void* dt, int64_t dt_row_stride,
+                    const float* dt_bias, const float* a_log2e, const float* d, void* y, int64_t y_row_stride, float* state,
+                    const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs,
+                    int num_tokens, int heads, int groups, int num_states, int vdim, int32_t* dev_status, void* stream);
+int mvb_gated_group_norm(int dtype, const void* y, int64_t y_row_stride, const void* z, int64_t z_row_stride, const float* weight, void* out,
+                         int64_t out_row_stride, int rows, int width, int groups, float eps, void* stream);
+int mvb_row_norm_rope_kv_write(int dtype, void* q, int64_t q_row_stride, void* k, int64_t k_row_stride, void* v, int64_t v_row_stride,
+                               const void* q_weight, const void* k_weight, int q_dim, int k_dim, int v_dim, float eps,
+                               const int64_t* positions, const float* cos_sin, int64_t max_pos, const int32_t* slot_mapping, void* k_cache,
+                               void* v_cache, int64_t num_slots, int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                               int kv_in_place, int32_t* dev_status, void* stream);
 
 #ifdef __cplusplus
 }

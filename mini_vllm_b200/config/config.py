@@ -157,3 +157,10 @@ def sunulorn_shape(layers: list[dict], width: int, vocab: int, embedding_scale: 
     return sunulorn_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
                             "embedding": {"scale": width ** 0.5 if embedding_scale is None else embedding_scale}}, None, dtype,
                            max_position_embeddings)
+
+
+def rasezen_shape(layers: list[dict], width: int, vocab: int, eps: float = 1e-6, max_position_embeddings: int = 32768,
+                  dtype: torch.dtype = torch.bfloat16) -> SimpleNamespace:
+    """A Rasezen description without a checkpoint; ``layers`` as in its config.json."""
+    from .native import rasezen_config
+    return rasezen_config({"layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps}}, None, dtype, max_position_embeddings)

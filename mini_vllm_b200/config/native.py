@@ -74,7 +74,17 @@ def sunulorn_config(config: dict, shapes: dict[str, list[int]] | None = None, dt
         max_position_embeddings=max_position_embeddings, eos_token_id=config.get("eos_token_id"))
 
 
-_READERS = {"Fupupel": fupupel_config, "Vebonex": vebonex_config, "Sunulorn": sunulorn_config}
+def rasezen_config(config: dict, shapes: dict[str, list[int]] | None = None, dtype: torch.dtype = torch.bfloat16,
+                   max_position_embeddings: int = 4096) -> SimpleNamespace:
+    """Positions are rotated, so the engine's longest request sets how many there are."""
+    layers = copy.deepcopy(config["layers"])
+    return SimpleNamespace(
+        architectures=["Rasezen"], dtype=dtype, layers=layers, num_hidden_layers=len(layers), hidden_size=config["width"],
+        vocab_size=config["vocab"], rms_norm_eps=config["norm"]["eps"], max_position_embeddings=max_position_embeddings,
+        eos_token_id=config.get("eos_token_id"))
+
+
+_READERS = {"Fupupel": fupupel_config, "Vebonex": vebonex_config, "Sunulorn": sunulorn_config, "Rasezen": rasezen_config}
 
 
 def read_native(path: str, dtype: torch.dtype | None, max_position_embeddings: int) -> Any:

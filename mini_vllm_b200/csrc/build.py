@@ -20,7 +20,8 @@ LIB = PKG / "libmini_vllm_b200.so"
 OBJ_DIR = CSRC / "build"
 SOURCES = ["api.cu", "pack.cu", "rope_kv_write.cu", "decode_attn.cu", "prefill_attn.cu", "prefill_attn_ext.cu", "sampler.cu", "fused_ops.cu", "lm_head_argmax.cu",
            "residual_ops.cu", "short_conv.cu", "selective_scan.cu", "gated_delta.cu", "any_attn.cu",
-           "hyper_ops.cu", "linear_attn.cu", "latent_attn.cu", "moe.cu"]
+           "hyper_ops.cu", "linear_attn.cu", "latent_attn.cu", "moe.cu",
+           "state_space.cu", "row_norm_rope.cu"]
 HEADERS = ["common.cuh", "dtype.cuh", "chunk_common.cuh", "head_norm.cuh", "decode_plan.cuh", "delta_chunks.cuh", "linear_chunks.cuh", "host_util.cuh", "scan.cuh", "prefill_attn.cuh", "rope_any.cuh", str(ROOT / "include" / "mini_vllm_b200.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo", "--extended-lambda",
               "-Xcompiler", "-fPIC", "-I", str(ROOT / "include"), "-I", str(CSRC)]

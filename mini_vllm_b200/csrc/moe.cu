@@ -1,11 +1,14 @@
 // Mixture of experts: each token goes through the `top` experts that score highest, small gated feed-forwards with weights of their own.
 //
-//   route    z = router logits (fp32): a warp per token picks the largest, keeps sigmoid(z) as the weight, and counts.  Counts meet in
-//            shared memory first, one atomic per block and expert after that; the block that finishes last turns them into the sorted
-//            layout (first row of every expert) and into row tiles (expert, first row, rows) of at most `block_rows`.
+//   route    z = router logits (fp32): a warp per token picks the largest scores, keeps them as weights (times a factor), and counts.  A
+//            score is sigmoid(z), or the softmax of z over all outputs; a correction per output may be added for the choice alone.  The
+//            outputs behind the experts are identity experts: they give a token its own row back, so their weights are only added up.
+//            Counts meet in shared memory first, one atomic per block and expert after that; the block that finishes last turns them
+//            into the sorted layout (first row of every expert) and into row tiles (expert, first row, rows) of at most `block_rows`.
 //   gather   rows of h in the sorted order
-//   gemm 1   [gate; up] of an expert times its rows, with the weight on the expert's input and the gated unit in the epilogue:
-//            y = g sigmoid(alpha g) (u + offset), g = min(w gate, limit), u = clamp(w up, -limit, limit)
+//   gemm 1   [gate; up] of an expert times its rows, with the gated unit in the epilogue and the weight on the expert's input, or on its
+//            output: y = g sigmoid(alpha g) (u + offset), g = min(w gate, limit), u = clamp(w up, -limit, limit), or w times that with
+//            the plain gate and up
 //   gemm 2   down projection.  The sum over a token's experts is taken by whoever reads the rows (residual_ops.cu), in a fixed order.
 //
 // The sizes of the groups never reach the host, so a step with experts is one CUDA graph whatever the tokens are.
@@ -42,9 +45,14 @@ struct RouteParams {
   int32_t* offsets;             // [experts + 1]: first sorted row of an expert
   int32_t* tile_offsets;        // [experts + 1]: first tile of an expert; the last entry is the number of tiles
   int4* tiles;                  // [max_tiles] (expert, first row, rows, 0)
+  int outputs;                  // router outputs: experts + identity experts
+  int softmax;
+  const float* correction;      // [outputs] or nullptr
+  float scale;                  // factor of the weights
+  float* identity;              // [tokens]: sum of a token's identity weights; nullptr: there are none
 };
 
-template <int EPL>              // experts per lane
+template <int EPL>              // router outputs per lane
 __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteParams p) {
   __shared__ int local[kMaxExperts];
   __shared__ int is_last;
@@ -53,9 +61,29 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RoutePar
   __syncthreads();
   for (int t = blockIdx.x * warps + warp; t < p.tokens; t += gridDim.x * warps) {
     const float* row = p.logits + t * p.logits_stride;
-    float z[EPL];
+    float z[EPL], own = 0.f;                                 // z: what is compared
 #pragma unroll
-    for (int i = 0; i < EPL; ++i) z[i] = i * 32 + lane < p.experts ? row[i * 32 + lane] : -INFINITY;
+    for (int i = 0; i < EPL; ++i) z[i] = i * 32 + lane < p.outputs ? row[i * 32 + lane] : -INFINITY;
+    float top_z = 0.f, inv = 1.f;                            // softmax: e^(z - top_z) inv
+    if (p.softmax) {
+      top_z = z[0];
+#pragma unroll
+      for (int i = 1; i < EPL; ++i) top_z = fmaxf(top_z, z[i]);
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, off));
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < EPL; ++i) sum += expf(z[i] - top_z);
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      inv = 1.f / sum;
+    }
+    auto score = [&](float x) { return p.softmax ? expf(x - top_z) * inv : sigmoid_f(x); };
+    if (p.correction != nullptr) {                           // (without one the logits' order is the scores')
+#pragma unroll
+      for (int i = 0; i < EPL; ++i)
+        if (i * 32 + lane < p.outputs) z[i] = score(z[i]) + p.correction[i * 32 + lane];
+    }
     uint32_t taken = 0;
     for (int k = 0; k < p.top; ++k) {
       float best = -INFINITY;
@@ -63,7 +91,7 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RoutePar
 #pragma unroll
       for (int i = 0; i < EPL; ++i) {
         const int e = i * 32 + lane;
-        if (e < p.experts && !((taken >> i) & 1u) && (who == 0x7fffffff || z[i] > best)) { best = z[i]; who = e; }
+        if (e < p.outputs && !((taken >> i) & 1u) && (who == 0x7fffffff || z[i] > best)) { best = z[i]; who = e; }
       }
 #pragma unroll
       for (int off = 16; off > 0; off >>= 1) {
@@ -74,11 +102,14 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RoutePar
       if ((who & 31) == lane) taken |= 1u << (who >> 5);
       if (lane == 0) {
         const int64_t at = static_cast<int64_t>(t) * p.top + k;
+        const float w = score(row[who]) * p.scale;
         p.ids[at] = who;
-        p.weights[at] = sigmoid_f(best);
-        p.ranks[at] = atomicAdd(&local[who], 1);
+        p.weights[at] = w;
+        if (who < p.experts) p.ranks[at] = atomicAdd(&local[who], 1);
+        else own += w;
       }
     }
+    if (p.identity != nullptr && lane == 0) p.identity[t] = own;
   }
   __syncthreads();
   for (int e = tid; e < p.experts; e += kRouteThreads)
@@ -87,7 +118,8 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RoutePar
   for (int t = blockIdx.x * warps + warp; t < p.tokens; t += gridDim.x * warps)
     for (int k = lane; k < p.top; k += 32) {
       const int64_t at = static_cast<int64_t>(t) * p.top + k;
-      p.ranks[at] += local[p.ids[at]];
+      const int e = p.ids[at];
+      p.ranks[at] = e < p.experts ? p.ranks[at] + local[e] : -1;
     }
   __threadfence();
   __syncthreads();
@@ -131,10 +163,15 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ h
   }
   for (int j0 = 0; j0 < top; j0 += 32) {
     const int n = min(32, top - j0);
-    const int slot = lane < n ? offsets[ids[at + j0 + lane]] + ranks[at + j0 + lane] : 0;
-    if (part == 0 && lane < n) { slots[at + j0 + lane] = slot; row_weights[slot] = weights[at + j0 + lane]; }
+    const int rank = lane < n ? ranks[at + j0 + lane] : -1, slot = rank < 0 ? -1 : offsets[ids[at + j0 + lane]] + rank;
+    if (part == 0 && lane < n) {
+      slots[at + j0 + lane] = slot;
+      if (slot >= 0) row_weights[slot] = weights[at + j0 + lane];
+    }
     for (int j = 0; j < n; ++j) {
-      T* dst = out + static_cast<int64_t>(__shfl_sync(0xffffffffu, slot, j)) * out_stride;
+      const int to = __shfl_sync(0xffffffffu, slot, j);
+      if (to < 0) continue;                                  // an identity expert
+      T* dst = out + static_cast<int64_t>(to) * out_stride;
       if (vec) {
 #pragma unroll
         for (int i = 0; i < N; ++i)
@@ -152,6 +189,7 @@ struct GroupParams {
   const int4* tiles;
   int max_tiles;
   const float* row_weights;     // [sorted rows] or nullptr (gated form)
+  bool weigh_output;
   void* out; int64_t out_stride;
   int m, blocks, k;             // rows of a weight block, items per row tile, inner size
   float limit, neg_alpha_log2e, offset;
@@ -160,8 +198,9 @@ struct GroupParams {
 };
 
 __device__ __forceinline__ float gated_unit(float gate, float up, float w, const GroupParams& p) {
-  const float g = fminf(gate * w, p.limit), u = fminf(fmaxf(up * w, -p.limit), p.limit);
-  return g * fast_rcp(1.f + fast_exp2(p.neg_alpha_log2e * g)) * (u + p.offset);      // g -> -inf: 0
+  const float in = p.weigh_output ? 1.f : w, g = fminf(gate * in, p.limit), u = fminf(fmaxf(up * in, -p.limit), p.limit);
+  const float y = g * fast_rcp(1.f + fast_exp2(p.neg_alpha_log2e * g)) * (u + p.offset);      // g -> -inf: 0
+  return p.weigh_output ? y * w : y;
 }
 
 constexpr int kMoeThreads = 10 * 32;                          // producer, MMA, eight epilogue warps
@@ -403,27 +442,38 @@ static int launch_moe_gemm(const CUtensorMap& wm, const CUtensorMap& xm, const G
 
 }  // namespace mvb
 
-extern "C" int mvb_moe_route(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int top, int block_rows,
-                             int max_tiles, int32_t* counters, int32_t* ids, float* weights, int32_t* ranks, int32_t* offsets,
-                             int32_t* tile_offsets, int32_t* tiles, void* stream) {
+extern "C" int mvb_moe_route_ext(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int num_identity, int top,
+                                 int softmax, const float* correction, float weight_scale, int block_rows, int max_tiles,
+                                 int32_t* counters, int32_t* ids, float* weights, int32_t* ranks, int32_t* offsets, int32_t* tile_offsets,
+                                 int32_t* tiles, float* identity_weights, void* stream) {
   using namespace mvb;
   if (!logits || !counters || !ids || !weights || !ranks || !offsets || !tile_offsets || !tiles) return kInvalidArgument;
-  if (num_tokens <= 0 || num_experts <= 0 || top <= 0 || top > num_experts || block_rows <= 0) return kInvalidArgument;
-  if (num_experts > kMaxExperts || static_cast<int64_t>(num_tokens) * top > 0x7fffffffLL) return kUnsupportedShape;
+  if (num_tokens <= 0 || num_experts <= 0 || num_identity < 0 || top <= 0 || top > num_experts + num_identity || block_rows <= 0)
+    return kInvalidArgument;
+  if (num_identity > 0 && identity_weights == nullptr) return kInvalidArgument;
+  if (num_experts + num_identity > kMaxExperts || static_cast<int64_t>(num_tokens) * top > 0x7fffffffLL) return kUnsupportedShape;
   const int64_t rows = static_cast<int64_t>(num_tokens) * top, part = rows < num_experts ? rows : num_experts;
   if (max_tiles < rows / block_rows + part || !is_aligned(tiles, 16)) return kInvalidArgument;
+  const int outputs = num_experts + num_identity;
   const RouteParams p{logits, logits_row_stride, num_tokens, num_experts, top, block_rows, max_tiles, counters, ids, weights, ranks, offsets,
-                      tile_offsets, reinterpret_cast<int4*>(tiles)};
+                      tile_offsets, reinterpret_cast<int4*>(tiles), outputs, softmax, correction, weight_scale, identity_weights};
   const int warps = kRouteThreads / 32;
   int grid = (num_tokens + warps - 1) / warps;
   if (grid > 4 * sm_count()) grid = 4 * sm_count();
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (num_experts <= 32) moe_route_kernel<1><<<grid, kRouteThreads, 0, st>>>(p);
-  else if (num_experts <= 64) moe_route_kernel<2><<<grid, kRouteThreads, 0, st>>>(p);
-  else if (num_experts <= 128) moe_route_kernel<4><<<grid, kRouteThreads, 0, st>>>(p);
-  else if (num_experts <= 256) moe_route_kernel<8><<<grid, kRouteThreads, 0, st>>>(p);
+  if (outputs <= 32) moe_route_kernel<1><<<grid, kRouteThreads, 0, st>>>(p);
+  else if (outputs <= 64) moe_route_kernel<2><<<grid, kRouteThreads, 0, st>>>(p);
+  else if (outputs <= 128) moe_route_kernel<4><<<grid, kRouteThreads, 0, st>>>(p);
+  else if (outputs <= 256) moe_route_kernel<8><<<grid, kRouteThreads, 0, st>>>(p);
   else moe_route_kernel<32><<<grid, kRouteThreads, 0, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+extern "C" int mvb_moe_route(const float* logits, int64_t logits_row_stride, int num_tokens, int num_experts, int top, int block_rows,
+                             int max_tiles, int32_t* counters, int32_t* ids, float* weights, int32_t* ranks, int32_t* offsets,
+                             int32_t* tile_offsets, int32_t* tiles, void* stream) {
+  return mvb_moe_route_ext(logits, logits_row_stride, num_tokens, num_experts, 0, top, 0, nullptr, 1.f, block_rows, max_tiles, counters,
+                           ids, weights, ranks, offsets, tile_offsets, tiles, nullptr, stream);
 }
 
 extern "C" int mvb_moe_gather(int dtype, const void* h, int64_t h_row_stride, const int32_t* ids, const float* weights,
@@ -461,7 +511,7 @@ extern "C" int mvb_moe_gemm(int dtype, const void* x, int64_t x_row_stride, int6
   if (dtype != kBf16 && dtype != kF32) return kInvalidArgument;
   if (num_rows == 0 || max_tiles == 0) return kOk;
   if (num_rows > 0x7fffffffLL || max_tiles > 65535 || !is_aligned(tiles, 16)) return kUnsupportedShape;
-  GroupParams p{num_tiles, reinterpret_cast<const int4*>(tiles), max_tiles, row_weights, out, out_row_stride, m, 0, k, limit,
+  GroupParams p{num_tiles, reinterpret_cast<const int4*>(tiles), max_tiles, row_weights, gated == 2, out, out_row_stride, m, 0, k, limit,
                 -alpha * 1.4426950408889634f, offset, nullptr, 0, nullptr, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dtype == kF32) {

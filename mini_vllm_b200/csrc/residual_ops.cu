@@ -1,5 +1,5 @@
 // Decoder glue around an fp32 residual stream (activations in bf16 or fp32): embedding lookup + first norm, branch
-// norm + residual add + next norm, the clamped gated activation, and the tanh cap of the logits.
+// norm + residual add + next norm, the clamped gated activation, xIELU, and the tanh cap of the logits.
 //
 // One CTA per row for the norms; a row stays in registers between the reductions, so the residual stream is read and
 // written once per sublayer.  Roofline: HBM at prefill (rows * hidden * (8 + 2 * sizeof(T)) bytes for the add + norm),
@@ -23,9 +23,11 @@ struct NormParams {
   int width;
   float eps;
   // the form with two norms of the same stream (PAIR): a factor of the looked-up row, further rows to add (row `row` of the stream
-  // gets extra[extra_index[row, j]], j < num_extra), and a second weight and output (nullptr: none)
+  // gets extra[extra_index[row, j]], j < num_extra, none for an index of -1, and own_weights[row] times its row of `own`), and a second
+  // weight and output (nullptr: none)
   float table_scale;
   const void* extra; const int32_t* extra_index; int num_extra; int64_t extra_stride, extra_rows;
+  const void* own; int64_t own_stride; const float* own_weights;
   const void* weight2;
   void* out2;
   int* dev_status;
@@ -80,6 +82,7 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p)
   if constexpr (PAIR) {
     for (int e = 0; e < p.num_extra; ++e) {
       const int32_t r = p.extra_index[static_cast<int64_t>(row) * p.num_extra + e];
+      if (r == -1) continue;
       if (r < 0 || r >= p.extra_rows) {
         if (threadIdx.x == 0) report(p.dev_status, kDevBadPosition, row);
         continue;
@@ -93,6 +96,19 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const NormParams p)
         load_vec<T, V>(erow + i * V, a);
 #pragma unroll
         for (int j = 0; j < V; ++j) v[k][j] += a[j];
+      }
+    }
+    const float own = p.own_weights != nullptr ? p.own_weights[row] : 0.f;
+    if (own != 0.f) {
+      const T* orow = static_cast<const T*>(p.own) + row * p.own_stride;
+#pragma unroll
+      for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x + k * nt;
+        if (i >= nvec) continue;
+        float a[V];
+        load_vec<T, V>(orow + i * V, a);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[k][j] = fmaf(own, a[j], v[k][j]);
       }
     }
   }
@@ -169,7 +185,7 @@ static int launch_norm(const NormParams& p, int rows, cudaStream_t st) {
   constexpr int V = kVec<T>;
   const bool vec = p.width % V == 0 && p.width % 4 == 0 && p.y_stride % V == 0 && is_aligned(p.x, 16) && is_aligned(p.y, 16) &&
                    is_aligned(p.y_weight, 16) && is_aligned(p.weight, 16) && is_aligned(p.out, 16) &&
-                   p.extra_stride % V == 0 && is_aligned(p.extra, 16) && is_aligned(p.weight2, 16) && is_aligned(p.out2, 16);
+                   p.extra_stride % V == 0 && is_aligned(p.extra, 16) && p.own_stride % V == 0 && is_aligned(p.own, 16) && is_aligned(p.weight2, 16) && is_aligned(p.out2, 16);
   return vec ? launch_norm_v<T, V, PAIR>(p, rows, st) : launch_norm_v<T, 1, PAIR>(p, rows, st);
 }
 
@@ -211,6 +227,44 @@ static int launch_glu(const void* gu, int64_t is, void* out, int64_t os, int row
   auto to = static_cast<T*>(out);
   if (vec) clamped_glu_kernel<T, V><<<dim3(bx, by), 128, 0, st>>>(tg, is, to, os, rows, inter, limit, alpha, offset, tr, gate_stride);
   else clamped_glu_kernel<T, 1><<<dim3(bx, by), 128, 0, st>>>(tg, is, to, os, rows, inter, limit, alpha, offset, tr, gate_stride);
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+// xIELU: act[0] z^2 + z / 2 for z > 0, act[1] (e^z - 1 - z) + z / 2 for z <= 0
+template <class T, int V>
+__global__ void __launch_bounds__(128) xielu_kernel(const T* __restrict__ in, int64_t in_stride, T* __restrict__ out, int64_t out_stride,
+                                                    int rows, int cols, const float* __restrict__ act) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
+  if (c >= cols) return;
+  const float above = act[0], below = act[1];
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    float z[V];
+    load_vec<T, V>(in + t * in_stride + c, z);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float n = fminf(z[i], 0.f);
+      float e;                                    // e^n - 1 - n, where a small n would leave the difference nothing but rounding
+      if (sizeof(T) == 2) e = n > -0.25f ? n * n * fmaf(n, fmaf(n, fmaf(n, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f)
+                                         : fast_exp2(n * 1.4426950408889634f) - 1.f - n;
+      else e = expm1f(n) - n;
+      z[i] = (z[i] > 0.f ? above * z[i] * z[i] : below * e) + 0.5f * z[i];
+    }
+    store_vec<T, V>(out + t * out_stride + c, z);
+  }
+}
+
+template <class T>
+static int launch_xielu(const void* in, int64_t is, void* out, int64_t os, int rows, int cols, const float* act, cudaStream_t st) {
+  constexpr int V = kVec<T>;
+  const bool vec = cols % V == 0 && is % V == 0 && os % V == 0 && is_aligned(in, 16) && is_aligned(out, 16);
+  const int v = vec ? V : 1, bx = (cols + 128 * v - 1) / (128 * v);
+  int by = rows, cap = (sm_count() * 16 + bx - 1) / bx;
+  if (by > cap) by = cap;
+  if (by > 65535) by = 65535;
+  auto ti = static_cast<const T*>(in);
+  auto to = static_cast<T*>(out);
+  if (vec) xielu_kernel<T, V><<<dim3(bx, by), 128, 0, st>>>(ti, is, to, os, rows, cols, act);
+  else xielu_kernel<T, 1><<<dim3(bx, by), 128, 0, st>>>(ti, is, to, os, rows, cols, act);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
@@ -268,7 +322,8 @@ extern "C" int mvb_residual_norm(int dtype, float* x, const void* y, int64_t y_r
   using namespace mvb;
   if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
   if (rows == 0) return kOk;
-  const NormParams p{x, y, y_row_stride, nullptr, 0, y_weight, weight, out, row_ends, width, eps, 1.f, nullptr, nullptr, 0, 0, 0, nullptr, nullptr, nullptr};
+  const NormParams p{x, y, y_row_stride, nullptr, 0, y_weight, weight, out, row_ends, width, eps, 1.f, nullptr, nullptr, 0, 0, 0, nullptr, 0, nullptr, nullptr,
+                     nullptr, nullptr};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
 }
@@ -280,7 +335,7 @@ extern "C" int mvb_embed_norm(int dtype, const int64_t* ids, const void* table, 
     return kInvalidArgument;
   if (rows == 0) return kOk;
   const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, 1.f, nullptr, nullptr, 0, 0, 0, nullptr,
-                     nullptr, dev_status};
+                     0, nullptr, nullptr, nullptr, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_norm<__nv_bfloat16>(p, rows, st) : launch_norm<float>(p, rows, st);
 }
@@ -311,8 +366,24 @@ extern "C" int mvb_embed_norm_pair(int dtype, const int64_t* ids, const void* ta
     return kInvalidArgument;
   if ((weight2 == nullptr) != (out2 == nullptr)) return kInvalidArgument;
   if (rows == 0) return kOk;
-  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, scale, nullptr, nullptr, 0, 0, 0, weight2, out2,
+  const NormParams p{x, table, width, ids, vocab, nullptr, weight, out, nullptr, width, eps, scale, nullptr, nullptr, 0, 0, 0, nullptr, 0, nullptr, weight2, out2,
                      dev_status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == kBf16 ? launch_norm<__nv_bfloat16, true>(p, rows, st) : launch_norm<float, true>(p, rows, st);
+}
+
+extern "C" int mvb_residual_norm_pair_ext(int dtype, float* x, const void* y, int64_t y_row_stride, const void* extra,
+                                          int64_t extra_row_stride, int64_t extra_rows, const int32_t* extra_index, int num_extra,
+                                          const void* own, int64_t own_row_stride, const float* own_weights, const void* weight, void* out,
+                                          const void* weight2, void* out2, const int32_t* row_ends, int rows, int width, float eps,
+                                          int32_t* dev_status, void* stream) {
+  using namespace mvb;
+  if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
+  if ((weight2 == nullptr) != (out2 == nullptr) || num_extra < 0 || (num_extra > 0 && (!extra || !extra_index))) return kInvalidArgument;
+  if (own_weights != nullptr && own == nullptr) return kInvalidArgument;
+  if (rows == 0) return kOk;
+  const NormParams p{x, y, y_row_stride, nullptr, 0, nullptr, weight, out, row_ends, width, eps, 1.f, extra, extra_index, num_extra,
+                     extra_row_stride, extra_rows, own, own_row_stride, own_weights, weight2, out2, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_norm<__nv_bfloat16, true>(p, rows, st) : launch_norm<float, true>(p, rows, st);
 }
@@ -321,14 +392,18 @@ extern "C" int mvb_residual_norm_pair(int dtype, float* x, const void* y, int64_
                                       int64_t extra_row_stride, int64_t extra_rows, const int32_t* extra_index, int num_extra,
                                       const void* weight, void* out, const void* weight2, void* out2, const int32_t* row_ends, int rows,
                                       int width, float eps, int32_t* dev_status, void* stream) {
+  return mvb_residual_norm_pair_ext(dtype, x, y, y_row_stride, extra, extra_row_stride, extra_rows, extra_index, num_extra, nullptr, 0,
+                                    nullptr, weight, out, weight2, out2, row_ends, rows, width, eps, dev_status, stream);
+}
+
+extern "C" int mvb_xielu(int dtype, const void* in, int64_t in_row_stride, void* out, int64_t out_row_stride, int rows, int cols,
+                         const float* act, void* stream) {
   using namespace mvb;
-  if (!x || !y || !weight || !out || rows < 0 || width <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
-  if ((weight2 == nullptr) != (out2 == nullptr) || num_extra < 0 || (num_extra > 0 && (!extra || !extra_index))) return kInvalidArgument;
+  if (!in || !out || !act || rows < 0 || cols <= 0 || (dtype != kBf16 && dtype != kF32)) return kInvalidArgument;
   if (rows == 0) return kOk;
-  const NormParams p{x, y, y_row_stride, nullptr, 0, nullptr, weight, out, row_ends, width, eps, 1.f, extra, extra_index, num_extra,
-                     extra_row_stride, extra_rows, weight2, out2, dev_status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return dtype == kBf16 ? launch_norm<__nv_bfloat16, true>(p, rows, st) : launch_norm<float, true>(p, rows, st);
+  return dtype == kBf16 ? launch_xielu<__nv_bfloat16>(in, in_row_stride, out, out_row_stride, rows, cols, act, st)
+                        : launch_xielu<float>(in, in_row_stride, out, out_row_stride, rows, cols, act, st);
 }
 
 extern "C" int mvb_cap_logits(int in_dtype, int out_dtype, const void* in, int64_t in_row_stride, void* out,

@@ -1,4 +1,4 @@
-"""Decoder assembled layer by layer from mixer branches (attention, latent attention, selective scan, gated delta rule, gated linear
+"""Decoder assembled layer by layer from mixer branches (attention, latent attention, selective scan, state space, gated delta rule, gated linear
 attention, matrix-memory LSTM), a feed-forward of its own kind, and an fp32 residual of its own kind (``layers/residual.py``), with
 optional tanh caps on the logits.
 

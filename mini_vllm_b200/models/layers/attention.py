@@ -101,9 +101,10 @@ class FlashAttention(nn.Module):
 
     def forward_fused(self, ctx: Context, q: torch.Tensor, k: torch.Tensor | None, v: torch.Tensor | None, positions: torch.Tensor,
                       cos_sin_cache: torch.Tensor | None, out: torch.Tensor | None = None, head_gate: torch.Tensor | None = None,
-                      norm: tuple[int, float] | None = None) -> torch.Tensor:
+                      norm: tuple[int, float] | None = None, row_norm: ops.RowNorm | None = None) -> torch.Tensor:
         """q, k NOT yet rotated: RoPE (in place on q and k) + cache write in one kernel, then attention.  ``cos_sin_cache`` None: no
-        rotation; ``norm`` (size, eps): q and k are divided by their root mean square behind it.  With a ``source`` k and v are None."""
+        rotation; ``norm`` (size, eps): q and k are divided by their root mean square behind it; ``row_norm``: norms in front of it, in
+        the same kernel.  With a ``source`` k and v are None."""
         if self.source is not None:
             k, v = ctx.shared.get(self.source, (None, None))          # this step's own, for prompts without earlier tokens
             if cos_sin_cache is not None or norm is not None:
@@ -112,7 +113,9 @@ class FlashAttention(nn.Module):
         else:
             cached = (ctx.slot_mapping, self.k_cache, self.v_cache) if self._has_cache() else (None, None, None)
             in_place = ctx.prefill and ctx.block_table is None
-            if norm is not None or (cos_sin_cache is None and q.dtype != torch.bfloat16):
+            if row_norm is not None:
+                ops.row_norm_rope_kv_write(q, k, v, row_norm, positions, cos_sin_cache, *cached, kv_in_place=in_place, status=ctx.status)
+            elif norm is not None or (cos_sin_cache is None and q.dtype != torch.bfloat16):
                 ops.rope_norm_kv_write(q, k, v, positions, cos_sin_cache, *cached, k_in_place=in_place, norm_dim=norm[0] if norm else 0,
                                        eps=norm[1] if norm else 0.0, status=ctx.status)
             else:

@@ -1,7 +1,7 @@
 """Mixer branches for decoders whose layers are assembled from parts.
 
-A branch is one token mixer (attention, latent attention, selective scan, gated delta rule, gated linear attention, matrix-memory
-LSTM) without its outer projections: it declares how
+A branch is one token mixer (attention, latent attention, selective scan, state space, gated delta rule, gated linear attention,
+matrix-memory LSTM) without its outer projections: it declares how
 many rows it needs in the layer's packed input projection and how many columns it brings to the packed output
 projection, and works between the two.  ``PackedMixer`` puts any number of branches side by side on the same input: ONE
 input GEMM over the concatenated rows, the branches, ONE output GEMM over the concatenated columns, which also adds the
@@ -89,6 +89,8 @@ class AttentionBranch(Branch):
     * ``taps``: a causal convolution over time on the channels of q and k, in front of the rotation (its inputs are per-sequence state)
     * ``keys_are_values``: v is k in front of the rotation (``vdim`` = ``dim``)
     * ``norm_eps``: q and k are divided by their root mean square behind the rotation
+    * ``row_norm_eps``: the rows of q and of k, all heads together, are normalised in front of the rotation, with weights
+    * ``value_norm_eps``: every value head is divided by its root mean square
     * ``in_bias``, ``out_bias``: the projections have biases (the gate's has none)
     * ``keep_first``: first tokens that the window never drops
     * ``sink``: "zero" or "learned" - a score per head in the softmax's denominator; ``slopes``: a bias by distance, per head
@@ -105,8 +107,12 @@ class AttentionBranch(Branch):
                  padded: int, window: int | None = None, softcap: float | None = None, factor: float = 1.0, interleaved: bool = False,
                  taps: int = 0, keys_are_values: bool = False, norm_eps: float | None = None, in_bias: bool = False,
                  out_bias: bool = False, keep_first: int = 0, sink: str | None = None, slopes: torch.Tensor | None = None,
-                 gate: str | None = None, source: "AttentionBranch | None" = None):
+                 gate: str | None = None, source: "AttentionBranch | None" = None, row_norm_eps: float | None = None,
+                 value_norm_eps: float | None = None):
         super().__init__()
+        row_eps = row_norm_eps if row_norm_eps is not None else value_norm_eps
+        if row_eps is not None and (norm_eps is not None or source is not None or value_norm_eps not in (None, row_eps)):
+            raise ValueError("norms in front of the rotation have one epsilon, no norm behind it, and keys of their own")
         if keys_are_values and vdim != dim:
             raise ValueError(f"values that are the keys have their size, not {vdim} beside {dim}")
         if source is not None and (source.kv_heads, source.dim, source.vdim, source.d) != (kv_heads, dim, vdim, padded):
@@ -131,6 +137,10 @@ class AttentionBranch(Branch):
         self.in_sizes = [heads * padded] + [kv_heads * padded] * len(self.made) + [self.gate_rows]
         self.in_rows = sum(self.in_sizes)
         self.out_cols = self.out_used = heads * padded
+        self.row_norm, self.normed_rows = row_eps, row_norm_eps is not None
+        self.value_dim = 0 if value_norm_eps is None else vdim
+        if self.normed_rows:
+            self.q_norm, self.k_norm = weight(heads * padded), weight(kv_heads * padded)
         self.taps = taps
         if taps:
             self.conv_weight = weight(taps, self.qk)
@@ -170,6 +180,9 @@ class AttentionBranch(Branch):
         if self.taps:
             conv = [self._heads(w(n + ".conv"), n, c) for n, c in (("q", self.heads), ("k", self.kv_heads))]
             self.conv_weight.copy_(torch.cat(conv).flip(1).T)
+        if self.normed_rows:
+            self.q_norm.copy_(self._heads(w("q.norm"), "q", self.heads))
+            self.k_norm.copy_(self._heads(w("k.norm"), "k", self.kv_heads))
         if self.gate == "value":
             rows.append(self._heads(w("g"), "v", self.heads))
         elif self.gate == "head":
@@ -203,8 +216,12 @@ class AttentionBranch(Branch):
         k, v = kv or (None, None)
         o = out.unflatten(1, (h, d))
         mixed = torch.empty(o.shape, dtype=o.dtype, device=o.device) if self.gate == "value" else o
+        row_norm = None
+        if self.row_norm is not None:
+            weights = (self.q_norm, self.k_norm) if self.normed_rows else (None, None)
+            row_norm = ops.RowNorm(*weights, h * self.dim, g * self.dim, self.value_dim, self.row_norm)
         self.attn.forward_fused(ctx, q, k, v, positions, None if self.rotary is None else self.rotary.cos_sin_cache, out=mixed,
-                                head_gate=gate[:, :h] if self.gate == "head" else None, norm=self.norm)
+                                head_gate=gate[:, :h] if self.gate == "head" else None, norm=self.norm, row_norm=row_norm)
         if self.gate == "value":
             ops.gate_mul(mixed.flatten(1), gate, out)
 
@@ -247,6 +264,57 @@ class SelectiveScanBranch(Branch):
         ops.selective_scan(u[:, :self.inner], dt, proj[:, self.ip:self.ip + self.inner], x[:, self.rp:self.rp + self.states],
                            x[:, self.rp + self.sp:self.rp + self.sp + self.states], self.dt_bias, self.a_log2e, self.skip,
                            out[:, :self.inner], self.scan_state, ctx.state_slots, cu, positions, status=ctx.status)
+
+
+class StateSpaceBranch(Branch):
+    """Mamba-2: a short convolution on values, keys and queries, one decay and step per head, keys and queries shared by groups of heads,
+    and a norm behind the output gate over equal parts of the row."""
+
+    def __init__(self, heads: int, groups: int, states: int, vdim: int, taps: int, norm_groups: int, eps: float):
+        super().__init__()
+        if heads % groups or heads * vdim % norm_groups:
+            raise ValueError(f"{heads} heads of {vdim} values do not split into {groups} groups and {norm_groups} norm groups")
+        self.heads, self.groups, self.states, self.vdim, self.taps = heads, groups, states, vdim, taps
+        self.norm_groups, self.eps, self.inner = norm_groups, eps, heads * vdim
+        self.ip, self.gp, self.hp = pad8(self.inner), pad8(groups * states), pad8(heads)
+        self.channels = self.ip + 2 * self.gp                                 # conv channels: x | B | C
+        self.in_sizes = [self.ip, self.channels, self.hp]                     # z | x B C | dt
+        self.in_rows, self.out_cols, self.out_used = sum(self.in_sizes), self.ip, self.inner
+        self.conv_weight, self.conv_bias = weight(taps, self.channels), weight(self.channels)
+        self.dt_bias, self.a_log2e, self.skip = weight_f32(heads), weight_f32(heads), weight_f32(heads)
+        self.norm_weight = weight_f32(self.inner)
+        self.conv_state = self.memory = None
+
+    def state_specs(self, dtype):
+        return {"conv_state": ((self.taps - 1, self.channels), dtype),
+                "memory": ((self.heads, self.states, -(-self.vdim // 4) * 4), torch.float32)}
+
+    def _channels(self, t: torch.Tensor) -> torch.Tensor:
+        """Rows of x, B and C, each padded to its place."""
+        gn = self.groups * self.states
+        return torch.cat([pad_rows(p, n) for p, n in zip(t.split([self.inner, gn, gn]), (self.ip, self.gp, self.gp))])
+
+    def load(self, w: Weights):
+        z, xbc, dt = w("in").split([self.inner, self.inner + 2 * self.groups * self.states, self.heads])
+        self.conv_weight.copy_(self._channels(w("conv")).flip(1).T)
+        self.conv_bias.copy_(self._channels(w("conv.b").unsqueeze(1)).squeeze(1))
+        self.dt_bias.copy_(w("dt_bias").float())
+        self.a_log2e.copy_(-torch.exp(w("A_log").float()) * LOG2E)
+        self.skip.copy_(w("D").float())
+        self.norm_weight.copy_(w("norm").float())
+        return torch.cat([pad_rows(z, self.ip), self._channels(xbc), pad_rows(dt, self.hp)]), pad_cols(w("o"), self.out_cols)
+
+    def forward(self, ctx, proj, out, positions):
+        cu, gn = ragged(ctx), self.groups * self.states
+        z, xbc, dt = proj.split(self.in_sizes, dim=1)
+        u = ops.short_conv_silu(xbc, self.conv_weight, self.conv_bias, self.conv_state, ctx.state_slots, cu, positions, status=ctx.status)
+        x, b, c = u.split([self.ip, self.gp, self.gp], dim=1)
+        b, c = (t[:, :gn].unflatten(1, (self.groups, self.states)) for t in (b, c))
+        y = torch.empty(u.shape[0], self.ip, dtype=u.dtype, device=u.device)
+        x, o = (t[:, :self.inner].unflatten(1, (self.heads, self.vdim)) for t in (x, y))
+        ops.state_space(x, b, c, dt[:, :self.heads], self.dt_bias, self.a_log2e, self.skip, o, self.memory, ctx.state_slots, cu, positions,
+                        status=ctx.status)
+        ops.gated_group_norm(y[:, :self.inner], z[:, :self.inner], self.norm_weight, out[:, :self.inner], self.norm_groups, self.eps)
 
 
 class GatedDeltaBranch(Branch):

@@ -6,12 +6,24 @@ weights) comes back as rows to be added to the residual stream (``routed``).
 """
 from __future__ import annotations
 
+from dataclasses import dataclass, replace
+
 import torch
 import torch.nn.functional as F
 from torch import nn
 
 from ... import ops
-from .branches import Weights, pad8, pad_cols, pad_rows, weight
+from .branches import Weights, pad8, pad_cols, pad_rows, weight, weight_f32
+
+
+@dataclass(frozen=True)
+class Routed:
+    """What routed experts add to the residual stream: token t gets ``rows[slots[t, j]]`` for every j (a slot of -1: nothing) and, with
+    identity experts, ``own_weights[t]`` times its own input row."""
+    rows: torch.Tensor
+    slots: torch.Tensor
+    own: torch.Tensor | None = None
+    own_weights: torch.Tensor | None = None
 
 
 class GatedFeed(nn.Module):
@@ -40,26 +52,57 @@ class GatedFeed(nn.Module):
         return None
 
 
-class ExpertFeed(nn.Module):
-    """Each token through the ``top`` of ``experts`` gated units that score highest; the score, a sigmoid, multiplies the expert's input.
-    ``shared`` (a ``GatedFeed``) runs for every token beside them."""
+class XieluFeed(nn.Module):
+    """``p z^2 + z / 2`` for z = up h > 0, ``(1/2 + q) (e^z - 1 - z) + z / 2`` below, p and q the softplus of two learned numbers."""
 
-    def __init__(self, width: int, inter: int, experts: int, top: int, limit: float, alpha: float, offset: float,
-                 shared: GatedFeed | None = None):
+    def __init__(self, width: int, inter: int):
         super().__init__()
-        if not 0 < top <= experts:
-            raise ValueError(f"{top} of {experts} experts cannot be chosen")
+        self.ip = self.out_cols = pad8(inter)                                     # padding: 0 gives 0
+        self.up, self.act = weight(self.ip, width), weight_f32(2)
+
+    @torch.no_grad()
+    def load(self, w: Weights) -> torch.Tensor:
+        self.up.copy_(pad_rows(w("up"), self.ip))
+        self.act.copy_(F.softplus(w("act").float()) + torch.tensor([0.0, 0.5], device=self.act.device))
+        return pad_cols(w("down"), self.ip)
+
+    def write(self, h: torch.Tensor, out: torch.Tensor) -> None:
+        ops.xielu(F.linear(h, self.up), self.act, out=out)
+
+    def routed(self, h: torch.Tensor, status: torch.Tensor | None) -> None:
+        return None
+
+
+class ExpertFeed(nn.Module):
+    """Each token through the ``top`` of ``experts`` gated units that score highest.  ``shared`` (a ``GatedFeed``) runs for every token
+    beside them.
+
+    Options: ``softmax`` - scores are the softmax over all router outputs instead of sigmoids; ``corrected`` - a number per output is
+    added for the choice alone; ``scale`` - a factor of the scores as weights; ``weigh_output`` - the weight multiplies the expert's output
+    instead of its input; ``identity`` - so many further router outputs return the token's own row."""
+
+    def __init__(self, width: int, inter: int, experts: int, top: int, limit: float = float("inf"), alpha: float = 1.0, offset: float = 0.0,
+                 shared: GatedFeed | None = None, softmax: bool = False, corrected: bool = False, scale: float = 1.0,
+                 weigh_output: bool = False, identity: int = 0):
+        super().__init__()
+        if not 0 < top <= experts + identity:
+            raise ValueError(f"{top} of {experts + identity} experts cannot be chosen")
         self.width, self.inter, self.ip, self.top, self.unit, self.shared = width, inter, pad8(inter), top, (limit, alpha, offset), shared
+        self.experts, self.weigh_output = experts, weigh_output
+        self.correction = weight_f32(experts + identity) if corrected else None
+        self.routing = ops.Routing(softmax, None, scale, identity)
         self.out_cols = 0 if shared is None else shared.out_cols
         kp = width if torch.get_default_dtype() == torch.float32 else pad8(width)      # (TMA rows start at 16-byte boundaries)
-        self.router = weight(experts, width)
+        self.router = weight(experts + identity, width)
         self.gate_up, self.down = weight(experts, 2, self.ip, kp), weight(experts, width, self.ip)
         self.register_buffer("counters", torch.zeros(experts + 1, dtype=torch.int32), persistent=False)
 
     @torch.no_grad()
     def load(self, w: Weights) -> torch.Tensor | None:
         self.router.copy_(w("router"))
-        for e in range(self.router.shape[0]):
+        if self.correction is not None:
+            self.correction.copy_(w("correction").float())
+        for e in range(self.experts):
             for i, name in enumerate(("gate", "up")):
                 self.gate_up[e, i].copy_(pad_cols(pad_rows(w(f"e{e}.{name}"), self.ip), self.gate_up.shape[3]))
             self.down[e].copy_(pad_cols(w(f"e{e}.down"), self.ip))
@@ -69,12 +112,11 @@ class ExpertFeed(nn.Module):
         if self.shared is not None:
             self.shared.write(h, out)
 
-    def routed(self, h: torch.Tensor, status: torch.Tensor | None) -> tuple[torch.Tensor, torch.Tensor]:
-        """(expert outputs in sorted order, the rows of each token)"""
+    def routed(self, h: torch.Tensor, status: torch.Tensor | None) -> Routed:
         if h.dtype == torch.float32:
             logits = F.linear(h, self.router)
         else:
             logits = torch.mm(h, self.router.T, out_dtype=torch.float32)
-        x, rows = ops.moe_sort(h, logits, self.top, self.counters)
-        y = ops.moe_gemm(x, self.gate_up, rows, self.width, gated=self.unit, status=status)
-        return ops.moe_gemm(y, self.down, rows, self.ip, status=status), rows.slots
+        x, rows = ops.moe_sort(h, logits, self.top, self.counters, replace(self.routing, correction=self.correction))
+        y = ops.moe_gemm(x, self.gate_up, rows, self.width, gated=self.unit, weigh_output=self.weigh_output, status=status)
+        return Routed(ops.moe_gemm(y, self.down, rows, self.ip, status=status), rows.slots, h, rows.identity)

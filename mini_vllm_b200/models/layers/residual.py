@@ -7,7 +7,8 @@ per sublayer:
 * ``SandwichStream``: one fp32 stream, a norm in front of and behind every sublayer;
 * ``HyperStream``: several fp32 streams.  A sublayer reads a weighted sum of them; afterwards every stream becomes a weighted sum of all
   old ones plus its own multiple of the output.  Norms in equal consecutive groups, learned positions added to the embedding;
-* ``ParallelStream``: one fp32 stream, from which a mixer and a feed-forward side by side read through norms of their own.
+* ``ParallelStream``: one fp32 stream, from which a mixer and a feed-forward side by side read through norms of their own or through one
+  they share.
 """
 from __future__ import annotations
 
@@ -106,36 +107,36 @@ class ParallelConnection(nn.Module):
 
     @torch.no_grad()
     def load(self, prefix: str, index: int, w: Weights) -> None:
-        self.norm.copy_(w(f"{prefix}norm{index}"))
+        self.norm.copy_(w(f"{prefix}norm{index}"))                    # (a single number is every coordinate's)
         if self.feed_norm is not None:
             self.feed_norm.copy_(w(f"{prefix}norm{index + 1}"))
 
 
 class ParallelStream(nn.Module):
-    """A sublayer's input is a pair of normalised rows (the second None without a feed-forward); its output what one GEMM adds up, with the
-    rows of routed experts beside it, if there are any."""
+    """A sublayer's input is a pair of normalised rows (the second None without a feed-forward, the same as the first with
+    ``shared_norm``); its output what one GEMM adds up, with what routed experts add beside it, if there are any."""
 
-    def __init__(self, width: int, eps: float, embedding_scale: float = 1.0):
+    def __init__(self, width: int, eps: float, embedding_scale: float = 1.0, shared_norm: bool = False):
         super().__init__()
-        self.width, self.eps, self.embedding_scale = width, eps, embedding_scale
+        self.width, self.eps, self.embedding_scale, self.shared_norm = width, eps, embedding_scale, shared_norm
 
     def connection(self, norms: int = 2) -> nn.Module:
-        return ParallelConnection(self.width, norms)
+        return ParallelConnection(self.width, 1 if self.shared_norm else norms)
 
     def load(self, w: Weights) -> None:
         pass
 
     def start(self, ctx, ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, first: ParallelConnection):
         x, h, h_feed = ops.embed_norm_pair(ids, table, self.embedding_scale, first.norm, first.feed_norm, self.eps, status=ctx.status)
-        return x, (h, h_feed)
+        return x, (h, h if self.shared_norm else h_feed)
 
     def advance(self, x: torch.Tensor, y, done: ParallelConnection, following: ParallelConnection | None, final_norm: torch.Tensor,
                 rows: torch.Tensor | None = None):
         summed, routed = y
         norm, feed_norm = (final_norm, None) if following is None else (following.norm, following.feed_norm)
-        extra, index = routed or (None, None)
-        h = ops.residual_norm_pair(x, summed, norm, feed_norm, self.eps, extra, index, row_ends=rows)
-        return h[0] if following is None else h
+        more = {} if routed is None else {"extra": routed.rows, "extra_index": routed.slots, "own": routed.own, "own_weights": routed.own_weights}
+        h, h_feed = ops.residual_norm_pair(x, summed, norm, feed_norm, self.eps, row_ends=rows, **more)
+        return h if following is None else (h, h if self.shared_norm else h_feed)
 
     @staticmethod
     def total(x: torch.Tensor) -> torch.Tensor:

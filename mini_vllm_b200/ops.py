@@ -576,6 +576,48 @@ def rope_norm_kv_write(q: torch.Tensor, k: torch.Tensor | None, v: torch.Tensor 
     LaunchCounter.add(1)
 
 
+@dataclass(frozen=True)
+class RowNorm:
+    """Norms in front of the rotation: q and k over the root mean square of their whole row (``q_dim``, ``k_dim`` used coordinates) times
+    weights [heads * head_dim] (None: neither), values over that of their head's ``v_dim`` used coordinates (0: not)."""
+    q_weight: torch.Tensor | None
+    k_weight: torch.Tensor | None
+    q_dim: int
+    k_dim: int
+    v_dim: int
+    eps: float
+
+
+def row_norm_rope_kv_write(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, norm: RowNorm, positions: torch.Tensor,
+                           cos_sin: torch.Tensor | None, slot_mapping: torch.Tensor | None, k_cache: torch.Tensor | None,
+                           v_cache: torch.Tensor | None, kv_in_place: bool = True, status: torch.Tensor | None = None) -> None:
+    """``norm``, then the rotation (``cos_sin`` None: none), then the cache write; q in place, k and v too if asked.  Either dtype, any even
+    head size."""
+    code = _dtype_of(q, "q")
+    _same(q.dtype, k=k, v=v, q_weight=norm.q_weight, k_weight=norm.k_weight)
+    _same(torch.float32, cos_sin=cos_sin)
+    _need(positions, torch.int64, "positions")
+    for t, n in ((q, "q"), (k, "k"), (v, "v")):
+        _heads_contiguous(t, n)
+    (tokens, hq, d), hkv, num_slots = q.shape, k.shape[1], 0
+    assert k.shape == v.shape == (tokens, hkv, d) and (cos_sin is None or (cos_sin.is_contiguous() and cos_sin.shape[1] == d))
+    for w, heads in ((norm.q_weight, hq), (norm.k_weight, hkv)):
+        assert w is None or (w.is_contiguous() and w.numel() == heads * d)
+    if slot_mapping is not None:
+        _need(slot_mapping, torch.int32, "slot_mapping")
+        _same(q.dtype, k_cache=k_cache, v_cache=v_cache)
+        assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[-2:] == (hkv, d)
+        num_slots = k_cache.shape[0] * k_cache.shape[1]
+    cached = slot_mapping is not None
+    rc = _cabi.load().mvb_row_norm_rope_kv_write(
+        code, _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(norm.q_weight), _ptr(norm.k_weight), norm.q_dim,
+        norm.k_dim, norm.v_dim, float(norm.eps), _ptr(positions), _ptr(cos_sin), 0 if cos_sin is None else cos_sin.shape[0],
+        _ptr(slot_mapping), _ptr(k_cache) if cached else None, _ptr(v_cache) if cached else None, num_slots, tokens, hq, hkv, d,
+        1 if kv_in_place else 0, _ptr(status), _stream())
+    _cabi.check(rc, "mvb_row_norm_rope_kv_write")
+    LaunchCounter.add(1)
+
+
 def residual_norm(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, y_weight: torch.Tensor | None = None,
                   row_ends: torch.Tensor | None = None) -> torch.Tensor:
     """fp32 residual stream: ``x += y`` (or ``x += rmsnorm(y, y_weight)``) in place, returns ``rmsnorm(x, weight)`` in y's
@@ -615,12 +657,12 @@ def embed_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps
 
 def residual_norm_pair(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, weight2: torch.Tensor | None, eps: float,
                        extra: torch.Tensor | None = None, extra_index: torch.Tensor | None = None,
-                       row_ends: torch.Tensor | None = None,
+                       row_ends: torch.Tensor | None = None, own: torch.Tensor | None = None, own_weights: torch.Tensor | None = None,
                        status: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
-    """``x += y`` in place, and ``extra[extra_index[row, j]]`` for every j; returns the norms of x with ``weight`` and ``weight2`` (None:
-    None) in y's dtype.  ``row_ends`` as in ``residual_norm``."""
+    """``x += y`` in place, and ``extra[extra_index[row, j]]`` for every j (an index of -1: nothing), and ``own_weights[row] own[row]``;
+    returns the norms of x with ``weight`` and ``weight2`` (None: None) in y's dtype.  ``row_ends`` as in ``residual_norm``."""
     code = _dtype_of(y, "y")
-    _need(x, torch.float32, "x"); _same(y.dtype, weight=weight, weight2=weight2, extra=extra)
+    _need(x, torch.float32, "x"); _same(y.dtype, weight=weight, weight2=weight2, extra=extra, own=own)
     assert x.dim() == 2 and x.is_contiguous() and y.shape == x.shape and y.stride(1) == 1
     rows, width = x.shape
     if row_ends is not None:
@@ -631,15 +673,18 @@ def residual_norm_pair(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, w
         _need(extra_index, torch.int32, "extra_index")
         count = extra_index.shape[1]
         assert extra_index.shape[0] == x.shape[0] and extra_index.is_contiguous() and extra.shape[1] >= width and extra.stride(1) == 1
+    if own_weights is not None:
+        _need(own_weights, torch.float32, "own_weights")
+        assert own.shape == x.shape and own.stride(1) == 1 and own_weights.is_contiguous() and own_weights.numel() == x.shape[0]
     out = torch.empty(rows, width, dtype=y.dtype, device=x.device)
     out2 = None if weight2 is None else torch.empty_like(out)
     if rows == 0:
         return out, out2
-    rc = _cabi.load().mvb_residual_norm_pair(
+    rc = _cabi.load().mvb_residual_norm_pair_ext(
         code, _ptr(x), _ptr(y), y.stride(0), _ptr(extra), 0 if extra is None else extra.stride(0), 0 if extra is None else extra.shape[0],
-        _ptr(extra_index), count, _ptr(weight), _ptr(out), _ptr(weight2), _ptr(out2), _ptr(row_ends), rows, width, float(eps), _ptr(status),
-        _stream())
-    _cabi.check(rc, "mvb_residual_norm_pair")
+        _ptr(extra_index), count, _ptr(own) if own_weights is not None else None, 0 if own is None else own.stride(0), _ptr(own_weights),
+        _ptr(weight), _ptr(out), _ptr(weight2), _ptr(out2), _ptr(row_ends), rows, width, float(eps), _ptr(status), _stream())
+    _cabi.check(rc, "mvb_residual_norm_pair_ext")
     LaunchCounter.add(1)
     return out, out2
 
@@ -683,6 +728,20 @@ def glu(gate_up: torch.Tensor, intermediate: int, limit: float = float("inf"), a
 def clamped_glu(gate_up: torch.Tensor, intermediate: int, limit: float, alpha: float) -> torch.Tensor:
     """``glu`` with one added to the clamped up projection."""
     return glu(gate_up, intermediate, limit, alpha, 1.0)
+
+
+def xielu(z: torch.Tensor, act: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``act[0] z^2 + z / 2`` for z > 0, ``act[1] (e^z - 1 - z) + z / 2`` for z <= 0 (``act``: fp32 [2])."""
+    code = _dtype_of(z, "z")
+    _need(act, torch.float32, "act")
+    if out is None:
+        out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    _same(z.dtype, out=out)
+    assert z.dim() == 2 and z.stride(1) == 1 and out.shape == z.shape and out.stride(1) == 1 and act.numel() == 2
+    rc = _cabi.load().mvb_xielu(code, _ptr(z), z.stride(0), _ptr(out), out.stride(0), z.shape[0], z.shape[1], _ptr(act), _stream())
+    _cabi.check(rc, "mvb_xielu")
+    LaunchCounter.add(1)
+    return out
 
 
 def cap_logits(logits: torch.Tensor, cap: float, out_dtype: torch.dtype) -> torch.Tensor:
@@ -771,6 +830,45 @@ def selective_scan(u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, b: torch.
         _ptr(dt_bias), _ptr(a_log2e), _ptr(d), _ptr(out), out.stride(0), st, sl, n, _ptr(cu_seqlens_q), _ptr(positions),
         num_seqs, tokens, channels, b.shape[1], a_log2e.shape[1], _ptr(status), _stream())
     _cabi.check(rc, "mvb_selective_scan")
+    LaunchCounter.add(1)
+    return out
+
+
+def state_space(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log2e: torch.Tensor,
+                d: torch.Tensor, out: torch.Tensor, state: torch.Tensor | None, state_slots: torch.Tensor | None,
+                cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor, status: torch.Tensor | None = None) -> torch.Tensor:
+    """``S <- e^(a dt) S + dt b x^T``, ``out = S^T c + d x`` per head, dt = softplus(raw + bias): x and out [T, heads, vdim], b and c
+    [T, groups, N], raw ``dt`` [T, heads]; fp32 ``dt_bias``, ``a_log2e`` (a times log2(e)) and ``d`` [heads]; ``state`` fp32
+    [slots, heads, N, vdim padded to 4]."""
+    code = _dtype_of(x, "x")
+    _same(x.dtype, b=b, c=c, dt=dt, out=out)
+    _same(torch.float32, dt_bias=dt_bias, a_log2e=a_log2e, d=d, state=state)
+    _need(positions, torch.int64, "positions")
+    for t, name in ((x, "x"), (b, "b"), (c, "c"), (out, "out")):
+        _heads_contiguous(t, name)
+    (tokens, heads, vdim), (groups, n) = x.shape, b.shape[1:]
+    assert x.stride(0) == b.stride(0) == c.stride(0) or tokens <= 1
+    assert b.shape == c.shape == (tokens, groups, n) and out.shape == x.shape and dt.shape == (tokens, heads) and dt.stride(1) == 1
+    assert state is None or state.shape[1:] == (heads, n, -(-vdim // 4) * 4)
+    st, sl, slots = _state_args(state, state_slots)
+    num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
+    rc = _cabi.load().mvb_state_space(
+        code, _ptr(x), _ptr(b), _ptr(c), x.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log2e), _ptr(d), _ptr(out),
+        out.stride(0), st, sl, slots, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, heads, groups, n, vdim, _ptr(status), _stream())
+    _cabi.check(rc, "mvb_state_space")
+    LaunchCounter.add(1)
+    return out
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    """``u / rms(u) * weight`` with ``u = y silu(z)``, the root mean square over each of ``groups`` equal parts of the row (fp32 weight)."""
+    code = _dtype_of(y, "y")
+    _same(y.dtype, z=z, out=out); _need(weight, torch.float32, "weight")
+    rows, width = y.shape
+    assert z.shape == out.shape == y.shape and y.stride(1) == z.stride(1) == out.stride(1) == 1 and weight.numel() == width
+    rc = _cabi.load().mvb_gated_group_norm(code, _ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), out.stride(0), rows,
+                                           width, groups, float(eps), _stream())
+    _cabi.check(rc, "mvb_gated_group_norm")
     LaunchCounter.add(1)
     return out
 
@@ -1023,6 +1121,18 @@ class ExpertRows:
     num_tiles: torch.Tensor       # int32 [1]
     block_rows: int
     experts: int
+    identity: torch.Tensor | None = None      # fp32 [T]: what a token's identity experts weigh together
+
+
+@dataclass(frozen=True)
+class Routing:
+    """How router logits become choices and weights: scores are sigmoids or the ``softmax`` over all outputs; the choice is by score plus
+    ``correction`` (fp32 [outputs]; None: by score); the weight is the score times ``scale``.  The last ``identity`` outputs are experts
+    that return a token's own row."""
+    softmax: bool = False
+    correction: torch.Tensor | None = None
+    scale: float = 1.0
+    identity: int = 0
 
 
 def moe_block_rows(rows: int, experts: int, dtype: torch.dtype) -> int:
@@ -1032,12 +1142,14 @@ def moe_block_rows(rows: int, experts: int, dtype: torch.dtype) -> int:
     return 128 if rows >= 40 * experts else 64 if rows >= 16 * experts else 32
 
 
-def moe_sort(h: torch.Tensor, logits: torch.Tensor, top: int, counters: torch.Tensor) -> tuple[torch.Tensor, ExpertRows]:
-    """Picks each token's ``top`` experts by the fp32 ``logits`` [T, E] (weight: the sigmoid) and gathers the rows of ``h`` expert by
-    expert.  ``counters``: int32 [E + 1], zero, left zero."""
+def moe_sort(h: torch.Tensor, logits: torch.Tensor, top: int, counters: torch.Tensor,
+             routing: Routing = Routing()) -> tuple[torch.Tensor, ExpertRows]:
+    """Picks each token's ``top`` experts by the fp32 ``logits`` [T, E + identity] and gathers the rows of ``h`` expert by expert.
+    ``counters``: int32 [E + 1], zero, left zero."""
     code = _dtype_of(h, "h")
-    _need(logits, torch.float32, "logits"); _need(counters, torch.int32, "counters")
-    (tokens, width), experts, dev, lib = h.shape, logits.shape[1], h.device, _cabi.load()
+    _need(logits, torch.float32, "logits"); _need(counters, torch.int32, "counters"); _same(torch.float32, correction=routing.correction)
+    (tokens, width), experts, dev, lib = h.shape, logits.shape[1] - routing.identity, h.device, _cabi.load()
+    assert routing.correction is None or routing.correction.numel() == logits.shape[1]
     assert h.stride(1) == 1 and logits.shape[0] == tokens and logits.stride(1) == 1 and counters.numel() > experts
     rows = tokens * top
     block_rows = moe_block_rows(rows, experts, h.dtype)
@@ -1046,21 +1158,23 @@ def moe_sort(h: torch.Tensor, logits: torch.Tensor, top: int, counters: torch.Te
     picked = torch.empty(2, rows, dtype=torch.float32, device=dev)       # weights by token, by sorted row
     offsets = torch.empty(2, experts + 1, dtype=torch.int32, device=dev)
     tiles = torch.empty(max_tiles, 4, dtype=torch.int32, device=dev)
-    rc = lib.mvb_moe_route(_ptr(logits), logits.stride(0), tokens, experts, top, block_rows, max_tiles, _ptr(counters), _ptr(ints[0]),
-                           _ptr(picked[0]), _ptr(ints[1]), _ptr(offsets[0]), _ptr(offsets[1]), _ptr(tiles), _stream())
-    _cabi.check(rc, "mvb_moe_route")
+    identity = torch.empty(tokens, dtype=torch.float32, device=dev) if routing.identity else None
+    rc = lib.mvb_moe_route_ext(_ptr(logits), logits.stride(0), tokens, experts, routing.identity, top, int(routing.softmax),
+                               _ptr(routing.correction), float(routing.scale), block_rows, max_tiles, _ptr(counters), _ptr(ints[0]),
+                               _ptr(picked[0]), _ptr(ints[1]), _ptr(offsets[0]), _ptr(offsets[1]), _ptr(tiles), _ptr(identity), _stream())
+    _cabi.check(rc, "mvb_moe_route_ext")
     x = torch.empty(rows, -(-width // 8) * 8, dtype=h.dtype, device=dev)[:, :width]
     rc = lib.mvb_moe_gather(code, _ptr(h), h.stride(0), _ptr(ints[0]), _ptr(picked[0]), _ptr(ints[1]), _ptr(offsets[0]), _ptr(x),
                             x.stride(0), _ptr(ints[2]), _ptr(picked[1]), tokens, top, width, _stream())
     _cabi.check(rc, "mvb_moe_gather")
     LaunchCounter.add(2)
-    return x, ExpertRows(ints[2].view(tokens, top), picked[1], tiles, offsets[1, experts:], block_rows, experts)
+    return x, ExpertRows(ints[2].view(tokens, top), picked[1], tiles, offsets[1, experts:], block_rows, experts, identity)
 
 
 def moe_gemm(x: torch.Tensor, weight: torch.Tensor, rows: ExpertRows, k: int,
-             gated: tuple[float, float, float] | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
+             gated: tuple[float, float, float] | None = None, weigh_output: bool = False, status: torch.Tensor | None = None) -> torch.Tensor:
     """Each expert's product over its sorted rows: ``weight`` [E, m, K] or, ``gated`` = (limit, alpha, offset), [E, 2, m, K] with the
-    gated unit behind it and the token's weight on the expert's input.  K >= k is what a weight row is padded to."""
+    gated unit behind it and the token's weight on the expert's input, or on the unit's output (``weigh_output``).  K >= k is what a weight row is padded to."""
     code = _dtype_of(x, "x")
     _same(x.dtype, weight=weight)
     m = weight.shape[-2]
@@ -1069,7 +1183,7 @@ def moe_gemm(x: torch.Tensor, weight: torch.Tensor, rows: ExpertRows, k: int,
     out = torch.empty(x.shape[0], -(-m // 8) * 8, dtype=x.dtype, device=x.device)[:, :m]
     limit, alpha, offset = gated or (0.0, 0.0, 0.0)
     rc = _cabi.load().mvb_moe_gemm(
-        code, _ptr(x), x.stride(0), x.shape[0], _ptr(weight), weight.shape[-1], rows.experts, m, k, 0 if gated is None else 1, float(limit),
+        code, _ptr(x), x.stride(0), x.shape[0], _ptr(weight), weight.shape[-1], rows.experts, m, k, 0 if gated is None else 2 if weigh_output else 1, float(limit),
         float(alpha), float(offset), None if gated is None else _ptr(rows.weights), _ptr(rows.num_tiles), _ptr(rows.tiles),
         rows.tiles.shape[0], rows.block_rows, _ptr(out), out.stride(0), _ptr(status), _stream())
     _cabi.check(rc, "mvb_moe_gemm")
