@@ -979,6 +979,125 @@ def sunulorn_kernel_legs(dev, peaks) -> dict:
     return leg.rows
 
 
+# ---- Rasezen: beside Sunulorn, Fupupel and Qwen3 layers of about as many active weights, and the kernels of its own ----------------
+def rasezen_bench_shape(size: str, window: int = 1024):
+    """Layers in turn: state space + dense, window + experts, state space + experts, window + dense.  State-space layers have twice the width
+    in heads of 64, 128 states and 8 groups; the dense feed-forward has as many weights as a gated one of ``ff``, the experts as in
+    ``sunulorn_bench_shape`` with two identity experts more."""
+    from mini_vllm_b200.config import rasezen_shape
+    width, heads, kv, ff, layers = FUPUPEL_SIZES[size]
+    space = {"heads": 2 * width // 64, "groups": 8, "state": 128, "vdim": 64, "conv": 4, "norm_groups": 8}
+    attn = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window}, "rot": {"base": 1e6, "dims": 128}}
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": SUNULORN_EXPERTS, "top": SUNULORN_TOP, "identity": 2, "scale": 2.0},
+           "shared": {"ff": ff // 2}}
+    turn = [("mamba2", space, dense), ("attention", attn, moe), ("mamba2", space, moe), ("attention", attn, dense)]
+    return rasezen_shape([dict(zip(("type", "mixer", "mlp"), turn[i % 4])) for i in range(layers)], width, 32768)
+
+
+def rasezen_throughput(sizes=tuple(FUPUPEL_SIZES)) -> dict:
+    return engine_throughput((f"{size}_{name}", hf) for size in sizes
+                             for name, hf in (("rasezen", rasezen_bench_shape(size)), ("sunulorn", sunulorn_bench_shape(size)),
+                                              ("fupupel", fupupel_bench_shape(size)), ("qwen3", qwen3_twin(size))))
+
+
+def rasezen_kernel_legs(dev, peaks) -> dict:
+    """Each kernel of the design against its roofline, next to the like kernel of the other models.  Width 2048, state-space layers of 64
+    heads of 64 (and, for the comparison, 16 of 128) with 128 states, 16 attention heads of 128 (8 KV heads), 16 experts of 1536 with
+    2 per token and 2 identity experts, 8192 prefill tokens, 256 decode rows."""
+    from mini_vllm_b200 import ops
+    from mini_vllm_b200.models.layers.rotary import build_cos_sin_cache
+    bf, leg = torch.bfloat16, Legs(dev, peaks)
+    rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
+    width, tokens, n, eps, inner = 2048, 8192, 128, 1e-6, 4096
+
+    def recurrences(tag, rows, cu, pos, slots, nbuf):
+        for heads, vdim, groups in ((64, 64, 8), (16, 128, 16)):
+            cols, keys = heads * vdim, groups * n
+            xbc, dt = [rnd(rows, cols + 2 * keys) for _ in range(nbuf)], rnd(rows, heads)
+            bias, a, d = torch.full((heads,), -4.0, device=dev), -torch.rand(heads, device=dev) * 8 - 1, torch.ones(heads, device=dev)
+            states, y = [torch.randn(slots.numel(), heads, n, vdim, device=dev) * 0.01 for _ in range(nbuf)], torch.empty(rows, heads, vdim, device=dev, dtype=bf)
+
+            def run(i):
+                x, b, c = xbc[i].split([cols, keys, keys], dim=1)
+                ops.state_space(x.unflatten(1, (heads, vdim)), b.unflatten(1, (groups, n)), c.unflatten(1, (groups, n)), dt, bias, a, d, y, states[i],
+                                slots, cu, pos)
+            work = {"byts": rows * heads * n * vdim * 8} if cu is None else {"byts": rows * (2 * cols + 2 * keys) * 2, "fp32": rows * heads * n * vdim * 2}
+            leg(f"state_space_{heads}x{vdim}_{tag}", run, nbuf, **work)
+            del xbc, states
+        heads, d = 16, 128
+        q, k, v, o, gate = (rnd(rows, heads, d) for _ in range(5))
+        bc, hb, w = rnd(rows, heads), torch.full((heads,), 4.0, device=dev), torch.ones(heads * d, device=dev)
+        states = [(torch.randn(slots.numel(), heads, d, d, device=dev) * 0.01, torch.zeros(slots.numel(), heads, d, device=dev),
+                   torch.zeros(slots.numel(), heads, device=dev)) for _ in range(nbuf)]
+        work = {"byts": rows * heads * d * d * 8} if cu is None else {"byts": rows * heads * d * 10, "fp32": rows * heads * d * d * 2}
+        leg(f"mlstm_16x128_{tag}", lambda i: ops.mlstm(q, k, v, bc, hb, bc, hb, 15.0, gate.flatten(1), w, o, states[i], slots, cu, pos, d ** -0.5, eps),
+            nbuf, **work)
+        del states
+        u, dt, z, y = (rnd(rows, inner) for _ in range(4))
+        b, c = rnd(rows, 32).split([16, 16], dim=1)
+        bias, a, skip = torch.full((inner,), -4.0, device=dev), -torch.rand(inner, 16, device=dev) * 8 - 1, torch.ones(inner, device=dev)
+        states = [torch.zeros(slots.numel(), inner, 16, device=dev) for _ in range(nbuf)]
+        work = {"byts": rows * inner * 16 * 8} if cu is None else {"byts": rows * inner * 8, "mufu": rows * inner * 16}
+        leg(f"selective_scan_{inner}x16_{tag}", lambda i: ops.selective_scan(u, dt, z, b, c, bias, a, skip, y, states[i], slots, cu, pos), nbuf, **work)
+
+    for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        recurrences(tag, tokens, cu, torch.cat([torch.arange(m, device=dev) for m in lens]), torch.arange(len(lens), dtype=torch.int32, device=dev), 2)
+    recurrences("decode256", 256, None, torch.full((256,), 1199, device=dev), torch.arange(256, dtype=torch.int32, device=dev), 2)
+
+    heads, kv, d, ff = 16, 8, 128, 9216
+    proj = [rnd(tokens, (heads + 2 * kv) * d) for _ in range(4)]
+    cut = lambda x: tuple(t.unflatten(1, (-1, d)) for t in x.split([heads * d, kv * d, kv * d], dim=1))
+    pools = [torch.zeros(2, tokens // 256 + 2, 256, kv, d, device=dev, dtype=bf) for _ in range(4)]
+    table, ones = build_cos_sin_cache(128, 8192, 1e6, head_dim=128).to(dev), torch.ones(d, device=dev, dtype=bf)
+    norm = ops.RowNorm(torch.ones(heads * d, device=dev, dtype=bf), torch.ones(kv * d, device=dev, dtype=bf), heads * d, kv * d, d, eps)
+    for rows in (tokens, 256):
+        pos, slots = torch.arange(rows, device=dev), torch.randperm(rows, device=dev).to(torch.int32)
+        byts = rows * (heads + 2 * kv) * d * 2 * 2
+        part = lambda i: cut(proj[i][:rows])
+        leg(f"qk_norm_rope_kv_write_{rows}", lambda i: ops.qk_norm_rope_kv_write(*part(i), ones, ones, eps, False, pos, table, slots, *pools[i],
+                                                                               k_in_place=False), 4, byts=byts)
+        leg(f"row_norm_rope_kv_write_{rows}", lambda i: ops.row_norm_rope_kv_write(*part(i), norm, pos, table, slots, *pools[i], kv_in_place=False), 4,
+            byts=byts)
+    del pools, proj
+    for rows, m in ((tokens, 3), (256, 48)):
+        # the state-space layer's convolution and norm
+        chan = inner + 2 * 8 * n
+        us, cu = [rnd(rows, chan) for _ in range(min(m, 8))], None if rows == 256 else torch.tensor([0, rows], dtype=torch.int32, device=dev)
+        w4, bias, state = rnd(4, chan), rnd(chan), torch.zeros(256, 3, chan, device=dev, dtype=bf)
+        pos, sl = torch.arange(rows, device=dev), torch.arange(256 if cu is None else 1, dtype=torch.int32, device=dev)
+        leg(f"short_conv_silu_{rows}", lambda i: ops.short_conv_silu(us[i], w4, bias, state, sl, cu, pos), len(us),
+            byts=rows * chan * 4 + (rows * chan * 12 if cu is None else 0))
+        del us
+        ys, zs, os = ([rnd(rows, inner) for _ in range(m)] for _ in range(3))
+        w = torch.ones(inner, device=dev)
+        leg(f"gated_group_norm_8_{rows}", lambda i: ops.gated_group_norm(ys[i], zs[i], w, os[i], 8, eps), m, byts=rows * inner * 6)
+        leg(f"gated_group_norm_1_{rows}", lambda i: ops.gated_group_norm(ys[i], zs[i], w, os[i], 1, eps), m, byts=rows * inner * 6)
+        leg(f"gate_mul_{rows}", lambda i: ops.gate_mul(ys[i], zs[i], os[i]), m, byts=rows * inner * 6)
+        del ys, zs, os
+        zs, os, act = [rnd(rows, ff) for _ in range(m)], [rnd(rows, ff) for _ in range(m)], torch.ones(2, device=dev)
+        leg(f"act_mul_{rows}", lambda i: ops.act_mul(zs[i], ff // 2, False, out=os[i][:, :ff // 2]), m, byts=rows * ff * 3)
+        leg(f"xielu_{rows}", lambda i: ops.xielu(zs[i], act, out=os[i]), m, byts=rows * ff * 4)
+        del zs, os
+        xs, ys, hs, w = [torch.randn(rows, width, device=dev) for _ in range(m)], [rnd(rows, width) for _ in range(m)], [rnd(rows, width) for _ in range(m)], ones.new_ones(width)
+        extra, index, own = rnd(rows * 2, width), torch.randperm(rows * 2, device=dev).view(rows, 2).to(torch.int32), torch.rand(rows, device=dev)
+        own[torch.rand(rows, device=dev) > 0.25] = 0                 # one token in four has an identity expert, and one expert's row less
+        index2 = torch.where((own != 0)[:, None] & (torch.arange(2, device=dev) == 0), -1, index)
+        leg(f"residual_norm_experts_{rows}", lambda i: ops.residual_norm_pair(xs[i], ys[i], w, None, eps, extra, index), m, byts=rows * width * 16)
+        leg(f"residual_norm_experts_identity_{rows}", lambda i: ops.residual_norm_pair(xs[i], ys[i], w, None, eps, extra, index2, own=hs[i],
+                                                                                     own_weights=own), m, byts=rows * width * 16)
+        del xs, ys, hs, extra
+        E, top = SUNULORN_EXPERTS, SUNULORN_TOP
+        h, counters, logits = rnd(rows, width), torch.zeros(E + 1, dtype=torch.int32, device=dev), torch.randn(rows, E + 2, device=dev)
+        routing = ops.Routing(True, torch.zeros(E + 2, device=dev), 2.0, 2)
+        taken = rows * top * E / (E + 2)
+        leg(f"moe_route_and_gather_{rows}", lambda i: ops.moe_sort(h, logits[:, :E], top, counters), 4,
+            byts=rows * (1 + top) * width * 2)
+        leg(f"moe_route_and_gather_identity_{rows}", lambda i: ops.moe_sort(h, logits, top, counters, routing), 4, byts=(rows + taken) * width * 2)
+    return leg.rows
+
+
 # ---- CPU leg: the oracle restatement of the reference path on the host cores ------------------------
 class CpuReference:
     """The oracle model (restatement of the reference's PyTorch path, pinned to the reference's own engine loop by
@@ -1099,6 +1218,8 @@ def main():
                     help="the same for the Vebonex design, beside Fupupel and Qwen3")
     ap.add_argument("--sunulorn", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
                     help="the same for the Sunulorn design, beside Qwen3")
+    ap.add_argument("--rasezen", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
+                    help="the same for the Rasezen design, beside Qwen3")
     ap.add_argument("--engine-steps", type=int, default=0,
                     help="profiling aid: prefill + N decode steps of the workload without CUDA graphs, then exit")
     args = ap.parse_args()
@@ -1146,6 +1267,15 @@ def main():
         if args.sunulorn in ("all", "engine"):
             line["engine"] = sunulorn_throughput()
         print(json.dumps({"sunulorn": line}))
+        return
+    if args.rasezen:
+        torch.cuda.set_device(0)
+        line = {}
+        if args.rasezen in ("all", "kernels"):
+            line["kernels"] = rasezen_kernel_legs(torch.device("cuda", 0), measured_peaks()[0])
+        if args.rasezen in ("all", "engine"):
+            line["engine"] = rasezen_throughput()
+        print(json.dumps({"rasezen": line}))
         return
     if args.kernel_legs:
         peaks, _ = measured_peaks()

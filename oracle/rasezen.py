@@ -83,13 +83,12 @@ def attention(q, k, v, scale: float, seen: torch.Tensor) -> torch.Tensor:
 def state_space(x, b, c, dt, a, d) -> torch.Tensor:
     """x [T, heads, vdim], b and c [T, groups, N], dt [T, heads] (positive), a and d [heads] (a negative) -> [T, heads, vdim]:
     S <- e^{a dt} S + dt b x^T, y = S^T c + d x, token by token."""
-    heads, group = x.shape[1], x.shape[1] // b.shape[1]
-    y = torch.empty_like(x)
-    for h in range(heads):
-        S = torch.zeros(b.shape[2], x.shape[2], dtype=x.dtype)
-        for t in range(x.shape[0]):
-            S = torch.exp(a[h] * dt[t, h]) * S + dt[t, h] * torch.outer(b[t, h // group], x[t, h])
-            y[t, h] = S.T @ c[t, h // group] + d[h] * x[t, h]
+    group_of = torch.arange(x.shape[1]) // (x.shape[1] // b.shape[1])
+    S, y = torch.zeros(x.shape[1], b.shape[2], x.shape[2], dtype=x.dtype), torch.empty_like(x)
+    for t in range(x.shape[0]):
+        key, query = b[t, group_of], c[t, group_of]                  # [heads, N]
+        S = torch.exp(a * dt[t])[:, None, None] * S + dt[t, :, None, None] * key[:, :, None] * x[t, :, None, :]
+        y[t] = (query[:, :, None] * S).sum(1) + d[:, None] * x[t]
     return y
 
 

@@ -329,7 +329,8 @@ def test_experts(cuda, dtype, tokens, experts, top, width, inter, skew):
     feed.load(lambda n: w[n].to(cuda))
     status, hd = ops.new_status(cuda), h.to(cuda)
     for _ in range(3):                                               # later calls find the counters as the first left them
-        y, slots = feed.routed(hd, status)
+        out = feed.routed(hd, status)
+        y, slots = out.rows, out.slots
         assert sorted(slots.flatten().tolist()) == list(range(tokens * top))
         got = y[slots.flatten().long()].view(tokens, top, width).double().sum(1)
         assert rel(got, want) < (2e-2 if dtype == BF else 2e-5)
@@ -354,10 +355,10 @@ def test_experts_in_a_graph_follow_the_tokens(cuda):
     feed.routed(h, None)
     graph = torch.cuda.CUDAGraph()
     with torch.cuda.graph(graph):
-        y, slots = feed.routed(h, None)
+        out = feed.routed(h, None)
     for k in range(4):
         h.copy_((torch.randn(n, width, generator=g) + (3 * (k % 2)) * feed.router[k].float().cpu()).to(BF).to(cuda))
         graph.replay()
-        got = y[slots.flatten().long()].view(n, top, width).float().sum(1)
-        y2, s2 = feed.routed(h, None)
-        assert torch.equal(got, y2[s2.flatten().long()].view(n, top, width).float().sum(1))
+        got = out.rows[out.slots.flatten().long()].view(n, top, width).float().sum(1)
+        again = feed.routed(h, None)
+        assert torch.equal(got, again.rows[again.slots.flatten().long()].view(n, top, width).float().sum(1))
