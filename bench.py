@@ -1011,7 +1011,7 @@ def rasezen_kernel_legs(dev, peaks) -> dict:
     rnd = lambda *shape, scale=1.0: (torch.randn(*shape, device=dev) * scale).to(bf)
     width, tokens, n, eps, inner = 2048, 8192, 128, 1e-6, 4096
 
-    def recurrences(tag, rows, cu, pos, slots, nbuf):
+    def recurrences(tag, rows, cu, pos, slots, nbuf, longest=0):
         for heads, vdim, groups in ((64, 64, 8), (16, 128, 16)):
             cols, keys = heads * vdim, groups * n
             xbc, dt = [rnd(rows, cols + 2 * keys) for _ in range(nbuf)], rnd(rows, heads)
@@ -1021,7 +1021,7 @@ def rasezen_kernel_legs(dev, peaks) -> dict:
             def run(i):
                 x, b, c = xbc[i].split([cols, keys, keys], dim=1)
                 ops.state_space(x.unflatten(1, (heads, vdim)), b.unflatten(1, (groups, n)), c.unflatten(1, (groups, n)), dt, bias, a, d, y, states[i],
-                                slots, cu, pos)
+                                slots, cu, pos, longest)
             work = {"byts": rows * heads * n * vdim * 8} if cu is None else {"byts": rows * (2 * cols + 2 * keys) * 2, "fp32": rows * heads * n * vdim * 2}
             leg(f"state_space_{heads}x{vdim}_{tag}", run, nbuf, **work)
             del xbc, states
@@ -1043,7 +1043,8 @@ def rasezen_kernel_legs(dev, peaks) -> dict:
 
     for tag, lens in (("4x2048", [2048] * 4), ("1x8192", [8192])):
         cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
-        recurrences(tag, tokens, cu, torch.cat([torch.arange(m, device=dev) for m in lens]), torch.arange(len(lens), dtype=torch.int32, device=dev), 2)
+        recurrences(tag, tokens, cu, torch.cat([torch.arange(m, device=dev) for m in lens]), torch.arange(len(lens), dtype=torch.int32, device=dev), 2,
+                    max(lens))
     recurrences("decode256", 256, None, torch.full((256,), 1199, device=dev), torch.arange(256, dtype=torch.int32, device=dev), 2)
 
     heads, kv, d, ff = 16, 8, 128, 9216

@@ -577,7 +577,9 @@ int mvb_moe_gemm(int dtype, const void* x, int64_t x_row_stride, int64_t num_row
 /*
  * mvb_state_space: per head, S <- e^(a dt) S + dt B x^T, y = S^T C + D x, dt = softplus(raw + dt_bias); head h uses the B and C of group
  *   h / (heads / groups).  x [num_tokens, heads, vdim], b and c [num_tokens, groups, num_states <= 256] with one row stride; fp32
- *   dt_bias, a_log2e (= a log2(e), a <= 0) and d [heads]; state fp32 [num_slots, heads, num_states, vdim rounded up to 4].
+ *   dt_bias, a_log2e (= a log2(e), a <= 0) and d [heads]; state fp32 [num_slots, heads, num_states, vdim rounded up to 4]; scratch of
+ *   mvb_state_space_scratch_bytes (often 0).  longest: tokens of the step's longest sequence, by which a ragged step decides whether to
+ *   cut sequences into segments (0: never).
  * mvb_gated_group_norm: out = u / rms(u) * weight with u = y silu(z), the root mean square over each of `groups` equal consecutive parts
  *   of a row of `width`.
  * mvb_row_norm_rope_kv_write: q and k are divided by the root mean square of their whole row (q_dim, k_dim used coordinates) and
@@ -587,7 +589,9 @@ int mvb_moe_gemm(int dtype, const void* x, int64_t x_row_stride, int64_t num_row
 int mvb_state_space(int dtype, const void* x, const void* b, const void* c, int64_t xbc_row_stride, const void* dt, int64_t dt_row_stride,
                     const float* dt_bias, const float* a_log2e, const float* d, void* y, int64_t y_row_stride, float* state,
                     const int32_t* state_slots, int64_t num_slots, const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs,
-                    int num_tokens, int heads, int groups, int num_states, int vdim, int32_t* dev_status, void* stream);
+                    int num_tokens, int longest, int heads, int groups, int num_states, int vdim, void* scratch, size_t scratch_bytes,
+                    int32_t* dev_status, void* stream);
+size_t mvb_state_space_scratch_bytes(int dtype, int num_tokens, int num_seqs, int longest, int heads, int num_states, int vdim, int ragged);
 int mvb_gated_group_norm(int dtype, const void* y, int64_t y_row_stride, const void* z, int64_t z_row_stride, const float* weight, void* out,
                          int64_t out_row_stride, int rows, int width, int groups, float eps, void* stream);
 int mvb_row_norm_rope_kv_write(int dtype, void* q, int64_t q_row_stride, void* k, int64_t k_row_stride, void* v, int64_t v_row_stride,

@@ -98,8 +98,9 @@ SIGNATURES = {
     "mvb_moe_route_ext": (i32, [vp, i64, i32, i32, i32, i32, i32, vp, f32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp]),
     "mvb_moe_gather": (i32, [i32, vp, i64, vp, vp, vp, vp, vp, i64, vp, vp, i32, i32, i32, vp]),
     "mvb_moe_gemm": (i32, [i32, vp, i64, i64, vp, i64, i32, i32, i32, i32, f32, f32, f32, vp, vp, vp, i32, i32, vp, i64, vp, vp]),
-    "mvb_state_space": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, vp,
-                              vp]),
+    "mvb_state_space": (i32, [i32, vp, vp, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp,
+                              sz, vp, vp]),
+    "mvb_state_space_scratch_bytes": (sz, [i32, i32, i32, i32, i32, i32, i32, i32]),
     "mvb_gated_group_norm": (i32, [i32, vp, i64, vp, i64, vp, vp, i64, i32, i32, i32, f32, vp]),
     "mvb_row_norm_rope_kv_write": (i32, [i32, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, f32, vp, vp, i64, vp, vp, vp, i64, i32,
                                          i32, i32, i32, i32, vp, vp]),

@@ -11,10 +11,13 @@
 //   S  <- e^{F_64} S0 + sum_s B_s (e^{F_64 - F_s} dt_s x_s)^T
 // All exponents are <= 0, so no factor exceeds 1 whatever the steps are.  A CTA walks the chunks of one sequence for one head and 16
 // value columns per warp; S^T stays in the accumulator registers of its warp, whose fragments are operand fragments of the next
-// chunk's product as they stand.  C B^T is computed once per CTA, in 16 x 16 blocks handed round the warps, and passes through shared
+// chunk's product as they stand.  C B^T is computed once per CTA, its rows shared out over the warps, and passes through shared
 // memory; B, C and x of the next chunk arrive by cp.async meanwhile.  x, B and C are bf16 and enter exactly; M, S and the scaled
 // values enter as bf16 high + low part (16 significant bits per factor, fp32 accumulation); the state itself is never rounded below
 // fp32.
+// Few (sequence, head) pairs with long prompts would leave most SMs idle, so there the sequences are cut into segments that are walked
+// at the same time: a first pass of the same kernel leaves what each segment alone adds to the state (STATES), ssd_join_kernel turns that
+// into the state in front of every segment, and the second pass starts from there.
 // Ragged step, fp32 (ssd_tokens_kernel): token by token in plain fp32.
 // One token per sequence (ssd_step_kernel): a CTA per (sequence, head) reads the state once and writes it once.
 //
@@ -38,8 +41,12 @@ struct SsdParams {
   const int32_t* cu; const int64_t* positions;
   int num_seqs, tokens, heads, per_group, n, vdim, vp;
   bool vec;                                    // rows of x, b and c may be read, and those of y written, as 16-byte vectors
+  int seg;                                     // tokens of a segment (0: sequences are walked whole)
+  float *seg_state, *seg_keep;                 // [segment slots, heads, N, vp], [segment slots, heads]
   int* dev_status;
 };
+// sequence s owns segment slots seg_base(first row, s) ..: never overlapping, no prefix sum needed
+__device__ __forceinline__ int seg_base(const SsdParams& p, int s) { return p.cu[s] / p.seg + s; }
 
 __device__ __forceinline__ int64_t ssd_slot(const SsdParams& p, int s) {
   if (p.state == nullptr) return -1;
@@ -206,29 +213,51 @@ __device__ __forceinline__ void stmatrix_x4_trans(uint32_t addr, const uint32_t 
                ::"r"(addr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
 }
 
-template <int KS, int WARPS>                    // 16 KS state channels, 16 WARPS value columns
+template <int KS, int WARPS, bool STATES>       // 16 KS state channels, 16 WARPS value columns
 struct SsdCfg {
   static constexpr int NROW = 16 * KS + 8, XROW = 16 * WARPS + 8, MROW = kSsdChunk + 8;      // (odd numbers of 16-byte units: no bank conflicts)
-  static constexpr int B = 0, C = kSsdChunk * NROW, X = 2 * kSsdChunk * NROW, STAGE = X + kSsdChunk * XROW;       // in bf16 numbers
-  static constexpr int SMEM = (2 * STAGE + 2 * kSsdChunk * MROW) * 2;
+  static constexpr int B = 0, X = kSsdChunk * NROW, C = X + kSsdChunk * XROW, STAGE = STATES ? C : C + kSsdChunk * NROW;      // in bf16 numbers
+  static constexpr int SMEM = (2 * STAGE + (STATES ? 0 : 2 * kSsdChunk * MROW)) * 2;
   static constexpr int THREADS = WARPS * 32;
 };
 
-template <int KS, int WARPS>
-__global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(const SsdParams p) {
-  using G = SsdCfg<KS, WARPS>;
+// STATES: only what the segment adds to the state (and what it leaves of the one before) is wanted
+template <int KS, int WARPS, bool STATES>
+__global__ void __launch_bounds__(SsdCfg<KS, WARPS, STATES>::THREADS) ssd_chunk_kernel(const SsdParams p) {
+  using G = SsdCfg<KS, WARPS, STATES>;
   constexpr int Q = kSsdChunk;
   extern __shared__ __align__(128) uint8_t smem[];
   __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(smem);
   __nv_bfloat16* m_hi = stages + 2 * G::STAGE;
   __nv_bfloat16* m_lo = m_hi + Q * G::MROW;
   __shared__ float f_s[2][Q], dt_s[2][Q];         // F_t (log2), dt_t; per chunk parity
-  const int s = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin;
-  if (n_tok <= 0) return;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int s = blockIdx.z, begin = 0, end = 0;
+  if (p.seg == 0) {
+    begin = p.cu[s]; end = p.cu[s + 1];
+  } else {                                        // the sequence and the rows of a segment slot
+    int lo = 0, hi = p.num_seqs;
+    while (hi - lo > 1) {
+      const int mid = (lo + hi) >> 1;
+      if (seg_base(p, mid) <= s) lo = mid; else hi = mid;
+    }
+    begin = p.cu[lo] + (s - seg_base(p, lo)) * p.seg;
+    end = min(begin + p.seg, p.cu[lo + 1]);
+    s = lo;
+  }
+  const int n_tok = end - begin;
+  const bool last = end == p.cu[s + 1];
+  if (n_tok <= 0 || (STATES && last)) return;
   const int n_chunks = (n_tok + Q - 1) / Q, p0 = (blockIdx.x * WARPS + warp) * 16;           // the warp's first value column
-  const int64_t slot = ssd_slot(p, s);
-  const bool fresh = slot < 0 || p.positions[begin] == 0;
+  const int64_t slot = ssd_slot(p, s), states = static_cast<int64_t>(p.n) * p.vp;
+  const float* from = nullptr;                    // the state in front, and where the one behind goes (nullptr: nowhere)
+  float* to = last && slot >= 0 ? p.state + (slot * p.heads + h) * states : nullptr;
+  if (p.seg != 0) {
+    float* here = p.seg_state + (static_cast<int64_t>(blockIdx.z) * p.heads + h) * states;
+    if (STATES) to = here; else from = here;
+  } else if (slot >= 0 && p.positions[begin] != 0) {
+    from = to;
+  }
   const float a = p.a_log2e[h], skip = p.d[h];
   const int64_t group = static_cast<int64_t>(h / p.per_group) * p.n, col0 = static_cast<int64_t>(h) * p.vdim + blockIdx.x * (WARPS * 16);
   const int cols = min(WARPS * 16, p.vdim - blockIdx.x * (WARPS * 16));                      // value columns there are
@@ -256,7 +285,7 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
   auto fetch = [&](int chunk) {
     __nv_bfloat16* st = stages + (chunk & 1) * G::STAGE;
     fetch_rows(st + G::B, G::NROW, bg, p.n, 16 * KS, chunk);
-    fetch_rows(st + G::C, G::NROW, cg, p.n, 16 * KS, chunk);
+    if constexpr (!STATES) fetch_rows(st + G::C, G::NROW, cg, p.n, 16 * KS, chunk);
     fetch_rows(st + G::X, G::XROW, xg, cols, 16 * WARPS, chunk);
     cp_async_commit();
   };
@@ -285,15 +314,14 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
   // S^T: rows p0 + lane / 4 (+ 8), columns 8 j + 2 (lane mod 4) (+ 1)
   const int dq = (lane & 3) * 2, r0 = lane >> 2;
   auto in_state = [&](int j, int i) { return 8 * j + dq + (i & 1) < p.n && p0 + r0 + (i & 2) * 4 < p.vdim; };
-  auto state_at = [&](int j, int i) {
-    return p.state + ((slot * p.heads + h) * static_cast<int64_t>(p.n) + 8 * j + dq + (i & 1)) * p.vp + p0 + r0 + (i & 2) * 4;
-  };
+  auto state_at = [&](int j, int i) { return static_cast<int64_t>(8 * j + dq + (i & 1)) * p.vp + p0 + r0 + (i & 2) * 4; };
   float S[2 * KS][4];
 #pragma unroll
   for (int j = 0; j < 2 * KS; ++j)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) S[j][i] = !fresh && in_state(j, i) ? *state_at(j, i) : 0.f;
+    for (int i = 0; i < 4; ++i) S[j][i] = from != nullptr && in_state(j, i) ? from[state_at(j, i)] : 0.f;
 
+  float kept = 0.f;                               // STATES: sum of the chunks' log decays
   for (int chunk = 0; chunk < n_chunks; ++chunk) {
     const int nt = min(Q, n_tok - chunk * Q), nb = (nt + 15) / 16;                           // tokens, blocks of 16 of them
     const __nv_bfloat16* st = stages + (chunk & 1) * G::STAGE;
@@ -304,74 +332,91 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
       fetch(chunk + 1);
       if (warp == 0) { raw0 = raw_step(chunk + 1, 2 * lane); raw1 = raw_step(chunk + 1, 2 * lane + 1); }
     }
-    // M: 16 x 16 blocks on and below the diagonal, in turn
-    for (int blk = warp; blk < nb * (nb + 1) / 2; blk += WARPS) {
-      int tb = 0;
-      while ((tb + 1) * (tb + 2) / 2 <= blk) ++tb;
-      const int sb = blk - tb * (tb + 1) / 2;
-      float g[2][4];
+    if constexpr (!STATES) {
+      // M: a warp takes rows of 16 x 16 blocks on and below the diagonal (two warps: the first and the last row, and the two between)
+#pragma unroll 1
+      for (int turn = 0; turn < 4 / WARPS; ++turn) {
+        const int tb = WARPS == 4 ? warp : WARPS == 2 ? (turn == 0 ? 3 - warp : warp) : turn;
+        if (tb >= nb) continue;
+        float g[8][4];
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < 8; ++n)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) g[n][i] = 0.f;
-      const uint32_t ca = smem_u32(st + G::C + (tb * 16 + (lane & 15)) * G::NROW + (lane >> 4) * 8);
-      const uint32_t ba = smem_u32(st + G::B + (sb * 16 + (lane & 7) + (lane >> 4) * 8) * G::NROW + ((lane >> 3) & 1) * 8);
+          for (int i = 0; i < 4; ++i) g[n][i] = 0.f;
+        const uint32_t ca = smem_u32(st + G::C + (tb * 16 + (lane & 15)) * G::NROW + (lane >> 4) * 8);
+        const uint32_t ba = smem_u32(st + G::B + ((lane & 7) + (lane >> 4) * 8) * G::NROW + ((lane >> 3) & 1) * 8);
 #pragma unroll
-      for (int ks = 0; ks < KS; ++ks) {
-        uint32_t cf[4], bf[4];
-        ldmatrix_x4(cf, ca + ks * 32);
-        ldmatrix_x4(bf, ba + ks * 32);
-        mma_bf16_16816(g[0], cf, bf[0], bf[1]);
-        mma_bf16_16816(g[1], cf, bf[2], bf[3]);
-      }
+        for (int ks = 0; ks < KS; ++ks) {
+          uint32_t cf[4];
+          ldmatrix_x4(cf, ca + ks * 32);
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int t = tb * 16 + r0 + half * 8, c = sb * 16 + n * 8 + dq;
-          const float ft = F[t];
-          float v[2];
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            v[i] = c + i <= t ? g[n][half * 2 + i] * fast_exp2(ft - F[c + i]) * D[c + i] : 0.f;
-            if (c + i == t) v[i] += skip;
+          for (int sb = 0; sb < 4; ++sb) {
+            if (sb > tb) break;
+            uint32_t bf[4];
+            ldmatrix_x4(bf, ba + (sb * 16 * G::NROW + ks * 16) * 2);
+            mma_bf16_16816(g[2 * sb], cf, bf[0], bf[1]);
+            mma_bf16_16816(g[2 * sb + 1], cf, bf[2], bf[3]);
           }
-          uint32_t hi, lo;
-          split_pair(v[0], v[1], hi, lo);
-          *reinterpret_cast<uint32_t*>(m_hi + t * G::MROW + c) = hi;
-          *reinterpret_cast<uint32_t*>(m_lo + t * G::MROW + c) = lo;
         }
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+          if (n > 2 * tb + 1) break;
+          const int c = n * 8 + dq;
+          const float f0 = F[c], f1 = F[c + 1], d0 = D[c], d1 = D[c + 1];
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int t = tb * 16 + r0 + half * 8;
+            const float ft = F[t];
+            float v0 = c <= t ? g[n][half * 2] * fast_exp2(ft - f0) * d0 : 0.f, v1 = c + 1 <= t ? g[n][half * 2 + 1] * fast_exp2(ft - f1) * d1 : 0.f;
+            if (c == t) v0 += skip;
+            if (c + 1 == t) v1 += skip;
+            uint32_t hi, lo;
+            split_pair(v0, v1, hi, lo);
+            *reinterpret_cast<uint32_t*>(m_hi + t * G::MROW + c) = hi;
+            *reinterpret_cast<uint32_t*>(m_lo + t * G::MROW + c) = lo;
+          }
+        }
+      }
     }
     if (warp == 0 && chunk + 1 < n_chunks) steps(chunk + 1);
-    __syncthreads();                              // M is complete
+    if constexpr (!STATES) __syncthreads();       // M is complete
     // y^T = e^{F_t} S0^T C^T + x^T M^T, 64 tokens wide
     float o[8][4];
 #pragma unroll
     for (int n = 0; n < 8; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
-    const uint32_t cb = smem_u32(st + G::C + ((lane & 7) + (lane >> 4) * 8) * G::NROW + ((lane >> 3) & 1) * 8);
+    if constexpr (!STATES) {
+      const uint32_t cb = smem_u32(st + G::C + ((lane & 7) + (lane >> 4) * 8) * G::NROW + ((lane >> 3) & 1) * 8);
 #pragma unroll
-    for (int ks = 0; ks < KS; ++ks) {
-      Split f;
-      split_tile(S[2 * ks], S[2 * ks + 1], f);
+      for (int ks = 0; ks < KS; ++ks) {
+        Split f;
+        split_tile(S[2 * ks], S[2 * ks + 1], f);
+        uint32_t cf[4][4];                          // (products that add to one accumulator are kept far apart)
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        if (n >= nb) break;
-        uint32_t cf[4];
-        ldmatrix_x4(cf, cb + (n * 16 * G::NROW + ks * 16) * 2);
-        mma_bf16_16816(o[2 * n], f.hi, cf[0], cf[1]);
-        mma_bf16_16816(o[2 * n + 1], f.hi, cf[2], cf[3]);
-        mma_bf16_16816(o[2 * n], f.lo, cf[0], cf[1]);
-        mma_bf16_16816(o[2 * n + 1], f.lo, cf[2], cf[3]);
+        for (int n = 0; n < 4; ++n)
+          if (n < nb) ldmatrix_x4(cf[n], cb + (n * 16 * G::NROW + ks * 16) * 2);
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          if (n >= nb) break;
+          mma_bf16_16816(o[2 * n], f.hi, cf[n][0], cf[n][1]);
+          mma_bf16_16816(o[2 * n + 1], f.hi, cf[n][2], cf[n][3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          if (n >= nb) break;
+          mma_bf16_16816(o[2 * n], f.lo, cf[n][0], cf[n][1]);
+          mma_bf16_16816(o[2 * n + 1], f.lo, cf[n][2], cf[n][3]);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const float e0 = fast_exp2(F[n * 8 + dq]), e1 = fast_exp2(F[n * 8 + dq + 1]);
+        o[n][0] *= e0; o[n][1] *= e1; o[n][2] *= e0; o[n][3] *= e1;
       }
     }
-#pragma unroll
-    for (int n = 0; n < 8; ++n) {
-      const float e0 = fast_exp2(F[n * 8 + dq]), e1 = fast_exp2(F[n * 8 + dq + 1]);
-      o[n][0] *= e0; o[n][1] *= e1; o[n][2] *= e0; o[n][3] *= e1;
-    }
     const float f_end = F[Q - 1], keep = fast_exp2(f_end);
+    kept += f_end;
 #pragma unroll
     for (int j = 0; j < 2 * KS; ++j)
 #pragma unroll
@@ -386,15 +431,15 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
       uint32_t xf[4];
       ldmatrix_x4_trans(xf, xa + k * 16 * G::XROW * 2);
 #pragma unroll
-      for (int n = k; n < 4; ++n) {
-        if (n >= nb) break;
-        uint32_t hi[4], lo[4];
-        ldmatrix_x4(hi, ma + (n * 16 * G::MROW + k * 16) * 2);
-        ldmatrix_x4(lo, ma + LOW + (n * 16 * G::MROW + k * 16) * 2);
-        mma_bf16_16816(o[2 * n], xf, hi[0], hi[1]);
-        mma_bf16_16816(o[2 * n + 1], xf, hi[2], hi[3]);
-        mma_bf16_16816(o[2 * n], xf, lo[0], lo[1]);
-        mma_bf16_16816(o[2 * n + 1], xf, lo[2], lo[3]);
+      for (int low = 0; low < (STATES ? 0 : 2); ++low) {
+#pragma unroll
+        for (int n = k; n < 4; ++n) {
+          if (n >= nb) break;
+          uint32_t m[4];
+          ldmatrix_x4(m, ma + low * LOW + (n * 16 * G::MROW + k * 16) * 2);
+          mma_bf16_16816(o[2 * n], xf, m[0], m[1]);
+          mma_bf16_16816(o[2 * n + 1], xf, m[2], m[3]);
+        }
       }
       Split w;                                    // the same values times e^{F_64 - F_s} dt_s
 #pragma unroll
@@ -404,16 +449,25 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
         split_pair(bf16_lo(xf[2 * half]) * w0, bf16_hi(xf[2 * half]) * w1, w.hi[2 * half], w.lo[2 * half]);
         split_pair(bf16_lo(xf[2 * half + 1]) * w0, bf16_hi(xf[2 * half + 1]) * w1, w.hi[2 * half + 1], w.lo[2 * half + 1]);
       }
+      constexpr int JB = KS % 4 == 0 ? 4 : KS % 3 == 0 ? 3 : KS % 2 == 0 ? 2 : 1;
 #pragma unroll
-      for (int j = 0; j < KS; ++j) {
-        uint32_t bf[4];
-        ldmatrix_x4_trans(bf, bb + (k * 16 * G::NROW + j * 16) * 2);
-        mma_bf16_16816(S[2 * j], w.hi, bf[0], bf[1]);
-        mma_bf16_16816(S[2 * j + 1], w.hi, bf[2], bf[3]);
-        mma_bf16_16816(S[2 * j], w.lo, bf[0], bf[1]);
-        mma_bf16_16816(S[2 * j + 1], w.lo, bf[2], bf[3]);
+      for (int j0 = 0; j0 < KS; j0 += JB) {
+        uint32_t bf[JB][4];
+#pragma unroll
+        for (int j = 0; j < JB; ++j) ldmatrix_x4_trans(bf[j], bb + (k * 16 * G::NROW + (j0 + j) * 16) * 2);
+#pragma unroll
+        for (int j = 0; j < JB; ++j) {
+          mma_bf16_16816(S[2 * (j0 + j)], w.hi, bf[j][0], bf[j][1]);
+          mma_bf16_16816(S[2 * (j0 + j) + 1], w.hi, bf[j][2], bf[j][3]);
+        }
+#pragma unroll
+        for (int j = 0; j < JB; ++j) {
+          mma_bf16_16816(S[2 * (j0 + j)], w.lo, bf[j][0], bf[j][1]);
+          mma_bf16_16816(S[2 * (j0 + j) + 1], w.lo, bf[j][2], bf[j][3]);
+        }
       }
     }
+    if constexpr (STATES) continue;
     // y goes out through the warp's own columns of x, which nobody needs any more
     __syncwarp();
     __nv_bfloat16* out_s = stages + (chunk & 1) * G::STAGE + G::X + warp * 16;
@@ -438,12 +492,34 @@ __global__ void __launch_bounds__(SsdCfg<KS, WARPS>::THREADS) ssd_chunk_kernel(c
         if ((e & 15) < mine) yg[(e >> 4) * p.y_stride + (e & 15)] = out_s[(e >> 4) * G::XROW + (e & 15)];
     }
   }
-  if (slot < 0) return;
+  if (to == nullptr) return;
+  if (STATES && blockIdx.x == 0 && tid == 0) p.seg_keep[static_cast<int64_t>(blockIdx.z) * p.heads + h] = fast_exp2(kept);
 #pragma unroll
   for (int j = 0; j < 2 * KS; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-      if (in_state(j, i)) *state_at(j, i) = S[j][i];
+      if (in_state(j, i)) to[state_at(j, i)] = S[j][i];
+}
+
+// What each segment adds, and leaves of what was there, becomes the state in front of it.  A thread owns four state entries.
+__global__ void __launch_bounds__(256) ssd_join_kernel(const SsdParams p) {
+  const int s = blockIdx.z, h = blockIdx.y, i = (blockIdx.x * 256 + threadIdx.x) * 4;
+  const int64_t states = static_cast<int64_t>(p.n) * p.vp;
+  const int begin = p.cu[s], n_tok = p.cu[s + 1] - begin, segments = (n_tok + p.seg - 1) / p.seg;
+  if (i >= states || segments <= 0) return;
+  const int64_t slot = ssd_slot(p, s), first = seg_base(p, s);
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (slot >= 0 && p.positions[begin] != 0) S = *reinterpret_cast<const float4*>(p.state + (slot * p.heads + h) * states + i);
+#pragma unroll 4
+  for (int k = 0; k < segments; ++k) {
+    const int64_t at = (first + k) * p.heads + h;
+    float4* here = reinterpret_cast<float4*>(p.seg_state + at * states + i);
+    if (k + 1 == segments) { *here = S; break; }
+    const float4 added = *here;
+    const float keep = p.seg_keep[at];
+    *here = S;
+    S.x = fmaf(S.x, keep, added.x); S.y = fmaf(S.y, keep, added.y); S.z = fmaf(S.z, keep, added.z); S.w = fmaf(S.w, keep, added.w);
+  }
 }
 
 // ---- launches ------------------------------------------------------------------------------------------------
@@ -464,22 +540,45 @@ static int launch_ssd_step(const SsdParams& p, cudaStream_t st) {
   return (p.n + 7) / 8 * quads <= 256 ? go(std::integral_constant<int, 8>{}) : go(std::integral_constant<int, 16>{});
 }
 
-template <int KS, int WARPS>
-static int launch_ssd_chunks(const SsdParams& p, cudaStream_t st) {
-  using G = SsdCfg<KS, WARPS>;
+// Segment length of a ragged step (0: whole sequences).  Worth its first pass, about half of the second's work, where the longest
+// sequence would be walked for twice as long as an even share of all tokens takes: two CTAs of 64 columns fit an SM.
+static int ssd_segment(int tokens, int longest, int heads, int vdim) {
+  const int64_t work = static_cast<int64_t>(tokens) * heads * ((vdim + 63) / 64), room = 2 * sm_count();
+  if (longest < 1024 || longest > tokens || longest * room <= 2 * work) return 0;
+  int seg = 256;
+  while (seg < 1024 && work / (2 * seg) >= 2 * room) seg *= 2;
+  return seg;
+}
+static int64_t ssd_segment_slots(int tokens, int num_seqs, int seg) { return tokens / seg + num_seqs; }
+
+template <int KS, int WARPS, bool STATES>
+static int launch_ssd_pass(const SsdParams& p, cudaStream_t st) {
+  using G = SsdCfg<KS, WARPS, STATES>;
   struct Tag {};
-  auto kernel = &ssd_chunk_kernel<KS, WARPS>;
+  auto kernel = &ssd_chunk_kernel<KS, WARPS, STATES>;
   const int rc = opt_in_dynamic_smem<Tag>(reinterpret_cast<const void*>(kernel), G::SMEM);
   if (rc != kOk) return rc;
-  kernel<<<dim3((p.vdim + 16 * WARPS - 1) / (16 * WARPS), p.heads, p.num_seqs), G::THREADS, G::SMEM, st>>>(p);
+  const unsigned z = p.seg == 0 ? p.num_seqs : static_cast<unsigned>(ssd_segment_slots(p.tokens, p.num_seqs, p.seg));
+  kernel<<<dim3((p.vdim + 16 * WARPS - 1) / (16 * WARPS), p.heads, z), G::THREADS, G::SMEM, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
+}
+
+template <int KS, int WARPS>
+static int launch_ssd_chunks(const SsdParams& p, cudaStream_t st) {
+  if (p.seg != 0) {
+    const int rc = launch_ssd_pass<KS, WARPS, true>(p, st);
+    if (rc != kOk) return rc;
+    ssd_join_kernel<<<dim3((p.n * p.vp / 4 + 255) / 256, p.heads, p.num_seqs), 256, 0, st>>>(p);
+    if (cudaGetLastError() != cudaSuccess) return kLaunchFailed;
+  }
+  return launch_ssd_pass<KS, WARPS, false>(p, st);
 }
 
 template <int KS>
 static int launch_ssd_columns(const SsdParams& p, cudaStream_t st) {
   const int tiles = (p.vdim + 15) / 16;
   // few (sequence, head) pairs: narrower CTAs, so that they spread over the SMs
-  const int64_t pairs = static_cast<int64_t>(p.heads) * p.num_seqs;
+  const int64_t pairs = static_cast<int64_t>(p.heads) * (p.seg == 0 ? p.num_seqs : ssd_segment_slots(p.tokens, p.num_seqs, p.seg));
   if (tiles >= 3 && pairs * ((tiles + 3) / 4) >= sm_count()) return launch_ssd_chunks<KS, 4>(p, st);
   return tiles >= 2 ? launch_ssd_chunks<KS, 2>(p, st) : launch_ssd_chunks<KS, 1>(p, st);
 }
@@ -493,7 +592,7 @@ static int launch_ssd_tokens(const SsdParams& p, cudaStream_t st) {
 template <class T>
 static int launch_ssd(const SsdParams& p, cudaStream_t st) {
   if (p.cu == nullptr) return launch_ssd_step<T>(p, st);
-  if (p.heads > 65535 || p.num_seqs > 65535) return kUnsupportedShape;
+  if (p.heads > 65535 || p.num_seqs > 65535 || (p.seg != 0 && ssd_segment_slots(p.tokens, p.num_seqs, p.seg) > 65535)) return kUnsupportedShape;
   if constexpr (sizeof(T) == 2) {
     switch (chunk_ks(p.n)) {
       case 1: return launch_ssd_columns<1>(p, st);
@@ -610,11 +709,20 @@ static int launch_group_norm(const GroupNormParams& p, cudaStream_t st) {
 
 }  // namespace mvb
 
+extern "C" size_t mvb_state_space_scratch_bytes(int dtype, int num_tokens, int num_seqs, int longest, int heads, int num_states, int vdim,
+                                                int ragged) {
+  using namespace mvb;
+  if (!ragged || dtype != kBf16 || num_seqs <= 0 || heads <= 0 || num_states <= 0 || vdim <= 0) return 0;
+  const int seg = ssd_segment(num_tokens, longest, heads, vdim);
+  if (seg == 0) return 0;
+  return static_cast<size_t>(ssd_segment_slots(num_tokens, num_seqs, seg)) * heads * (static_cast<size_t>(num_states) * ((vdim + 3) / 4 * 4) + 1) * sizeof(float);
+}
+
 extern "C" int mvb_state_space(int dtype, const void* x, const void* b, const void* c, int64_t xbc_row_stride, const void* dt,
                                int64_t dt_row_stride, const float* dt_bias, const float* a_log2e, const float* d, void* y,
                                int64_t y_row_stride, float* state, const int32_t* state_slots, int64_t num_slots,
-                               const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int heads, int groups,
-                               int num_states, int vdim, int32_t* dev_status, void* stream) {
+                               const int32_t* cu_seqlens_q, const int64_t* positions, int num_seqs, int num_tokens, int longest, int heads,
+                               int groups, int num_states, int vdim, void* scratch, size_t scratch_bytes, int32_t* dev_status, void* stream) {
   using namespace mvb;
   if (!x || !b || !c || !dt || !dt_bias || !a_log2e || !d || !y || !positions) return kInvalidArgument;
   if (num_seqs < 0 || num_tokens < 0 || heads <= 0 || groups <= 0 || heads % groups != 0 || num_states <= 0 || vdim <= 0) return kInvalidArgument;
@@ -626,8 +734,16 @@ extern "C" int mvb_state_space(int dtype, const void* x, const void* b, const vo
   if (num_tokens == 0 || num_seqs == 0) return kOk;
   const bool vec = vdim % 8 == 0 && num_states % 8 == 0 && xbc_row_stride % 8 == 0 && y_row_stride % 8 == 0 && is_aligned(x, 16) &&
                    is_aligned(b, 16) && is_aligned(c, 16) && is_aligned(y, 16);
-  const SsdParams p{x, b, c, xbc_row_stride, dt, dt_row_stride, dt_bias, a_log2e, d, y, y_row_stride, state, state_slots, num_slots,
-                    cu_seqlens_q, positions, num_seqs, num_tokens, heads, heads / groups, num_states, vdim, (vdim + 3) / 4 * 4, vec, dev_status};
+  SsdParams p{x, b, c, xbc_row_stride, dt, dt_row_stride, dt_bias, a_log2e, d, y, y_row_stride, state, state_slots, num_slots,
+                    cu_seqlens_q, positions, num_seqs, num_tokens, heads, heads / groups, num_states, vdim, (vdim + 3) / 4 * 4, vec, 0, nullptr,
+              nullptr, dev_status};
+  if (dtype == kBf16 && cu_seqlens_q != nullptr) p.seg = ssd_segment(num_tokens, longest, heads, vdim);
+  if (p.seg != 0) {
+    if (!scratch || scratch_bytes < mvb_state_space_scratch_bytes(dtype, num_tokens, num_seqs, longest, heads, num_states, vdim, 1)) return kInvalidArgument;
+    if (!is_aligned(scratch, 16)) return kMisaligned;
+    p.seg_state = static_cast<float*>(scratch);
+    p.seg_keep = p.seg_state + ssd_segment_slots(num_tokens, num_seqs, p.seg) * heads * num_states * p.vp;
+  }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == kBf16 ? launch_ssd<__nv_bfloat16>(p, st) : launch_ssd<float>(p, st);
 }

@@ -313,7 +313,7 @@ class StateSpaceBranch(Branch):
         y = torch.empty(u.shape[0], self.ip, dtype=u.dtype, device=u.device)
         x, o = (t[:, :self.inner].unflatten(1, (self.heads, self.vdim)) for t in (x, y))
         ops.state_space(x, b, c, dt[:, :self.heads], self.dt_bias, self.a_log2e, self.skip, o, self.memory, ctx.state_slots, cu, positions,
-                        status=ctx.status)
+                        longest=ctx.max_seqlen_q if ctx.prefill else 0, status=ctx.status)
         ops.gated_group_norm(y[:, :self.inner], z[:, :self.inner], self.norm_weight, out[:, :self.inner], self.norm_groups, self.eps)
 
 

@@ -836,10 +836,11 @@ def selective_scan(u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, b: torch.
 
 def state_space(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log2e: torch.Tensor,
                 d: torch.Tensor, out: torch.Tensor, state: torch.Tensor | None, state_slots: torch.Tensor | None,
-                cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor, status: torch.Tensor | None = None) -> torch.Tensor:
+                cu_seqlens_q: torch.Tensor | None, positions: torch.Tensor, longest: int = 0,
+                status: torch.Tensor | None = None) -> torch.Tensor:
     """``S <- e^(a dt) S + dt b x^T``, ``out = S^T c + d x`` per head, dt = softplus(raw + bias): x and out [T, heads, vdim], b and c
     [T, groups, N], raw ``dt`` [T, heads]; fp32 ``dt_bias``, ``a_log2e`` (a times log2(e)) and ``d`` [heads]; ``state`` fp32
-    [slots, heads, N, vdim padded to 4]."""
+    [slots, heads, N, vdim padded to 4].  ``longest``: tokens of the step's longest sequence; few long ones are cut into segments."""
     code = _dtype_of(x, "x")
     _same(x.dtype, b=b, c=c, dt=dt, out=out)
     _same(torch.float32, dt_bias=dt_bias, a_log2e=a_log2e, d=d, state=state)
@@ -852,11 +853,15 @@ def state_space(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Ten
     assert state is None or state.shape[1:] == (heads, n, -(-vdim // 4) * 4)
     st, sl, slots = _state_args(state, state_slots)
     num_seqs = tokens if cu_seqlens_q is None else cu_seqlens_q.numel() - 1
-    rc = _cabi.load().mvb_state_space(
+    lib, ragged = _cabi.load(), cu_seqlens_q is not None
+    need = lib.mvb_state_space_scratch_bytes(code, tokens, num_seqs, longest, heads, n, vdim, int(ragged))
+    scratch = torch.empty(need, dtype=torch.uint8, device=x.device) if need else None
+    rc = lib.mvb_state_space(
         code, _ptr(x), _ptr(b), _ptr(c), x.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log2e), _ptr(d), _ptr(out),
-        out.stride(0), st, sl, slots, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, heads, groups, n, vdim, _ptr(status), _stream())
+        out.stride(0), st, sl, slots, _ptr(cu_seqlens_q), _ptr(positions), num_seqs, tokens, longest, heads, groups, n, vdim, _ptr(scratch), need,
+        _ptr(status), _stream())
     _cabi.check(rc, "mvb_state_space")
-    LaunchCounter.add(1)
+    LaunchCounter.add(3 if need else 1)
     return out
 
 

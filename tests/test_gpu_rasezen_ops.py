@@ -30,7 +30,7 @@ def run_state_space(cuda, seqs, heads, dt_bias, a, d, portions, dtype, slots=Tru
         x, b, c, dt = (v[:, :f.shape[1]] for v, f in zip(wide.split(pad, dim=1), flat))
         out = torch.full((pos.numel(), pad[0]), math.nan, dtype=dtype, device=cuda)[:, :flat[0].shape[1]].unflatten(1, (heads, vdim))
         ops.state_space(x.unflatten(1, (heads, vdim)), *(t.unflatten(1, (-1, n)) for t in (b, c)), dt, *consts, out, state, slot if slots else None,
-                        cu, pos, status=status)
+                        cu, pos, longest=max(hi - lo for _, lo, hi in entries) if cu is not None else 0, status=status)
         at = 0
         for i, lo, hi in entries:
             got[i][lo:hi] = out[at:at + hi - lo].double().cpu()
@@ -92,6 +92,21 @@ def test_a_remembered_token(cuda, dtype, at):
     for portions in ([[10 ** 6]], [[max(at, 1), 1, 2]], [[at + 1, 63]], [[1]]):
         got = run_state_space(cuda, [s], 1, bias, a, d, portions, dtype)[0]
         assert rel(got[192:], want[192:]) < (5e-3 if dtype == BF else 1e-5)
+
+
+@pytest.mark.parametrize("heads,groups,n,vdim", [(2, 1, 16, 16), (3, 1, 40, 72), (2, 2, 128, 24)])
+@pytest.mark.parametrize("portions,slots", [([[10 ** 6]], True), ([[10 ** 6]], False), ([[1100, 64, 300], [70, 1], [1], [1200]], True)])
+def test_long_sequences_in_segments(cuda, heads, groups, n, vdim, portions, slots):
+    """Long sequences beside short ones are cut into segments that are walked at once: the same outputs, and the same state for what
+    follows, as one by one."""
+    from mini_vllm_b200 import _cabi
+    g, lens = gen(n), [1500, 71, 1, 1290]
+    assert _cabi.load().mvb_state_space_scratch_bytes(0, sum(lens), len(lens), max(lens), heads, n, vdim, 1) > 0
+    mk = lambda *s: torch.randn(*s, generator=g).to(BF)
+    seqs = [{"x": mk(t, heads, vdim), "b": mk(t, groups, n), "c": mk(t, groups, n), "dt": mk(t, heads)} for t in lens]
+    dt_bias, a, d = torch.full((heads,), -3.0), -torch.exp(torch.linspace(-9, 1, heads)), torch.ones(heads)      # from long memories to short
+    for x, s in zip(run_state_space(cuda, seqs, heads, dt_bias, a, d, portions, BF, slots=slots), seqs):
+        assert rel(x, want_state_space(s, dt_bias, a, d)) < 6e-3
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
