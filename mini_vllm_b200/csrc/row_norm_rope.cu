@@ -203,7 +203,8 @@ __global__ void __launch_bounds__(256) row_rope_any_kernel(const RowRopeParams p
 template <int PPH>
 static int launch_row_rope(const RowRopeParams& p, cudaStream_t st) {
   const int tasks = (p.hq + 2 * p.hkv) * PPH;
-  const int items = tasks <= 384 ? 1 : tasks <= 1024 ? 2 : 4;
+  // many tokens: small blocks with more loads in flight per thread; few: the shortest path for each
+  const int items = p.tokens >= 1024 ? (tasks <= 128 ? 2 : 4) : tasks <= 384 ? 1 : tasks <= 1024 ? 2 : 4;
   const int nt = ((tasks + items - 1) / items + 31) / 32 * 32;
   if (nt > 512) return kUnsupportedShape;
   if (items == 1) row_rope_kernel<1, PPH><<<p.tokens, nt, 0, st>>>(p);
