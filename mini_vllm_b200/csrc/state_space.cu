@@ -19,7 +19,8 @@
 // at the same time: a first pass of the same kernel leaves what each segment alone adds to the state (STATES), ssd_join_kernel turns that
 // into the state in front of every segment, and the second pass starts from there.
 // Ragged step, fp32 (ssd_tokens_kernel): token by token in plain fp32.
-// One token per sequence (ssd_step_kernel): a CTA per (sequence, head) reads the state once and writes it once.
+// One token per sequence (ssd_step_kernel): a CTA per sequence and up to 64 columns of a head, the state read once and
+// written once.
 //
 // gated_group_norm_kernel finishes the mixer: y silu(z), over the root mean square of each of `groups` equal parts of the row, times w.
 //
@@ -27,8 +28,6 @@
 #include "chunk_common.cuh"
 #include "host_util.cuh"
 #include "mini_vllm_b200.h"
-
-#include <type_traits>
 
 namespace mvb {
 
@@ -68,63 +67,57 @@ template <class T> __device__ __forceinline__ float ssd_advance(float S, float d
 }
 
 // ---- one token per sequence ------------------------------------------------------------------------------
-template <class T, int RPT>
-__global__ void __launch_bounds__(512) ssd_step_kernel(const SsdParams p, int tile_cols) {
+// A CTA has tile_cols columns of a head, a thread kStepRows rows x 4 columns.
+constexpr int kStepRows = 8;
+
+template <class T>
+__global__ void __launch_bounds__(512, 2) ssd_step_kernel(const SsdParams p, int tile_cols, int tiles) {
   extern __shared__ __align__(16) float sm[];
-  const int s = blockIdx.y, h = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
-  const int quads = tile_cols / 4, row_groups = (p.n + RPT - 1) / RPT;
+  const int s = blockIdx.y, h = blockIdx.x / tiles, col0 = blockIdx.x % tiles * tile_cols, tid = threadIdx.x, nt = blockDim.x;
+  const int quads = tile_cols / 4, row_groups = (p.n + kStepRows - 1) / kStepRows;
   float* red = sm;                              // [row groups][tile_cols]
   float* b_s = red + row_groups * tile_cols;    // [n], times dt
   float* c_s = b_s + p.n;
   const int64_t slot = ssd_slot(p, s);
   const bool fresh = slot < 0 || p.positions[s] == 0;
-  const int rg = tid / quads, cq = tid % quads;
-  const int64_t hbase = (slot * p.heads + h) * static_cast<int64_t>(p.n);
+  const int rg = tid / quads, cq = tid % quads, c = col0 + cq * 4;
+  const int rows = rg < row_groups && c < p.vp ? (p.n - rg + row_groups - 1) / row_groups : 0;      // rows rg, rg + row_groups, ...
+  const int64_t down = static_cast<int64_t>(row_groups) * p.vp;
+  float* at = p.state + ((slot * p.heads + h) * static_cast<int64_t>(p.n) + rg) * p.vp + c;
+  float4 S[kStepRows];
+#pragma unroll
+  for (int r = 0; r < kStepRows; ++r) {         // the state first: it is what the kernel waits for
+    S[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!fresh && r < rows) S[r] = __ldcs(reinterpret_cast<const float4*>(at + r * down));
+  }
+  const float dt = ssd_dt<T>(p, s, h), decay = ssd_decay<T>(p.a_log2e[h] * dt);
+  const int64_t group = s * p.stride + static_cast<int64_t>(h / p.per_group) * p.n;
+  for (int i = tid; i < p.n; i += nt) {
+    b_s[i] = to_f(static_cast<const T*>(p.b)[group + i]) * dt;
+    c_s[i] = to_f(static_cast<const T*>(p.c)[group + i]);
+  }
   const T* xrow = static_cast<const T*>(p.x) + s * p.stride + static_cast<int64_t>(h) * p.vdim;
-  float decay = 0.f;
-  for (int col0 = 0; col0 < p.vp; col0 += tile_cols) {
-    const int c = col0 + cq * 4;
-    const bool active = rg < row_groups && c < p.vp;
-    float4 S[RPT];
+  float x[4];
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) {             // the state first: it is what the kernel waits for
-      const int row = rg + r * row_groups;
-      S[r] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (active && !fresh && row < p.n) S[r] = *reinterpret_cast<const float4*>(p.state + (hbase + row) * p.vp + c);
-    }
-    float x[4];
+  for (int j = 0; j < 4; ++j) x[j] = rows > 0 && c + j < p.vdim ? to_f(xrow[c + j]) : 0.f;
+  __syncthreads();
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) x[j] = active && c + j < p.vdim ? to_f(xrow[c + j]) : 0.f;
-    if (col0 == 0) {
-      const float dt = ssd_dt<T>(p, s, h);
-      decay = ssd_decay<T>(p.a_log2e[h] * dt);
-      const int64_t at = s * p.stride + static_cast<int64_t>(h / p.per_group) * p.n;
-      for (int i = tid; i < p.n; i += nt) {
-        b_s[i] = to_f(static_cast<const T*>(p.b)[at + i]) * dt;
-        c_s[i] = to_f(static_cast<const T*>(p.c)[at + i]);
-      }
-      __syncthreads();
-    }
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-      const int row = rg + r * row_groups;
-      if (!active || row >= p.n) continue;
-      const float k = b_s[row], q = c_s[row];
-      S[r].x = ssd_advance<T>(S[r].x, decay, k * x[0]); S[r].y = ssd_advance<T>(S[r].y, decay, k * x[1]);
-      S[r].z = ssd_advance<T>(S[r].z, decay, k * x[2]); S[r].w = ssd_advance<T>(S[r].w, decay, k * x[3]);
-      acc.x = fmaf(S[r].x, q, acc.x); acc.y = fmaf(S[r].y, q, acc.y); acc.z = fmaf(S[r].z, q, acc.z); acc.w = fmaf(S[r].w, q, acc.w);
-      if (slot >= 0) *reinterpret_cast<float4*>(p.state + (hbase + row) * p.vp + c) = S[r];
-    }
-    if (active) *reinterpret_cast<float4*>(red + rg * tile_cols + cq * 4) = acc;
-    __syncthreads();
-    if (tid < tile_cols && col0 + tid < p.vdim) {
-      float y = 0.f;
-      for (int w = 0; w < row_groups; ++w) y += red[w * tile_cols + tid];
-      y = fmaf(p.d[h], to_f(xrow[col0 + tid]), y);
-      static_cast<T*>(p.y)[s * p.y_stride + static_cast<int64_t>(h) * p.vdim + col0 + tid] = from_f<T>(y);
-    }
-    __syncthreads();                            // red is about to be used again
+  for (int r = 0; r < kStepRows; ++r) {
+    if (r >= rows) break;
+    const float k = b_s[rg + r * row_groups], q = c_s[rg + r * row_groups];
+    S[r].x = ssd_advance<T>(S[r].x, decay, k * x[0]); S[r].y = ssd_advance<T>(S[r].y, decay, k * x[1]);
+    S[r].z = ssd_advance<T>(S[r].z, decay, k * x[2]); S[r].w = ssd_advance<T>(S[r].w, decay, k * x[3]);
+    acc.x = fmaf(S[r].x, q, acc.x); acc.y = fmaf(S[r].y, q, acc.y); acc.z = fmaf(S[r].z, q, acc.z); acc.w = fmaf(S[r].w, q, acc.w);
+    if (slot >= 0) __stcs(reinterpret_cast<float4*>(at + r * down), S[r]);
+  }
+  if (rg < row_groups) *reinterpret_cast<float4*>(red + rg * tile_cols + cq * 4) = acc;
+  __syncthreads();
+  if (tid < tile_cols && col0 + tid < p.vdim) {
+    float y = 0.f;
+    for (int w = 0; w < row_groups; ++w) y += red[w * tile_cols + tid];
+    y = fmaf(p.d[h], to_f(xrow[col0 + tid]), y);
+    static_cast<T*>(p.y)[s * p.y_stride + static_cast<int64_t>(h) * p.vdim + col0 + tid] = from_f<T>(y);
   }
 }
 
@@ -510,34 +503,38 @@ __global__ void __launch_bounds__(256) ssd_join_kernel(const SsdParams p) {
   const int64_t slot = ssd_slot(p, s), first = seg_base(p, s);
   float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
   if (slot >= 0 && p.positions[begin] != 0) S = *reinterpret_cast<const float4*>(p.state + (slot * p.heads + h) * states + i);
-#pragma unroll 4
-  for (int k = 0; k < segments; ++k) {
-    const int64_t at = (first + k) * p.heads + h;
-    float4* here = reinterpret_cast<float4*>(p.seg_state + at * states + i);
-    if (k + 1 == segments) { *here = S; break; }
-    const float4 added = *here;
-    const float keep = p.seg_keep[at];
-    *here = S;
-    S.x = fmaf(S.x, keep, added.x); S.y = fmaf(S.y, keep, added.y); S.z = fmaf(S.z, keep, added.z); S.w = fmaf(S.w, keep, added.w);
+  constexpr int U = 8;                            // segments whose parts are requested before the first is used
+  for (int k0 = 0; k0 < segments; k0 += U) {
+    float4 added[U];
+    float keep[U];
+#pragma unroll
+    for (int j = 0; j < U; ++j)
+      if (k0 + j + 1 < segments) {
+        added[j] = *reinterpret_cast<const float4*>(p.seg_state + ((first + k0 + j) * p.heads + h) * states + i);
+        keep[j] = p.seg_keep[(first + k0 + j) * p.heads + h];
+      }
+#pragma unroll
+    for (int j = 0; j < U; ++j) {
+      if (k0 + j >= segments) return;
+      *reinterpret_cast<float4*>(p.seg_state + ((first + k0 + j) * p.heads + h) * states + i) = S;
+      if (k0 + j + 1 == segments) return;
+      S.x = fmaf(S.x, keep[j], added[j].x); S.y = fmaf(S.y, keep[j], added[j].y);
+      S.z = fmaf(S.z, keep[j], added[j].z); S.w = fmaf(S.w, keep[j], added[j].w);
+    }
   }
 }
 
 // ---- launches ------------------------------------------------------------------------------------------------
 template <class T>
 static int launch_ssd_step(const SsdParams& p, cudaStream_t st) {
-  const int tile = p.vp < 128 ? p.vp : 128, quads = tile / 4;
+  const int tile = p.vp < 64 ? p.vp : 64, tiles = (p.vp + tile - 1) / tile, quads = tile / 4;
   if (p.num_seqs > 65535) return kUnsupportedShape;
-  auto go = [&](auto tag) -> int {
-    constexpr int RPT = decltype(tag)::value;
-    const int row_groups = (p.n + RPT - 1) / RPT;
-    int nt = (row_groups * quads + 31) / 32 * 32;
-    if (nt < (tile + 31) / 32 * 32) nt = (tile + 31) / 32 * 32;      // a thread per column at the end
-    const size_t smem = (2 * static_cast<size_t>(p.n) + static_cast<size_t>(row_groups) * tile) * sizeof(float);
-    if (nt > 512 || smem > 47 * 1024) return kUnsupportedShape;
-    ssd_step_kernel<T, RPT><<<dim3(p.heads, p.num_seqs), nt, smem, st>>>(p, tile);
-    return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
-  };
-  return (p.n + 7) / 8 * quads <= 256 ? go(std::integral_constant<int, 8>{}) : go(std::integral_constant<int, 16>{});
+  const int row_groups = (p.n + kStepRows - 1) / kStepRows;
+  int nt = (row_groups * quads + 31) / 32 * 32;                      // N <= 256 and 16 quads at most: never more than 512 threads
+  if (nt < (tile + 31) / 32 * 32) nt = (tile + 31) / 32 * 32;        // a thread per column at the end
+  const size_t smem = (2 * static_cast<size_t>(p.n) + static_cast<size_t>(row_groups) * tile) * sizeof(float);
+  ssd_step_kernel<T><<<dim3(p.heads * tiles, p.num_seqs), nt, smem, st>>>(p, tile, tiles);
+  return cudaGetLastError() == cudaSuccess ? kOk : kLaunchFailed;
 }
 
 // Segment length of a ragged step (0: whole sequences).  Worth its first pass, about half of the second's work, where the longest
@@ -624,7 +621,7 @@ struct GroupNormParams {
   float eps;
 };
 
-// TPR threads per part (32: several parts per block, no shared memory), ITEMS vectors per thread; a part longer than that (LOOP) is
+// A warp per part, eight parts per block, or (WIDE) a block per part; a thread keeps ITEMS vectors, and what a part has beyond them is
 // read a second time
 template <class T, int V, int ITEMS, bool WIDE>
 __global__ void __launch_bounds__(256) gated_group_norm_kernel(const GroupNormParams p) {
