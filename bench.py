@@ -1220,7 +1220,7 @@ def main():
     ap.add_argument("--sunulorn", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
                     help="the same for the Sunulorn design, beside Qwen3")
     ap.add_argument("--rasezen", nargs="?", const="all", default=None, choices=["all", "engine", "kernels"],
-                    help="the same for the Rasezen design, beside Qwen3")
+                    help="the same for the Rasezen design, beside Sunulorn, Fupupel and Qwen3")
     ap.add_argument("--engine-steps", type=int, default=0,
                     help="profiling aid: prefill + N decode steps of the workload without CUDA graphs, then exit")
     args = ap.parse_args()

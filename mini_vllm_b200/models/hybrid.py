@@ -1,6 +1,6 @@
-"""Decoder assembled layer by layer from mixer branches (attention, latent attention, selective scan, state space, gated delta rule, gated linear
-attention, matrix-memory LSTM), a feed-forward of its own kind, and an fp32 residual of its own kind (``layers/residual.py``), with
-optional tanh caps on the logits.
+"""Decoder assembled layer by layer from mixer branches (attention, latent attention, selective scan, state space, gated delta rule,
+gated linear attention, matrix-memory LSTM), a feed-forward of its own kind, and an fp32 residual of its own kind
+(``layers/residual.py``), with optional tanh caps on the logits.
 
 The step contract is ``DecoderLM``'s (``models/decoder.py``): ``forward(ctx, input_ids, positions, head)``, one row per
 sequence - or per entry of ``ctx.logit_rows`` - and the same loader, executor, KV pool, CUDA graphs and sampler.  Recurrent

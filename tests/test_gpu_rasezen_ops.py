@@ -46,7 +46,7 @@ def want_state_space(s, dt_bias, a, d):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("heads,groups,n,vdim", [(4, 2, 16, 16), (3, 3, 20, 12), (4, 1, 128, 64), (2, 1, 48, 32), (5, 1, 7, 9), (2, 2, 256, 40),
+@pytest.mark.parametrize("heads,groups,n,vdim", [(4, 2, 16, 16), (3, 3, 20, 12), (4, 1, 128, 64), (2, 1, 56, 32), (5, 1, 7, 9), (2, 2, 256, 40),
                                                  (1, 1, 1, 1), (6, 2, 64, 136), (80, 8, 24, 56), (2, 1, 180, 72)])
 @pytest.mark.parametrize("portions", list(PORTIONS))
 def test_state_space(cuda, dtype, heads, groups, n, vdim, portions):
@@ -67,7 +67,7 @@ def test_state_space_at_its_extremes(cuda, dtype, dt_bias, log_a):
     """Steps of nothing, decays to zero within a token (exponents far below what fp32 holds), and memories that lose nothing."""
     g, heads = gen(5), 2
     mk = lambda *s: torch.randn(*s, generator=g).to(dtype)
-    seqs = [{"x": mk(t, heads, 32), "b": mk(t, 1, 48), "c": mk(t, 1, 48), "dt": mk(t, heads)} for t in (200, 65)]
+    seqs = [{"x": mk(t, heads, 40), "b": mk(t, 1, 24), "c": mk(t, 1, 24), "dt": mk(t, heads)} for t in (200, 65)]
     bias, a, d = torch.full((heads,), dt_bias), torch.full((heads,), -math.exp(log_a)), torch.tensor([0.0, 1.0])
     for portions in ("whole", "single", "long"):
         for x, s in zip(run_state_space(cuda, seqs, heads, bias, a, d, portions, dtype), seqs):
